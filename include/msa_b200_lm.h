@@ -1,0 +1,128 @@
+/*
+ * msa_b200_lm -- C ABI of the kernels behind the layered decoder designs (libmsa_b200_lm.so): residual / norm steps,
+ * windowed latent attention, the gated delta rule, and mixtures of small experts.
+ *
+ * Conventions are those of msa_b200.h (raw device pointers owned by the caller, asynchronous on `stream`, strides in
+ * elements, MSA_OK or a negative code with msa_last_error()).  `dtype` is the type of activations and weights
+ * (MSA_BF16 or MSA_F32); norms, scores, gates, states and the residual are 32-bit in both.
+ *
+ * Packed step.  A step runs n_tok tokens of n_seq sequences, packed one sequence after the other: sequence s owns the
+ * rows cu[s] .. cu[s+1]-1, continues at position start[s] and keeps its state in slot slot[s].  The first n_decode
+ * sequences bring exactly one token each.
+ */
+#ifndef MSA_B200_LM_H
+#define MSA_B200_LM_H
+
+#include "msa_b200.h"
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+/* x_out[r] = base + branch;  h_out[r] = rmsnorm(x_out[r]) * w_next;  cat_out[r] = x_out[r] rounded to dtype.
+ *   base    row r of base [.., width] fp32 with base_stride (0: one vector for all rows), or null
+ *   branch  null, or B = row r of y (y_dtype), or the weighted sum over k < top of rows inv[r*top+k] of y with
+ *           weights mix[r*top+k] (inv != null); with w_branch: rmsnorm(B) * w_branch
+ *   rows    optional: output row r works on input row rows[r] of base
+ * Any of x_out, h_out (with w_next), cat_out may be null. */
+int msa_lm_residual_norm(const float* base, int64_t base_stride, const void* y, int32_t y_dtype, int64_t y_stride,
+                         const int32_t* inv, const float* mix, int32_t top, const float* w_branch, const float* w_next,
+                         float eps, const int32_t* rows, int32_t n_rows, int32_t width, float* x_out, void* h_out,
+                         void* cat_out, int64_t cat_stride, int32_t dtype, void* stream);
+
+/* x_out[r] = table[token[r]] (fp32), h_out = rmsnorm(x_out) * w_next, cat0 / cat1[r] = the row in dtype (either null).
+ * Tokens outside 0 .. vocab-1 read row 0 and count in status[2]. */
+int msa_lm_embed(const void* table, const int32_t* token, int32_t n_rows, int32_t width, int32_t vocab,
+                 const float* w_next, float eps, float* x_out, void* h_out, void* cat0, void* cat1, int64_t cat_stride,
+                 int32_t* status, int32_t dtype, void* stream);
+
+/* out[r, j] = silu(gu[r, j]) * gu[r, ff + j]. */
+int msa_lm_silu_mul(const void* gu, int64_t gu_stride, int32_t n_rows, int32_t ff, void* out, int32_t dtype, void* stream);
+
+/* ---- windowed latent attention ------------------------------------------------------------------------------------
+ * proj row = [heads * (dim + rot) query | rank latent | rot shared key part].  The kernel normalises the latent with
+ * w_norm, rotates the key part and (in place) every head's rotated query part, and writes [latent | key part] to the
+ * sequence's ring (decode rows: ring[slot][position % ring_rows]) or to the packed context of the step (the others:
+ * row ctx_off[s - n_decode] + min(start, window - 1) + t).  It also copies the ring rows that a continued portion still
+ * sees (positions start - min(start, window-1) .. start-1) into the context, n_old rows in all; old_off is their prefix
+ * sum over the non-decode sequences. */
+int msa_lm_latent_prep(void* proj, int64_t proj_stride, const float* w_norm, float eps, const float* inv_freq,
+                       int32_t heads, int32_t dim, int32_t rot, int32_t rank, const int32_t* pos, const int32_t* tok_seq,
+                       const int32_t* slot, const int32_t* start, const int32_t* cu, const int32_t* ctx_off,
+                       const int32_t* old_off, int32_t n_tok, int32_t n_seq, int32_t n_decode, int32_t n_old,
+                       int32_t window, void* ring, int64_t ring_rows, void* ctx, int32_t dtype, void* stream);
+
+/* The last min(tokens, ring_rows) context rows of every non-decode sequence go to its ring. */
+int msa_lm_ring_store(const void* ctx, int32_t row_width, const int32_t* slot, const int32_t* start, const int32_t* cu,
+                      const int32_t* ctx_off, int32_t n_seq, int32_t n_decode, int32_t max_len, int32_t window, void* ring,
+                      int64_t ring_rows, int32_t dtype, void* stream);
+
+/* General windowed attention (any sizes, both dtypes).  A query is [qa (da) | qb (db)], a key [ka | kb]; strides per row
+ * and per head (a head stride of 0 shares the operand).  Queries: rows cu[s] .. of the sequences seq0 .. seq1-1, token t
+ * at position start[s] + t.  Keys: ring_rows > 0: position j in row slot[s] * ring_rows + j % ring_rows; else context row
+ * ctx_off[s - seq0] + (j - first), first = start[s] - min(start[s], window-1).  Position i sees 0 <= i - j < window.
+ * out row stride out_stride, head stride out_head. */
+typedef struct {
+  const void* qa; int64_t qa_row, qa_head;
+  const void* qb; int64_t qb_row, qb_head;
+  const void* ka; int64_t ka_row, ka_head;
+  const void* kb; int64_t kb_row, kb_head;
+  const void* v;  int64_t v_row, v_head;
+  void* out;      int64_t out_row, out_head;
+  const int32_t *slot, *start, *cu, *ctx_off;
+  int64_t ring_rows;
+  int32_t seq0, seq1, max_len, heads, da, db, dv, window;
+  int32_t qa_dtype, out_dtype, dtype;   /* qa and out may be fp32 beside bf16 keys and values */
+  float scale;
+} msa_lm_attn_args;
+int msa_lm_window_attn(const msa_lm_attn_args* args, void* stream);
+
+/* ---- gated delta rule ---------------------------------------------------------------------------------------------
+ * proj row = [kv_heads*dim q | kv_heads*dim k | heads*vdim v | heads*vdim gate | heads beta | heads decay].
+ * Convolution weights conv_w [2*kv_heads*dim + heads*vdim, taps] fp32.  Conv state [slots, 2, taps-1, channels] in dtype:
+ * the inputs of the taps-1 positions before position p live in half p & 1.  Recurrent state [slots, heads, dim, vdim]
+ * fp32.  A sequence at position 0 starts from zero whatever its slot held. */
+typedef struct {
+  const void* proj; int64_t proj_stride;
+  const float *conv_w, *a_log, *dt_bias, *w_norm;
+  void* conv_state;
+  float* state;
+  const int32_t *pos, *tok_seq, *slot, *start, *cu;
+  int32_t n_tok, n_seq, n_decode;
+  int32_t heads, kv_heads, dim, vdim, taps;
+  float eps;
+  int32_t dtype;
+} msa_lm_delta_args;
+
+/* Decode sequences: convolution, unit norms, gates, state update, read-out, gated norm -> out [n_decode, heads*vdim]. */
+int msa_lm_delta_decode(const msa_lm_delta_args* a, void* out, int64_t out_stride, void* stream);
+/* The other sequences: convolution + silu + unit norms -> qk [rows, 2, kv_heads, dim] fp32 (q scaled by dim^-1/2),
+ * v [rows, heads, vdim] fp32, gates [rows, 2, heads] fp32 (log decay, beta); rows count from the first non-decode token. */
+int msa_lm_delta_prep(const msa_lm_delta_args* a, float* qk, float* v, float* gates, void* stream);
+/* Convolution inputs of the last taps-1 positions -> conv_state. */
+int msa_lm_delta_conv_store(const msa_lm_delta_args* a, void* stream);
+/* The recurrence token by token -> o [rows, heads, vdim] fp32; advances the state. */
+int msa_lm_delta_scan(const msa_lm_delta_args* a, const float* qk, const float* v, const float* gates, float* o, void* stream);
+/* out = o / rms(o) * w_norm * silu(gate) for the non-decode rows. */
+int msa_lm_delta_out(const msa_lm_delta_args* a, const float* o, void* out, int64_t out_stride, void* stream);
+
+/* ---- mixtures of experts -------------------------------------------------------------------------------------------
+ * Router logits (fp32) + bias -> the top experts of every row (ties: lower index) and the softmax over their logits. */
+int msa_lm_moe_topk(const float* logits, int64_t stride, const float* bias, int32_t n_rows, int32_t experts, int32_t top,
+                    int32_t* idx, float* weight, void* stream);
+/* Groups the n_rows*top choices by expert: src[i] = row of the i-th grouped entry, inv[r*top+k] = its place,
+ * off[e] .. off[e+1] the entries of expert e, tiles [max_tiles, 2] = (expert, first entry) of every tile of tile_rows
+ * entries (expert -1: unused). */
+int msa_lm_moe_sort(const int32_t* idx, int32_t n_rows, int32_t top, int32_t experts, int32_t tile_rows, int32_t* src,
+                    int32_t* inv, int32_t* off, int32_t* tiles, int32_t max_tiles, void* stream);
+/* Grouped product over the tiles of msa_lm_moe_sort (tile_rows = 32): out[i] = x[src ? src[i] : i] . w[e]^T with
+ * w [experts, n_out, k].  act = 1: w holds gate rows then up rows (n_out = 2*ff) and out[i, ff] = g * sigmoid(1.702 g) *
+ * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit). */
+int msa_lm_moe_gemm(const void* x, int64_t x_stride, const int32_t* src, const void* w, const int32_t* off,
+                    const int32_t* tiles, int32_t max_tiles, int32_t n_out, int32_t k, int32_t act, float limit, void* out,
+                    int64_t out_stride, int32_t out_dtype, int32_t dtype, void* stream);
+
+#ifdef __cplusplus
+}
+#endif
+#endif

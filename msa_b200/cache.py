@@ -8,6 +8,8 @@ Only the protocol the path uses is kept -- per-layer ``cache_kwargs``, ``meta``,
 from __future__ import annotations
 
 import os
+from dataclasses import dataclass
+from typing import Dict, Hashable, List, Optional, Sequence, Tuple
 
 import torch
 
@@ -63,6 +65,183 @@ class SparseCacheOnCPU(SparseCache):
 
     def update_router_kcache(self, key_states, layer_idx):
         return super().update_router_kcache(self._cpu(key_states), layer_idx)
+
+
+@dataclass(frozen=True)
+class RingSpec:
+    """A windowed layer's state: the last rows of ``width`` elements (``window`` None: every row)."""
+    width: int
+    window: Optional[int]
+
+
+@dataclass(frozen=True)
+class RecurrentSpec:
+    """A recurrent layer's state: a ``[heads, dim, vdim]`` fp32 matrix per head and the last ``taps - 1`` inputs of its
+    convolution over ``channels`` channels (double-buffered by the parity of the sequence's position)."""
+    heads: int
+    dim: int
+    vdim: int
+    channels: int
+    taps: int
+
+
+class SequenceStateCache(SparseCache):
+    """Slots of per-sequence state for models whose layers keep bounded state (rings, recurrent matrices).
+
+    One slot holds a sequence's state in every layer run; ``acquire`` / ``release`` hand slots out and take them back.
+    Nothing is cleared: the kernels take a sequence at position 0 as empty and never read a ring row that the sequence
+    has not written.  ``specs`` lists the runs in order (``model.state_specs()``); a ring has
+    ``min(window, max_len)`` rows.  The protocol of ``SparseCache`` (``meta``, ``record_kwargs``) stays usable, so the
+    interleave loop drives a model on this cache unchanged."""
+
+    def __init__(self, specs: Sequence, n_slots: int, max_len: int, device, dtype: torch.dtype):
+        super().__init__()
+        if n_slots < 1 or max_len < 1:
+            raise ValueError("SequenceStateCache needs at least one slot and one position")
+        self.specs, self.n_slots, self.max_len, self.device, self.dtype = list(specs), n_slots, max_len, torch.device(device), dtype
+        self.ring: Dict[int, torch.Tensor] = {}
+        self.state: Dict[int, torch.Tensor] = {}
+        self.conv: Dict[int, torch.Tensor] = {}
+        for i, s in enumerate(self.specs):
+            if isinstance(s, RingSpec):
+                rows = max_len if s.window is None else min(s.window, max_len)
+                self.ring[i] = torch.zeros((n_slots, rows, s.width), dtype=dtype, device=device)
+            else:
+                self.state[i] = torch.zeros((n_slots, s.heads, s.dim, s.vdim), dtype=torch.float32, device=device)
+                self.conv[i] = torch.zeros((n_slots, 2, s.taps - 1, s.channels), dtype=dtype, device=device)
+        self._free: List[int] = list(range(n_slots - 1, -1, -1))
+        self._slot: Dict[Hashable, int] = {}
+        self._length: Dict[Hashable, int] = {}
+
+    @property
+    def free_slots(self) -> int:
+        return len(self._free)
+
+    def __contains__(self, seq: Hashable) -> bool:
+        return seq in self._slot
+
+    def acquire(self, seq: Hashable) -> int:
+        if seq in self._slot:
+            raise KeyError(f"sequence {seq!r} already holds a slot")
+        if not self._free:
+            raise RuntimeError(f"all {self.n_slots} slots are taken")
+        self._slot[seq], self._length[seq] = self._free.pop(), 0
+        return self._slot[seq]
+
+    def release(self, seq: Hashable) -> None:
+        self._free.append(self._slot.pop(seq))
+        del self._length[seq]
+
+    def slot(self, seq: Hashable) -> int:
+        return self._slot[seq]
+
+    def length(self, seq: Hashable) -> int:
+        return self._length[seq]
+
+    def advance(self, seq: Hashable, n: int) -> None:
+        self._length[seq] += n
+
+    def state_bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for d in (self.ring, self.state, self.conv) for t in d.values())
+
+
+@dataclass
+class ContextView:
+    """Context bookkeeping of one step for one attention window: where each portion's context starts (``ctx_off``,
+    prefix sums) and how many earlier rows it begins with (``old_off``, prefix sums)."""
+    window: int
+    ctx_off: Optional[torch.Tensor]
+    old_off: Optional[torch.Tensor]
+    n_ctx: int
+    n_old: int
+
+
+class PackedStep:
+    """The tokens of one step, packed: single-token continuations (decode) first, then the portions.
+
+    ``entries`` = ``(sequence, token ids, wanted places)``; the sequences must hold slots in ``cache``.  ``want_rows``
+    lists the packed rows whose logits are asked for, in the order of the entries."""
+
+    def __init__(self, entries: Sequence[Tuple[Hashable, Sequence[int], Sequence[int]]], cache: SequenceStateCache, windows: Sequence[Optional[int]]):
+        entries = [(s, list(t), list(w)) for s, t, w in entries]
+        if len({s for s, _, _ in entries}) != len(entries):
+            raise ValueError("a sequence appears twice in one step")
+        for s, t, w in entries:
+            if not t:
+                raise ValueError(f"sequence {s!r} brings no tokens")
+            if cache.length(s) + len(t) > cache.max_len:
+                raise ValueError(f"sequence {s!r} would hold {cache.length(s) + len(t)} tokens, the cache has room for {cache.max_len}")
+            if any(not 0 <= i < len(t) for i in w):
+                raise ValueError(f"sequence {s!r}: a wanted place lies outside its {len(t)} tokens")
+        order = sorted(range(len(entries)), key=lambda i: len(entries[i][1]) > 1)      # stable: decode entries first
+        token, pos, tok_seq, slot, start, cu, row0 = [], [], [], [], [], [0], {}
+        for k, i in enumerate(order):
+            s, t, _ = entries[i]
+            p0 = cache.length(s)
+            row0[i] = len(token)
+            token += t
+            pos += range(p0, p0 + len(t))
+            tok_seq += [k] * len(t)
+            slot.append(cache.slot(s))
+            start.append(p0)
+            cu.append(len(token))
+        self.seqs = [(s, len(t)) for s, t, _ in entries]
+        self.n_tok, self.n_seq = len(token), len(order)
+        self.n_decode = sum(len(t) == 1 for _, t, _ in entries)
+        self.max_len = max([len(t) for _, t, _ in entries if len(t) > 1], default=0)
+        want = [row0[i] + w for i, (_, _, ws) in enumerate(entries) for w in ws]
+        views = []
+        for window in windows:
+            size = cache.max_len if window is None else min(window, cache.max_len)
+            ctx, old = [0], [0]
+            for k in range(self.n_decode, self.n_seq):
+                o = min(start[k], size - 1)
+                old.append(old[-1] + o)
+                ctx.append(ctx[-1] + o + cu[k + 1] - cu[k])
+            views.append((window, size, ctx, old))
+        # one host-to-device copy for all tables
+        parts = [token, pos, tok_seq, slot, start, cu, want] + [x for v in views for x in v[2:]]
+        flat = torch.tensor([x for p in parts for x in p], dtype=torch.int32)
+        if cache.device.type == "cuda":
+            flat = flat.pin_memory()
+        flat = flat.to(cache.device, non_blocking=True)
+        at, dev = 0, []
+        for p in parts:
+            dev.append(flat[at:at + len(p)])
+            at += len(p)
+        self.token, self.pos, self.tok_seq, self.slot, self.start, self.cu, self.want_rows = dev[:7]
+        self.views = {w: ContextView(size, dev[7 + 2 * i], dev[8 + 2 * i], ctx[-1], old[-1])
+                      for i, (w, size, ctx, old) in enumerate(views)}
+
+    def commit(self, cache: SequenceStateCache) -> None:
+        """The step has been launched: its sequences have grown."""
+        for s, n in self.seqs:
+            cache.advance(s, n)
+
+
+class DecodeStep:
+    """A step of one token for each of ``n`` sequences with tables that stay at fixed device addresses, so that a CUDA
+    graph of the step can be replayed: ``fill`` rewrites them, the sampled tokens may be fed back on the device."""
+
+    def __init__(self, n: int, cache: SequenceStateCache, windows: Sequence[Optional[int]]):
+        dev = cache.device
+        i = dict(dtype=torch.int32, device=dev)
+        self.n_tok = self.n_seq = self.n_decode = n
+        self.max_len = 0
+        self.table = torch.zeros((3, n), **i)
+        self.token, self.pos, self.slot = self.table[0], self.table[1], self.table[2]
+        self.start = self.pos
+        self.tok_seq = torch.arange(n, **i)
+        self.cu = torch.arange(n + 1, **i)
+        self.want_rows = torch.arange(n, **i)
+        self.views = {w: ContextView(cache.max_len if w is None else min(w, cache.max_len), None, None, 0, 0) for w in windows}
+        self._host = torch.zeros((3, n), dtype=torch.int32)
+        if dev.type == "cuda":
+            self._host = self._host.pin_memory()
+
+    def fill(self, tokens: Sequence[int], positions: Sequence[int], slots: Sequence[int]) -> None:
+        self._host[0], self._host[1], self._host[2] = torch.tensor(tokens), torch.tensor(positions), torch.tensor(slots)
+        self.table.copy_(self._host, non_blocking=True)
 
 
 class SharedPooledCache:

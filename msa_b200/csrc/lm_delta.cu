@@ -1,0 +1,394 @@
+// Gated delta rule: short causal convolution, unit norms, gates, the recurrence in fp32, and the gated output norm.
+//
+// Per sequence slot a layer keeps the matrix state [heads, dim, vdim] (fp32) and the last taps-1 inputs of the
+// convolution.  The convolution inputs are double-buffered by the parity of the sequence's position, so a decode launch
+// can read the old ones in every block while it writes the new ones.
+//
+// One step of a head, with S the state before it, reads S once for both products:
+//     c = S^T k,  r = S^T q;   u = beta (v - g c);   S <- g S + k u^T;   o = g r + (q.k) u
+#include "lm_common.cuh"
+
+namespace msa {
+
+struct DeltaLayout {
+  int nqk, nv, chan;   // kv_heads*dim, heads*vdim, 2*nqk + nv
+  __host__ __device__ explicit DeltaLayout(const msa_lm_delta_args& a)
+      : nqk(a.kv_heads * a.dim), nv(a.heads * a.vdim), chan(2 * a.kv_heads * a.dim + a.heads * a.vdim) {}
+};
+
+// Convolution of channel c at token n (row of proj), t tokens into its portion that starts at position p0; then silu.
+template <typename T>
+__device__ __forceinline__ float conv_silu(const msa_lm_delta_args& a, const T* state_half, int chan, long long n, int t,
+                                           int p0, int c) {
+  const T* proj = reinterpret_cast<const T*>(a.proj);
+  const float* w = a.conv_w + (long long)c * a.taps;
+  float acc = 0.f;
+  for (int i = 0; i < a.taps; ++i) {
+    const int lag = a.taps - 1 - i;
+    if (t - lag >= 0) acc = fmaf(w[i], to_f(proj[(n - lag) * a.proj_stride + c]), acc);
+    else if (p0 + t - lag >= 0) acc = fmaf(w[i], to_f(state_half[(long long)(a.taps - 1 + t - lag) * chan + c]), acc);
+  }
+  return silu_f(acc);
+}
+template <typename T>
+__device__ __forceinline__ const T* conv_half(const msa_lm_delta_args& a, int chan, int slot, int p) {
+  return reinterpret_cast<const T*>(a.conv_state) + ((long long)slot * 2 + (p & 1)) * (a.taps - 1) * chan;
+}
+
+// ---- prefill: convolution, unit norms, gates ---------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_prep_kernel(const msa_lm_delta_args a, float* __restrict__ qk, float* __restrict__ v, float* __restrict__ gates) {
+  const DeltaLayout L(a);
+  const int row = blockIdx.x;                       // counts from the first non-decode token
+  const long long n = (long long)a.n_decode + row;
+  const int s = a.tok_seq[n], t = (int)(n - a.cu[s]), p0 = a.start[s];
+  const T* half = conv_half<T>(a, L.chan, a.slot[s], p0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int hd = warp; hd < 2 * a.kv_heads; hd += 8) {   // heads of q, then of k
+    float* dst = qk + (long long)row * 2 * L.nqk + (long long)hd * a.dim;
+    float ss = 0.f;
+    for (int i = lane; i < a.dim; i += 32) {
+      const float x = conv_silu<T>(a, half, L.chan, n, t, p0, hd * a.dim + i);
+      dst[i] = x;
+      ss += x * x;
+    }
+    ss = warp_sum_f(ss);
+    const float sc = (hd < a.kv_heads ? 1.f / sqrtf((float)a.dim) : 1.f) / sqrtf(ss + 1e-6f);
+    for (int i = lane; i < a.dim; i += 32) dst[i] *= sc;
+  }
+  for (int i = threadIdx.x; i < L.nv; i += blockDim.x)
+    v[(long long)row * L.nv + i] = conv_silu<T>(a, half, L.chan, n, t, p0, 2 * L.nqk + i);
+  const T* g = reinterpret_cast<const T*>(a.proj) + n * a.proj_stride + 2 * L.nqk + 2 * L.nv;
+  for (int h = threadIdx.x; h < a.heads; h += blockDim.x) {
+    gates[(long long)row * 2 * a.heads + h] = -expf(a.a_log[h]) * softplus_f(to_f(g[a.heads + h]) + a.dt_bias[h]);
+    gates[(long long)row * 2 * a.heads + a.heads + h] = sigmoid_f(to_f(g[h]));
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) delta_conv_store_kernel(const msa_lm_delta_args a) {
+  const DeltaLayout L(a);
+  const int s = a.n_decode + blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= L.chan) return;
+  const int len = a.cu[s + 1] - a.cu[s], p0 = a.start[s], keep = a.taps - 1;
+  const T* proj = reinterpret_cast<const T*>(a.proj);
+  const T* old = conv_half<T>(a, L.chan, a.slot[s], p0);
+  T* dst = reinterpret_cast<T*>(a.conv_state) + ((long long)a.slot[s] * 2 + ((p0 + len) & 1)) * keep * L.chan;
+  // ascending: an entry that comes from the old half (possibly the same memory) is read before it is overwritten
+  for (int j = 0; j < keep; ++j) {
+    const int t = len - keep + j;                   // token of the portion, negative: before it
+    T x = from_f<T>(0.f);
+    if (t >= 0) x = proj[((long long)a.cu[s] + t) * a.proj_stride + c];
+    else if (p0 + t >= 0) x = old[(long long)(keep + t) * L.chan + c];
+    dst[(long long)j * L.chan + c] = x;
+  }
+}
+
+// ---- prefill: the recurrence, token by token ------------------------------------------------------------------------
+// 8 lanes share a state column (R rows each, in registers); a warp covers 4 columns, a block of 4 warps 16.  Tokens are
+// staged in shared memory 16 at a time.
+constexpr int kScTok = 16, kScCols = 16, kScThreads = 128;
+
+template <int R>
+__global__ void __launch_bounds__(kScThreads)
+delta_scan_kernel(const msa_lm_delta_args a, const float* __restrict__ qk, const float* __restrict__ v,
+                  const float* __restrict__ gates, float* __restrict__ o) {
+  constexpr int D = 8 * R;
+  __shared__ __align__(16) float s_q[kScTok][D], s_k[kScTok][D];
+  __shared__ float s_v[kScTok][kScCols], s_o[kScTok][kScCols], s_g[kScTok], s_b[kScTok], s_qk[kScTok];
+  const DeltaLayout L(a);
+  const int s = a.n_decode + blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * kScCols;
+  const int hk = h / (a.heads / a.kv_heads);
+  const int len = a.cu[s + 1] - a.cu[s];
+  const long long row0 = a.cu[s] - a.n_decode;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int part = lane & 7, cl = warp * 4 + (lane >> 3), col = c0 + cl;
+  float* S = a.state + (((long long)a.slot[s] * a.heads + h) * a.dim) * a.vdim;
+  float st[R];
+  const bool fresh = a.start[s] == 0;
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int d = part * R + r;
+    st[r] = (!fresh && d < a.dim && col < a.vdim) ? S[(long long)d * a.vdim + col] : 0.f;
+  }
+  for (int t0 = 0; t0 < len; t0 += kScTok) {
+    const int nt = min(kScTok, len - t0);
+    __syncthreads();
+    for (int i = threadIdx.x; i < nt * D; i += kScThreads) {
+      const int t = i / D, d = i % D;
+      const float* src = qk + (row0 + t0 + t) * 2 * L.nqk + (long long)hk * a.dim + d;
+      s_q[t][d] = d < a.dim ? src[0] : 0.f;
+      s_k[t][d] = d < a.dim ? src[L.nqk] : 0.f;
+    }
+    for (int i = threadIdx.x; i < nt * kScCols; i += kScThreads) {
+      const int t = i / kScCols, c = i % kScCols;
+      s_v[t][c] = c0 + c < a.vdim ? v[(row0 + t0 + t) * L.nv + (long long)h * a.vdim + c0 + c] : 0.f;
+    }
+    if (threadIdx.x < nt) {
+      const float* g = gates + (row0 + t0 + threadIdx.x) * 2 * a.heads + h;
+      s_g[threadIdx.x] = expf(g[0]);
+      s_b[threadIdx.x] = g[a.heads];
+    }
+    __syncthreads();
+    for (int t = warp; t < nt; t += kScThreads / 32) {
+      float d = 0.f;
+      for (int i = lane; i < D; i += 32) d = fmaf(s_q[t][i], s_k[t][i], d);
+      d = warp_sum_f(d);
+      if (lane == 0) s_qk[t] = d;
+    }
+    __syncthreads();
+    for (int t = 0; t < nt; ++t) {
+      float k[R], c = 0.f, r_ = 0.f;
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        k[r] = s_k[t][part * R + r];
+        c = fmaf(st[r], k[r], c);
+        r_ = fmaf(st[r], s_q[t][part * R + r], r_);
+      }
+#pragma unroll
+      for (int w = 1; w < 8; w <<= 1) {
+        c += __shfl_xor_sync(0xffffffffu, c, w);
+        r_ += __shfl_xor_sync(0xffffffffu, r_, w);
+      }
+      const float g = s_g[t], u = s_b[t] * (s_v[t][cl] - g * c);
+#pragma unroll
+      for (int r = 0; r < R; ++r) st[r] = fmaf(k[r], u, g * st[r]);
+      if (part == 0) s_o[t][cl] = fmaf(g, r_, s_qk[t] * u);
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < nt * kScCols; i += kScThreads) {
+      const int t = i / kScCols, c = i % kScCols;
+      if (c0 + c < a.vdim) o[(row0 + t0 + t) * L.nv + (long long)h * a.vdim + c0 + c] = s_o[t][c];
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int d = part * R + r;
+    if (d < a.dim && col < a.vdim) S[(long long)d * a.vdim + col] = st[r];
+  }
+}
+
+// out = o / rms(o) * w * silu(gate); one warp per (row, head).
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_out_kernel(const msa_lm_delta_args a, const float* __restrict__ o, T* __restrict__ out, long long out_stride, long long n) {
+  const DeltaLayout L(a);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * 8 + warp;
+  if (item >= n * a.heads) return;
+  const long long row = item / a.heads;
+  const int h = (int)(item % a.heads);
+  const float* src = o + row * L.nv + (long long)h * a.vdim;
+  const T* gate = reinterpret_cast<const T*>(a.proj) + (a.n_decode + row) * a.proj_stride + 2 * L.nqk + L.nv + (long long)h * a.vdim;
+  float ss = 0.f;
+  for (int i = lane; i < a.vdim; i += 32) ss += src[i] * src[i];
+  const float inv = 1.f / sqrtf(warp_sum_f(ss) / (float)a.vdim + a.eps);
+  for (int i = lane; i < a.vdim; i += 32)
+    out[row * out_stride + (long long)h * a.vdim + i] = from_f<T>(src[i] * inv * a.w_norm[i] * silu_f(to_f(gate[i])));
+}
+
+// ---- decode: everything between the projections and the output product -----------------------------------------------
+// One block per (sequence, head).  Threads form a grid of row groups x column vectors over the state; the state is read
+// (twice, the second time from L1 / L2) and written once.
+constexpr int kDdThreads = 256;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(kDdThreads)
+delta_decode_kernel(const msa_lm_delta_args a, T* __restrict__ out, long long out_stride, int groups) {
+  extern __shared__ float sm[];
+  __shared__ float s_part[32];
+  const DeltaLayout L(a);
+  const int b = blockIdx.y, h = blockIdx.x, group = a.heads / a.kv_heads, hk = h / group;
+  const int dk = a.dim, dv = a.vdim, keep = a.taps - 1;
+  float* s_q = sm;                        // [dk]
+  float* s_k = s_q + dk;                  // [dk]
+  float* s_v = s_k + dk;                  // [dv], then the output row
+  float* s_c = s_v + dv;                  // [groups][dv]
+  float* s_r = s_c + groups * dv;         // [groups][dv]
+  const int slot = a.slot[b], p = a.pos[b];
+  const T* proj = reinterpret_cast<const T*>(a.proj) + (long long)b * a.proj_stride;
+  const T* old = conv_half<T>(a, L.chan, slot, p);
+  T* fresh = reinterpret_cast<T*>(a.conv_state) + ((long long)slot * 2 + ((p + 1) & 1)) * keep * L.chan;
+  for (int i = threadIdx.x; i < 2 * dk + dv; i += kDdThreads) {
+    const int c = i < dk ? hk * dk + i : (i < 2 * dk ? L.nqk + hk * dk + (i - dk) : 2 * L.nqk + h * dv + (i - 2 * dk));
+    const bool writer = i >= 2 * dk || h % group == 0;
+    const float* w = a.conv_w + (long long)c * a.taps;
+    float acc = 0.f;
+    for (int j = 0; j < keep; ++j) {
+      const T x = p - keep + j >= 0 ? old[(long long)j * L.chan + c] : from_f<T>(0.f);
+      acc = fmaf(w[j], to_f(x), acc);
+      if (writer && j > 0) fresh[(long long)(j - 1) * L.chan + c] = x;
+    }
+    const T x = proj[c];
+    acc = fmaf(w[keep], to_f(x), acc);
+    if (writer && keep > 0) fresh[(long long)(keep - 1) * L.chan + c] = x;
+    sm[i] = silu_f(acc);
+  }
+  __syncthreads();
+  float qq = 0.f, kk = 0.f, qk = 0.f;
+  for (int i = threadIdx.x; i < dk; i += kDdThreads) {
+    qq += s_q[i] * s_q[i];
+    kk += s_k[i] * s_k[i];
+    qk += s_q[i] * s_k[i];
+  }
+  qq = block_sum(qq, s_part);
+  kk = block_sum(kk, s_part);
+  qk = block_sum(qk, s_part);
+  const float sq = 1.f / (sqrtf((float)dk) * sqrtf(qq + 1e-6f)), sk = 1.f / sqrtf(kk + 1e-6f);
+  qk *= sq * sk;
+  const float beta = sigmoid_f(to_f(proj[2 * L.nqk + 2 * L.nv + h]));
+  const float g = expf(-expf(a.a_log[h]) * softplus_f(to_f(proj[2 * L.nqk + 2 * L.nv + a.heads + h]) + a.dt_bias[h]));
+  float* S = a.state + (((long long)slot * a.heads + h) * dk) * dv;
+  const bool zero = p == 0;
+  const int cols = dv / V, rg = threadIdx.x / cols, cv = (threadIdx.x % cols) * V;   // groups * cols <= blockDim
+  const bool active = rg < groups;
+  // columns are walked in one sweep when they fit the block; otherwise cols > blockDim is split over `cs`
+  for (int cs = 0; cs < cols; cs += kDdThreads) {
+    const int c = cols > kDdThreads ? (cs + threadIdx.x) * V : cv;
+    const int g0 = cols > kDdThreads ? 0 : rg;
+    const bool on = cols > kDdThreads ? cs + (int)threadIdx.x < cols : active;
+    if (on) {
+      float ac[V], ar[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) ac[e] = ar[e] = 0.f;
+      if (!zero)
+#pragma unroll 4
+        for (int d = g0; d < dk; d += groups) {
+          float x[V];
+          if constexpr (V == 4) { const float4 f = load4(S + (long long)d * dv + c); x[0] = f.x; x[1] = f.y; x[2] = f.z; x[3] = f.w; }
+          else x[0] = S[(long long)d * dv + c];
+          const float kd = s_k[d], qd = s_q[d];
+#pragma unroll
+          for (int e = 0; e < V; ++e) { ac[e] = fmaf(x[e], kd, ac[e]); ar[e] = fmaf(x[e], qd, ar[e]); }
+        }
+#pragma unroll
+      for (int e = 0; e < V; ++e) { s_c[g0 * dv + c + e] = ac[e]; s_r[g0 * dv + c + e] = ar[e]; }
+    }
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < dv; i += kDdThreads) {
+    float c = 0.f, r = 0.f;
+    for (int j = 0; j < groups; ++j) { c += s_c[j * dv + i]; r += s_r[j * dv + i]; }
+    const float u = beta * (s_v[i] - g * (c * sk)), o = fmaf(g, r * sq, qk * u);
+    s_c[i] = u * sk;      // group 0's entry: read by this thread alone
+    s_v[i] = o;
+    ss += o * o;
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, s_part) / (float)dv + a.eps);   // its barriers publish s_c and s_v
+  __syncthreads();
+  for (int cs = 0; cs < cols; cs += kDdThreads) {
+    const int c = cols > kDdThreads ? (cs + threadIdx.x) * V : cv;
+    const int g0 = cols > kDdThreads ? 0 : rg;
+    const bool on = cols > kDdThreads ? cs + (int)threadIdx.x < cols : active;
+    if (on) {
+#pragma unroll 4
+      for (int d = g0; d < dk; d += groups) {
+        float x[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] = 0.f;
+        if (!zero) {
+          if constexpr (V == 4) { const float4 f = load4(S + (long long)d * dv + c); x[0] = f.x; x[1] = f.y; x[2] = f.z; x[3] = f.w; }
+          else x[0] = S[(long long)d * dv + c];
+        }
+        const float kd = s_k[d];
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] = fmaf(kd, s_c[c + e], g * x[e]);
+        if constexpr (V == 4) store4(S + (long long)d * dv + c, make_float4(x[0], x[1], x[2], x[3]));
+        else S[(long long)d * dv + c] = x[0];
+      }
+    }
+  }
+  const T* gate = proj + 2 * L.nqk + L.nv + (long long)h * dv;
+  for (int i = threadIdx.x; i < dv; i += kDdThreads)
+    out[(long long)b * out_stride + (long long)h * dv + i] = from_f<T>(s_v[i] * inv * a.w_norm[i] * silu_f(to_f(gate[i])));
+}
+
+inline int delta_check(const msa_lm_delta_args* a, const char* what) {
+  MSA_REQUIRE(a, "%s: null arguments", what);
+  MSA_REQUIRE(dtype_ok(a->dtype) && a->proj && a->conv_w && a->a_log && a->dt_bias && a->w_norm && a->state && a->slot &&
+                  a->start && a->cu && a->pos && a->tok_seq, "%s: null pointer or bad dtype", what);
+  MSA_REQUIRE(a->taps >= 1 && (a->taps == 1 || a->conv_state), "%s: convolution state missing", what);
+  MSA_REQUIRE(a->heads > 0 && a->kv_heads > 0 && a->heads % a->kv_heads == 0 && a->dim > 0 && a->vdim > 0,
+              "%s: bad head counts or sizes", what);
+  MSA_REQUIRE(a->n_decode >= 0 && a->n_decode <= a->n_seq && a->n_tok >= a->n_decode, "%s: bad counts", what);
+  return MSA_OK;
+}
+
+}  // namespace msa
+
+using namespace msa;
+
+extern "C" int msa_lm_delta_decode(const msa_lm_delta_args* a, void* out, int64_t out_stride, void* stream) {
+  MSA_OK_OR_RETURN(delta_check(a, "delta_decode"));
+  MSA_REQUIRE(out, "delta_decode: null output");
+  if (a->n_decode == 0) return MSA_OK;
+  const int v = a->vdim % 4 == 0 && aligned16(a->state) ? 4 : 1;
+  const int cols = a->vdim / v;
+  const int groups = cols >= kDdThreads ? 1 : kDdThreads / cols;
+  const size_t smem = (size_t)4 * (2 * a->dim + a->vdim + 2 * groups * a->vdim);
+  const dim3 grid((unsigned)a->heads, (unsigned)a->n_decode);
+  MSA_LM_DISPATCH(a->dtype, {
+    if (v == 4) {
+      static DeviceSmem st4;
+      MSA_OK_OR_RETURN(ensure_dynamic_smem(delta_decode_kernel<T, 4>, smem, st4));
+      delta_decode_kernel<T, 4><<<grid, kDdThreads, smem, (cudaStream_t)stream>>>(*a, (T*)out, out_stride, groups);
+    } else {
+      static DeviceSmem st1;
+      MSA_OK_OR_RETURN(ensure_dynamic_smem(delta_decode_kernel<T, 1>, smem, st1));
+      delta_decode_kernel<T, 1><<<grid, kDdThreads, smem, (cudaStream_t)stream>>>(*a, (T*)out, out_stride, groups);
+    }
+  });
+  MSA_LAUNCH_OK("delta_decode_kernel");
+  return MSA_OK;
+}
+
+extern "C" int msa_lm_delta_prep(const msa_lm_delta_args* a, float* qk, float* v, float* gates, void* stream) {
+  MSA_OK_OR_RETURN(delta_check(a, "delta_prep"));
+  MSA_REQUIRE(qk && v && gates, "delta_prep: null output");
+  const int rows = a->n_tok - a->n_decode;
+  if (rows == 0) return MSA_OK;
+  MSA_LM_DISPATCH(a->dtype, { delta_prep_kernel<T><<<rows, 256, 0, (cudaStream_t)stream>>>(*a, qk, v, gates); });
+  MSA_LAUNCH_OK("delta_prep_kernel");
+  return MSA_OK;
+}
+
+extern "C" int msa_lm_delta_conv_store(const msa_lm_delta_args* a, void* stream) {
+  MSA_OK_OR_RETURN(delta_check(a, "delta_conv_store"));
+  if (a->n_seq == a->n_decode || a->taps == 1) return MSA_OK;
+  const DeltaLayout L(*a);
+  const dim3 grid((unsigned)((L.chan + 255) / 256), (unsigned)(a->n_seq - a->n_decode));
+  MSA_LM_DISPATCH(a->dtype, { delta_conv_store_kernel<T><<<grid, 256, 0, (cudaStream_t)stream>>>(*a); });
+  MSA_LAUNCH_OK("delta_conv_store_kernel");
+  return MSA_OK;
+}
+
+extern "C" int msa_lm_delta_scan(const msa_lm_delta_args* a, const float* qk, const float* v, const float* gates, float* o,
+                                 void* stream) {
+  MSA_OK_OR_RETURN(delta_check(a, "delta_scan"));
+  MSA_REQUIRE(qk && v && gates && o, "delta_scan: null pointer");
+  MSA_REQUIRE(a->dim <= 256, "delta_scan: dim must be at most 256");
+  if (a->n_seq == a->n_decode) return MSA_OK;
+  const dim3 grid((unsigned)((a->vdim + kScCols - 1) / kScCols), (unsigned)a->heads, (unsigned)(a->n_seq - a->n_decode));
+  cudaStream_t st = (cudaStream_t)stream;
+  if (a->dim <= 32) delta_scan_kernel<4><<<grid, kScThreads, 0, st>>>(*a, qk, v, gates, o);
+  else if (a->dim <= 64) delta_scan_kernel<8><<<grid, kScThreads, 0, st>>>(*a, qk, v, gates, o);
+  else if (a->dim <= 128) delta_scan_kernel<16><<<grid, kScThreads, 0, st>>>(*a, qk, v, gates, o);
+  else delta_scan_kernel<32><<<grid, kScThreads, 0, st>>>(*a, qk, v, gates, o);
+  MSA_LAUNCH_OK("delta_scan_kernel");
+  return MSA_OK;
+}
+
+extern "C" int msa_lm_delta_out(const msa_lm_delta_args* a, const float* o, void* out, int64_t out_stride, void* stream) {
+  MSA_OK_OR_RETURN(delta_check(a, "delta_out"));
+  MSA_REQUIRE(o && out, "delta_out: null pointer");
+  const long long rows = a->n_tok - a->n_decode;
+  if (rows == 0) return MSA_OK;
+  const long long blocks = (rows * a->heads + 7) / 8;
+  MSA_LM_DISPATCH(a->dtype, {
+    delta_out_kernel<T><<<(unsigned)blocks, 256, 0, (cudaStream_t)stream>>>(*a, o, (T*)out, out_stride, rows);
+  });
+  MSA_LAUNCH_OK("delta_out_kernel");
+  return MSA_OK;
+}

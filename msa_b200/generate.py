@@ -46,6 +46,18 @@ def _process_logits(logits: torch.Tensor, temperature: Optional[float], top_p: O
     return logits
 
 
+def choose_tokens(logits: torch.Tensor, temperature: Sequence[Optional[float]], top_p: Sequence[Optional[float]],
+                  generators: Sequence[Optional[torch.Generator]]) -> list:
+    """One token per row of ``logits``, as host integers: greedy where the row's temperature is 0 or None, else sampled
+    after temperature and nucleus filtering from the row's own generator."""
+    tokens = logits.argmax(dim=-1)
+    for i, t in enumerate(temperature):
+        if t is not None and t > 0:
+            probs = F.softmax(_process_logits(logits[i:i + 1].float(), t, top_p[i]), dim=-1)
+            tokens[i] = torch.multinomial(probs, num_samples=1, generator=generators[i])[0, 0]
+    return tokens.tolist()
+
+
 @torch.no_grad()
 def interleave_generate(model, input_ids: torch.Tensor, attention_mask: torch.Tensor, doc_ids: torch.Tensor,
                         position_ids: torch.Tensor, past_key_values, *, eos_token_ids: Sequence[int], pad_token_id: int,

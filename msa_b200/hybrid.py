@@ -1,0 +1,342 @@
+"""Layered decoder designs: a stack whose layers each name their mixer and feed-forward, on the package's kernels.
+
+The configuration (``hybrid_config``) lists the layers; a mixer is a class below with its weights, its per-sequence
+state (``state_spec``) and its forward step.  A step works on packed tokens of many sequences (``cache.PackedStep``):
+matrix products run over all of them at once, the mixers treat single-token continuations and longer portions by their
+own kernels.  The residual stream is fp32; between two products one launch does branch norm, residual add, next norm
+and rounding (``lm_ops.residual_norm``), including the weighted sum over a mixture's experts.
+
+``HybridForCausalLM.step`` is the serving entry (scheduler, trace replay, benchmark); ``forward`` takes the keyword
+arguments of ``MSAForCausalLM.forward``, so that the interleave loop can drive either.
+"""
+from __future__ import annotations
+
+import glob
+import os
+from types import SimpleNamespace
+from typing import Dict, List, Optional
+
+import torch
+
+from . import lm_ops as K
+from .cache import DecodeStep, PackedStep, RecurrentSpec, RingSpec, SequenceStateCache
+from .hybrid_config import HybridConfig
+
+
+class Weights:
+    """Checkpoint tensors by name; every tensor must be taken exactly once."""
+
+    def __init__(self, tensors: Dict[str, torch.Tensor], device, dtype: torch.dtype):
+        self._t, self._left, self.device, self.dtype = tensors, set(tensors), device, dtype
+
+    def raw(self, name: str, *shape: int) -> torch.Tensor:
+        if name not in self._t:
+            raise KeyError(f"checkpoint lacks {name}")
+        t = self._t[name]
+        if tuple(t.shape) != shape:
+            raise ValueError(f"{name} has shape {tuple(t.shape)}, the configuration says {shape}")
+        self._left.discard(name)
+        return t
+
+    def matrix(self, name: str, *shape: int) -> torch.Tensor:
+        return self.raw(name, *shape).to(device=self.device, dtype=self.dtype).contiguous()
+
+    def vector(self, name: str, *shape: int) -> torch.Tensor:
+        return self.raw(name, *shape).to(device=self.device, dtype=torch.float32).contiguous()
+
+    def stack(self, names_rows, cols: int) -> torch.Tensor:
+        """Matrices with a common input, stacked by output rows: one product instead of several."""
+        return torch.cat([self.raw(n, r, cols) for n, r in names_rows]).to(device=self.device, dtype=self.dtype).contiguous()
+
+    def check_all_used(self) -> None:
+        if self._left:
+            raise ValueError(f"checkpoint tensors the configuration does not name: {sorted(self._left)[:5]}")
+
+
+class LatentAttention:
+    """Windowed attention over a cached low-rank latent.  Portions expand keys and values for their context and attend
+    per head; single tokens fold the key expansion into the query and attend over the latents themselves."""
+
+    def __init__(self, spec, w: Weights, prefix: str, width: int, eps: float):
+        s = self.spec = spec
+        self.eps = eps
+        self.w_in = w.stack([(prefix + "q", s.heads * (s.dim + s.rot_dim)), (prefix + "dkv", s.kv_rank + s.rot_dim)], width)
+        self.norm = w.vector(prefix + "dkv.norm", s.kv_rank)
+        self.w_kv = w.stack([(prefix + "uk", s.heads * s.dim), (prefix + "uv", s.heads * s.vdim)], s.kv_rank)
+        self.w_uk = self.w_kv[:s.heads * s.dim].view(s.heads, s.dim, s.kv_rank)
+        self.w_uv = self.w_kv[s.heads * s.dim:].view(s.heads, s.vdim, s.kv_rank)
+        self.w_o = w.matrix(prefix + "o", width, s.heads * s.vdim)
+        i = torch.arange(s.rot_dim // 2, dtype=torch.float64)
+        self.inv_freq = (s.rot_base ** (-2.0 * i / max(s.rot_dim, 1))).to(torch.float32).to(self.w_in.device)
+
+    @property
+    def state_spec(self) -> RingSpec:
+        return RingSpec(self.spec.kv_rank + self.spec.rot_dim, self.spec.window)
+
+    def mix(self, proj: torch.Tensor, step, cache: SequenceStateCache, run: int) -> torch.Tensor:
+        s, n, nd = self.spec, step.n_tok, step.n_decode
+        ring, view = cache.ring[run], step.views[s.window]
+        out = torch.empty((n, s.heads * s.vdim), dtype=proj.dtype, device=proj.device)
+        ctx = torch.empty((view.n_ctx, s.kv_rank + s.rot_dim), dtype=proj.dtype, device=proj.device) if n > nd else None
+        K.latent_prep(proj, s, self.norm, self.inv_freq, self.eps, step, view, ring, ctx)
+        q = proj[:, :s.heads * (s.dim + s.rot_dim)].view(n, s.heads, s.dim + s.rot_dim)
+        if nd:
+            self._decode(q[:nd], step, view, ring, out[:nd])
+        if n > nd:
+            kv = K.matmul(ctx[:, :s.kv_rank], self.w_kv)
+            k = kv[:, :s.heads * s.dim].view(-1, s.heads, s.dim)
+            v = kv[:, s.heads * s.dim:].view(-1, s.heads, s.vdim)
+            kr = ctx[:, s.kv_rank:].unsqueeze(1) if s.rot_dim else None
+            qp = q[nd:]
+            K.window_attn(qp[..., :s.dim], qp[..., s.dim:] if s.rot_dim else None, k, kr, v, out[nd:].view(n - nd, s.heads, s.vdim),
+                          scale=s.scale, window=view.window, start=step.start, cu=step.cu, seq0=nd, seq1=step.n_seq,
+                          max_len=step.max_len, ctx_off=view.ctx_off)
+            K.ring_store(ctx, step, view, ring)
+        return out
+
+    def _decode(self, q, step, view, ring, out) -> None:
+        s, n = self.spec, q.shape[0]
+        f32 = dict(out_dtype=torch.float32) if q.dtype != torch.float32 else {}
+        qa = torch.bmm(q[..., :s.dim].transpose(0, 1), self.w_uk, **f32)                  # [heads, n, rank]
+        lat = torch.empty((n, s.heads, s.kv_rank), dtype=q.dtype, device=q.device)
+        rows = ring.view(-1, 1, s.kv_rank + s.rot_dim)
+        K.window_attn(qa.transpose(0, 1), q[..., s.dim:] if s.rot_dim else None, rows[..., :s.kv_rank],
+                      rows[..., s.kv_rank:] if s.rot_dim else None, rows[..., :s.kv_rank], lat, scale=s.scale,
+                      window=view.window, start=step.start, cu=step.cu, seq0=0, seq1=n, max_len=1, slot=step.slot,
+                      ring_rows=ring.shape[1])
+        out.view(n, s.heads, s.vdim).copy_(torch.bmm(lat.transpose(0, 1), self.w_uv.transpose(1, 2)).transpose(0, 1))
+
+
+class GatedDelta:
+    """Gated delta rule behind a short causal convolution."""
+
+    def __init__(self, spec, w: Weights, prefix: str, width: int, eps: float):
+        s = self.spec = spec
+        self.eps = eps
+        qk, v = s.kv_heads * s.dim, s.heads * s.vdim
+        self.w_in = w.stack([(prefix + "q", qk), (prefix + "k", qk), (prefix + "v", v), (prefix + "g", v),
+                             (prefix + "b", s.heads), (prefix + "a", s.heads)], width)
+        self.conv = torch.cat([w.vector(prefix + n + ".conv", r, s.taps) for n, r in (("q", qk), ("k", qk), ("v", v))]).contiguous()
+        self.a_log, self.dt_bias = w.vector(prefix + "A_log", s.heads), w.vector(prefix + "dt_bias", s.heads)
+        self.norm = w.vector(prefix + "norm", s.vdim)
+        self.w_o = w.matrix(prefix + "o", width, v)
+
+    @property
+    def state_spec(self) -> RecurrentSpec:
+        s = self.spec
+        return RecurrentSpec(s.heads, s.dim, s.vdim, s.channels, s.taps)
+
+    def mix(self, proj: torch.Tensor, step, cache: SequenceStateCache, run: int) -> torch.Tensor:
+        return K.delta_mix(proj, self.spec, self, cache.conv[run], cache.state[run], self.eps, step)
+
+
+class DenseFeedForward:
+    def __init__(self, spec, w: Weights, prefix: str, width: int):
+        self.ff = spec.ff
+        self.w_gate_up = w.stack([(prefix + "gate", spec.ff), (prefix + "up", spec.ff)], width)
+        self.w_down = w.matrix(prefix + "down", width, spec.ff)
+
+    def branch(self, h: torch.Tensor) -> dict:
+        return dict(y=K.matmul(K.silu_mul(K.matmul(h, self.w_gate_up), self.ff), self.w_down))
+
+
+class MixtureFeedForward:
+    """Top-k mixture of small clamped experts; the weighted sum over a token's experts is left to the residual step."""
+
+    def __init__(self, spec, w: Weights, prefix: str, width: int):
+        s = self.spec = spec
+        self.router = w.matrix(prefix + "router", s.experts, width)
+        self.bias = w.vector(prefix + "router.b", s.experts)
+        dev, dt = w.device, w.dtype
+        self.w_gate_up = torch.empty((s.experts, 2 * s.ff, width), dtype=dt, device=dev)
+        self.w_down = torch.empty((s.experts, width, s.ff), dtype=dt, device=dev)
+        for e in range(s.experts):
+            p = f"{prefix}e{e}."
+            self.w_gate_up[e, :s.ff] = w.raw(p + "gate", s.ff, width)
+            self.w_gate_up[e, s.ff:] = w.raw(p + "up", s.ff, width)
+            self.w_down[e] = w.raw(p + "down", width, s.ff)
+
+    def branch(self, h: torch.Tensor) -> dict:
+        s, n = self.spec, h.shape[0]
+        idx, mix = K.moe_topk(K.matmul(h, self.router, torch.float32), self.bias, s.top)
+        src, inv, off, tiles = K.moe_sort(idx, s.experts)
+        act = K.moe_gemm(h, src, self.w_gate_up, off, tiles, entries=n * s.top, act=True, limit=s.limit)
+        y = K.moe_gemm(act, None, self.w_down, off, tiles, entries=n * s.top, act=False)
+        return dict(y=y, inv=inv, mix=mix)
+
+
+MIXERS = {"latent_attention": LatentAttention, "delta": GatedDelta}
+FEED_FORWARDS = {"dense": DenseFeedForward, "moe": MixtureFeedForward}
+
+
+class HybridForCausalLM:
+    """Weights, layer runs and the packed step."""
+
+    def __init__(self, config: HybridConfig, tensors: Dict[str, torch.Tensor], device, dtype: torch.dtype = torch.bfloat16):
+        self.config, self.device, self.dtype = config, torch.device(device), dtype
+        torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False     # 32-bit accumulation throughout
+        w = Weights(tensors, self.device, dtype)
+        c, width = config, config.width
+        self.embed = w.matrix("embed", c.vocab, width)
+        self.final_norm = w.vector("final.norm", width)
+        if c.loop is not None:
+            self.loop_in = w.matrix("loop.in", width, 2 * width)
+            self.loop_step = w.vector("loop.step", c.loop.times, width)
+        self.layers: List[SimpleNamespace] = []
+        for i, spec in enumerate(c.layers):
+            p = f"l{i}."
+            layer = SimpleNamespace(
+                mixer=MIXERS[spec.mixer.kind](spec.mixer, w, p + "mix.", width, c.eps), norm1=w.vector(p + "norm1", width),
+                norm1b=w.vector(p + "norm1b", width), ff=None)
+            if spec.mlp is not None:
+                layer.ff = FEED_FORWARDS[spec.mlp.kind](spec.mlp, w, p + "mlp.", width)
+                layer.norm2, layer.norm2b = w.vector(p + "norm2", width), w.vector(p + "norm2b", width)
+            elif p + "norm2" in tensors:       # a layer without a feed-forward has no use for its norms
+                w.vector(p + "norm2", width), w.vector(p + "norm2b", width)
+            self.layers.append(layer)
+        w.check_all_used()
+        self.status = torch.zeros(4, dtype=torch.int32, device=self.device)
+        self._program = self._compile()
+        self.on_layer = None       # hook(run, x): the stream after every layer run (debugging)
+
+    @classmethod
+    def from_pretrained(cls, path: str, device, dtype: torch.dtype = torch.bfloat16) -> "HybridForCausalLM":
+        from safetensors.torch import load_file
+        tensors: Dict[str, torch.Tensor] = {}
+        for shard in sorted(glob.glob(os.path.join(path, "*.safetensors"))):
+            tensors.update(load_file(shard))
+        return cls(HybridConfig.from_pretrained(path), tensors, device, dtype)
+
+    # ------------------------------------------------------------------ structure
+    def _compile(self):
+        """The run as a list of (kind, run, layer, pass): what is norm-ed for whom follows from the next entry."""
+        prog, loop = [], self.config.loop
+        for run, (i, t) in enumerate(self.config.runs()):
+            if loop is not None and t is not None and i == loop.start:
+                prog.append(("enter", run, i, t))
+            prog.append(("mix", run, i, t))
+            if self.layers[i].ff is not None:
+                prog.append(("ff", run, i, t))
+        return prog + [("final", None, None, None)]
+
+    def _next_norm(self, k: int) -> Optional[torch.Tensor]:
+        kind, _, i, _ = self._program[k]
+        return {"mix": lambda: self.layers[i].norm1, "ff": lambda: self.layers[i].norm2}.get(kind, lambda: None)()
+
+    def state_specs(self):
+        return [self.layers[i].mixer.state_spec for i, _ in self.config.runs()]
+
+    def new_cache(self, n_slots: int, max_len: int) -> SequenceStateCache:
+        return SequenceStateCache(self.state_specs(), n_slots, max_len, self.device, self.dtype)
+
+    # ------------------------------------------------------------------ the step
+    @torch.no_grad()
+    def step(self, step, cache: SequenceStateCache) -> torch.Tensor:
+        """Runs the step's tokens from the states in ``cache`` and advances those; fp32 logits ``[wanted, vocab]``."""
+        c, eps, dt = self.config, self.config.eps, self.dtype
+        cat = torch.empty((step.n_tok, 2 * c.width), dtype=dt, device=self.device) if c.loop is not None else None
+        x, h = K.embed(self.embed, step.token, self._next_norm(0), eps, cat=cat, cat_both=self._program[0][0] == "enter",
+                       status=self.status)
+        for k, (kind, run, i, t) in enumerate(self._program[:-1]):
+            nxt = self._next_norm(k + 1)
+            if kind == "enter":
+                y = K.matmul(cat, self.loop_in, torch.float32)
+                h = K.residual_norm(self.loop_step[t], y, None, nxt, eps, dt, x_out=x, broadcast=True)
+                continue
+            layer = self.layers[i]
+            if kind == "mix":
+                proj = K.matmul(h, layer.mixer.w_in)
+                branch, wb = dict(y=K.matmul(layer.mixer.mix(proj, step, cache, run), layer.mixer.w_o)), layer.norm1b
+            else:
+                branch, wb = layer.ff.branch(h), layer.norm2b
+            left = cat if self._program[k + 1][0] == "enter" else None
+            h = K.residual_norm(x, branch.pop("y"), wb, nxt, eps, dt, x_out=x, cat=left, **branch)
+            if self.on_layer is not None and self._program[k + 1][1] != run:
+                self.on_layer(run, x)
+        h = K.residual_norm(x, None, None, self.final_norm, eps, dt, rows=step.want_rows)
+        return K.matmul(h, self.embed, torch.float32)
+
+    def run(self, entries, cache: SequenceStateCache) -> torch.Tensor:
+        """``entries`` = (sequence, tokens, wanted places): one step, states advanced."""
+        step = PackedStep(entries, cache, self.config.windows)
+        logits = self.step(step, cache)
+        step.commit(cache)
+        return logits
+
+    # ------------------------------------------------------------------ the call of the interleave loop
+    @torch.no_grad()
+    def forward(self, input_ids=None, attention_mask=None, position_ids=None, past_key_values=None, doc_ids=None,
+                use_cache=True, logits_to_keep: int = 1, **unused):
+        """``MSAForCausalLM.forward``'s call on a batch of rows: row b continues sequence b of ``past_key_values`` (a
+        ``SequenceStateCache``) with its unmasked tokens; returns the logits of the last ``logits_to_keep`` columns
+        (masked columns: zeros).  Positions follow from the sequence; ``doc_ids`` has no meaning here."""
+        bsz, width = input_ids.shape
+        mask = torch.ones_like(input_ids) if attention_mask is None else attention_mask[:, -width:]
+        ids, mask = input_ids.tolist(), mask.bool().tolist()
+        keep = logits_to_keep or width
+        entries, places = [], []
+        for b in range(bsz):
+            cols = [j for j in range(width) if mask[b][j]]
+            if not cols:
+                continue
+            if b not in past_key_values:
+                past_key_values.acquire(b)
+            want = [n for n, j in enumerate(cols) if j >= width - keep]
+            entries.append((b, [ids[b][j] for j in cols], want))
+            places += [(b, cols[n] - (width - keep)) for n in want]
+        logits = torch.zeros((bsz, keep, self.config.vocab), dtype=torch.float32, device=self.device)
+        if entries:
+            got = self.run(entries, past_key_values)
+            if places:
+                b, j = zip(*places)
+                logits[list(b), list(j)] = got
+        return SimpleNamespace(logits=logits, past_key_values=past_key_values if use_cache else None)
+
+    __call__ = forward
+
+    def check_status(self) -> None:
+        """Raises if a step met token ids outside the vocabulary or a kernel gave up waiting."""
+        st = self.status.tolist()
+        if st[0] or st[2]:
+            self.status.zero_()
+            raise RuntimeError(f"kernel status {st}: wait code {st[0]}, {st[2]} token ids outside the vocabulary")
+
+
+class GraphedDecode:
+    """Decode steps of a fixed number of sequences as one CUDA graph.  ``run`` feeds tokens from the host,
+    ``replay`` continues on the device with what the last step chose (greedy)."""
+
+    def __init__(self, model: HybridForCausalLM, cache: SequenceStateCache, n: int):
+        self.model, self.cache, self.n = model, cache, n
+        self.tables = DecodeStep(n, cache, model.config.windows)
+        self.logits = self.next = None
+        self.graph = torch.cuda.CUDAGraph()
+        # the warm-up and capture passes run on slots 0 .. n-1 at position 0 and leave garbage there: callers capture
+        # before they acquire slots, or pass slots that are free
+        side = torch.cuda.Stream(model.device)
+        side.wait_stream(torch.cuda.current_stream(model.device))
+
+        def body():
+            logits = model.step(self.tables, cache)
+            return logits, logits.argmax(dim=-1).to(torch.int32)
+        free = list(cache._free)
+        if len(free) < n:
+            raise RuntimeError(f"capturing a decode step of {n} sequences needs {n} free slots")
+        self.tables.fill([0] * n, [0] * n, free[:n])
+        with torch.cuda.stream(side):
+            for _ in range(2):
+                body()
+        torch.cuda.current_stream(model.device).wait_stream(side)
+        with torch.cuda.graph(self.graph):
+            self.logits, self.next = body()
+
+    def run(self, tokens, positions, slots) -> torch.Tensor:
+        self.tables.fill(tokens, positions, slots)
+        self.graph.replay()
+        return self.logits
+
+    def replay(self) -> torch.Tensor:
+        self.tables.token.copy_(self.next)
+        self.tables.pos.add_(1)
+        self.graph.replay()
+        return self.next

@@ -60,29 +60,35 @@ class BlockModelInput:
     chunk_sizes: List[int]
 
 
-def default_model_factory(model_path: str, device):
-    """Tokenizer and decoder stack from a checkpoint directory in the reference's format (``config.json`` with an
+def load_msa_checkpoint(model_path: str, device, dtype: torch.dtype = torch.bfloat16):
+    """The memory decoder stack from a checkpoint directory in the reference's format (``config.json`` with an
     ``msa_config`` entry, safetensors weights)."""
     import glob
     import json
 
     from safetensors.torch import load_file
-    from transformers import AutoTokenizer
 
     from .configuration import MSAConfig
     from .model import MSAForCausalLM
-    tokenizer = AutoTokenizer.from_pretrained(model_path)
     with open(os.path.join(model_path, "config.json")) as f:
         raw = json.load(f)
     config = MSAConfig(**{k: v for k, v in raw.items() if k not in ("architectures", "model_type", "auto_map")})
-    model = MSAForCausalLM(config).to(torch.bfloat16)
+    model = MSAForCausalLM(config).to(dtype)
     state = {}
     for shard in sorted(glob.glob(os.path.join(model_path, "*.safetensors"))):
         state.update(load_file(shard))
     missing, unexpected = model.load_state_dict(state, strict=False)
     if missing:
         raise RuntimeError(f"{model_path}: checkpoint lacks {missing[:5]} ...")
-    return model.to(device).eval(), tokenizer
+    return model.to(device).eval()
+
+
+def default_model_factory(model_path: str, device):
+    """``(model, tokenizer)`` of a checkpoint directory: the model of the design its config.json names
+    (``registry.load_model``); a directory without tokenizer files gets the number tokenizer."""
+    from .registry import load_model
+    from .tools import load_tokenizer
+    return load_model(model_path, device), load_tokenizer(model_path)
 
 
 class PrefillStage1Worker:
