@@ -236,12 +236,17 @@ class DecodeStep:
         self.want_rows = torch.arange(n, **i)
         self.views = {w: ContextView(cache.max_len if w is None else min(w, cache.max_len), None, None, 0, 0) for w in windows}
         self._host = torch.zeros((3, n), dtype=torch.int32)
+        self._copied = None
         if dev.type == "cuda":
-            self._host = self._host.pin_memory()
+            self._host, self._copied = self._host.pin_memory(), torch.cuda.Event()
 
     def fill(self, tokens: Sequence[int], positions: Sequence[int], slots: Sequence[int]) -> None:
-        self._host[0], self._host[1], self._host[2] = torch.tensor(tokens), torch.tensor(positions), torch.tensor(slots)
+        if self._copied is not None:
+            self._copied.synchronize()        # the copy of the last fill has left the host buffer
+        self._host.copy_(torch.tensor([tokens, positions, slots], dtype=torch.int32))
         self.table.copy_(self._host, non_blocking=True)
+        if self._copied is not None:
+            self._copied.record()
 
 
 class SharedPooledCache:

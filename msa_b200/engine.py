@@ -17,6 +17,11 @@ answers requests with the Memory-Interleave loop (``msa_b200.generate``).  Token
 ``(model_path, device) -> (model, tokenizer)`` (``msa_b200.prefill.default_model_factory`` unless
 ``model_config.envs["MSA_B200_MODEL_FACTORY"] = "module:function"`` names another); ``MSAEngine(...,
 service_main=...)`` swaps the whole service process (the tests run the protocol with a text-only stand-in).
+
+A checkpoint whose design is served from per-sequence state slots (``registry.Design.serves == "states"``) takes the
+same ``generate`` call without a memory file: prompts are texts or token lists, nothing is templated or padded, and each
+service process (``state_service_main``) feeds its share to a continuous-batching ``scheduler.Scheduler`` that serves
+all requests in flight together; the texts are the generated tokens alone.
 """
 from __future__ import annotations
 
@@ -58,6 +63,10 @@ class GenerateConfig:
     top_p: float = 0.9
     temperature: float = 0.0
     qa_mode: bool = False
+    # models served from state slots
+    state_slots: int = 64         # sequences in flight per GPU
+    max_context: int = 8192       # prompt and generated tokens of one sequence
+    seed: Optional[int] = None    # sampling: row i of a request draws from seed + i
 
     def __post_init__(self):
         if isinstance(self.template, str):
@@ -100,6 +109,7 @@ class GenerateResponse:
     gpu_id: int = 0
     generated_texts: List[str] = None
     recall_topk: Optional[Dict[int, List]] = None
+    error: Optional[str] = None
 
 
 @dataclass
@@ -143,15 +153,25 @@ def _resolve_factory(envs: Optional[dict]):
     return default_model_factory
 
 
+def _serves(model_path: str) -> str:
+    """What the checkpoint at ``model_path`` is served with; a path without config.json belongs to a factory of the
+    memory model."""
+    if not os.path.exists(os.path.join(model_path, "config.json")):
+        return "memory"
+    from .registry import design_of
+    return design_of(model_path).serves
+
+
 class MSAEngine:
-    def __init__(self, generate_config: GenerateConfig, model_config: ModelConfig, memory_config: MemoryConfig,
+    def __init__(self, generate_config: GenerateConfig, model_config: ModelConfig, memory_config: Optional[MemoryConfig] = None,
                  service_main: Optional[Callable] = None, tokenizer=None, start: bool = True):
         if not generate_config.devices:
             # NCCL wants the global device numbering; select GPUs with CUDA_VISIBLE_DEVICES (src/msa_service.py:1376-1379)
             generate_config.devices = list(range(torch.cuda.device_count()))
         self.world_size = generate_config.world
         self.generate_config, self.model_config, self.memory_config = generate_config, model_config, memory_config
-        self._service_main = service_main or MSAEngine.service_main
+        self.serves = _serves(model_config.model_path)
+        self._service_main = service_main or (state_service_main if self.serves == "states" else MSAEngine.service_main)
         self.tokenizer = tokenizer
         self.worker_processes: List[mp.Process] = []
         self.worker_qs: Dict[int, Any] = {}
@@ -174,17 +194,20 @@ class MSAEngine:
     def initialize(self):
         if self.tokenizer is None:
             _, self.tokenizer = None, self._load_tokenizer()
-        self._prepare_template()
-        self._load_memory_file()
-        self._wait_ready_signal()          # every service is up before the buckets are sent
-        self._process_buckets()
+        if self.serves == "states":
+            self._wait_ready_signal()
+        else:
+            self._prepare_template()
+            self._load_memory_file()
+            self._wait_ready_signal()      # every service is up before the buckets are sent
+            self._process_buckets()
         self.running = True                # the receiver starts only after the buckets are processed
         self.recv_rsp_thread = threading.Thread(target=self.receive_response, daemon=True)
         self.recv_rsp_thread.start()
 
     def _load_tokenizer(self):
-        from transformers import AutoTokenizer
-        return AutoTokenizer.from_pretrained(self.model_config.model_path)
+        from .tools import load_tokenizer
+        return load_tokenizer(self.model_config.model_path)
 
     def start_workers(self):
         for gpu_id in self.generate_config.devices:
@@ -345,6 +368,8 @@ class MSAEngine:
         (``3 + doc_top_k``) for every prompt; a GPU's share is left-padded to its own longest prompt, padding repeats
         the first position and has doc id 0 and mask 0."""
         world = self.generate_config.world
+        if self.serves == "states":
+            return self._prepare_state_requests(prompts, msg_id)
         bsz = (len(prompts) + world - 1) // world
         if self.generate_config.max_batch_size > 0 and bsz > self.generate_config.max_batch_size:
             raise ValueError(f"Batch size exceeds maximum allowed batch size {self.generate_config.max_batch_size}")
@@ -372,12 +397,27 @@ class MSAEngine:
                                             require_recall_topk=require_recall_topk))
         return requests, pads
 
+    def _prepare_state_requests(self, prompts, msg_id: int):
+        """Prompts (texts or token lists) dealt over the GPUs in runs; no padding, no fill-ins: a GPU's share may be empty."""
+        cfg = self.generate_config
+        rows = [list(p) if not isinstance(p, str) else list(self.tokenizer(p, add_special_tokens=False)["input_ids"]) for p in prompts]
+        for ids in rows:
+            if not ids:
+                raise ValueError("empty query is not acceptable")
+            if len(ids) + cfg.max_generate_tokens > cfg.max_context:
+                raise ValueError(f"{len(ids)} prompt tokens and {cfg.max_generate_tokens} new ones exceed max_context {cfg.max_context}")
+        share = (len(rows) + cfg.world - 1) // cfg.world
+        if cfg.max_batch_size > 0 and share > cfg.max_batch_size:
+            raise ValueError(f"Batch size exceeds maximum allowed batch size {cfg.max_batch_size}")
+        return [GenerateRequest(msg_id=msg_id, seq_id=i, prompts=list(prompts[i * share:(i + 1) * share]),
+                                input_ids=rows[i * share:(i + 1) * share]) for i in range(cfg.world)], 0
+
     # ------------------------------------------------------------------ requests and responses
     def default_callback(self, texts, recall_topk, userdata):
         self.sync_rsp = (texts, recall_topk, userdata)
         self.sync_event.set()
 
-    def generate(self, prompts: Union[str, List[str]], userdata=None, require_recall_topk: bool = False,
+    def generate(self, prompts: Union[str, List[str], List[List[int]]], userdata=None, require_recall_topk: bool = False,
                  callback: Optional[GenerateReceiver] = None):
         """Blocking without ``callback`` (returns ``(texts, recall_topk, userdata)``); with one, returns at once and
         the receiver thread calls ``callback(texts, recall_topk, userdata)``.  At most four requests are in flight."""
@@ -395,6 +435,8 @@ class MSAEngine:
         if sync:
             self.sync_event.wait()
             self.sync_event.clear()
+            if isinstance(self.sync_rsp, Exception):
+                raise self.sync_rsp
             return self.sync_rsp
 
     def receive_response(self):
@@ -412,7 +454,12 @@ class MSAEngine:
                     done = self.requests.pop(rsp.msg_id)
             if done is not None:
                 self.limiter.release()
-                done.respond()
+                errors = [r.error for r in done.responses if r.error]
+                if errors and done.callback == self.default_callback:       # the blocking caller raises it
+                    self.sync_rsp = RuntimeError(errors[0])
+                    self.sync_event.set()
+                else:
+                    done.respond()
 
     # ------------------------------------------------------------------ the per-GPU process
     @staticmethod
@@ -468,6 +515,71 @@ class MSAEngine:
                 print(f"[subprocess {gpu_id}] error: {e}")
                 import traceback
                 traceback.print_exc()
+
+
+def state_service_main(gpu_id: int, request_queue, response_queue, generate_config: GenerateConfig,
+                       model_config: ModelConfig, memory_config=None):
+    """One GPU's process for a model on state slots: requests that arrive while others run join the next step."""
+    from .scheduler import Scheduler, SequenceRequest
+    for k, v in (model_config.envs or {}).items():
+        os.environ[k] = v
+    torch.cuda.set_device(gpu_id)
+    if (model_config.envs or {}).get("MSA_B200_MODEL_FACTORY") or os.environ.get("MSA_B200_MODEL_FACTORY"):
+        model, tokenizer = _resolve_factory(model_config.envs)(model_config.model_path, f"cuda:{gpu_id}")
+    else:
+        from .registry import load_model
+        from .tools import load_tokenizer
+        model = load_model(model_config.model_path, f"cuda:{gpu_id}", getattr(torch, model_config.dtype))
+        tokenizer = load_tokenizer(model_config.model_path)
+    sched = Scheduler(model, max_batch=generate_config.state_slots, max_len=generate_config.max_context)
+    eos = getattr(tokenizer, "eos_token_id", None)
+    eos = [] if eos is None else ([eos] if isinstance(eos, int) else list(eos))
+    open_requests: Dict[Any, dict] = {}
+
+    def answer(key, error=None):
+        st = open_requests.pop(key)
+        texts = [] if error else tokenizer.batch_decode([r.output for r in st["rows"]])
+        response_queue.put(GenerateResponse(msg_id=st["cmd"].msg_id, seq_id=st["cmd"].seq_id, gpu_id=gpu_id,
+                                            generated_texts=texts, error=error))
+
+    ProtocolConstants.send(response_queue, MEMORY_WORKER_READY, block=False)
+    closing = False
+    while not (closing and not sched.busy):
+        try:
+            while not closing:
+                cmd = request_queue.get(block=not sched.busy)
+                if cmd is None:
+                    closing = True
+                    break
+                key = (cmd.msg_id, cmd.seq_id)
+                rows = [SequenceRequest(tokens=ids, max_new_tokens=generate_config.max_generate_tokens, eos_token_ids=eos,
+                                        temperature=generate_config.temperature, top_p=generate_config.top_p, tag=key,
+                                        seed=None if generate_config.seed is None else generate_config.seed + i)
+                        for i, ids in enumerate(cmd.input_ids)]
+                open_requests[key] = {"cmd": cmd, "rows": rows}
+                try:
+                    for r in rows:
+                        sched.check(r)
+                    for r in rows:
+                        sched.submit(r)
+                except ValueError as e:
+                    answer(key, f"{type(e).__name__}: {e}")
+                    continue
+                if not rows:
+                    answer(key)
+        except queue.Empty:
+            pass
+        try:
+            for r in sched.step():
+                if all(x.finished for x in open_requests[r.tag]["rows"]):
+                    answer(r.tag)
+        except Exception as e:        # a failed step fails every request in flight, not the process
+            import traceback
+            traceback.print_exc()
+            for key in list(open_requests):
+                for r in open_requests[key]["rows"]:
+                    sched.cancel(r.id)
+                answer(key, f"{type(e).__name__}: {e}")
 
 
 def create_generate_args(generate_config: GenerateConfig) -> dict:

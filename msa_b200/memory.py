@@ -41,6 +41,7 @@ class ModelConfig:
     template_token_id: int = -2
     template_id_num: int = 3
     envs: Optional[dict] = None     # environment of the stage-1 worker process (get_model_envs in the reference)
+    dtype: str = "bfloat16"         # models served from state slots: "bfloat16" or "float32"
 
 
 @dataclass

@@ -44,7 +44,8 @@ class Scheduler:
         self._seen: Dict[int, int] = {}
 
     # ------------------------------------------------------------------ requests
-    def submit(self, request: SequenceRequest) -> int:
+    def check(self, request: SequenceRequest) -> None:
+        """Raises ``ValueError`` for a request that cannot be served."""
         if not request.tokens:
             raise ValueError("a request needs at least one token")
         if request.max_new_tokens < 1:
@@ -53,6 +54,9 @@ class Scheduler:
             raise ValueError(f"{len(request.tokens)} + {request.max_new_tokens} tokens do not fit the {self.cache.max_len} a slot holds")
         if min(request.tokens) < 0 or max(request.tokens) >= self.model.config.vocab:
             raise ValueError("token id outside the vocabulary")
+
+    def submit(self, request: SequenceRequest) -> int:
+        self.check(request)
         request.id = next(self._ids)
         self.waiting.append(request)
         return request.id

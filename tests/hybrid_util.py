@@ -1,0 +1,146 @@
+"""Small random models of the layered decoder designs, and the comparisons the tests share."""
+import json
+import os
+
+import torch
+
+from oracle import hybrid_oracle as O
+
+
+def latent(heads, dim, rot, vdim, rank, window, base=500.0, scale=None):
+    return {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank, "scale": scale or (dim + rot) ** -0.5,
+            "rot": {"base": base, "dims": rot}, "mask": {"size": window}}
+
+
+def delta(heads, kv_heads, dim, vdim, conv):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}
+
+
+def dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(experts, top, ff, limit):
+    return {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff, "limit": limit}}
+
+
+def layer(kind, mixer, mlp):
+    return {"type": kind, "mixer": mixer, "mlp": mlp}
+
+
+def config(width, vocab, layers, loop=None, eps=1e-5):
+    return {"architecture": "Mutuvik", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": layers, "loop": loop}
+
+
+# uneven sizes everywhere, two windows, a layer without a feed-forward, a loop in the middle with a tail behind it
+MIXED = config(88, 211, [
+    layer("delta", delta(4, 2, 24, 20, 4), dense(112)),
+    layer("latent_attention", latent(3, 20, 12, 28, 44, 17), moe(7, 2, 36, 1.5)),
+    layer("latent_attention", latent(5, 8, 6, 12, 20, 33, base=77.0), None),
+    layer("delta", delta(6, 3, 16, 36, 2), moe(4, 3, 20, 0.7)),
+    layer("latent_attention", latent(2, 16, 8, 16, 24, 9), dense(52)),
+], loop={"start": 1, "stop": 4, "times": 3}, eps=3e-4)
+
+# odd sizes: nothing is a multiple of 4; the loop starts with the first layer and runs once; window 1 and a wide one
+ODD = config(51, 97, [
+    layer("latent_attention", latent(3, 5, 2, 7, 13, 1), moe(3, 1, 11, 3.0)),
+    layer("delta", delta(3, 1, 9, 7, 3), dense(33)),
+    layer("latent_attention", latent(1, 3, 4, 5, 9, 400), moe(5, 5, 9, 1.0)),
+], loop={"start": 0, "stop": 2, "times": 1})
+
+# no loop; sizes that the tensor-core kernels take
+WIDE = config(256, 320, [
+    layer("delta", delta(4, 2, 128, 128, 4), moe(8, 2, 128, 2.5)),
+    layer("latent_attention", latent(4, 128, 64, 128, 256, 96, base=10000.0), moe(6, 3, 64, 1.0)),
+    layer("delta", delta(2, 2, 64, 64, 4), dense(256)),
+    layer("latent_attention", latent(8, 64, 32, 64, 128, 160, base=10000.0), dense(128)),
+])
+
+CONFIGS = {"mixed": MIXED, "odd": ODD, "wide": WIDE}
+
+
+def make_weights(cfg, seed=0, sharp=2.0):
+    """bf16 tensors by name.  ``sharp`` scales the attention queries: peaked weights let a single wrong key show."""
+    g = torch.Generator().manual_seed(seed)
+    w, width = {}, cfg["width"]
+    mat = lambda n, r, c, s=1.0: w.__setitem__(n, torch.randn(r, c, generator=g) * (s / c ** 0.5))
+    vec = lambda n, k, mean, std: w.__setitem__(n, mean + std * torch.randn(k, generator=g))
+    w["embed"] = torch.randn(cfg["vocab"], width, generator=g)
+    if cfg["loop"]:
+        mat("loop.in", width, 2 * width)
+        w["loop.step"] = 0.5 * torch.randn(cfg["loop"]["times"], width, generator=g)
+    for i, entry in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", entry["mixer"]
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if entry["mlp"] else ()):
+            vec(p + n, width, 1.0, 0.2)
+        x = p + "mix."
+        if entry["type"] == "delta":
+            qk, v = m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
+            for n, r in (("q", qk), ("k", qk), ("v", v)):
+                mat(x + n, r, width)
+                w[x + n + ".conv"] = torch.randn(r, m["conv"], generator=g) * 0.6
+            mat(x + "g", v, width)
+            mat(x + "b", m["heads"], width)
+            mat(x + "a", m["heads"], width)
+            w[x + "A_log"] = torch.rand(m["heads"], generator=g) * 3 - 3.5
+            vec(x + "dt_bias", m["heads"], 0.0, 1.0)
+            vec(x + "norm", m["vdim"], 1.0, 0.2)
+            mat(x + "o", width, v)
+        else:
+            mat(x + "q", m["heads"] * (m["dim"] + m["rot_dim"]), width, sharp)
+            mat(x + "dkv", m["kv_rank"] + m["rot_dim"], width)
+            vec(x + "dkv.norm", m["kv_rank"], 1.0, 0.2)
+            mat(x + "uk", m["heads"] * m["dim"], m["kv_rank"])
+            mat(x + "uv", m["heads"] * m["vdim"], m["kv_rank"])
+            mat(x + "o", width, m["heads"] * m["vdim"])
+        f = entry["mlp"]
+        if f and f["kind"] == "dense":
+            for n, r, c in (("gate", f["ff"], width), ("up", f["ff"], width), ("down", width, f["ff"])):
+                mat(p + "mlp." + n, r, c)
+        elif f:
+            e_ff = f["expert"]["ff"]
+            mat(p + "mlp.router", f["router"]["experts"], width)
+            vec(p + "mlp.router.b", f["router"]["experts"], 0.0, 0.7)
+            for e in range(f["router"]["experts"]):
+                for n, r, c in (("gate", e_ff, width), ("up", e_ff, width), ("down", width, e_ff)):
+                    mat(f"{p}mlp.e{e}.{n}", r, c, 1.5)
+    vec("final.norm", width, 1.0, 0.2)
+    return {k: v.to(torch.bfloat16) for k, v in w.items()}
+
+
+def save(cfg, weights, path):
+    from safetensors.torch import save_file
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    save_file({k: v.contiguous() for k, v in weights.items()}, os.path.join(path, "model.safetensors"))
+
+
+def tokens_of(cfg, n, seed):
+    return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+def row_errors(got, want):
+    """Per row: rms of the difference over the rms of the wanted rows."""
+    got, want = got.double().cpu(), want.double().cpu()
+    return (got - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
+
+
+def model_weights(name, seed, dtype):
+    """Whole-model comparisons in bf16 cannot rest on close calls of a router: there the biases decide most choices."""
+    w = make_weights(CONFIGS[name], seed)
+    if dtype == torch.bfloat16:
+        for k in w:
+            if k.endswith("router.b"):
+                w[k] = w[k] * 6
+    return w
+
+
+_ORACLE = {}
+
+
+def oracle_logits(name, seed, toks, dtype=torch.float32):
+    key = (name, seed, tuple(toks), dtype)
+    if key not in _ORACLE:
+        _ORACLE[key] = O.forward(CONFIGS[name], model_weights(name, seed, dtype), toks)
+    return _ORACLE[key]
