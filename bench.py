@@ -63,8 +63,9 @@ def parse():
     ap.add_argument("--short", action="store_true", help="secondary workloads: take --steps / --warmup as given (profiling runs)")
     ap.add_argument("--decode-batch", type=int, default=32, help="route-decode workload: sequences per step (<= 128)")
     ap.add_argument("--workload", default="routing",
-                    choices=["routing", "pooling", "decode", "fetch", "route-decode", "prefill", "stage1", "generate"],
+                    choices=["routing", "pooling", "decode", "fetch", "route-decode", "prefill", "stage1", "generate", "hybrid"],
                     help="routing = the headline (default); the others time one secondary kernel each")
+    ap.add_argument("--hybrid-sizes", default="2k,4k", help="hybrid workload: model sizes to run")
     return ap.parse_args()
 
 
@@ -1402,6 +1403,274 @@ def generate_timeline(torch, model, router_ids, dev, with_fetch=True):
         return {"error": f"{type(e).__name__}: {e}"}
 
 
+# ------------------------------------------------------------------------------------------
+# layered decoder (windowed latent attention, gated delta rule, experts, looped layers) beside the memory decoder
+# ------------------------------------------------------------------------------------------
+HYBRID_SIZES = {   # width, heads, kv heads of the delta layers, window, dense ff, experts, top, expert ff
+    "2k": dict(width=2048, heads=16, kv=8, window=1024, ff=6144, experts=32, top=4, eff=1536),
+    "4k": dict(width=4096, heads=32, kv=16, window=2048, ff=12288, experts=64, top=8, eff=1536),
+}
+
+
+def hybrid_config(z, vocab=32768):
+    delta = {"type": "delta", "mixer": {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128, "conv": 4}}
+    latent = {"type": "latent_attention", "mixer": {
+        "heads": z["heads"], "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
+        "rot": {"base": 10000.0, "dims": 64}, "mask": {"size": z["window"]}}}
+    moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["eff"], "limit": 7.0}}
+    return {"architecture": "Mutuvik", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-5},
+            "layers": [{**delta, "mlp": {"kind": "dense", "ff": z["ff"]}}, {**latent, "mlp": moe}, {**delta, "mlp": moe}, {**latent, "mlp": moe}],
+            "loop": {"start": 1, "stop": 4, "times": 2}}
+
+
+def hybrid_model(torch, dev, z):
+    from msa_b200.hybrid import HybridForCausalLM, Weights
+    from msa_b200.hybrid_config import HybridConfig
+    gen = torch.Generator(device=dev)
+    gen.manual_seed(3)
+
+    class Drawn(Weights):
+        def raw(self, name, *shape):
+            t = torch.randn(shape, generator=gen, device=dev, dtype=torch.float32)
+            if len(shape) == 2 and not name.endswith(".conv") and name not in ("embed", "loop.step"):
+                t *= shape[1] ** -0.5
+            elif "norm" in name:
+                t = 1 + 0.1 * t
+            elif name.endswith("A_log"):
+                t -= 1.0
+            return t.to(torch.bfloat16)
+    return HybridForCausalLM(HybridConfig.parse(hybrid_config(z)), Drawn({}, dev, torch.bfloat16), dev)
+
+
+def hybrid_kernels(torch, dev, model, z, pk, decode_b):
+    """Every kernel of the design alone: time, algorithmic flops and bytes, and the fraction of the bound that applies
+    (the larger of flops over the burst bf16 rate and bytes over the copy bandwidth)."""
+    import ctypes
+
+    from msa_b200 import _cabi_lm as A, lm_ops as K
+    from msa_b200.cache import DecodeStep, PackedStep
+    rows, heads, width, window = {}, z["heads"], z["width"], z["window"]
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+
+    def leg(name, fn, flops, nbytes, reps=10):
+        for _ in range(3):
+            fn()
+        ts = []
+        for _ in range(reps):
+            flush.zero_()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1))
+        ms = statistics.median(ts)
+        t_f, t_b = flops / (pk["tflops_burst"] * 1e9), nbytes / (pk["hbm_gbs"] * 1e6)
+        rows[name] = {"us": round(ms * 1e3, 1), "bound": "tensor" if t_f > t_b else "hbm", "bound_us": round(max(t_f, t_b) * 1e3, 1),
+                      "frac": round(max(t_f, t_b) / ms, 3)}
+
+    n_seq, t = 4, 2048
+    n = n_seq * t
+    cache = model.new_cache(max(n_seq, decode_b) + 1, 4096)
+    for i in range(n_seq):
+        cache.acquire(i)
+    step = PackedStep([(i, [1] * t, []) for i in range(n_seq)], cache, model.config.windows)
+    lat, dlt, moe = model.layers[1].mixer, model.layers[0].mixer, model.layers[1].ff
+    view = step.views[window]
+    bf = dict(dtype=torch.bfloat16, device=dev)
+    h = torch.randn((n, width), **bf)
+    x = torch.randn((n, width), dtype=torch.float32, device=dev)
+    y = torch.randn((n, width), **bf)
+    leg("residual_norm", lambda: K.residual_norm(x, y, model.layers[0].norm1b, model.layers[0].norm2, 1e-5, torch.bfloat16, x_out=x),
+        0, n * width * 12)
+    s = lat.spec
+    proj = K.matmul(h, lat.w_in)
+    ctx = torch.empty((n, s.kv_rank + s.rot_dim), **bf)
+    leg("latent_prep", lambda: K.latent_prep(proj, s, lat.norm, lat.inv_freq, 1e-5, step, view, cache.ring[1], ctx), 0,
+        n * 2 * (2 * heads * s.rot_dim + 2 * (s.kv_rank + s.rot_dim)))
+    kv = K.matmul(ctx[:, :s.kv_rank], lat.w_kv)
+    out = torch.empty((n, heads * s.vdim), **bf)
+    pairs = n_seq * sum(min(i + 1, window) for i in range(t))
+    leg("window_attn_tc (prompt)", lambda: K.window_attn_tc(proj, kv, ctx, s, out, step, view, model.status),
+        2.0 * pairs * heads * (s.dim + s.rot_dim + s.vdim), n * heads * 2 * (s.dim + s.rot_dim + s.dim + 2 * s.vdim))
+    leg("ring_store", lambda: K.ring_store(ctx, step, view, cache.ring[1]), 0, n_seq * min(t, window) * (s.kv_rank + s.rot_dim) * 4)
+    d = dlt.spec
+    projd = K.matmul(h, dlt.w_in)
+    args = K.delta_args(projd, d, dlt, cache.conv[0], cache.state[0], 1e-5, step)
+    f32 = dict(dtype=torch.float32, device=dev)
+    qk, v, gates, o = (torch.empty((n, c), **f32) for c in (2 * d.kv_heads * d.dim, heads * d.vdim, 2 * heads, heads * d.vdim))
+    outd, st = torch.empty((n, heads * d.vdim), **bf), A.stream_ptr(dev)
+    p = A.ptr
+    leg("delta_prep", lambda: A.call("msa_lm_delta_prep", ctypes.byref(args), p(qk), p(v), p(gates), st), 0, n * d.channels * 6)
+    leg("delta_scan", lambda: K.delta_recurrence(args, qk, v, gates, o, model.status), n * heads * d.dim * d.vdim * 6.0, n * 4 * (d.channels + heads * d.vdim))
+    leg("delta_out", lambda: A.call("msa_lm_delta_out", ctypes.byref(args), p(o), p(outd), outd.stride(0), st), 0, n * heads * d.vdim * 8)
+    m = moe.spec
+    logits = K.matmul(h, moe.router, torch.float32)
+    leg("moe_topk", lambda: K.moe_topk(logits, moe.bias, m.top), 0, n * m.experts * 4)
+    idx, mix = K.moe_topk(logits, moe.bias, m.top)
+    leg("moe_sort", lambda: K.moe_sort(idx, m.experts, 128), 0, n * m.top * 12)
+    src, inv, off, tiles = K.moe_sort(idx, m.experts, 128)
+    ent = n * m.top
+    act = K.moe_gemm_tc(h, src, moe.w_gate_up, off, tiles, entries=ent, act=True, limit=7.0, status=model.status)
+    leg("moe_gemm_tc gate/up + activation (prompt)", lambda: K.moe_gemm_tc(h, src, moe.w_gate_up, off, tiles, entries=ent, act=True, limit=7.0, status=model.status),
+        2.0 * ent * width * 2 * m.ff, moe.w_gate_up.numel() * 2 + n * width * 2 + ent * m.ff * 2)
+    ye = K.moe_gemm_tc(act, None, moe.w_down, off, tiles, entries=ent, act=False, status=model.status)
+    leg("moe_gemm_tc down (prompt)", lambda: K.moe_gemm_tc(act, None, moe.w_down, off, tiles, entries=ent, act=False, status=model.status),
+        2.0 * ent * width * m.ff, moe.w_down.numel() * 2 + ent * (m.ff + width) * 2)
+    leg("residual_norm over experts", lambda: K.residual_norm(x, ye, model.layers[1].norm2b, model.layers[2].norm1, 1e-5, torch.bfloat16, x_out=x, inv=inv, mix=mix),
+        0, n * width * 10 + ent * width * 2)
+    leg("cuBLAS in-projection (reference)", lambda: K.matmul(h, dlt.w_in), 2.0 * n * width * dlt.w_in.shape[0], (n * width + dlt.w_in.numel() + n * dlt.w_in.shape[0]) * 2)
+    # decode: every sequence past its window
+    for i in range(n_seq):
+        cache.release(i)
+    b = decode_b
+    ds = DecodeStep(b, cache, model.config.windows)
+    ds.fill([1] * b, [window + 5] * b, list(range(b)))
+    hb = torch.randn((b, width), **bf)
+    pl, pd = K.matmul(hb, lat.w_in), K.matmul(hb, dlt.w_in)
+    q = pl[:, :heads * (s.dim + s.rot_dim)].view(b, heads, s.dim + s.rot_dim)
+    qa = torch.bmm(q[..., :s.dim].transpose(0, 1), lat.w_uk)
+    lo = torch.empty((b, heads, s.kv_rank), **bf)
+    leg(f"latent_decode + merge (batch {b})", lambda: K.latent_decode(qa.transpose(0, 1), q[..., s.dim:], cache.ring[1], ds.slot, ds.start, lo, window=window, scale=s.scale),
+        2.0 * b * window * heads * (2 * s.kv_rank + s.rot_dim), b * window * (s.kv_rank + s.rot_dim) * 2)
+    da = K.delta_args(pd, d, dlt, cache.conv[0], cache.state[0], 1e-5, ds)
+    od = torch.empty((b, heads * d.vdim), **bf)
+    leg(f"delta_decode (batch {b})", lambda: A.call("msa_lm_delta_decode", ctypes.byref(da), p(od), od.stride(0), st), 0,
+        b * heads * d.dim * d.vdim * 8 + b * d.channels * 2 * (2 * d.taps))
+    lg = K.matmul(hb, moe.router, torch.float32)
+    idx, mix = K.moe_topk(lg, moe.bias, m.top)
+    src, inv, off, tiles = K.moe_sort(idx, m.experts, 128)
+    used = int((off[1:] > off[:-1]).sum())
+    leg(f"moe_topk + moe_sort (batch {b})", lambda: K.moe_sort(K.moe_topk(lg, moe.bias, m.top)[0], m.experts, 128), 0, b * m.experts * 4)
+    leg(f"moe_gemm_tc gate/up (batch {b})", lambda: K.moe_gemm_tc(hb, src, moe.w_gate_up, off, tiles, entries=b * m.top, act=True, limit=7.0, status=model.status),
+        2.0 * b * m.top * width * 2 * m.ff, used * 2 * m.ff * width * 2)
+    ab = K.moe_gemm_tc(hb, src, moe.w_gate_up, off, tiles, entries=b * m.top, act=True, limit=7.0, status=model.status)
+    leg(f"moe_gemm_tc down (batch {b})", lambda: K.moe_gemm_tc(ab, None, moe.w_down, off, tiles, entries=b * m.top, act=False, status=model.status),
+        2.0 * b * m.top * width * m.ff, used * m.ff * width * 2)
+    model.check_status()
+    return rows
+
+
+def closest_kernels(torch, dev, pk):
+    """The memory decoder's kernels of the same roles, timed in the same run."""
+    from msa_b200 import ops
+    out = {}
+    a = leg_stage1_attention(torch, ops, dev, pk)
+    out["doc_attn_tc (prompt attention)"] = {"us": round(a["ms"] * 1e3, 1), "bound": "tensor", "frac": round(a["frac"], 3)}
+    a = leg_decode(torch, ops, dev, pk, 200, 3)
+    out["sparse_decode_attn"] = {"us": round(a["ms"] * 1e3, 1), "bound": "hbm", "frac": round(a["frac"], 3)}
+    n, w = 8192, 4096
+    x, y = (torch.randn((n, w), dtype=torch.bfloat16, device=dev) for _ in range(2))
+    wt = torch.ones(w, dtype=torch.bfloat16, device=dev)
+    ms = _time_ms(torch, lambda: ops.add_rmsnorm(x, y, wt, 1e-6), 20, 3)
+    out["add_rmsnorm"] = {"us": round(ms * 1e3, 1), "bound": "hbm", "frac": round(n * w * 8 / (ms * pk["hbm_gbs"] * 1e6), 3)}
+    gu = torch.randn((n, 2 * w), dtype=torch.bfloat16, device=dev)
+    ms = _time_ms(torch, lambda: ops.silu_mul(gu, w), 20, 3)
+    out["silu_mul"] = {"us": round(ms * 1e3, 1), "bound": "hbm", "frac": round(n * w * 6 / (ms * pk["hbm_gbs"] * 1e6), 3)}
+    return out
+
+
+def closest_model(torch, dev, z, runs, decode_batches, steps, warmup):
+    """Prompt and decode throughput of the memory decoder (Qwen3-shaped) with the same width, layer runs, attention span,
+    active feed-forward width and vocabulary; no routing, no retrieval."""
+    from msa_b200.cache import SparseCacheOnCPU
+    from msa_b200.configuration import MSAConfig
+    from msa_b200.decoder import DecoderShape, SparseDecodeModel
+    from msa_b200.model import MSAForCausalLM
+    out = {}
+    shape = DecoderShape(num_layers=runs, hidden=z["width"], n_q_heads=z["width"] // 128, n_kv_heads=8, ffn=z["ff"], vocab=32768)
+    for b in decode_batches:
+        m = SparseDecodeModel(shape, None, [], b, z["window"] - 3, 4 * (steps + warmup) + 16, 0, dev)
+        for _ in range(3):
+            m.step()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            m.step()
+        m.reset()
+        ms = _time_ms(torch, graph.replay, steps, warmup)
+        out[f"decode_batch_{b}"] = {"ms_per_step": ms, "tokens_per_s": b / ms * 1e3}
+        del graph, m
+        torch.cuda.empty_cache()
+    cfg = MSAConfig(hidden_size=z["width"], num_hidden_layers=runs, num_attention_heads=z["width"] // 128, num_key_value_heads=8,
+                    head_dim=128, intermediate_size=z["ff"], vocab_size=32768, rms_norm_eps=1e-6, rope_theta=1e6,
+                    msa_config=dict(router_layer_idx="999", pooling_kernel_size=64, top_k_docs=2, head_reduce_method="mean",
+                                    query_reduce_method="max", chunk_reduce_method="max", decouple_router=False,
+                                    decouple_pooling_mode="mean", aux_loss=False, aux_loss_method="INFONCE", rewrite_position=False))
+    with torch.device(dev):
+        model = MSAForCausalLM(cfg).to(torch.bfloat16).eval()
+    n_seq, t = 4, 2048
+    ids = torch.randint(0, 32768, (1, n_seq * t), device=dev)
+    docs = torch.arange(1, n_seq + 1, device=dev).repeat_interleave(t)[None]
+    pos = torch.arange(t, device=dev).repeat(n_seq)[None]
+    mask = torch.ones_like(ids)
+
+    def prompt():
+        cache = SparseCacheOnCPU()
+        for l in range(runs):
+            cache.record_kwargs(l, {"stage": "prefill_stage1"})
+        with torch.no_grad():
+            model.model(input_ids=ids, attention_mask=mask, position_ids=pos, past_key_values=cache, doc_ids=docs)
+    ms = _time_ms(torch, prompt, max(3, steps // 5), 3)
+    out["prompt_4x2048"] = {"ms": ms, "tokens_per_s": n_seq * t / ms * 1e3}
+    del model
+    torch.cuda.empty_cache()
+    return out
+
+
+def run_hybrid(args):
+    """Prompt and decode throughput of the layered decoder at a few sizes, its kernels one by one, and the memory
+    decoder at equal size.  Prompts: 4 x 2,048 tokens in one step, logits of each last token; decode: one token for every
+    sequence from a full window, CUDA graph, tokens fed back on the device."""
+    import torch
+    from msa_b200 import _cabi_lm as A
+    from msa_b200.cache import PackedStep
+    from msa_b200.hybrid import GraphedDecode
+    torch.cuda.set_device(0)
+    dev, pk = torch.device("cuda", 0), peaks()
+    steps, warmup = max(args.steps, 20), max(args.warmup, 3)
+    sampler = ClockSampler(0)
+    sampler.start()
+    sizes, launches, batches = {}, 0, (1, 32, 128)
+    for name in args.hybrid_sizes.split(","):
+        z = HYBRID_SIZES[name]
+        model = hybrid_model(torch, dev, z)
+        runs = len(model.config.runs())
+        r = {"layer_runs": runs}
+        n_seq, t = 4, 2048
+        cache = model.new_cache(n_seq, t)
+        for i in range(n_seq):
+            cache.acquire(i)
+        ids = torch.randint(0, 32768, (n_seq, t)).tolist()
+        step = PackedStep([(i, ids[i], [t - 1]) for i in range(n_seq)], cache, model.config.windows)
+        l0 = A.launches
+        model.step(step, cache)
+        launches += (A.launches - l0) * (max(3, steps // 2) + 3)
+        ms = _time_ms(torch, lambda: model.step(step, cache), max(3, steps // 2), 3)
+        r["prompt_4x2048"] = {"ms": ms, "tokens_per_s": n_seq * t / ms * 1e3}
+        del cache, step
+        for b in batches:
+            cache = model.new_cache(b, z["window"] + 4 * (steps + warmup) + 64)
+            g = GraphedDecode(model, cache, b)
+            g.tables.fill([1] * b, [z["window"] + 3] * b, list(range(b)))
+            ms = _time_ms(torch, g.replay, steps, warmup)
+            r[f"decode_batch_{b}"] = {"ms_per_step": ms, "tokens_per_s": b / ms * 1e3}
+            model.check_status()
+            del g, cache
+            torch.cuda.empty_cache()
+        r["kernels"] = hybrid_kernels(torch, dev, model, z, pk, 32)
+        del model
+        torch.cuda.empty_cache()
+        r["memory_decoder"] = closest_model(torch, dev, z, runs, batches, steps, warmup)
+        sizes[name] = r
+    closest = closest_kernels(torch, dev, pk)
+    first = sizes[args.hybrid_sizes.split(",")[-1]]
+    print(json.dumps({"metric": "layered decoder prompt tokens/s", "value": first["prompt_4x2048"]["tokens_per_s"], "unit": "tokens/s",
+                      "n_gpus": 1, "steps": steps, "warmup": warmup, "ms_per_step": first["prompt_4x2048"]["ms"], "higher_is_better": True,
+                      "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic, random weights",
+                      "config": {"workload": "hybrid", "sizes": {k: HYBRID_SIZES[k] for k in sizes}, "l2": "kernel legs flush L2"},
+                      "gpu_launches": launches, "clocks": sampler.stop(), "peaks": pk, "results": sizes, "memory_decoder_kernels": closest}))
+
+
 def run_generate(args):
     import torch
     import torch.distributed as dist
@@ -1450,6 +1719,8 @@ if __name__ == "__main__":
         run_reference(a)
     elif a.workload == "generate":
         run_generate(a)
+    elif a.workload == "hybrid":
+        run_hybrid(a)
     elif a.workload != "routing":
         run_secondary(a)
     else:

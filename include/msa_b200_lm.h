@@ -77,6 +77,25 @@ typedef struct {
 } msa_lm_attn_args;
 int msa_lm_window_attn(const msa_lm_attn_args* args, void* stream);
 
+/* The same for a prompt portion on tcgen05 (bf16; dim 64 or 128, rot 0 or 64, vdim 64 or 128).  q rows [n_rows,
+ * heads*(dim+rot)] (row 0 = packed row row0 = cu[seq0]), kv rows [n_ctx, heads*dim keys | heads*vdim values], ctx rows
+ * [n_ctx, rank | rot].  A wait that runs out sets status[0]. */
+int msa_lm_window_attn_tc_supported(int32_t dim, int32_t rot, int32_t vdim);
+int msa_lm_window_attn_tc(const void* q, int64_t q_row, int32_t n_rows, const void* kv, int64_t kv_row, const void* ctx,
+                          int64_t ctx_row, int32_t n_ctx, int32_t heads, int32_t dim, int32_t rot, int32_t vdim,
+                          int32_t rank, const int32_t* start, const int32_t* cu, const int32_t* ctx_off, int32_t seq0,
+                          int32_t seq1, int32_t row0, int32_t max_len, int32_t window, float scale, void* out,
+                          int64_t out_row, int32_t* status, void* stream);
+
+/* Decode attention over the rings on tensor cores (bf16; rank a multiple of 128 up to 512, rot 0, 32 or 64): sequence i
+ * of n at position pos[i] attends with qa [n, heads, rank] and qb [n, heads, rot] (row / head strides) to its ring's
+ * visible rows; out [n, heads, rank].  splits > 1: part_o [n, heads, splits, rank], part_ml [n, heads, splits, 2] fp32. */
+int msa_lm_latent_decode_supported(int32_t rank, int32_t rot);
+int msa_lm_latent_decode(const void* qa, int64_t qa_row, int64_t qa_head, const void* qb, int64_t qb_row, int64_t qb_head,
+                         const void* ring, int64_t ring_rows, const int32_t* slot, const int32_t* pos, int32_t n,
+                         int32_t heads, int32_t rank, int32_t rot, int32_t window, int32_t splits, float scale, void* out,
+                         float* part_o, float* part_ml, void* stream);
+
 /* ---- gated delta rule ---------------------------------------------------------------------------------------------
  * proj row = [kv_heads*dim q | kv_heads*dim k | heads*vdim v | heads*vdim gate | heads beta | heads decay].
  * Convolution weights conv_w [2*kv_heads*dim + heads*vdim, taps] fp32.  Conv state [slots, 2, taps-1, channels] in dtype:
@@ -121,6 +140,12 @@ int msa_lm_moe_sort(const int32_t* idx, int32_t n_rows, int32_t top, int32_t exp
 int msa_lm_moe_gemm(const void* x, int64_t x_stride, const int32_t* src, const void* w, const int32_t* off,
                     const int32_t* tiles, int32_t max_tiles, int32_t n_out, int32_t k, int32_t act, float limit, void* out,
                     int64_t out_stride, int32_t out_dtype, int32_t dtype, void* stream);
+
+/* The same on tcgen05 (bf16; tiles of msa_lm_moe_sort with tile_rows = 128; k, output columns and strides multiples of 8):
+ * x has x_rows rows, out is bf16.  A wait that runs out sets status[0]. */
+int msa_lm_moe_gemm_tc(const void* x, int64_t x_stride, int32_t x_rows, const int32_t* src, const void* w, int32_t experts,
+                       const int32_t* off, const int32_t* tiles, int32_t max_tiles, int32_t n_out, int32_t k, int32_t act,
+                       float limit, void* out, int64_t out_stride, int32_t* status, void* stream);
 
 #ifdef __cplusplus
 }

@@ -66,6 +66,81 @@ delta_prep_kernel(const msa_lm_delta_args a, float* __restrict__ qk, float* __re
   }
 }
 
+// The same with four channels per lane and the convolution's history in registers: a warp walks 16 rows of one unit (a
+// head of q or k, or 128 channels of v), so every input is loaded once.
+constexpr int kPrepRows = 16;
+
+template <typename T> __device__ __forceinline__ float silu_act(float z) { return silu_f(z); }
+template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256)
+delta_prep_vec_kernel(const msa_lm_delta_args a, float* __restrict__ qk, float* __restrict__ v, float* __restrict__ gates) {
+  const DeltaLayout L(a);
+  const int row0 = blockIdx.x * kPrepRows, n_rows = a.n_tok - a.n_decode;
+  const int row1 = min(row0 + kPrepRows, n_rows);
+  const T* proj = reinterpret_cast<const T*>(a.proj);
+  if (blockIdx.y == 0) {
+    for (int i = threadIdx.x; i < (row1 - row0) * a.heads; i += 256) {
+      const int row = row0 + i / a.heads, h = i % a.heads;
+      const T* g = proj + (long long)(a.n_decode + row) * a.proj_stride + 2 * L.nqk + 2 * L.nv;
+      gates[(long long)row * 2 * a.heads + h] = -expf(a.a_log[h]) * softplus_f(to_f(g[a.heads + h]) + a.dt_bias[h]);
+      gates[(long long)row * 2 * a.heads + a.heads + h] = sigmoid_f(to_f(g[h]));
+    }
+  }
+  const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const bool is_v = unit >= 2 * a.kv_heads;
+  const int c0 = is_v ? (unit - 2 * a.kv_heads) * 128 + lane * 4 : lane * 4;          // within v, or within the head
+  if (is_v ? (unit - 2 * a.kv_heads) * 128 >= L.nv : false) return;
+  const bool on = is_v ? c0 < L.nv : c0 < a.dim;
+  const int c = is_v ? 2 * L.nqk + c0 : unit * a.dim + c0;
+  float w[TAPS][4];
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) w[j][e] = on ? a.conv_w[(long long)(c + e) * TAPS + j] : 0.f;
+  const float post = unit < a.kv_heads ? 1.f / sqrtf((float)a.dim) : 1.f;
+  float4 hist[TAPS];      // hist[j] = input `TAPS - 1 - j` tokens back
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) hist[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int row = row0; row < row1; ++row) {
+    const long long n = (long long)a.n_decode + row;
+    const int s = a.tok_seq[n], t = (int)(n - a.cu[s]);
+    if (row == row0 || t == 0) {
+      const int p0 = a.start[s];
+      const T* half = conv_half<T>(a, L.chan, a.slot[s], p0);
+#pragma unroll
+      for (int j = 1; j < TAPS; ++j) {                  // what the shift below turns into lags TAPS-1 .. 1
+        const int lag = TAPS - j;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (on) {
+          if (t - lag >= 0) x = load4(proj + (n - lag) * a.proj_stride + c);
+          else if (p0 + t - lag >= 0) x = load4(half + (long long)(TAPS - 1 + t - lag) * L.chan + c);
+        }
+        hist[j] = x;
+      }
+    }
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; ++j) hist[j] = hist[j + 1];
+    hist[TAPS - 1] = on ? load4(proj + n * a.proj_stride + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    float y[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      y[0] = fmaf(w[j][0], hist[j].x, y[0]); y[1] = fmaf(w[j][1], hist[j].y, y[1]);
+      y[2] = fmaf(w[j][2], hist[j].z, y[2]); y[3] = fmaf(w[j][3], hist[j].w, y[3]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) y[e] = silu_act<T>(y[e]);
+    if (is_v) {
+      if (on) store4(v + (long long)row * L.nv + c0, make_float4(y[0], y[1], y[2], y[3]));
+    } else {
+      const float ss = warp_sum_f(on ? y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3] : 0.f);
+      const float sc = post / sqrtf(ss + 1e-6f);
+      if (on) store4(qk + (long long)row * 2 * L.nqk + (long long)unit * a.dim + c0, make_float4(y[0] * sc, y[1] * sc, y[2] * sc, y[3] * sc));
+    }
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) delta_conv_store_kernel(const msa_lm_delta_args a) {
   const DeltaLayout L(a);
@@ -172,7 +247,7 @@ delta_scan_kernel(const msa_lm_delta_args a, const float* __restrict__ qk, const
 // out = o / rms(o) * w * silu(gate); one warp per (row, head).
 template <typename T>
 __global__ void __launch_bounds__(256)
-delta_out_kernel(const msa_lm_delta_args a, const float* __restrict__ o, T* __restrict__ out, long long out_stride, long long n) {
+delta_out_kernel(const msa_lm_delta_args a, const float* __restrict__ o, T* __restrict__ out, long long out_stride, long long n, bool vec) {
   const DeltaLayout L(a);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * 8 + warp;
@@ -182,6 +257,17 @@ delta_out_kernel(const msa_lm_delta_args a, const float* __restrict__ o, T* __re
   const float* src = o + row * L.nv + (long long)h * a.vdim;
   const T* gate = reinterpret_cast<const T*>(a.proj) + (a.n_decode + row) * a.proj_stride + 2 * L.nqk + L.nv + (long long)h * a.vdim;
   float ss = 0.f;
+  if (vec) {
+    for (int i = lane * 4; i < a.vdim; i += 128) { const float4 x = load4(src + i); ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w; }
+    const float inv = 1.f / sqrtf(warp_sum_f(ss) / (float)a.vdim + a.eps);
+    for (int i = lane * 4; i < a.vdim; i += 128) {
+      const float4 x = load4(src + i), w = load4(a.w_norm + i), z = load4(gate + i);
+      store4(out + row * out_stride + (long long)h * a.vdim + i,
+             make_float4(x.x * inv * w.x * silu_act<T>(z.x), x.y * inv * w.y * silu_act<T>(z.y), x.z * inv * w.z * silu_act<T>(z.z),
+                         x.w * inv * w.w * silu_act<T>(z.w)));
+    }
+    return;
+  }
   for (int i = lane; i < a.vdim; i += 32) ss += src[i] * src[i];
   const float inv = 1.f / sqrtf(warp_sum_f(ss) / (float)a.vdim + a.eps);
   for (int i = lane; i < a.vdim; i += 32)
@@ -349,6 +435,23 @@ extern "C" int msa_lm_delta_prep(const msa_lm_delta_args* a, float* qk, float* v
   MSA_REQUIRE(qk && v && gates, "delta_prep: null output");
   const int rows = a->n_tok - a->n_decode;
   if (rows == 0) return MSA_OK;
+  const DeltaLayout L(*a);
+  const int e4 = 4 * (int)dtype_size(a->dtype);
+  const bool vec = a->taps >= 2 && a->taps <= 4 && a->dim % 4 == 0 && a->dim <= 128 && a->vdim % 4 == 0 && a->proj_stride % 4 == 0 &&
+                   reinterpret_cast<uintptr_t>(a->proj) % e4 == 0 && reinterpret_cast<uintptr_t>(a->conv_state) % e4 == 0 &&
+                   aligned16(qk) && aligned16(v);
+  if (vec) {
+    const int units = 2 * a->kv_heads + (L.nv + 127) / 128;
+    const dim3 grid((unsigned)((rows + kPrepRows - 1) / kPrepRows), (unsigned)((units + 7) / 8));
+    cudaStream_t st = (cudaStream_t)stream;
+    MSA_LM_DISPATCH(a->dtype, {
+      if (a->taps == 2) delta_prep_vec_kernel<T, 2><<<grid, 256, 0, st>>>(*a, qk, v, gates);
+      else if (a->taps == 3) delta_prep_vec_kernel<T, 3><<<grid, 256, 0, st>>>(*a, qk, v, gates);
+      else delta_prep_vec_kernel<T, 4><<<grid, 256, 0, st>>>(*a, qk, v, gates);
+    });
+    MSA_LAUNCH_OK("delta_prep_vec_kernel");
+    return MSA_OK;
+  }
   MSA_LM_DISPATCH(a->dtype, { delta_prep_kernel<T><<<rows, 256, 0, (cudaStream_t)stream>>>(*a, qk, v, gates); });
   MSA_LAUNCH_OK("delta_prep_kernel");
   return MSA_OK;
@@ -387,7 +490,11 @@ extern "C" int msa_lm_delta_out(const msa_lm_delta_args* a, const float* o, void
   if (rows == 0) return MSA_OK;
   const long long blocks = (rows * a->heads + 7) / 8;
   MSA_LM_DISPATCH(a->dtype, {
-    delta_out_kernel<T><<<(unsigned)blocks, 256, 0, (cudaStream_t)stream>>>(*a, o, (T*)out, out_stride, rows);
+    const int e4 = 4 * (int)sizeof(T);
+    const bool vec = a->vdim % 4 == 0 && a->proj_stride % 4 == 0 && out_stride % 4 == 0 && aligned16(o) && aligned16(a->w_norm) &&
+                     reinterpret_cast<uintptr_t>(a->proj) % e4 == 0 && reinterpret_cast<uintptr_t>(out) % e4 == 0 &&
+                     (2 * a->kv_heads * a->dim) % 4 == 0;
+    delta_out_kernel<T><<<(unsigned)blocks, 256, 0, (cudaStream_t)stream>>>(*a, o, (T*)out, out_stride, rows, vec);
   });
   MSA_LAUNCH_OK("delta_out_kernel");
   return MSA_OK;

@@ -18,19 +18,11 @@ struct LatentPrepParams {
   void* ring; long long ring_rows; void* ctx;
 };
 
-template <typename T>
-__device__ __forceinline__ void rotate_pair(T* p, int i, float angle) {
-  float s, c;
-  sincosf(angle, &s, &c);
-  const float u = to_f(p[2 * i]), v = to_f(p[2 * i + 1]);
-  p[2 * i] = from_f<T>(u * c - v * s);
-  p[2 * i + 1] = from_f<T>(v * c + u * s);
-}
-
 // Blocks 0 .. n_tok-1: one token each; the blocks after them: one old ring row each.
 template <typename T>
 __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams p) {
   __shared__ float s_part[32];
+  extern __shared__ float2 s_turn[];       // cosine and sine of the token's angles
   const int width = p.rank + p.rot;
   if ((int)blockIdx.x >= p.n_tok) {
     const int o = (int)blockIdx.x - p.n_tok;
@@ -45,9 +37,19 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
   const int n = blockIdx.x, s = p.tok_seq[n], pos = p.pos[n];
   T* row = reinterpret_cast<T*>(p.proj) + (long long)n * p.proj_stride;
   const int hd = p.dim + p.rot, half = p.rot / 2;
+  for (int j = threadIdx.x; j < half; j += blockDim.x) {
+    float sn, cs;
+    sincosf((float)pos * p.inv_freq[j], &sn, &cs);
+    s_turn[j] = make_float2(cs, sn);
+  }
+  __syncthreads();
   for (int i = threadIdx.x; i < p.heads * half; i += blockDim.x) {
-    const int h = i / half, j = i % half;
-    rotate_pair(row + h * hd + p.dim, j, (float)pos * p.inv_freq[j]);
+    const int h = i / half, j = i - h * half;
+    T* q = row + h * hd + p.dim + 2 * j;
+    const float2 cs = s_turn[j];
+    const float u = to_f(q[0]), v = to_f(q[1]);
+    q[0] = from_f<T>(u * cs.x - v * cs.y);
+    q[1] = from_f<T>(v * cs.x + u * cs.y);
   }
   T* lat = row + p.heads * hd;
   T* dst;
@@ -62,11 +64,10 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
   const float inv = 1.f / sqrtf(block_sum(ss, s_part) / (float)p.rank + p.eps);
   for (int i = threadIdx.x; i < p.rank; i += blockDim.x) dst[i] = from_f<T>(to_f(lat[i]) * inv * p.w_norm[i]);
   for (int j = threadIdx.x; j < half; j += blockDim.x) {
-    float sn, cs;
-    sincosf((float)pos * p.inv_freq[j], &sn, &cs);
+    const float2 cs = s_turn[j];
     const float u = to_f(lat[p.rank + 2 * j]), v = to_f(lat[p.rank + 2 * j + 1]);
-    dst[p.rank + 2 * j] = from_f<T>(u * cs - v * sn);
-    dst[p.rank + 2 * j + 1] = from_f<T>(v * cs + u * sn);
+    dst[p.rank + 2 * j] = from_f<T>(u * cs.x - v * cs.y);
+    dst[p.rank + 2 * j + 1] = from_f<T>(v * cs.x + u * cs.y);
   }
 }
 
@@ -180,14 +181,14 @@ extern "C" int msa_lm_latent_prep(void* proj, int64_t proj_stride, const float* 
                                   int32_t n_decode, int32_t n_old, int32_t window, void* ring, int64_t ring_rows, void* ctx,
                                   int32_t dtype, void* stream) {
   MSA_REQUIRE(dtype_ok(dtype) && proj && w_norm && pos && tok_seq && slot && start && cu && ring, "latent_prep: null pointer");
-  MSA_REQUIRE(heads > 0 && dim >= 0 && rot >= 0 && rot % 2 == 0 && rank > 0 && window > 0, "latent_prep: bad sizes");
+  MSA_REQUIRE(heads > 0 && dim >= 0 && rot >= 0 && rot <= 4096 && rot % 2 == 0 && rank > 0 && window > 0, "latent_prep: bad sizes");
   MSA_REQUIRE(rot == 0 || inv_freq, "latent_prep: inv_freq missing");
   MSA_REQUIRE(ring_rows >= 1 && n_decode >= 0 && n_decode <= n_seq && n_tok >= n_decode && n_old >= 0, "latent_prep: bad counts");
   MSA_REQUIRE(n_seq == n_decode || (ctx && ctx_off && old_off), "latent_prep: portions need a context");
   if (n_tok == 0) return MSA_OK;
   LatentPrepParams p{proj, proj_stride, w_norm, eps, inv_freq, heads, dim, rot, rank, pos, tok_seq, slot, start, cu, ctx_off,
                      old_off, n_tok, n_seq, n_decode, window, ring, ring_rows, ctx};
-  MSA_LM_DISPATCH(dtype, { latent_prep_kernel<T><<<n_tok + n_old, 128, 0, (cudaStream_t)stream>>>(p); });
+  MSA_LM_DISPATCH(dtype, { latent_prep_kernel<T><<<n_tok + n_old, 128, (size_t)rot * 4, (cudaStream_t)stream>>>(p); });
   MSA_LAUNCH_OK("latent_prep_kernel");
   return MSA_OK;
 }

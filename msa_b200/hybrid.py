@@ -27,7 +27,11 @@ class Weights:
     """Checkpoint tensors by name; every tensor must be taken exactly once."""
 
     def __init__(self, tensors: Dict[str, torch.Tensor], device, dtype: torch.dtype):
-        self._t, self._left, self.device, self.dtype = tensors, set(tensors), device, dtype
+        self._t, self._left, self.device, self.dtype = tensors, set(tensors), torch.device(device), dtype
+        self.status = torch.zeros(4, dtype=torch.int32, device=device)     # shared by the kernels that report
+
+    def has(self, name: str) -> bool:
+        return name in self._t
 
     def raw(self, name: str, *shape: int) -> torch.Tensor:
         if name not in self._t:
@@ -44,9 +48,13 @@ class Weights:
     def vector(self, name: str, *shape: int) -> torch.Tensor:
         return self.raw(name, *shape).to(device=self.device, dtype=torch.float32).contiguous()
 
-    def stack(self, names_rows, cols: int) -> torch.Tensor:
-        """Matrices with a common input, stacked by output rows: one product instead of several."""
-        return torch.cat([self.raw(n, r, cols) for n, r in names_rows]).to(device=self.device, dtype=self.dtype).contiguous()
+    def stack(self, names_rows, cols: int, pad: bool = False) -> torch.Tensor:
+        """Matrices with a common input, stacked by output rows: one product instead of several.  ``pad``: zero rows up to
+        a multiple of 8, so that every row of the product starts on a 16-byte boundary."""
+        m = torch.cat([self.raw(n, r, cols) for n, r in names_rows])
+        if pad and m.shape[0] % 8:
+            m = torch.cat([m, m.new_zeros((-m.shape[0] % 8, cols))])
+        return m.to(device=self.device, dtype=self.dtype).contiguous()
 
     def check_all_used(self) -> None:
         if self._left:
@@ -59,8 +67,9 @@ class LatentAttention:
 
     def __init__(self, spec, w: Weights, prefix: str, width: int, eps: float):
         s = self.spec = spec
-        self.eps = eps
-        self.w_in = w.stack([(prefix + "q", s.heads * (s.dim + s.rot_dim)), (prefix + "dkv", s.kv_rank + s.rot_dim)], width)
+        self.eps, self.status = eps, w.status
+        self.tc_prompt, self.tc_decode = K.window_attn_tc_supported(s, w.dtype), K.latent_decode_supported(s, w.dtype)
+        self.w_in = w.stack([(prefix + "q", s.heads * (s.dim + s.rot_dim)), (prefix + "dkv", s.kv_rank + s.rot_dim)], width, pad=True)
         self.norm = w.vector(prefix + "dkv.norm", s.kv_rank)
         self.w_kv = w.stack([(prefix + "uk", s.heads * s.dim), (prefix + "uv", s.heads * s.vdim)], s.kv_rank)
         self.w_uk = self.w_kv[:s.heads * s.dim].view(s.heads, s.dim, s.kv_rank)
@@ -84,6 +93,10 @@ class LatentAttention:
             self._decode(q[:nd], step, view, ring, out[:nd])
         if n > nd:
             kv = K.matmul(ctx[:, :s.kv_rank], self.w_kv)
+            if self.tc_prompt:
+                K.window_attn_tc(proj[nd:], kv, ctx, s, out[nd:], step, view, self.status)
+                K.ring_store(ctx, step, view, ring)
+                return out
             k = kv[:, :s.heads * s.dim].view(-1, s.heads, s.dim)
             v = kv[:, s.heads * s.dim:].view(-1, s.heads, s.vdim)
             kr = ctx[:, s.kv_rank:].unsqueeze(1) if s.rot_dim else None
@@ -96,6 +109,13 @@ class LatentAttention:
 
     def _decode(self, q, step, view, ring, out) -> None:
         s, n = self.spec, q.shape[0]
+        if self.tc_decode:
+            qa = torch.bmm(q[..., :s.dim].transpose(0, 1), self.w_uk)                     # [heads, n, rank]
+            lat = torch.empty((n, s.heads, s.kv_rank), dtype=q.dtype, device=q.device)
+            K.latent_decode(qa.transpose(0, 1), q[..., s.dim:] if s.rot_dim else None, ring, step.slot, step.start, lat,
+                            window=view.window, scale=s.scale)
+            out.view(n, s.heads, s.vdim).copy_(torch.bmm(lat.transpose(0, 1), self.w_uv.transpose(1, 2)).transpose(0, 1))
+            return
         f32 = dict(out_dtype=torch.float32) if q.dtype != torch.float32 else {}
         qa = torch.bmm(q[..., :s.dim].transpose(0, 1), self.w_uk, **f32)                  # [heads, n, rank]
         lat = torch.empty((n, s.heads, s.kv_rank), dtype=q.dtype, device=q.device)
@@ -112,10 +132,10 @@ class GatedDelta:
 
     def __init__(self, spec, w: Weights, prefix: str, width: int, eps: float):
         s = self.spec = spec
-        self.eps = eps
+        self.eps, self.status = eps, w.status
         qk, v = s.kv_heads * s.dim, s.heads * s.vdim
         self.w_in = w.stack([(prefix + "q", qk), (prefix + "k", qk), (prefix + "v", v), (prefix + "g", v),
-                             (prefix + "b", s.heads), (prefix + "a", s.heads)], width)
+                             (prefix + "b", s.heads), (prefix + "a", s.heads)], width, pad=True)
         self.conv = torch.cat([w.vector(prefix + n + ".conv", r, s.taps) for n, r in (("q", qk), ("k", qk), ("v", v))]).contiguous()
         self.a_log, self.dt_bias = w.vector(prefix + "A_log", s.heads), w.vector(prefix + "dt_bias", s.heads)
         self.norm = w.vector(prefix + "norm", s.vdim)
@@ -127,7 +147,7 @@ class GatedDelta:
         return RecurrentSpec(s.heads, s.dim, s.vdim, s.channels, s.taps)
 
     def mix(self, proj: torch.Tensor, step, cache: SequenceStateCache, run: int) -> torch.Tensor:
-        return K.delta_mix(proj, self.spec, self, cache.conv[run], cache.state[run], self.eps, step)
+        return K.delta_mix(proj, self.spec, self, cache.conv[run], cache.state[run], self.eps, step, self.status)
 
 
 class DenseFeedForward:
@@ -148,6 +168,7 @@ class MixtureFeedForward:
         self.router = w.matrix(prefix + "router", s.experts, width)
         self.bias = w.vector(prefix + "router.b", s.experts)
         dev, dt = w.device, w.dtype
+        self.status, self.tc = w.status, K.moe_tc_supported(dt, width, s.ff)
         self.w_gate_up = torch.empty((s.experts, 2 * s.ff, width), dtype=dt, device=dev)
         self.w_down = torch.empty((s.experts, width, s.ff), dtype=dt, device=dev)
         for e in range(s.experts):
@@ -159,6 +180,11 @@ class MixtureFeedForward:
     def branch(self, h: torch.Tensor) -> dict:
         s, n = self.spec, h.shape[0]
         idx, mix = K.moe_topk(K.matmul(h, self.router, torch.float32), self.bias, s.top)
+        if self.tc:
+            src, inv, off, tiles = K.moe_sort(idx, s.experts, K.MOE_TC_TILE_ROWS)
+            act = K.moe_gemm_tc(h, src, self.w_gate_up, off, tiles, entries=n * s.top, act=True, limit=s.limit, status=self.status)
+            return dict(y=K.moe_gemm_tc(act, None, self.w_down, off, tiles, entries=n * s.top, act=False, status=self.status),
+                        inv=inv, mix=mix)
         src, inv, off, tiles = K.moe_sort(idx, s.experts)
         act = K.moe_gemm(h, src, self.w_gate_up, off, tiles, entries=n * s.top, act=True, limit=s.limit)
         y = K.moe_gemm(act, None, self.w_down, off, tiles, entries=n * s.top, act=False)
@@ -172,10 +198,11 @@ FEED_FORWARDS = {"dense": DenseFeedForward, "moe": MixtureFeedForward}
 class HybridForCausalLM:
     """Weights, layer runs and the packed step."""
 
-    def __init__(self, config: HybridConfig, tensors: Dict[str, torch.Tensor], device, dtype: torch.dtype = torch.bfloat16):
+    def __init__(self, config: HybridConfig, tensors, device, dtype: torch.dtype = torch.bfloat16):
+        """``tensors``: the checkpoint's tensors by name, or a ``Weights`` that hands them out."""
         self.config, self.device, self.dtype = config, torch.device(device), dtype
         torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False     # 32-bit accumulation throughout
-        w = Weights(tensors, self.device, dtype)
+        w = tensors if isinstance(tensors, Weights) else Weights(tensors, self.device, dtype)
         c, width = config, config.width
         self.embed = w.matrix("embed", c.vocab, width)
         self.final_norm = w.vector("final.norm", width)
@@ -191,11 +218,11 @@ class HybridForCausalLM:
             if spec.mlp is not None:
                 layer.ff = FEED_FORWARDS[spec.mlp.kind](spec.mlp, w, p + "mlp.", width)
                 layer.norm2, layer.norm2b = w.vector(p + "norm2", width), w.vector(p + "norm2b", width)
-            elif p + "norm2" in tensors:       # a layer without a feed-forward has no use for its norms
+            elif w.has(p + "norm2"):       # a layer without a feed-forward has no use for its norms
                 w.vector(p + "norm2", width), w.vector(p + "norm2b", width)
             self.layers.append(layer)
         w.check_all_used()
-        self.status = torch.zeros(4, dtype=torch.int32, device=self.device)
+        self.status = w.status
         self._program = self._compile()
         self.on_layer = None       # hook(run, x): the stream after every layer run (debugging)
 

@@ -101,6 +101,44 @@ def window_attn(qa, qb, ka, kb, v, out, *, scale, window, start, cu, seq0, seq1,
     A.call("msa_lm_window_attn", C.byref(args), A.stream_ptr(qa.device))
 
 
+def window_attn_tc_supported(spec, dtype) -> bool:
+    return (dtype == torch.bfloat16 and spec.kv_rank % 8 == 0 and spec.scale > 0
+            and bool(A.lib().msa_lm_window_attn_tc_supported(spec.dim, spec.rot_dim, spec.vdim)))
+
+
+def window_attn_tc(proj, kv, ctx, spec, out, step, view, status):
+    """The portions of a step on the tensor cores: ``proj`` / ``out`` from the first portion row on."""
+    A.call("msa_lm_window_attn_tc", A.ptr(proj), _rows(proj), proj.shape[0], A.ptr(kv), _rows(kv), A.ptr(ctx), _rows(ctx),
+           ctx.shape[0], spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank, A.ptr(step.start), A.ptr(step.cu),
+           A.ptr(view.ctx_off), step.n_decode, step.n_seq, step.n_decode, step.max_len, view.window, float(spec.scale),
+           A.ptr(out), _rows(out), A.ptr(status), A.stream_ptr(proj.device))
+
+
+def latent_decode_supported(spec, dtype) -> bool:
+    return (dtype == torch.bfloat16 and spec.dim % 8 == 0
+            and bool(A.lib().msa_lm_latent_decode_supported(spec.kv_rank, spec.rot_dim)))
+
+
+def latent_decode_splits(n: int, heads: int, ring_rows: int, n_sm: int = 148) -> int:
+    """CTAs per sequence and head group: fill the GPU once, at least two 64-row tiles each."""
+    groups = (heads + 31) // 32 if heads > 16 else 1
+    return max(1, min(n_sm // max(n * groups, 1), (ring_rows + 127) // 128, 64))
+
+
+def latent_decode(qa, qb, ring, slot, pos, out, *, window, scale):
+    """``qa`` / ``qb`` / ``out`` ``[n, heads, d]`` views, ``ring`` ``[slots, rows, rank + rot]``."""
+    n, heads, rank = qa.shape
+    rot = 0 if qb is None else qb.shape[2]
+    splits = latent_decode_splits(n, heads, ring.shape[1])
+    part_o = part_ml = None
+    if splits > 1:
+        f = dict(dtype=torch.float32, device=qa.device)
+        part_o, part_ml = torch.empty((n, heads, splits, rank), **f), torch.empty((n, heads, splits, 2), **f)
+    A.call("msa_lm_latent_decode", A.ptr(qa), qa.stride(0), qa.stride(1), A.ptr(qb), 0 if qb is None else qb.stride(0),
+           0 if qb is None else qb.stride(1), A.ptr(ring), ring.shape[1], A.ptr(slot), A.ptr(pos), n, heads, rank, rot, window,
+           splits, float(scale), A.ptr(out), A.ptr(part_o), A.ptr(part_ml), A.stream_ptr(qa.device))
+
+
 # ---------------------------------------------------------------------------------------------- gated delta rule
 def delta_args(proj, spec, w, conv_state, state, eps, step) -> A.DeltaArgs:
     return A.DeltaArgs(proj=A.ptr(proj), proj_stride=_rows(proj), conv_w=A.ptr(w.conv), a_log=A.ptr(w.a_log),
@@ -111,7 +149,12 @@ def delta_args(proj, spec, w, conv_state, state, eps, step) -> A.DeltaArgs:
                        dtype=A.dtype_code(proj.dtype))
 
 
-def delta_mix(proj, spec, w, conv_state, state, eps, step) -> torch.Tensor:
+def delta_recurrence(args, qk, v, gates, o, status) -> None:
+    """The recurrence over the portions of a step."""
+    A.call("msa_lm_delta_scan", C.byref(args), A.ptr(qk), A.ptr(v), A.ptr(gates), A.ptr(o), A.stream_ptr(qk.device))
+
+
+def delta_mix(proj, spec, w, conv_state, state, eps, step, status) -> torch.Tensor:
     """From the projections to the input of the output product, ``[n_tok, heads*vdim]``; advances the states."""
     args = delta_args(proj, spec, w, conv_state, state, eps, step)
     dev, st = proj.device, A.stream_ptr(proj.device)
@@ -127,7 +170,7 @@ def delta_mix(proj, spec, w, conv_state, state, eps, step) -> torch.Tensor:
         o = torch.empty((rows, spec.heads * spec.vdim), **f)
         A.call("msa_lm_delta_prep", C.byref(args), A.ptr(qk), A.ptr(v), A.ptr(gates), st)
         A.call("msa_lm_delta_conv_store", C.byref(args), st)
-        A.call("msa_lm_delta_scan", C.byref(args), A.ptr(qk), A.ptr(v), A.ptr(gates), A.ptr(o), st)
+        delta_recurrence(args, qk, v, gates, o, status)
         tail = out[step.n_decode:]
         A.call("msa_lm_delta_out", C.byref(args), A.ptr(o), A.ptr(tail), _rows(tail), st)
     return out
@@ -166,4 +209,19 @@ def moe_gemm(x, src, w, off, tiles, *, entries, act, limit=0.0, out_dtype=None):
     A.call("msa_lm_moe_gemm", A.ptr(x), _rows(x), A.ptr(src), A.ptr(w), A.ptr(off), A.ptr(tiles), tiles.shape[0], n_out, k,
            1 if act else 0, float(limit), A.ptr(out), _rows(out), A.dtype_code(out.dtype), A.dtype_code(x.dtype),
            A.stream_ptr(x.device))
+    return out
+
+
+MOE_TC_TILE_ROWS = 128
+
+
+def moe_tc_supported(dtype, width, ff) -> bool:
+    return dtype == torch.bfloat16 and width % 8 == 0 and ff % 8 == 0
+
+
+def moe_gemm_tc(x, src, w, off, tiles, *, entries, act, limit=0.0, status):
+    experts, n_out, k = w.shape
+    out = torch.empty((entries, n_out // 2 if act else n_out), dtype=x.dtype, device=x.device)
+    A.call("msa_lm_moe_gemm_tc", A.ptr(x), _rows(x), x.shape[0], A.ptr(src), A.ptr(w), experts, A.ptr(off), A.ptr(tiles),
+           tiles.shape[0], n_out, k, 1 if act else 0, float(limit), A.ptr(out), _rows(out), A.ptr(status), A.stream_ptr(x.device))
     return out

@@ -133,6 +133,8 @@ def model_weights(name, seed, dtype):
         for k in w:
             if k.endswith("router.b"):
                 w[k] = w[k] * 6
+            elif k.endswith("mlp.router"):
+                w[k] = w[k] * 0.25
     return w
 
 
