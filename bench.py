@@ -1498,12 +1498,15 @@ def hybrid_kernels(torch, dev, model, z, pk, decode_b):
     projd = K.matmul(h, dlt.w_in)
     args = K.delta_args(projd, d, dlt, cache.conv[0], cache.state[0], 1e-5, step)
     f32 = dict(dtype=torch.float32, device=dev)
-    qk, v, gates, o = (torch.empty((n, c), **f32) for c in (2 * d.kv_heads * d.dim, heads * d.vdim, 2 * heads, heads * d.vdim))
-    outd, st = torch.empty((n, heads * d.vdim), **bf), A.stream_ptr(dev)
+    v, gates = torch.empty((n, heads * d.vdim), **f32), torch.empty((n, 2 * heads), **f32)
+    qk, outd, st = torch.empty((n, 4 * d.kv_heads * d.dim), **bf), torch.empty((n, heads * d.vdim), **bf), A.stream_ptr(dev)
     p = A.ptr
-    leg("delta_prep", lambda: A.call("msa_lm_delta_prep", ctypes.byref(args), p(qk), p(v), p(gates), st), 0, n * d.channels * 6)
-    leg("delta_scan", lambda: K.delta_recurrence(args, qk, v, gates, o, model.status), n * heads * d.dim * d.vdim * 6.0, n * 4 * (d.channels + heads * d.vdim))
-    leg("delta_out", lambda: A.call("msa_lm_delta_out", ctypes.byref(args), p(o), p(outd), outd.stride(0), st), 0, n * heads * d.vdim * 8)
+    leg("delta_prep", lambda: A.call("msa_lm_delta_prep_split", ctypes.byref(args), p(qk), p(v), p(gates), st), 0, n * d.channels * 6)
+    # flops of the chunked form, once each: S products, the triangular ones at half
+    c = 64
+    macs = n * heads * (3 * d.dim * d.vdim + c * d.vdim) + n * d.kv_heads * c * d.dim + n * heads * c * c / 6
+    leg("delta_chunk + delta_state", lambda: K.delta_chunks(args, d, step, qk, v, gates, outd), 2.0 * macs,
+        n * (d.kv_heads * d.dim * 8 + heads * d.vdim * (4 + 2 + 2)) + n_seq * heads * d.dim * d.vdim * 4)
     m = moe.spec
     logits = K.matmul(h, moe.router, torch.float32)
     leg("moe_topk", lambda: K.moe_topk(logits, moe.bias, m.top), 0, n * m.experts * 4)
@@ -1512,7 +1515,9 @@ def hybrid_kernels(torch, dev, model, z, pk, decode_b):
     src, inv, off, tiles = K.moe_sort(idx, m.experts, 128)
     ent = n * m.top
     act = K.moe_gemm_tc(h, src, moe.w_gate_up, off, tiles, entries=ent, act=True, limit=7.0, status=model.status)
-    leg("moe_gemm_tc gate/up + activation (prompt)", lambda: K.moe_gemm_tc(h, src, moe.w_gate_up, off, tiles, entries=ent, act=True, limit=7.0, status=model.status),
+    leg("gather_rows", lambda: K.gather_rows(h, src), 0, ent * width * 2 + n * width * 2)
+    hg = K.gather_rows(h, src)
+    leg("moe_gemm_tc gate/up + activation (prompt)", lambda: K.moe_gemm_tc(hg, None, moe.w_gate_up, off, tiles, entries=ent, act=True, limit=7.0, status=model.status),
         2.0 * ent * width * 2 * m.ff, moe.w_gate_up.numel() * 2 + n * width * 2 + ent * m.ff * 2)
     ye = K.moe_gemm_tc(act, None, moe.w_down, off, tiles, entries=ent, act=False, status=model.status)
     leg("moe_gemm_tc down (prompt)", lambda: K.moe_gemm_tc(act, None, moe.w_down, off, tiles, entries=ent, act=False, status=model.status),

@@ -118,6 +118,16 @@ int msa_lm_delta_decode(const msa_lm_delta_args* a, void* out, int64_t out_strid
 /* The other sequences: convolution + silu + unit norms -> qk [rows, 2, kv_heads, dim] fp32 (q scaled by dim^-1/2),
  * v [rows, heads, vdim] fp32, gates [rows, 2, heads] fp32 (log decay, beta); rows count from the first non-decode token. */
 int msa_lm_delta_prep(const msa_lm_delta_args* a, float* qk, float* v, float* gates, void* stream);
+/* The same with q and k as pairs of bf16 numbers: qk [rows, 2 (q, k), 2 (hi, lo), kv_heads, dim] (bf16 activations, 2 to 4
+ * taps, dim <= 128, dim and vdim multiples of 4). */
+int msa_lm_delta_prep_split(const msa_lm_delta_args* a, void* qk, float* v, float* gates, void* stream);
+/* The recurrence in chunks of 64 tokens on tensor cores, from msa_lm_delta_prep_split's outputs, with the gated output norm
+ * -> out (bf16); advances the state.  chunk_off: prefix sums of ceil(tokens / 64) over the non-decode sequences, n_chunks in
+ * all; tile: value columns per CTA (32, 64 or 128, divides vdim); o [rows, heads, vdim] fp32 scratch when tile < vdim. */
+int msa_lm_delta_chunk_supported(int32_t dim, int32_t vdim, int32_t taps);
+int64_t msa_lm_delta_chunk_workspace(int32_t n_chunks, int32_t heads);
+int msa_lm_delta_chunk(const msa_lm_delta_args* a, const void* qk, const float* v, const float* gates, const int32_t* chunk_off,
+                       int32_t n_chunks, int32_t tile, void* workspace, float* o, void* out, int64_t out_stride, void* stream);
 /* Convolution inputs of the last taps-1 positions -> conv_state. */
 int msa_lm_delta_conv_store(const msa_lm_delta_args* a, void* stream);
 /* The recurrence token by token -> o [rows, heads, vdim] fp32; advances the state. */
@@ -131,9 +141,13 @@ int msa_lm_moe_topk(const float* logits, int64_t stride, const float* bias, int3
                     int32_t* idx, float* weight, void* stream);
 /* Groups the n_rows*top choices by expert: src[i] = row of the i-th grouped entry, inv[r*top+k] = its place,
  * off[e] .. off[e+1] the entries of expert e, tiles [max_tiles, 2] = (expert, first entry) of every tile of tile_rows
- * entries (expert -1: unused). */
+ * entries (expert -1: unused).  counts: int32 [ceil(n_rows*top / 2048), experts] lets many choices be sorted by many
+ * blocks (null: one block). */
 int msa_lm_moe_sort(const int32_t* idx, int32_t n_rows, int32_t top, int32_t experts, int32_t tile_rows, int32_t* src,
-                    int32_t* inv, int32_t* off, int32_t* tiles, int32_t max_tiles, void* stream);
+                    int32_t* inv, int32_t* off, int32_t* tiles, int32_t max_tiles, int32_t* counts, void* stream);
+/* out[i] = x[src[i]] (rows of row_bytes, a multiple of 16). */
+int msa_lm_gather_rows(const void* x, int64_t x_stride_bytes, const int32_t* src, int32_t n, int32_t row_bytes, void* out,
+                       void* stream);
 /* Grouped product over the tiles of msa_lm_moe_sort (tile_rows = 32): out[i] = x[src ? src[i] : i] . w[e]^T with
  * w [experts, n_out, k].  act = 1: w holds gate rows then up rows (n_out = 2*ff) and out[i, ff] = g * sigmoid(1.702 g) *
  * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit). */

@@ -13,7 +13,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libmsa_b200_lm.so")
 
 EXPORTS = ["msa_lm_residual_norm", "msa_lm_embed", "msa_lm_silu_mul", "msa_lm_latent_prep", "msa_lm_ring_store",
-           "msa_lm_window_attn", "msa_lm_window_attn_tc_supported", "msa_lm_window_attn_tc", "msa_lm_latent_decode_supported", "msa_lm_latent_decode", "msa_lm_delta_decode", "msa_lm_delta_prep", "msa_lm_delta_conv_store", "msa_lm_delta_scan",
+           "msa_lm_window_attn", "msa_lm_window_attn_tc_supported", "msa_lm_window_attn_tc", "msa_lm_latent_decode_supported", "msa_lm_latent_decode", "msa_lm_delta_decode", "msa_lm_delta_prep", "msa_lm_delta_prep_split", "msa_lm_delta_chunk_supported", "msa_lm_delta_chunk_workspace", "msa_lm_delta_chunk", "msa_lm_gather_rows", "msa_lm_delta_conv_store", "msa_lm_delta_scan",
            "msa_lm_delta_out", "msa_lm_moe_topk", "msa_lm_moe_sort", "msa_lm_moe_gemm", "msa_lm_moe_gemm_tc"]
 
 vp, i32, i64, f32 = C.c_void_p, C.c_int32, C.c_int64, C.c_float
@@ -69,12 +69,17 @@ def lib() -> C.CDLL:
             "msa_lm_delta_scan": [dp, vp, vp, vp, vp, vp],
             "msa_lm_delta_out": [dp, vp, vp, i64, vp],
             "msa_lm_moe_topk": [vp, i64, vp, i32, i32, i32, vp, vp, vp],
-            "msa_lm_moe_sort": [vp, i32, i32, i32, i32, vp, vp, vp, vp, i32, vp],
+            "msa_lm_moe_sort": [vp, i32, i32, i32, i32, vp, vp, vp, vp, i32, vp, vp],
+            "msa_lm_gather_rows": [vp, i64, vp, i32, i32, vp, vp],
+            "msa_lm_delta_prep_split": [dp, vp, vp, vp, vp],
+            "msa_lm_delta_chunk_supported": [i32, i32, i32],
+            "msa_lm_delta_chunk_workspace": [i32, i32],
+            "msa_lm_delta_chunk": [dp, vp, vp, vp, vp, i32, i32, vp, vp, vp, i64, vp],
             "msa_lm_moe_gemm": [vp, i64, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp, i64, i32, i32, vp],
         }
         for name in EXPORTS:
             getattr(l, name).argtypes = sig[name]
-            getattr(l, name).restype = C.c_int
+            getattr(l, name).restype = i64 if name.endswith("_workspace") else C.c_int
         _lib = l
     return _lib
 

@@ -199,8 +199,12 @@ class PackedStep:
                 old.append(old[-1] + o)
                 ctx.append(ctx[-1] + o + cu[k + 1] - cu[k])
             views.append((window, size, ctx, old))
+        chunk_off = [0]                       # chunks of 64 tokens of the portions (the recurrent layers walk those)
+        for k in range(self.n_decode, self.n_seq):
+            chunk_off.append(chunk_off[-1] + (cu[k + 1] - cu[k] + 63) // 64)
+        self.n_chunks = chunk_off[-1]
         # one host-to-device copy for all tables
-        parts = [token, pos, tok_seq, slot, start, cu, want] + [x for v in views for x in v[2:]]
+        parts = [token, pos, tok_seq, slot, start, cu, want, chunk_off] + [x for v in views for x in v[2:]]
         flat = torch.tensor([x for p in parts for x in p], dtype=torch.int32)
         if cache.device.type == "cuda":
             flat = flat.pin_memory()
@@ -209,8 +213,8 @@ class PackedStep:
         for p in parts:
             dev.append(flat[at:at + len(p)])
             at += len(p)
-        self.token, self.pos, self.tok_seq, self.slot, self.start, self.cu, self.want_rows = dev[:7]
-        self.views = {w: ContextView(size, dev[7 + 2 * i], dev[8 + 2 * i], ctx[-1], old[-1])
+        self.token, self.pos, self.tok_seq, self.slot, self.start, self.cu, self.want_rows, self.chunk_off = dev[:8]
+        self.views = {w: ContextView(size, dev[8 + 2 * i], dev[9 + 2 * i], ctx[-1], old[-1])
                       for i, (w, size, ctx, old) in enumerate(views)}
 
     def commit(self, cache: SequenceStateCache) -> None:
@@ -227,7 +231,8 @@ class DecodeStep:
         dev = cache.device
         i = dict(dtype=torch.int32, device=dev)
         self.n_tok = self.n_seq = self.n_decode = n
-        self.max_len = 0
+        self.max_len = self.n_chunks = 0
+        self.chunk_off = None
         self.table = torch.zeros((3, n), **i)
         self.token, self.pos, self.slot = self.table[0], self.table[1], self.table[2]
         self.start = self.pos

@@ -66,77 +66,105 @@ delta_prep_kernel(const msa_lm_delta_args a, float* __restrict__ qk, float* __re
   }
 }
 
-// The same with four channels per lane and the convolution's history in registers: a warp walks 16 rows of one unit (a
+// The same with four channels per lane and the convolution's history in registers: a warp walks 8 rows of one unit (a
 // head of q or k, or 128 channels of v), so every input is loaded once.
-constexpr int kPrepRows = 16;
+constexpr int kPrepRows = 8;
 
 template <typename T> __device__ __forceinline__ float silu_act(float z) { return silu_f(z); }
 template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 
-template <typename T, int TAPS>
+// SPLIT: q and k leave as pairs of bf16 numbers whose sum they are, [rows, 2 (q, k), 2 (hi, lo), kv_heads, dim].
+template <typename T, int TAPS, bool SPLIT>
 __global__ void __launch_bounds__(256)
-delta_prep_vec_kernel(const msa_lm_delta_args a, float* __restrict__ qk, float* __restrict__ v, float* __restrict__ gates) {
+delta_prep_vec_kernel(const msa_lm_delta_args a, void* __restrict__ qk_out, float* __restrict__ v, float* __restrict__ gates) {
   const DeltaLayout L(a);
   const int row0 = blockIdx.x * kPrepRows, n_rows = a.n_tok - a.n_decode;
-  const int row1 = min(row0 + kPrepRows, n_rows);
-  const T* proj = reinterpret_cast<const T*>(a.proj);
+  const int n_here = min(kPrepRows, n_rows - row0);
+  const T* proj = reinterpret_cast<const T*>(a.proj) + ((long long)a.n_decode + row0) * a.proj_stride;   // row 0 of the block
   if (blockIdx.y == 0) {
-    for (int i = threadIdx.x; i < (row1 - row0) * a.heads; i += 256) {
-      const int row = row0 + i / a.heads, h = i % a.heads;
-      const T* g = proj + (long long)(a.n_decode + row) * a.proj_stride + 2 * L.nqk + 2 * L.nv;
-      gates[(long long)row * 2 * a.heads + h] = -expf(a.a_log[h]) * softplus_f(to_f(g[a.heads + h]) + a.dt_bias[h]);
-      gates[(long long)row * 2 * a.heads + a.heads + h] = sigmoid_f(to_f(g[h]));
+    for (int i = threadIdx.x; i < n_here * a.heads; i += 256) {
+      const int r = i / a.heads, h = i % a.heads;
+      const T* g = proj + (long long)r * a.proj_stride + 2 * L.nqk + 2 * L.nv;
+      float* dst = gates + (long long)(row0 + r) * 2 * a.heads + h;
+      dst[0] = -expf(a.a_log[h]) * softplus_f(to_f(g[a.heads + h]) + a.dt_bias[h]);
+      dst[a.heads] = sigmoid_f(to_f(g[h]));
     }
   }
   const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   const bool is_v = unit >= 2 * a.kv_heads;
-  const int c0 = is_v ? (unit - 2 * a.kv_heads) * 128 + lane * 4 : lane * 4;          // within v, or within the head
-  if (is_v ? (unit - 2 * a.kv_heads) * 128 >= L.nv : false) return;
+  const int seg = (unit - 2 * a.kv_heads) * 128;
+  if (is_v && seg >= L.nv) return;
+  const int c0 = is_v ? seg + lane * 4 : lane * 4;          // within v, or within the head
   const bool on = is_v ? c0 < L.nv : c0 < a.dim;
   const int c = is_v ? 2 * L.nqk + c0 : unit * a.dim + c0;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  // every input of the block's rows and of the TAPS-1 rows before them, all loads in flight at once
+  float4 x[kPrepRows + TAPS - 1];
+  const int s0 = a.tok_seq[a.n_decode + row0], first = a.n_decode + row0 - a.cu[s0], p0 = a.start[s0];
+  const T* half = conv_half<T>(a, L.chan, a.slot[s0], p0);
+#pragma unroll
+  for (int j = 0; j < TAPS - 1; ++j) {
+    const int t = first - (TAPS - 1) + j;                   // token of the portion that the block's first row continues
+    x[j] = zero;
+    if (on) {
+      if (t >= 0) x[j] = load4(proj + (long long)(j - (TAPS - 1)) * a.proj_stride + c);
+      else if (p0 + t >= 0) x[j] = load4(half + (long long)(TAPS - 1 + t) * L.chan + c);
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < kPrepRows; ++r) x[TAPS - 1 + r] = on && r < n_here ? load4(proj + (long long)r * a.proj_stride + c) : zero;
   float w[TAPS][4];
 #pragma unroll
   for (int j = 0; j < TAPS; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) w[j][e] = on ? a.conv_w[(long long)(c + e) * TAPS + j] : 0.f;
   const float post = unit < a.kv_heads ? 1.f / sqrtf((float)a.dim) : 1.f;
-  float4 hist[TAPS];      // hist[j] = input `TAPS - 1 - j` tokens back
 #pragma unroll
-  for (int j = 0; j < TAPS; ++j) hist[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-  for (int row = row0; row < row1; ++row) {
-    const long long n = (long long)a.n_decode + row;
-    const int s = a.tok_seq[n], t = (int)(n - a.cu[s]);
-    if (row == row0 || t == 0) {
-      const int p0 = a.start[s];
-      const T* half = conv_half<T>(a, L.chan, a.slot[s], p0);
+  for (int r = 0; r < kPrepRows; ++r) {
+    if (r >= n_here) break;
+    const long long row = row0 + r, n = a.n_decode + row;
+    float4 in[TAPS];
 #pragma unroll
-      for (int j = 1; j < TAPS; ++j) {                  // what the shift below turns into lags TAPS-1 .. 1
-        const int lag = TAPS - j;
-        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (on) {
-          if (t - lag >= 0) x = load4(proj + (n - lag) * a.proj_stride + c);
-          else if (p0 + t - lag >= 0) x = load4(half + (long long)(TAPS - 1 + t - lag) * L.chan + c);
+    for (int j = 0; j < TAPS; ++j) in[j] = x[r + j];
+    const int s = a.tok_seq[n];
+    if (s != s0) {                                          // a row of a later sequence: its own history where that is short
+      const int t = (int)(n - a.cu[s]);
+      if (t < TAPS - 1) {
+        const int q0 = a.start[s];
+        const T* h2 = conv_half<T>(a, L.chan, a.slot[s], q0);
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) {
+          const int lag = TAPS - 1 - j;
+          if (t - lag < 0) in[j] = on && q0 + t - lag >= 0 ? load4(h2 + (long long)(TAPS - 1 + t - lag) * L.chan + c) : zero;
         }
-        hist[j] = x;
       }
     }
-#pragma unroll
-    for (int j = 0; j + 1 < TAPS; ++j) hist[j] = hist[j + 1];
-    hist[TAPS - 1] = on ? load4(proj + n * a.proj_stride + c) : make_float4(0.f, 0.f, 0.f, 0.f);
     float y[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) {
-      y[0] = fmaf(w[j][0], hist[j].x, y[0]); y[1] = fmaf(w[j][1], hist[j].y, y[1]);
-      y[2] = fmaf(w[j][2], hist[j].z, y[2]); y[3] = fmaf(w[j][3], hist[j].w, y[3]);
+      y[0] = fmaf(w[j][0], in[j].x, y[0]); y[1] = fmaf(w[j][1], in[j].y, y[1]);
+      y[2] = fmaf(w[j][2], in[j].z, y[2]); y[3] = fmaf(w[j][3], in[j].w, y[3]);
     }
 #pragma unroll
     for (int e = 0; e < 4; ++e) y[e] = silu_act<T>(y[e]);
     if (is_v) {
-      if (on) store4(v + (long long)row * L.nv + c0, make_float4(y[0], y[1], y[2], y[3]));
+      if (on) store4(v + row * L.nv + c0, make_float4(y[0], y[1], y[2], y[3]));
+      continue;
+    }
+    const float ss = warp_sum_f(on ? y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3] : 0.f);
+    const float sc = post / sqrtf(ss + 1e-6f);
+    if (!on) continue;
+    const float4 q = make_float4(y[0] * sc, y[1] * sc, y[2] * sc, y[3] * sc);
+    if constexpr (SPLIT) {
+      const int is_k = unit >= a.kv_heads;
+      __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(qk_out) + row * 4 * L.nqk + (long long)is_k * 2 * L.nqk +
+                           (unit - is_k * a.kv_heads) * a.dim + c0;
+      const float4 hi = make_float4(__bfloat162float(__float2bfloat16_rn(q.x)), __bfloat162float(__float2bfloat16_rn(q.y)),
+                                    __bfloat162float(__float2bfloat16_rn(q.z)), __bfloat162float(__float2bfloat16_rn(q.w)));
+      store4(dst, hi);
+      store4(dst + L.nqk, make_float4(q.x - hi.x, q.y - hi.y, q.z - hi.z, q.w - hi.w));
     } else {
-      const float ss = warp_sum_f(on ? y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3] : 0.f);
-      const float sc = post / sqrtf(ss + 1e-6f);
-      if (on) store4(qk + (long long)row * 2 * L.nqk + (long long)unit * a.dim + c0, make_float4(y[0] * sc, y[1] * sc, y[2] * sc, y[3] * sc));
+      store4(reinterpret_cast<float*>(qk_out) + row * 2 * L.nqk + (long long)unit * a.dim + c0, q);
     }
   }
 }
@@ -170,6 +198,8 @@ __global__ void __launch_bounds__(kScThreads)
 delta_scan_kernel(const msa_lm_delta_args a, const float* __restrict__ qk, const float* __restrict__ v,
                   const float* __restrict__ gates, float* __restrict__ o) {
   constexpr int D = 8 * R;
+  // dimension d = part * R + r of a token lies at (r / 4) * 32 + part * 4 + r % 4: the eight lanes of a column read
+  // 128 consecutive bytes per vector
   __shared__ __align__(16) float s_q[kScTok][D], s_k[kScTok][D];
   __shared__ float s_v[kScTok][kScCols], s_o[kScTok][kScCols], s_g[kScTok], s_b[kScTok], s_qk[kScTok];
   const DeltaLayout L(a);
@@ -193,8 +223,9 @@ delta_scan_kernel(const msa_lm_delta_args a, const float* __restrict__ qk, const
     for (int i = threadIdx.x; i < nt * D; i += kScThreads) {
       const int t = i / D, d = i % D;
       const float* src = qk + (row0 + t0 + t) * 2 * L.nqk + (long long)hk * a.dim + d;
-      s_q[t][d] = d < a.dim ? src[0] : 0.f;
-      s_k[t][d] = d < a.dim ? src[L.nqk] : 0.f;
+      const int at = (d % R / 4) * 32 + d / R * 4 + d % 4;
+      s_q[t][at] = d < a.dim ? src[0] : 0.f;
+      s_k[t][at] = d < a.dim ? src[L.nqk] : 0.f;
     }
     for (int i = threadIdx.x; i < nt * kScCols; i += kScThreads) {
       const int t = i / kScCols, c = i % kScCols;
@@ -214,13 +245,16 @@ delta_scan_kernel(const msa_lm_delta_args a, const float* __restrict__ qk, const
     }
     __syncthreads();
     for (int t = 0; t < nt; ++t) {
-      float k[R], c = 0.f, r_ = 0.f;
+      float k[R], c = 0.f, r_ = 0.f, c2 = 0.f, r2 = 0.f;
 #pragma unroll
-      for (int r = 0; r < R; ++r) {
-        k[r] = s_k[t][part * R + r];
-        c = fmaf(st[r], k[r], c);
-        r_ = fmaf(st[r], s_q[t][part * R + r], r_);
+      for (int r = 0; r < R; r += 4) {
+        const float4 kv = load4(&s_k[t][r * 8 + part * 4]), qv = load4(&s_q[t][r * 8 + part * 4]);
+        k[r] = kv.x; k[r + 1] = kv.y; k[r + 2] = kv.z; k[r + 3] = kv.w;
+        c = fmaf(st[r], kv.x, c); c2 = fmaf(st[r + 1], kv.y, c2); c = fmaf(st[r + 2], kv.z, c); c2 = fmaf(st[r + 3], kv.w, c2);
+        r_ = fmaf(st[r], qv.x, r_); r2 = fmaf(st[r + 1], qv.y, r2); r_ = fmaf(st[r + 2], qv.z, r_); r2 = fmaf(st[r + 3], qv.w, r2);
       }
+      c += c2;
+      r_ += r2;
 #pragma unroll
       for (int w = 1; w < 8; w <<= 1) {
         c += __shfl_xor_sync(0xffffffffu, c, w);
@@ -250,10 +284,10 @@ __global__ void __launch_bounds__(256)
 delta_out_kernel(const msa_lm_delta_args a, const float* __restrict__ o, T* __restrict__ out, long long out_stride, long long n, bool vec) {
   const DeltaLayout L(a);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const long long item = (long long)blockIdx.x * 8 + warp;
-  if (item >= n * a.heads) return;
-  const long long row = item / a.heads;
-  const int h = (int)(item % a.heads);
+  const unsigned item = blockIdx.x * 8 + warp;
+  if (item >= (unsigned)(n * a.heads)) return;
+  const long long row = item / (unsigned)a.heads;
+  const int h = (int)(item % (unsigned)a.heads);
   const float* src = o + row * L.nv + (long long)h * a.vdim;
   const T* gate = reinterpret_cast<const T*>(a.proj) + (a.n_decode + row) * a.proj_stride + 2 * L.nqk + L.nv + (long long)h * a.vdim;
   float ss = 0.f;
@@ -279,7 +313,9 @@ delta_out_kernel(const msa_lm_delta_args a, const float* __restrict__ o, T* __re
 // (twice, the second time from L1 / L2) and written once.
 constexpr int kDdThreads = 256;
 
-template <typename T, int V>
+// HOLD > 0: a thread's part of the state (HOLD rows of one column vector) is loaded before anything else and stays in
+// registers, so the state is read once.
+template <typename T, int V, int HOLD>
 __global__ void __launch_bounds__(kDdThreads)
 delta_decode_kernel(const msa_lm_delta_args a, T* __restrict__ out, long long out_stride, int groups) {
   extern __shared__ float sm[];
@@ -290,9 +326,19 @@ delta_decode_kernel(const msa_lm_delta_args a, T* __restrict__ out, long long ou
   float* s_q = sm;                        // [dk]
   float* s_k = s_q + dk;                  // [dk]
   float* s_v = s_k + dk;                  // [dv], then the output row
-  float* s_c = s_v + dv;                  // [groups][dv]
+  float* s_c = sm + (2 * dk + dv + 3) / 4 * 4;   // [groups][dv]
   float* s_r = s_c + groups * dv;         // [groups][dv]
   const int slot = a.slot[b], p = a.pos[b];
+  float* S = a.state + (((long long)slot * a.heads + h) * dk) * dv;
+  float4 held[HOLD > 0 ? HOLD : 1];
+  const int hold_c = threadIdx.x % (dv / V) * V, hold_g = threadIdx.x / (dv / V);
+  if constexpr (HOLD > 0) {
+#pragma unroll
+    for (int i = 0; i < HOLD; ++i) {
+      const int d = hold_g + i * groups;
+      held[i] = p != 0 && hold_g < groups && d < dk ? load4(S + (long long)d * dv + hold_c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  }
   const T* proj = reinterpret_cast<const T*>(a.proj) + (long long)b * a.proj_stride;
   const T* old = conv_half<T>(a, L.chan, slot, p);
   T* fresh = reinterpret_cast<T*>(a.conv_state) + ((long long)slot * 2 + ((p + 1) & 1)) * keep * L.chan;
@@ -325,10 +371,25 @@ delta_decode_kernel(const msa_lm_delta_args a, T* __restrict__ out, long long ou
   qk *= sq * sk;
   const float beta = sigmoid_f(to_f(proj[2 * L.nqk + 2 * L.nv + h]));
   const float g = expf(-expf(a.a_log[h]) * softplus_f(to_f(proj[2 * L.nqk + 2 * L.nv + a.heads + h]) + a.dt_bias[h]));
-  float* S = a.state + (((long long)slot * a.heads + h) * dk) * dv;
   const bool zero = p == 0;
   const int cols = dv / V, rg = threadIdx.x / cols, cv = (threadIdx.x % cols) * V;   // groups * cols <= blockDim
   const bool active = rg < groups;
+  if constexpr (HOLD > 0) {
+    if (active) {
+      float4 ac = make_float4(0.f, 0.f, 0.f, 0.f), ar = ac;
+#pragma unroll
+      for (int i = 0; i < HOLD; ++i) {
+        const int d = rg + i * groups;
+        if (d < dk) {
+          const float kd = s_k[d], qd = s_q[d];
+          ac.x = fmaf(held[i].x, kd, ac.x); ac.y = fmaf(held[i].y, kd, ac.y); ac.z = fmaf(held[i].z, kd, ac.z); ac.w = fmaf(held[i].w, kd, ac.w);
+          ar.x = fmaf(held[i].x, qd, ar.x); ar.y = fmaf(held[i].y, qd, ar.y); ar.z = fmaf(held[i].z, qd, ar.z); ar.w = fmaf(held[i].w, qd, ar.w);
+        }
+      }
+      store4(s_c + rg * dv + cv, ac);
+      store4(s_r + rg * dv + cv, ar);
+    }
+  } else
   // columns are walked in one sweep when they fit the block; otherwise cols > blockDim is split over `cs`
   for (int cs = 0; cs < cols; cs += kDdThreads) {
     const int c = cols > kDdThreads ? (cs + threadIdx.x) * V : cv;
@@ -364,6 +425,20 @@ delta_decode_kernel(const msa_lm_delta_args a, T* __restrict__ out, long long ou
   }
   const float inv = 1.f / sqrtf(block_sum(ss, s_part) / (float)dv + a.eps);   // its barriers publish s_c and s_v
   __syncthreads();
+  if constexpr (HOLD > 0) {
+    if (active) {
+      const float4 u = load4(s_c + cv);
+#pragma unroll
+      for (int i = 0; i < HOLD; ++i) {
+        const int d = rg + i * groups;
+        if (d < dk) {
+          const float kd = s_k[d];
+          store4(S + (long long)d * dv + cv, make_float4(fmaf(kd, u.x, g * held[i].x), fmaf(kd, u.y, g * held[i].y),
+                                                         fmaf(kd, u.z, g * held[i].z), fmaf(kd, u.w, g * held[i].w)));
+        }
+      }
+    }
+  } else
   for (int cs = 0; cs < cols; cs += kDdThreads) {
     const int c = cols > kDdThreads ? (cs + threadIdx.x) * V : cv;
     const int g0 = cols > kDdThreads ? 0 : rg;
@@ -413,48 +488,63 @@ extern "C" int msa_lm_delta_decode(const msa_lm_delta_args* a, void* out, int64_
   const int v = a->vdim % 4 == 0 && aligned16(a->state) ? 4 : 1;
   const int cols = a->vdim / v;
   const int groups = cols >= kDdThreads ? 1 : kDdThreads / cols;
-  const size_t smem = (size_t)4 * (2 * a->dim + a->vdim + 2 * groups * a->vdim);
+  const size_t smem = (size_t)4 * ((2 * a->dim + a->vdim + 3) / 4 * 4 + 2 * groups * a->vdim);
+  const int hold = v == 4 && cols <= kDdThreads ? (a->dim + groups - 1) / groups : 99;
   const dim3 grid((unsigned)a->heads, (unsigned)a->n_decode);
   MSA_LM_DISPATCH(a->dtype, {
-    if (v == 4) {
-      static DeviceSmem st4;
-      MSA_OK_OR_RETURN(ensure_dynamic_smem(delta_decode_kernel<T, 4>, smem, st4));
-      delta_decode_kernel<T, 4><<<grid, kDdThreads, smem, (cudaStream_t)stream>>>(*a, (T*)out, out_stride, groups);
-    } else {
-      static DeviceSmem st1;
-      MSA_OK_OR_RETURN(ensure_dynamic_smem(delta_decode_kernel<T, 1>, smem, st1));
-      delta_decode_kernel<T, 1><<<grid, kDdThreads, smem, (cudaStream_t)stream>>>(*a, (T*)out, out_stride, groups);
-    }
+    auto launch = [&](auto kernel, DeviceSmem& configured) -> int {
+      MSA_OK_OR_RETURN(ensure_dynamic_smem(kernel, smem, configured));
+      kernel<<<grid, kDdThreads, smem, (cudaStream_t)stream>>>(*a, (T*)out, out_stride, groups);
+      return MSA_OK;
+    };
+    static DeviceSmem st8, st16, st4, st1;
+    if (hold <= 8) MSA_OK_OR_RETURN(launch(delta_decode_kernel<T, 4, 8>, st8));
+    else if (hold <= 16) MSA_OK_OR_RETURN(launch(delta_decode_kernel<T, 4, 16>, st16));
+    else if (v == 4) MSA_OK_OR_RETURN(launch(delta_decode_kernel<T, 4, 0>, st4));
+    else MSA_OK_OR_RETURN(launch(delta_decode_kernel<T, 1, 0>, st1));
   });
   MSA_LAUNCH_OK("delta_decode_kernel");
   return MSA_OK;
 }
+
+namespace {
+bool prep_vec_ok(const msa_lm_delta_args* a, const void* qk, const void* v) {
+  const int e4 = 4 * (int)dtype_size(a->dtype);
+  return a->taps >= 2 && a->taps <= 4 && a->dim % 4 == 0 && a->dim <= 128 && a->vdim % 4 == 0 && a->proj_stride % 4 == 0 &&
+         reinterpret_cast<uintptr_t>(a->proj) % e4 == 0 && reinterpret_cast<uintptr_t>(a->conv_state) % e4 == 0 && aligned16(qk) &&
+         aligned16(v);
+}
+template <typename T, bool SPLIT>
+int launch_prep_vec(const msa_lm_delta_args* a, void* qk, float* v, float* gates, cudaStream_t st) {
+  const DeltaLayout L(*a);
+  const int units = 2 * a->kv_heads + (L.nv + 127) / 128;
+  const dim3 grid((unsigned)((a->n_tok - a->n_decode + kPrepRows - 1) / kPrepRows), (unsigned)((units + 7) / 8));
+  if (a->taps == 2) delta_prep_vec_kernel<T, 2, SPLIT><<<grid, 256, 0, st>>>(*a, qk, v, gates);
+  else if (a->taps == 3) delta_prep_vec_kernel<T, 3, SPLIT><<<grid, 256, 0, st>>>(*a, qk, v, gates);
+  else delta_prep_vec_kernel<T, 4, SPLIT><<<grid, 256, 0, st>>>(*a, qk, v, gates);
+  MSA_LAUNCH_OK("delta_prep_vec_kernel");
+  return MSA_OK;
+}
+}  // namespace
 
 extern "C" int msa_lm_delta_prep(const msa_lm_delta_args* a, float* qk, float* v, float* gates, void* stream) {
   MSA_OK_OR_RETURN(delta_check(a, "delta_prep"));
   MSA_REQUIRE(qk && v && gates, "delta_prep: null output");
   const int rows = a->n_tok - a->n_decode;
   if (rows == 0) return MSA_OK;
-  const DeltaLayout L(*a);
-  const int e4 = 4 * (int)dtype_size(a->dtype);
-  const bool vec = a->taps >= 2 && a->taps <= 4 && a->dim % 4 == 0 && a->dim <= 128 && a->vdim % 4 == 0 && a->proj_stride % 4 == 0 &&
-                   reinterpret_cast<uintptr_t>(a->proj) % e4 == 0 && reinterpret_cast<uintptr_t>(a->conv_state) % e4 == 0 &&
-                   aligned16(qk) && aligned16(v);
-  if (vec) {
-    const int units = 2 * a->kv_heads + (L.nv + 127) / 128;
-    const dim3 grid((unsigned)((rows + kPrepRows - 1) / kPrepRows), (unsigned)((units + 7) / 8));
-    cudaStream_t st = (cudaStream_t)stream;
-    MSA_LM_DISPATCH(a->dtype, {
-      if (a->taps == 2) delta_prep_vec_kernel<T, 2><<<grid, 256, 0, st>>>(*a, qk, v, gates);
-      else if (a->taps == 3) delta_prep_vec_kernel<T, 3><<<grid, 256, 0, st>>>(*a, qk, v, gates);
-      else delta_prep_vec_kernel<T, 4><<<grid, 256, 0, st>>>(*a, qk, v, gates);
-    });
-    MSA_LAUNCH_OK("delta_prep_vec_kernel");
-    return MSA_OK;
+  if (prep_vec_ok(a, qk, v)) {
+    MSA_LM_DISPATCH(a->dtype, { return (launch_prep_vec<T, false>(a, qk, v, gates, (cudaStream_t)stream)); });
   }
   MSA_LM_DISPATCH(a->dtype, { delta_prep_kernel<T><<<rows, 256, 0, (cudaStream_t)stream>>>(*a, qk, v, gates); });
   MSA_LAUNCH_OK("delta_prep_kernel");
   return MSA_OK;
+}
+
+extern "C" int msa_lm_delta_prep_split(const msa_lm_delta_args* a, void* qk, float* v, float* gates, void* stream) {
+  MSA_OK_OR_RETURN(delta_check(a, "delta_prep_split"));
+  MSA_REQUIRE(qk && v && gates && a->dtype == MSA_BF16 && prep_vec_ok(a, qk, v), "delta_prep_split: unsupported sizes or alignment");
+  if (a->n_tok == a->n_decode) return MSA_OK;
+  return launch_prep_vec<__nv_bfloat16, true>(a, qk, v, gates, (cudaStream_t)stream);
 }
 
 extern "C" int msa_lm_delta_conv_store(const msa_lm_delta_args* a, void* stream) {
@@ -488,6 +578,7 @@ extern "C" int msa_lm_delta_out(const msa_lm_delta_args* a, const float* o, void
   MSA_REQUIRE(o && out, "delta_out: null pointer");
   const long long rows = a->n_tok - a->n_decode;
   if (rows == 0) return MSA_OK;
+  MSA_REQUIRE(rows * a->heads < (1ll << 31), "delta_out: too many rows");
   const long long blocks = (rows * a->heads + 7) / 8;
   MSA_LM_DISPATCH(a->dtype, {
     const int e4 = 4 * (int)sizeof(T);

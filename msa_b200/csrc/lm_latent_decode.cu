@@ -47,13 +47,18 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
   const int n_tiles = k1 > k0 ? (k1 - k0 + kLdKeys - 1) / kLdKeys : 0;
   const __nv_bfloat16* ring = p.ring + (long long)p.slot[b] * p.ring_rows * width;
 
+  const int n_ring = (int)p.ring_rows, lo_row = lo % n_ring;
+  const uint32_t k_base = (uint32_t)__cvta_generic_to_shared(s_k);
   auto load_tile = [&](int t) {
-    unsigned char* dst = s_k + (t & 1) * kLdKeys * pitch;
-    for (int i = threadIdx.x; i < kLdKeys * vecs; i += kLdThreads) {
-      const int r = i / vecs, c = i - r * vecs, k = k0 + t * kLdKeys + r;
-      const bool on = k < k1;
-      const long long row = on ? (lo + k) % p.ring_rows : 0;
-      cp_async16((uint32_t)__cvta_generic_to_shared(dst + r * pitch + c * 16), ring + row * width + c * 8, on ? 16u : 0u);
+    const uint32_t dst = k_base + (t & 1) * kLdKeys * pitch;
+#pragma unroll 4
+    for (int r = threadIdx.x >> 5; r < kLdKeys; r += kLdThreads / 32) {     // a warp per row
+      const int k = k0 + t * kLdKeys + r;
+      const uint32_t bytes = k < k1 ? 16u : 0u;
+      int row = lo_row + k;                                                 // both terms are below the ring's size
+      row = k < k1 ? (row >= n_ring ? row - n_ring : row) : 0;
+      const __nv_bfloat16* src = ring + (long long)row * width;
+      for (int c = threadIdx.x & 31; c < vecs; c += 32) cp_async16(dst + r * pitch + c * 16, src + c * 8, bytes);
     }
     cp_async_commit();
   };
@@ -85,11 +90,13 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     if (t + 1 < n_tiles) { load_tile(t + 1); cp_async_wait<1>(); } else cp_async_wait<0>();
     __syncthreads();
     const uint32_t kb = (uint32_t)__cvta_generic_to_shared(s_k + (t & 1) * kLdKeys * pitch);
-    float s[MT][4];
+    float s[MT][4], s2[MT][4];            // two chains per tile, added below
 #pragma unroll
-    for (int j = 0; j < MT; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
+    for (int j = 0; j < MT; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[j][e] = s2[j][e] = 0.f;
     const uint32_t b_addr = kb + brow * pitch + bcol;
-#pragma unroll 2
+#pragma unroll 4
     for (int k = 0; k < width; k += 32) {
       uint32_t a[4], a2[4], x[4], y[4];
       ldmatrix_x4(q_addr + k * 2, a[0], a[1], a[2], a[3]);
@@ -99,13 +106,17 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
         ldmatrix_x4(b_addr + k * 2 + 32, y[0], y[1], y[2], y[3]);
         mma_bf16_full(s[0], a, x[0], x[1]);
         mma_bf16_full(s[1], a, x[2], x[3]);
-        mma_bf16_full(s[0], a2, y[0], y[1]);
-        mma_bf16_full(s[1], a2, y[2], y[3]);
+        mma_bf16_full(s2[0], a2, y[0], y[1]);
+        mma_bf16_full(s2[1], a2, y[2], y[3]);
       } else {
         mma_bf16_full(s[0], a, x[0], x[1]);
-        mma_bf16_full(s[0], a2, x[2], x[3]);
+        mma_bf16_full(s2[0], a2, x[2], x[3]);
       }
     }
+#pragma unroll
+    for (int j = 0; j < MT; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[j][e] += s2[j][e];
     // s[j][0..1]: row g, keys (octet j of this warp) 2*tq, 2*tq+1; s[j][2..3]: row g+8
     const int valid = k1 - k0 - t * kLdKeys;
     float mx[2] = {-INFINITY, -INFINITY};
@@ -260,7 +271,7 @@ extern "C" int msa_lm_latent_decode(const void* qa, int64_t qa_row, int64_t qa_h
                                     const int32_t* pos, int32_t n, int32_t heads, int32_t rank, int32_t rot, int32_t window,
                                     int32_t splits, float scale, void* out, float* part_o, float* part_ml, void* stream) {
   MSA_REQUIRE(qa && ring && slot && pos && out && (rot == 0 || qb), "latent_decode: null pointer");
-  MSA_REQUIRE(msa_lm_latent_decode_supported(rank, rot) && heads > 0 && window > 0 && ring_rows > 0, "latent_decode: bad sizes");
+  MSA_REQUIRE(msa_lm_latent_decode_supported(rank, rot) && heads > 0 && window > 0 && ring_rows > 0 && ring_rows < (1ll << 30), "latent_decode: bad sizes");
   MSA_REQUIRE(splits >= 1 && splits <= 64 && (splits == 1 || (part_o && part_ml)), "latent_decode: bad splits");
   MSA_REQUIRE(aligned16(qa) && aligned16(ring) && aligned16(out) && (rot == 0 || aligned16(qb)) && qa_row % 8 == 0 &&
                   qa_head % 8 == 0 && qb_row % 8 == 0 && qb_head % 8 == 0, "latent_decode: rows must be 16-byte aligned");

@@ -82,6 +82,84 @@ moe_sort_kernel(const int32_t* __restrict__ idx, int n, int top, int experts, in
   }
 }
 
+// The same over many blocks: counts per block of 2,048 choices, then every block places its own from the counts before it.
+constexpr int kSortBlock = 2048;
+
+__global__ void __launch_bounds__(256)
+moe_count_kernel(const int32_t* __restrict__ idx, int n, int experts, int32_t* __restrict__ cnt) {
+  __shared__ int s_cnt[kMoeMaxExperts];
+  for (int e = threadIdx.x; e < experts; e += 256) s_cnt[e] = 0;
+  __syncthreads();
+  const int i1 = min(n, ((int)blockIdx.x + 1) * kSortBlock);
+  for (int i = blockIdx.x * kSortBlock + threadIdx.x; i < i1; i += 256) atomicAdd(&s_cnt[idx[i]], 1);
+  __syncthreads();
+  for (int e = threadIdx.x; e < experts; e += 256) cnt[blockIdx.x * experts + e] = s_cnt[e];
+}
+
+__global__ void __launch_bounds__(256)
+moe_place_kernel(const int32_t* __restrict__ idx, int n, int top, int experts, int tile_rows, const int32_t* __restrict__ cnt,
+                 int32_t* __restrict__ src, int32_t* __restrict__ inv, int32_t* __restrict__ off, int32_t* __restrict__ tiles,
+                 int max_tiles) {
+  __shared__ int s_total[kMoeMaxExperts + 1], s_next[kMoeMaxExperts], s_tile[kMoeMaxExperts + 1];
+  for (int e = threadIdx.x; e < experts; e += 256) {
+    int total = 0, before = 0;
+    for (int b = 0; b < (int)gridDim.x; ++b) {
+      const int c = cnt[b * experts + e];
+      if (b < (int)blockIdx.x) before += c;
+      total += c;
+    }
+    s_total[e] = total;
+    s_next[e] = before;
+  }
+  __syncthreads();
+  if (threadIdx.x < 32) {                               // one warp: prefix sums over the experts
+    int o = 0, t = 0;
+    for (int e0 = 0; e0 < experts; e0 += 32) {
+      const int e = e0 + threadIdx.x;
+      const int c = e < experts ? s_total[e] : 0, ct = (c + tile_rows - 1) / tile_rows;
+      int so = c, stl = ct;
+#pragma unroll
+      for (int d = 1; d < 32; d <<= 1) {
+        const int x = __shfl_up_sync(0xffffffffu, so, d), y = __shfl_up_sync(0xffffffffu, stl, d);
+        if ((int)threadIdx.x >= d) { so += x; stl += y; }
+      }
+      if (e < experts) { s_total[e] = o + so - c; s_tile[e] = t + stl - ct; }
+      o += __shfl_sync(0xffffffffu, so, 31);
+      t += __shfl_sync(0xffffffffu, stl, 31);
+    }
+    if (threadIdx.x == 0) { s_total[experts] = o; s_tile[experts] = t; }
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < experts; e += 256) s_next[e] += s_total[e];
+  if (blockIdx.x == 0) {
+    for (int e = threadIdx.x; e <= experts; e += 256) off[e] = s_total[e];
+    for (int e = threadIdx.x; e < experts; e += 256)
+      for (int t = s_tile[e]; t < s_tile[e + 1] && t < max_tiles; ++t) {
+        tiles[2 * t] = e;
+        tiles[2 * t + 1] = s_total[e] + (t - s_tile[e]) * tile_rows;
+      }
+    for (int t = s_tile[experts] + threadIdx.x; t < max_tiles; t += 256) { tiles[2 * t] = -1; tiles[2 * t + 1] = 0; }
+  }
+  __syncthreads();
+  const int i1 = min(n, ((int)blockIdx.x + 1) * kSortBlock);
+  for (int i = blockIdx.x * kSortBlock + threadIdx.x; i < i1; i += 256) {
+    const int at = atomicAdd(&s_next[idx[i]], 1);
+    src[at] = i / top;
+    inv[i] = at;
+  }
+}
+
+// out[i] = x[src[i]], 16 bytes per lane.
+__global__ void __launch_bounds__(256)
+gather_rows_kernel(const uint4* __restrict__ x, long long x_vecs, const int32_t* __restrict__ src, int n, int vecs, uint4* __restrict__ out) {
+  const int row = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (row >= n) return;
+  const uint4* from = x + (long long)src[row] * x_vecs;
+  uint4* to = out + (long long)row * vecs;
+#pragma unroll 4
+  for (int c = threadIdx.x & 31; c < vecs; c += 32) to[c] = from[c];
+}
+
 __device__ __forceinline__ float clamped_gate(float g, float u, float limit) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
@@ -150,13 +228,22 @@ extern "C" int msa_lm_moe_topk(const float* logits, int64_t stride, const float*
 }
 
 extern "C" int msa_lm_moe_sort(const int32_t* idx, int32_t n_rows, int32_t top, int32_t experts, int32_t tile_rows,
-                               int32_t* src, int32_t* inv, int32_t* off, int32_t* tiles, int32_t max_tiles, void* stream) {
+                               int32_t* src, int32_t* inv, int32_t* off, int32_t* tiles, int32_t max_tiles,
+                               int32_t* counts, void* stream) {
   MSA_REQUIRE(idx && src && inv && off && tiles && n_rows >= 0 && top > 0 && tile_rows > 0, "moe_sort: bad arguments");
   MSA_REQUIRE(experts > 0 && experts <= kMoeMaxExperts, "moe_sort: at most 1024 experts");
   const long long n = (long long)n_rows * top;
   MSA_REQUIRE(n < (1ll << 31), "moe_sort: too many rows");
   long long need = n / tile_rows + (n < experts ? n : experts);
   MSA_REQUIRE(max_tiles >= need, "moe_sort: room for %lld tiles needed", need);
+  if (counts && n > 2 * kSortBlock) {
+    const unsigned blocks = (unsigned)((n + kSortBlock - 1) / kSortBlock);
+    moe_count_kernel<<<blocks, 256, 0, (cudaStream_t)stream>>>(idx, (int)n, experts, counts);
+    MSA_LAUNCH_OK("moe_count_kernel");
+    moe_place_kernel<<<blocks, 256, 0, (cudaStream_t)stream>>>(idx, (int)n, top, experts, tile_rows, counts, src, inv, off, tiles, max_tiles);
+    MSA_LAUNCH_OK("moe_place_kernel");
+    return MSA_OK;
+  }
   moe_sort_kernel<<<1, 1024, 0, (cudaStream_t)stream>>>(idx, (int)n, top, experts, tile_rows, src, inv, off, tiles, max_tiles);
   MSA_LAUNCH_OK("moe_sort_kernel");
   return MSA_OK;
@@ -176,5 +263,15 @@ extern "C" int msa_lm_moe_gemm(const void* x, int64_t x_stride, const int32_t* s
     else moe_gemm_kernel<T, false><<<grid, 256, 0, (cudaStream_t)stream>>>((const T*)x, x_stride, src, (const T*)w, off, tiles, n_out, k, limit, out, out_stride, out_dtype);
   });
   MSA_LAUNCH_OK("moe_gemm_kernel");
+  return MSA_OK;
+}
+
+extern "C" int msa_lm_gather_rows(const void* x, int64_t x_stride_bytes, const int32_t* src, int32_t n, int32_t row_bytes, void* out,
+                                  void* stream) {
+  MSA_REQUIRE(x && src && out && n >= 0 && row_bytes > 0, "gather_rows: bad arguments");
+  MSA_REQUIRE(aligned16(x) && aligned16(out) && row_bytes % 16 == 0 && x_stride_bytes % 16 == 0, "gather_rows: 16-byte rows expected");
+  if (n == 0) return MSA_OK;
+  gather_rows_kernel<<<(unsigned)((n + 7) / 8), 256, 0, (cudaStream_t)stream>>>((const uint4*)x, x_stride_bytes / 16, src, n, row_bytes / 16, (uint4*)out);
+  MSA_LAUNCH_OK("gather_rows_kernel");
   return MSA_OK;
 }

@@ -132,7 +132,7 @@ class GatedDelta:
 
     def __init__(self, spec, w: Weights, prefix: str, width: int, eps: float):
         s = self.spec = spec
-        self.eps, self.status = eps, w.status
+        self.eps = eps
         qk, v = s.kv_heads * s.dim, s.heads * s.vdim
         self.w_in = w.stack([(prefix + "q", qk), (prefix + "k", qk), (prefix + "v", v), (prefix + "g", v),
                              (prefix + "b", s.heads), (prefix + "a", s.heads)], width, pad=True)
@@ -147,7 +147,7 @@ class GatedDelta:
         return RecurrentSpec(s.heads, s.dim, s.vdim, s.channels, s.taps)
 
     def mix(self, proj: torch.Tensor, step, cache: SequenceStateCache, run: int) -> torch.Tensor:
-        return K.delta_mix(proj, self.spec, self, cache.conv[run], cache.state[run], self.eps, step, self.status)
+        return K.delta_mix(proj, self.spec, self, cache.conv[run], cache.state[run], self.eps, step)
 
 
 class DenseFeedForward:
@@ -182,6 +182,8 @@ class MixtureFeedForward:
         idx, mix = K.moe_topk(K.matmul(h, self.router, torch.float32), self.bias, s.top)
         if self.tc:
             src, inv, off, tiles = K.moe_sort(idx, s.experts, K.MOE_TC_TILE_ROWS)
+            if n * s.top >= s.experts * K.MOE_GATHER_ROWS:
+                h, src = K.gather_rows(h, src), None
             act = K.moe_gemm_tc(h, src, self.w_gate_up, off, tiles, entries=n * s.top, act=True, limit=s.limit, status=self.status)
             return dict(y=K.moe_gemm_tc(act, None, self.w_down, off, tiles, entries=n * s.top, act=False, status=self.status),
                         inv=inv, mix=mix)

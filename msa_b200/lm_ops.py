@@ -149,12 +149,43 @@ def delta_args(proj, spec, w, conv_state, state, eps, step) -> A.DeltaArgs:
                        dtype=A.dtype_code(proj.dtype))
 
 
-def delta_recurrence(args, qk, v, gates, o, status) -> None:
-    """The recurrence over the portions of a step."""
-    A.call("msa_lm_delta_scan", C.byref(args), A.ptr(qk), A.ptr(v), A.ptr(gates), A.ptr(o), A.stream_ptr(qk.device))
+def delta_chunk_supported(spec, dtype) -> bool:
+    return dtype == torch.bfloat16 and bool(A.lib().msa_lm_delta_chunk_supported(spec.dim, spec.vdim, spec.taps))
 
 
-def delta_mix(proj, spec, w, conv_state, state, eps, step, status) -> torch.Tensor:
+def delta_tile(n_seq: int, heads: int, vdim: int, n_sm: int = 148) -> int:
+    """Value columns per CTA of the chunked recurrence: wide ones unless that leaves most of the GPU idle."""
+    best = 32
+    for t in (128, 64, 32):
+        if vdim % t == 0:
+            best = t
+            if n_seq * heads * (vdim // t) * 2 >= n_sm:
+                break
+    return best
+
+
+def delta_portions(args, spec, step, out) -> None:
+    """The portions of a step through the chunked kernels."""
+    dev, st = out.device, A.stream_ptr(out.device)
+    rows, heads = step.n_tok - step.n_decode, spec.heads
+    qk = torch.empty((rows, 4 * spec.kv_heads * spec.dim), dtype=torch.bfloat16, device=dev)
+    f = dict(dtype=torch.float32, device=dev)
+    v, gates = torch.empty((rows, heads * spec.vdim), **f), torch.empty((rows, 2 * heads), **f)
+    A.call("msa_lm_delta_prep_split", C.byref(args), A.ptr(qk), A.ptr(v), A.ptr(gates), st)
+    A.call("msa_lm_delta_conv_store", C.byref(args), st)
+    delta_chunks(args, spec, step, qk, v, gates, out)
+
+
+def delta_chunks(args, spec, step, qk, v, gates, out) -> None:
+    dev, heads = out.device, spec.heads
+    tile = delta_tile(step.n_seq - step.n_decode, heads, spec.vdim)
+    work = torch.empty(A.lib().msa_lm_delta_chunk_workspace(step.n_chunks, heads), dtype=torch.uint8, device=dev)
+    o = torch.empty_like(v) if tile != spec.vdim else None
+    A.call("msa_lm_delta_chunk", C.byref(args), A.ptr(qk), A.ptr(v), A.ptr(gates), A.ptr(step.chunk_off), step.n_chunks, tile,
+           A.ptr(work), A.ptr(o), A.ptr(out), _rows(out), A.stream_ptr(dev))
+
+
+def delta_mix(proj, spec, w, conv_state, state, eps, step) -> torch.Tensor:
     """From the projections to the input of the output product, ``[n_tok, heads*vdim]``; advances the states."""
     args = delta_args(proj, spec, w, conv_state, state, eps, step)
     dev, st = proj.device, A.stream_ptr(proj.device)
@@ -162,17 +193,21 @@ def delta_mix(proj, spec, w, conv_state, state, eps, step, status) -> torch.Tens
     if step.n_decode:
         A.call("msa_lm_delta_decode", C.byref(args), A.ptr(out), _rows(out), st)
     rows = step.n_tok - step.n_decode
-    if rows:
-        f = dict(dtype=torch.float32, device=dev)
-        qk = torch.empty((rows, 2 * spec.kv_heads * spec.dim), **f)
-        v = torch.empty((rows, spec.heads * spec.vdim), **f)
-        gates = torch.empty((rows, 2 * spec.heads), **f)
-        o = torch.empty((rows, spec.heads * spec.vdim), **f)
-        A.call("msa_lm_delta_prep", C.byref(args), A.ptr(qk), A.ptr(v), A.ptr(gates), st)
-        A.call("msa_lm_delta_conv_store", C.byref(args), st)
-        delta_recurrence(args, qk, v, gates, o, status)
-        tail = out[step.n_decode:]
-        A.call("msa_lm_delta_out", C.byref(args), A.ptr(o), A.ptr(tail), _rows(tail), st)
+    if not rows:
+        return out
+    tail = out[step.n_decode:]
+    if delta_chunk_supported(spec, proj.dtype):
+        delta_portions(args, spec, step, tail)
+        return out
+    f = dict(dtype=torch.float32, device=dev)
+    qk = torch.empty((rows, 2 * spec.kv_heads * spec.dim), **f)
+    v = torch.empty((rows, spec.heads * spec.vdim), **f)
+    gates = torch.empty((rows, 2 * spec.heads), **f)
+    o = torch.empty((rows, spec.heads * spec.vdim), **f)
+    A.call("msa_lm_delta_prep", C.byref(args), A.ptr(qk), A.ptr(v), A.ptr(gates), st)
+    A.call("msa_lm_delta_conv_store", C.byref(args), st)
+    A.call("msa_lm_delta_scan", C.byref(args), A.ptr(qk), A.ptr(v), A.ptr(gates), A.ptr(o), st)
+    A.call("msa_lm_delta_out", C.byref(args), A.ptr(o), A.ptr(tail), _rows(tail), st)
     return out
 
 
@@ -197,8 +232,9 @@ def moe_sort(idx, experts, tile_rows=MOE_TILE_ROWS):
     i = dict(dtype=torch.int32, device=dev)
     src, inv = torch.empty(n * top, **i), torch.empty((n, top), **i)
     off, tiles = torch.empty(experts + 1, **i), torch.empty((max_tiles, 2), **i)
+    counts = torch.empty(((n * top + 2047) // 2048, experts), **i) if n * top > 4096 else None
     A.call("msa_lm_moe_sort", A.ptr(idx), n, top, experts, tile_rows, A.ptr(src), A.ptr(inv), A.ptr(off), A.ptr(tiles),
-           max_tiles, A.stream_ptr(dev))
+           max_tiles, A.ptr(counts), A.stream_ptr(dev))
     return src, inv, off, tiles
 
 
@@ -213,6 +249,14 @@ def moe_gemm(x, src, w, off, tiles, *, entries, act, limit=0.0, out_dtype=None):
 
 
 MOE_TC_TILE_ROWS = 128
+MOE_GATHER_ROWS = 64      # entries per expert from which a copy of the grouped rows beats fetching them four at a time
+
+
+def gather_rows(x, src):
+    out = torch.empty((src.shape[0], x.shape[1]), dtype=x.dtype, device=x.device)
+    A.call("msa_lm_gather_rows", A.ptr(x), _rows(x) * x.element_size(), A.ptr(src), src.shape[0], x.shape[1] * x.element_size(),
+           A.ptr(out), A.stream_ptr(x.device))
+    return out
 
 
 def moe_tc_supported(dtype, width, ff) -> bool:

@@ -327,8 +327,7 @@ def test_unequal_requests_side_by_side_with_slots_used_again(name, dtype):
             if at[i] == len(toks[i]):
                 del at[i]
                 cache.release(i)
-    for i in toks:
-        close(torch.cat(got[i]), U.oracle_logits(name, 0, toks[i], dtype), dtype)
+    close(torch.cat([torch.cat(got[i]) for i in toks]), torch.cat([U.oracle_logits(name, 0, toks[i], dtype) for i in toks]), dtype)
 
 
 def test_batch_mates_do_not_change_a_sequence():
