@@ -1498,15 +1498,16 @@ def hybrid_kernels(torch, dev, model, z, pk, decode_b):
     projd = K.matmul(h, dlt.w_in)
     args = K.delta_args(projd, d, dlt, cache.conv[0], cache.state[0], 1e-5, step)
     f32 = dict(dtype=torch.float32, device=dev)
-    v, gates = torch.empty((n, heads * d.vdim), **f32), torch.empty((n, 2 * heads), **f32)
+    v, gates = torch.empty((n, heads * d.vdim), **bf), torch.empty((n, 2 * heads), **f32)
     qk, outd, st = torch.empty((n, 4 * d.kv_heads * d.dim), **bf), torch.empty((n, heads * d.vdim), **bf), A.stream_ptr(dev)
     p = A.ptr
-    leg("delta_prep", lambda: A.call("msa_lm_delta_prep_split", ctypes.byref(args), p(qk), p(v), p(gates), st), 0, n * d.channels * 6)
+    leg("delta_prep", lambda: A.call("msa_lm_delta_prep_split", ctypes.byref(args), p(qk), p(v), p(gates), st), 0,
+        n * (d.channels * 2 + 2 * d.kv_heads * d.dim * 4 + heads * d.vdim * 2))
     # flops of the chunked form, once each: S products, the triangular ones at half
     c = 64
     macs = n * heads * (3 * d.dim * d.vdim + c * d.vdim) + n * d.kv_heads * c * d.dim + n * heads * c * c / 6
     leg("delta_chunk + delta_state", lambda: K.delta_chunks(args, d, step, qk, v, gates, outd), 2.0 * macs,
-        n * (d.kv_heads * d.dim * 8 + heads * d.vdim * (4 + 2 + 2)) + n_seq * heads * d.dim * d.vdim * 4)
+        n * (d.kv_heads * d.dim * 8 + heads * d.vdim * (2 + 2 + 2)) + n_seq * heads * d.dim * d.vdim * 4)
     m = moe.spec
     logits = K.matmul(h, moe.router, torch.float32)
     leg("moe_topk", lambda: K.moe_topk(logits, moe.bias, m.top), 0, n * m.experts * 4)

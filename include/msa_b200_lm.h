@@ -98,7 +98,7 @@ int msa_lm_latent_decode(const void* qa, int64_t qa_row, int64_t qa_head, const 
 
 /* ---- gated delta rule ---------------------------------------------------------------------------------------------
  * proj row = [kv_heads*dim q | kv_heads*dim k | heads*vdim v | heads*vdim gate | heads beta | heads decay].
- * Convolution weights conv_w [2*kv_heads*dim + heads*vdim, taps] fp32.  Conv state [slots, 2, taps-1, channels] in dtype:
+ * Convolution weights conv_w [taps, 2*kv_heads*dim + heads*vdim] fp32.  Conv state [slots, 2, taps-1, channels] in dtype:
  * the inputs of the taps-1 positions before position p live in half p & 1.  Recurrent state [slots, heads, dim, vdim]
  * fp32.  A sequence at position 0 starts from zero whatever its slot held. */
 typedef struct {
@@ -118,15 +118,15 @@ int msa_lm_delta_decode(const msa_lm_delta_args* a, void* out, int64_t out_strid
 /* The other sequences: convolution + silu + unit norms -> qk [rows, 2, kv_heads, dim] fp32 (q scaled by dim^-1/2),
  * v [rows, heads, vdim] fp32, gates [rows, 2, heads] fp32 (log decay, beta); rows count from the first non-decode token. */
 int msa_lm_delta_prep(const msa_lm_delta_args* a, float* qk, float* v, float* gates, void* stream);
-/* The same with q and k as pairs of bf16 numbers: qk [rows, 2 (q, k), 2 (hi, lo), kv_heads, dim] (bf16 activations, 2 to 4
+/* The same with q and k as pairs of bf16 numbers: qk [rows, 2 (q, k), 2 (hi, lo), kv_heads, dim], v in bf16 (bf16 activations, 2 to 4
  * taps, dim <= 128, dim and vdim multiples of 4). */
-int msa_lm_delta_prep_split(const msa_lm_delta_args* a, void* qk, float* v, float* gates, void* stream);
+int msa_lm_delta_prep_split(const msa_lm_delta_args* a, void* qk, void* v, float* gates, void* stream);
 /* The recurrence in chunks of 64 tokens on tensor cores, from msa_lm_delta_prep_split's outputs, with the gated output norm
  * -> out (bf16); advances the state.  chunk_off: prefix sums of ceil(tokens / 64) over the non-decode sequences, n_chunks in
  * all; tile: value columns per CTA (32, 64 or 128, divides vdim); o [rows, heads, vdim] fp32 scratch when tile < vdim. */
 int msa_lm_delta_chunk_supported(int32_t dim, int32_t vdim, int32_t taps);
 int64_t msa_lm_delta_chunk_workspace(int32_t n_chunks, int32_t heads);
-int msa_lm_delta_chunk(const msa_lm_delta_args* a, const void* qk, const float* v, const float* gates, const int32_t* chunk_off,
+int msa_lm_delta_chunk(const msa_lm_delta_args* a, const void* qk, const void* v, const float* gates, const int32_t* chunk_off,
                        int32_t n_chunks, int32_t tile, void* workspace, float* o, void* out, int64_t out_stride, void* stream);
 /* Convolution inputs of the last taps-1 positions -> conv_state. */
 int msa_lm_delta_conv_store(const msa_lm_delta_args* a, void* stream);

@@ -30,23 +30,25 @@ struct WindowAttnTcParams {
   int q_row0;                            // packed row of the first query row of the map
   int q_head, k_head, v_head, v_col, r_col;   // column strides of a head, first value column, rotated column of the context
   float scale_log2e;
-  int max_mb;
-  long long n_items;
+  long long n_sh, n_items;               // sequences * heads; times the row blocks of the longest portion
   __nv_bfloat16* out; long long out_row;
   int32_t* status;
 };
 
+// Items are numbered from every portion's last row block to its first: the late ones see the most keys, and the
+// fixed-stride walk of the persistent CTAs then ends on short ones.
 struct WaItem { int len, r0, h, q_row, k_row, old, n_kt, a[kWaTiles], b[kWaTiles]; bool valid; };
 __device__ __forceinline__ WaItem wa_item(const WindowAttnTcParams& p, long long w) {
   WaItem it;
-  const int mb = (int)(w % p.max_mb);
-  const long long sh = w / p.max_mb;
+  const int x = (int)(w / p.n_sh);
+  const long long sh = w % p.n_sh;
   it.h = (int)(sh % p.heads);
   const int ps = (int)(sh / p.heads), s = p.seq0 + ps;
   const int c0 = p.cu[s];
   it.len = p.cu[s + 1] - c0;
-  it.r0 = mb * kWaRows * kWaTiles;
-  it.valid = it.r0 < it.len;
+  const int n_mb = (it.len + kWaRows * kWaTiles - 1) / (kWaRows * kWaTiles);
+  it.valid = x < n_mb;
+  it.r0 = (n_mb - 1 - x) * kWaRows * kWaTiles;
   it.old = min(p.start[s], p.window - 1);
   it.q_row = c0 - p.q_row0 + it.r0;
   const int j_lo = max(0, it.old + it.r0 - p.window + 1);
@@ -425,8 +427,8 @@ extern "C" int msa_lm_window_attn_tc(const void* q, int64_t q_row, int32_t n_row
   p.seq0 = seq0; p.heads = heads; p.window = window; p.q_row0 = row0;
   p.q_head = dim + rot; p.k_head = dim; p.v_head = vdim; p.v_col = heads * dim; p.r_col = rank;
   p.scale_log2e = scale * 1.4426950408889634f;
-  p.max_mb = (max_len + kWaRows * kWaTiles - 1) / (kWaRows * kWaTiles);
-  p.n_items = (long long)(seq1 - seq0) * heads * p.max_mb;
+  p.n_sh = (long long)(seq1 - seq0) * heads;
+  p.n_items = p.n_sh * ((max_len + kWaRows * kWaTiles - 1) / (kWaRows * kWaTiles));
   p.out = (__nv_bfloat16*)out; p.out_row = out_row; p.status = status;
   cudaStream_t st = (cudaStream_t)stream;
   const int key = (dim / 64) * 100 + (rot / 64) * 10 + vdim / 64;

@@ -6,6 +6,8 @@
 //
 // One step of a head, with S the state before it, reads S once for both products:
 //     c = S^T k,  r = S^T q;   u = beta (v - g c);   S <- g S + k u^T;   o = g r + (q.k) u
+#include <type_traits>
+
 #include "lm_common.cuh"
 
 namespace msa {
@@ -21,12 +23,12 @@ template <typename T>
 __device__ __forceinline__ float conv_silu(const msa_lm_delta_args& a, const T* state_half, int chan, long long n, int t,
                                            int p0, int c) {
   const T* proj = reinterpret_cast<const T*>(a.proj);
-  const float* w = a.conv_w + (long long)c * a.taps;
   float acc = 0.f;
   for (int i = 0; i < a.taps; ++i) {
     const int lag = a.taps - 1 - i;
-    if (t - lag >= 0) acc = fmaf(w[i], to_f(proj[(n - lag) * a.proj_stride + c]), acc);
-    else if (p0 + t - lag >= 0) acc = fmaf(w[i], to_f(state_half[(long long)(a.taps - 1 + t - lag) * chan + c]), acc);
+    const float w = a.conv_w[(long long)i * chan + c];
+    if (t - lag >= 0) acc = fmaf(w, to_f(proj[(n - lag) * a.proj_stride + c]), acc);
+    else if (p0 + t - lag >= 0) acc = fmaf(w, to_f(state_half[(long long)(a.taps - 1 + t - lag) * chan + c]), acc);
   }
   return silu_f(acc);
 }
@@ -73,10 +75,23 @@ constexpr int kPrepRows = 8;
 template <typename T> __device__ __forceinline__ float silu_act(float z) { return silu_f(z); }
 template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 
-// SPLIT: q and k leave as pairs of bf16 numbers whose sum they are, [rows, 2 (q, k), 2 (hi, lo), kv_heads, dim].
+// SPLIT: q and k leave as pairs of bf16 numbers whose sum they are, [rows, 2 (q, k), 2 (hi, lo), kv_heads, dim], and v in
+// bf16.
+template <typename T> struct Raw4;
+template <> struct Raw4<float> { using type = float4; };
+template <> struct Raw4<__nv_bfloat16> { using type = uint2; };
+__device__ __forceinline__ float4 widen(float4 v) { return v; }
+__device__ __forceinline__ float4 widen(uint2 r) {
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
 template <typename T, int TAPS, bool SPLIT>
 __global__ void __launch_bounds__(256)
-delta_prep_vec_kernel(const msa_lm_delta_args a, void* __restrict__ qk_out, float* __restrict__ v, float* __restrict__ gates) {
+delta_prep_vec_kernel(const msa_lm_delta_args a, void* __restrict__ qk_out, void* __restrict__ v_out, float* __restrict__ gates) {
+  using Raw = typename Raw4<T>::type;
+  auto raw = [](const T* p) { return *reinterpret_cast<const Raw*>(p); };
   const DeltaLayout L(a);
   const int row0 = blockIdx.x * kPrepRows, n_rows = a.n_tok - a.n_decode;
   const int n_here = min(kPrepRows, n_rows - row0);
@@ -97,9 +112,9 @@ delta_prep_vec_kernel(const msa_lm_delta_args a, void* __restrict__ qk_out, floa
   const int c0 = is_v ? seg + lane * 4 : lane * 4;          // within v, or within the head
   const bool on = is_v ? c0 < L.nv : c0 < a.dim;
   const int c = is_v ? 2 * L.nqk + c0 : unit * a.dim + c0;
-  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  const Raw zero{};
   // every input of the block's rows and of the TAPS-1 rows before them, all loads in flight at once
-  float4 x[kPrepRows + TAPS - 1];
+  Raw x[kPrepRows + TAPS - 1];
   const int s0 = a.tok_seq[a.n_decode + row0], first = a.n_decode + row0 - a.cu[s0], p0 = a.start[s0];
   const T* half = conv_half<T>(a, L.chan, a.slot[s0], p0);
 #pragma unroll
@@ -107,23 +122,21 @@ delta_prep_vec_kernel(const msa_lm_delta_args a, void* __restrict__ qk_out, floa
     const int t = first - (TAPS - 1) + j;                   // token of the portion that the block's first row continues
     x[j] = zero;
     if (on) {
-      if (t >= 0) x[j] = load4(proj + (long long)(j - (TAPS - 1)) * a.proj_stride + c);
-      else if (p0 + t >= 0) x[j] = load4(half + (long long)(TAPS - 1 + t) * L.chan + c);
+      if (t >= 0) x[j] = raw(proj + (long long)(j - (TAPS - 1)) * a.proj_stride + c);
+      else if (p0 + t >= 0) x[j] = raw(half + (long long)(TAPS - 1 + t) * L.chan + c);
     }
   }
 #pragma unroll
-  for (int r = 0; r < kPrepRows; ++r) x[TAPS - 1 + r] = on && r < n_here ? load4(proj + (long long)r * a.proj_stride + c) : zero;
-  float w[TAPS][4];
+  for (int r = 0; r < kPrepRows; ++r) x[TAPS - 1 + r] = on && r < n_here ? raw(proj + (long long)r * a.proj_stride + c) : zero;
+  float4 w[TAPS];
 #pragma unroll
-  for (int j = 0; j < TAPS; ++j)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) w[j][e] = on ? a.conv_w[(long long)(c + e) * TAPS + j] : 0.f;
+  for (int j = 0; j < TAPS; ++j) w[j] = on ? load4(a.conv_w + (long long)j * L.chan + c) : make_float4(0.f, 0.f, 0.f, 0.f);
   const float post = unit < a.kv_heads ? 1.f / sqrtf((float)a.dim) : 1.f;
 #pragma unroll
   for (int r = 0; r < kPrepRows; ++r) {
     if (r >= n_here) break;
     const long long row = row0 + r, n = a.n_decode + row;
-    float4 in[TAPS];
+    Raw in[TAPS];
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) in[j] = x[r + j];
     const int s = a.tok_seq[n];
@@ -135,20 +148,22 @@ delta_prep_vec_kernel(const msa_lm_delta_args a, void* __restrict__ qk_out, floa
 #pragma unroll
         for (int j = 0; j < TAPS - 1; ++j) {
           const int lag = TAPS - 1 - j;
-          if (t - lag < 0) in[j] = on && q0 + t - lag >= 0 ? load4(h2 + (long long)(TAPS - 1 + t - lag) * L.chan + c) : zero;
+          if (t - lag < 0) in[j] = on && q0 + t - lag >= 0 ? raw(h2 + (long long)(TAPS - 1 + t - lag) * L.chan + c) : zero;
         }
       }
     }
     float y[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) {
-      y[0] = fmaf(w[j][0], in[j].x, y[0]); y[1] = fmaf(w[j][1], in[j].y, y[1]);
-      y[2] = fmaf(w[j][2], in[j].z, y[2]); y[3] = fmaf(w[j][3], in[j].w, y[3]);
+      const float4 f = widen(in[j]);
+      y[0] = fmaf(w[j].x, f.x, y[0]); y[1] = fmaf(w[j].y, f.y, y[1]);
+      y[2] = fmaf(w[j].z, f.z, y[2]); y[3] = fmaf(w[j].w, f.w, y[3]);
     }
 #pragma unroll
     for (int e = 0; e < 4; ++e) y[e] = silu_act<T>(y[e]);
     if (is_v) {
-      if (on) store4(v + row * L.nv + c0, make_float4(y[0], y[1], y[2], y[3]));
+      using TV = typename std::conditional<SPLIT, __nv_bfloat16, float>::type;
+      if (on) store4(reinterpret_cast<TV*>(v_out) + row * L.nv + c0, make_float4(y[0], y[1], y[2], y[3]));
       continue;
     }
     const float ss = warp_sum_f(on ? y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3] : 0.f);
@@ -313,9 +328,8 @@ delta_out_kernel(const msa_lm_delta_args a, const float* __restrict__ o, T* __re
 // (twice, the second time from L1 / L2) and written once.
 constexpr int kDdThreads = 256;
 
-// HOLD > 0: a thread's part of the state (HOLD rows of one column vector) is loaded before anything else and stays in
-// registers, so the state is read once.
-template <typename T, int V, int HOLD>
+// STAGE: the state is copied to shared memory before anything else (cp.async) and read from there both times.
+template <typename T, int V, bool STAGE>
 __global__ void __launch_bounds__(kDdThreads)
 delta_decode_kernel(const msa_lm_delta_args a, T* __restrict__ out, long long out_stride, int groups) {
   extern __shared__ float sm[];
@@ -330,30 +344,36 @@ delta_decode_kernel(const msa_lm_delta_args a, T* __restrict__ out, long long ou
   float* s_r = s_c + groups * dv;         // [groups][dv]
   const int slot = a.slot[b], p = a.pos[b];
   float* S = a.state + (((long long)slot * a.heads + h) * dk) * dv;
-  float4 held[HOLD > 0 ? HOLD : 1];
-  const int hold_c = threadIdx.x % (dv / V) * V, hold_g = threadIdx.x / (dv / V);
-  if constexpr (HOLD > 0) {
-#pragma unroll
-    for (int i = 0; i < HOLD; ++i) {
-      const int d = hold_g + i * groups;
-      held[i] = p != 0 && hold_g < groups && d < dk ? load4(S + (long long)d * dv + hold_c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  float* s_state = sm + (2 * dk + dv + 3) / 4 * 4 + 2 * groups * dv;   // [dk][dv]
+  if constexpr (STAGE) {
+    if (p != 0) {
+      const uint32_t dst = (uint32_t)__cvta_generic_to_shared(s_state);
+      for (int i = threadIdx.x; i < dk * dv / 4; i += kDdThreads)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + i * 16), "l"(S + (long long)i * 4) : "memory");
+    } else {
+      for (int i = threadIdx.x; i < dk * dv / 4; i += kDdThreads) store4(s_state + i * 4, make_float4(0.f, 0.f, 0.f, 0.f));
     }
+    asm volatile("cp.async.commit_group;" ::: "memory");
   }
   const T* proj = reinterpret_cast<const T*>(a.proj) + (long long)b * a.proj_stride;
+  const float raw_beta = to_f(proj[2 * L.nqk + 2 * L.nv + h]), raw_decay = to_f(proj[2 * L.nqk + 2 * L.nv + a.heads + h]);
+  const float a_log = a.a_log[h], dt_bias = a.dt_bias[h];
+  const T* gate = proj + 2 * L.nqk + L.nv + (long long)h * dv;
+  const float gate0 = threadIdx.x < dv ? to_f(gate[threadIdx.x]) : 0.f, norm0 = threadIdx.x < dv ? a.w_norm[threadIdx.x] : 0.f;
   const T* old = conv_half<T>(a, L.chan, slot, p);
   T* fresh = reinterpret_cast<T*>(a.conv_state) + ((long long)slot * 2 + ((p + 1) & 1)) * keep * L.chan;
   for (int i = threadIdx.x; i < 2 * dk + dv; i += kDdThreads) {
     const int c = i < dk ? hk * dk + i : (i < 2 * dk ? L.nqk + hk * dk + (i - dk) : 2 * L.nqk + h * dv + (i - 2 * dk));
     const bool writer = i >= 2 * dk || h % group == 0;
-    const float* w = a.conv_w + (long long)c * a.taps;
+    const float* w = a.conv_w + c;
     float acc = 0.f;
     for (int j = 0; j < keep; ++j) {
       const T x = p - keep + j >= 0 ? old[(long long)j * L.chan + c] : from_f<T>(0.f);
-      acc = fmaf(w[j], to_f(x), acc);
+      acc = fmaf(w[(long long)j * L.chan], to_f(x), acc);
       if (writer && j > 0) fresh[(long long)(j - 1) * L.chan + c] = x;
     }
     const T x = proj[c];
-    acc = fmaf(w[keep], to_f(x), acc);
+    acc = fmaf(w[(long long)keep * L.chan], to_f(x), acc);
     if (writer && keep > 0) fresh[(long long)(keep - 1) * L.chan + c] = x;
     sm[i] = silu_f(acc);
   }
@@ -364,27 +384,34 @@ delta_decode_kernel(const msa_lm_delta_args a, T* __restrict__ out, long long ou
     kk += s_k[i] * s_k[i];
     qk += s_q[i] * s_k[i];
   }
-  qq = block_sum(qq, s_part);
-  kk = block_sum(kk, s_part);
-  qk = block_sum(qk, s_part);
+  qq = warp_sum_f(qq);
+  kk = warp_sum_f(kk);
+  qk = warp_sum_f(qk);
+  if ((threadIdx.x & 31) == 0) {
+    const int w = threadIdx.x >> 5;
+    s_part[w] = qq; s_part[8 + w] = kk; s_part[16 + w] = qk;
+  }
+  if constexpr (STAGE) asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  qq = kk = qk = 0.f;
+#pragma unroll
+  for (int w = 0; w < kDdThreads / 32; ++w) { qq += s_part[w]; kk += s_part[8 + w]; qk += s_part[16 + w]; }
   const float sq = 1.f / (sqrtf((float)dk) * sqrtf(qq + 1e-6f)), sk = 1.f / sqrtf(kk + 1e-6f);
   qk *= sq * sk;
-  const float beta = sigmoid_f(to_f(proj[2 * L.nqk + 2 * L.nv + h]));
-  const float g = expf(-expf(a.a_log[h]) * softplus_f(to_f(proj[2 * L.nqk + 2 * L.nv + a.heads + h]) + a.dt_bias[h]));
+  const float beta = sigmoid_f(raw_beta);
+  const float g = expf(-expf(a_log) * softplus_f(raw_decay + dt_bias));
   const bool zero = p == 0;
   const int cols = dv / V, rg = threadIdx.x / cols, cv = (threadIdx.x % cols) * V;   // groups * cols <= blockDim
   const bool active = rg < groups;
-  if constexpr (HOLD > 0) {
+  if constexpr (STAGE) {
     if (active) {
       float4 ac = make_float4(0.f, 0.f, 0.f, 0.f), ar = ac;
-#pragma unroll
-      for (int i = 0; i < HOLD; ++i) {
-        const int d = rg + i * groups;
-        if (d < dk) {
-          const float kd = s_k[d], qd = s_q[d];
-          ac.x = fmaf(held[i].x, kd, ac.x); ac.y = fmaf(held[i].y, kd, ac.y); ac.z = fmaf(held[i].z, kd, ac.z); ac.w = fmaf(held[i].w, kd, ac.w);
-          ar.x = fmaf(held[i].x, qd, ar.x); ar.y = fmaf(held[i].y, qd, ar.y); ar.z = fmaf(held[i].z, qd, ar.z); ar.w = fmaf(held[i].w, qd, ar.w);
-        }
+#pragma unroll 4
+      for (int d = rg; d < dk; d += groups) {
+        const float4 x = load4(s_state + d * dv + cv);
+        const float kd = s_k[d], qd = s_q[d];
+        ac.x = fmaf(x.x, kd, ac.x); ac.y = fmaf(x.y, kd, ac.y); ac.z = fmaf(x.z, kd, ac.z); ac.w = fmaf(x.w, kd, ac.w);
+        ar.x = fmaf(x.x, qd, ar.x); ar.y = fmaf(x.y, qd, ar.y); ar.z = fmaf(x.z, qd, ar.z); ar.w = fmaf(x.w, qd, ar.w);
       }
       store4(s_c + rg * dv + cv, ac);
       store4(s_r + rg * dv + cv, ar);
@@ -425,17 +452,14 @@ delta_decode_kernel(const msa_lm_delta_args a, T* __restrict__ out, long long ou
   }
   const float inv = 1.f / sqrtf(block_sum(ss, s_part) / (float)dv + a.eps);   // its barriers publish s_c and s_v
   __syncthreads();
-  if constexpr (HOLD > 0) {
+  if constexpr (STAGE) {
     if (active) {
       const float4 u = load4(s_c + cv);
-#pragma unroll
-      for (int i = 0; i < HOLD; ++i) {
-        const int d = rg + i * groups;
-        if (d < dk) {
-          const float kd = s_k[d];
-          store4(S + (long long)d * dv + cv, make_float4(fmaf(kd, u.x, g * held[i].x), fmaf(kd, u.y, g * held[i].y),
-                                                         fmaf(kd, u.z, g * held[i].z), fmaf(kd, u.w, g * held[i].w)));
-        }
+#pragma unroll 4
+      for (int d = rg; d < dk; d += groups) {
+        const float4 x = load4(s_state + d * dv + cv);
+        const float kd = s_k[d];
+        store4(S + (long long)d * dv + cv, make_float4(fmaf(kd, u.x, g * x.x), fmaf(kd, u.y, g * x.y), fmaf(kd, u.z, g * x.z), fmaf(kd, u.w, g * x.w)));
       }
     }
   } else
@@ -461,9 +485,10 @@ delta_decode_kernel(const msa_lm_delta_args a, T* __restrict__ out, long long ou
       }
     }
   }
-  const T* gate = proj + 2 * L.nqk + L.nv + (long long)h * dv;
-  for (int i = threadIdx.x; i < dv; i += kDdThreads)
-    out[(long long)b * out_stride + (long long)h * dv + i] = from_f<T>(s_v[i] * inv * a.w_norm[i] * silu_f(to_f(gate[i])));
+  for (int i = threadIdx.x; i < dv; i += kDdThreads) {
+    const float z = i == (int)threadIdx.x ? gate0 : to_f(gate[i]), w = i == (int)threadIdx.x ? norm0 : a.w_norm[i];
+    out[(long long)b * out_stride + (long long)h * dv + i] = from_f<T>(s_v[i] * inv * w * silu_f(z));
+  }
 }
 
 inline int delta_check(const msa_lm_delta_args* a, const char* what) {
@@ -489,19 +514,18 @@ extern "C" int msa_lm_delta_decode(const msa_lm_delta_args* a, void* out, int64_
   const int cols = a->vdim / v;
   const int groups = cols >= kDdThreads ? 1 : kDdThreads / cols;
   const size_t smem = (size_t)4 * ((2 * a->dim + a->vdim + 3) / 4 * 4 + 2 * groups * a->vdim);
-  const int hold = v == 4 && cols <= kDdThreads ? (a->dim + groups - 1) / groups : 99;
+  const bool stage = v == 4 && cols <= kDdThreads && (size_t)a->dim * a->vdim * 4 + smem <= 110 * 1024;
   const dim3 grid((unsigned)a->heads, (unsigned)a->n_decode);
   MSA_LM_DISPATCH(a->dtype, {
-    auto launch = [&](auto kernel, DeviceSmem& configured) -> int {
-      MSA_OK_OR_RETURN(ensure_dynamic_smem(kernel, smem, configured));
-      kernel<<<grid, kDdThreads, smem, (cudaStream_t)stream>>>(*a, (T*)out, out_stride, groups);
+    auto launch = [&](auto kernel, DeviceSmem& configured, size_t bytes) -> int {
+      MSA_OK_OR_RETURN(ensure_dynamic_smem(kernel, bytes, configured));
+      kernel<<<grid, kDdThreads, bytes, (cudaStream_t)stream>>>(*a, (T*)out, out_stride, groups);
       return MSA_OK;
     };
-    static DeviceSmem st8, st16, st4, st1;
-    if (hold <= 8) MSA_OK_OR_RETURN(launch(delta_decode_kernel<T, 4, 8>, st8));
-    else if (hold <= 16) MSA_OK_OR_RETURN(launch(delta_decode_kernel<T, 4, 16>, st16));
-    else if (v == 4) MSA_OK_OR_RETURN(launch(delta_decode_kernel<T, 4, 0>, st4));
-    else MSA_OK_OR_RETURN(launch(delta_decode_kernel<T, 1, 0>, st1));
+    static DeviceSmem staged, st4, st1;
+    if (stage) MSA_OK_OR_RETURN(launch(delta_decode_kernel<T, 4, true>, staged, smem + (size_t)a->dim * a->vdim * 4));
+    else if (v == 4) MSA_OK_OR_RETURN(launch(delta_decode_kernel<T, 4, false>, st4, smem));
+    else MSA_OK_OR_RETURN(launch(delta_decode_kernel<T, 1, false>, st1, smem));
   });
   MSA_LAUNCH_OK("delta_decode_kernel");
   return MSA_OK;
@@ -512,10 +536,10 @@ bool prep_vec_ok(const msa_lm_delta_args* a, const void* qk, const void* v) {
   const int e4 = 4 * (int)dtype_size(a->dtype);
   return a->taps >= 2 && a->taps <= 4 && a->dim % 4 == 0 && a->dim <= 128 && a->vdim % 4 == 0 && a->proj_stride % 4 == 0 &&
          reinterpret_cast<uintptr_t>(a->proj) % e4 == 0 && reinterpret_cast<uintptr_t>(a->conv_state) % e4 == 0 && aligned16(qk) &&
-         aligned16(v);
+         aligned16(v) && aligned16(a->conv_w);
 }
 template <typename T, bool SPLIT>
-int launch_prep_vec(const msa_lm_delta_args* a, void* qk, float* v, float* gates, cudaStream_t st) {
+int launch_prep_vec(const msa_lm_delta_args* a, void* qk, void* v, float* gates, cudaStream_t st) {
   const DeltaLayout L(*a);
   const int units = 2 * a->kv_heads + (L.nv + 127) / 128;
   const dim3 grid((unsigned)((a->n_tok - a->n_decode + kPrepRows - 1) / kPrepRows), (unsigned)((units + 7) / 8));
@@ -540,7 +564,7 @@ extern "C" int msa_lm_delta_prep(const msa_lm_delta_args* a, float* qk, float* v
   return MSA_OK;
 }
 
-extern "C" int msa_lm_delta_prep_split(const msa_lm_delta_args* a, void* qk, float* v, float* gates, void* stream) {
+extern "C" int msa_lm_delta_prep_split(const msa_lm_delta_args* a, void* qk, void* v, float* gates, void* stream) {
   MSA_OK_OR_RETURN(delta_check(a, "delta_prep_split"));
   MSA_REQUIRE(qk && v && gates && a->dtype == MSA_BF16 && prep_vec_ok(a, qk, v), "delta_prep_split: unsupported sizes or alignment");
   if (a->n_tok == a->n_decode) return MSA_OK;

@@ -36,7 +36,8 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
 
 struct DeltaChunkParams {
   const __nv_bfloat16* qk;      // [rows, 2 (q, k), 2 (hi, lo), kv_heads, dim]
-  const float *v, *gates;       // [rows, heads, vdim]; [rows, 2, heads]
+  const __nv_bfloat16* v;       // [rows, heads, vdim]
+  const float* gates;           // [rows, 2, heads]
   const int32_t *slot, *start, *cu, *chunk_off;   // chunk_off: prefix sums over the non-decode sequences
   int n_decode, n_seq, heads, kv_heads, dim, vdim, n_chunks;
   __nv_bfloat16* tm;            // [chunks, heads, 2 (T, M), 2 (hi, lo), 64, 64]
@@ -56,9 +57,10 @@ __global__ void __launch_bounds__(128) delta_chunk_kernel(const DeltaChunkParams
   extern __shared__ __align__(16) unsigned char sm[];
   unsigned char* s_q = sm;                               // hi, lo
   unsigned char* s_k = s_q + 2 * kDcRows * kPitch;       // hi, lo
-  float* s_kk = reinterpret_cast<float*>(s_k + 2 * kDcRows * kPitch);   // [64][65]
+  // over the operands once they are used up
+  float* s_a = reinterpret_cast<float*>(sm);             // [64][68]
+  float* s_kk = s_a + kDcRows * 68;                      // [64][65]
   float* s_qk = s_kk + kDcRows * 65;
-  float* s_a = reinterpret_cast<float*>(s_q);            // [64][68], over the operands once they are used up
   __shared__ float s_g[kDcRows], s_b[kDcRows];
   const int chunk = blockIdx.x, hk = blockIdx.y, group = p.heads / p.kv_heads;
   const int ps = owner_of(p.chunk_off, p.n_seq - p.n_decode, chunk), s = ps + p.n_decode;
@@ -109,6 +111,7 @@ __global__ void __launch_bounds__(128) delta_chunk_kernel(const DeltaChunkParams
         }
       }
     }
+    __syncthreads();
 #pragma unroll
     for (int j = 0; j < 8; ++j)
 #pragma unroll
@@ -189,30 +192,33 @@ struct DeltaStateSmem {
   static constexpr int kPk = DK * 2 + 16, kPv = DVT * 2 + 16;      // bytes per row
   static constexpr int kQ = 0, kK = kQ + 2 * kDcRows * kPk, kT = kK + 2 * kDcRows * kPk, kM = kT + 2 * kDcRows * kDcPitch,
                        kS = kM + 2 * kDcRows * kDcPitch;
-  static constexpr int kSBytes = 2 * (DK > kDcRows ? DK : kDcRows) * kPv;          // S, later the decayed U
-  static constexpr int kU = kS + kSBytes;
-  static constexpr int kVPitch = DVT * 4 + 16;                                     // V in fp32, later R and U
-  static constexpr int kUBytes = 2 * kDcRows * kPv > kDcRows * kVPitch ? 2 * kDcRows * kPv : kDcRows * kVPitch;
-  static constexpr int kTotal = kU + kUBytes;
+  static constexpr int kU = kS + 2 * (DK > kDcRows ? DK : kDcRows) * kPv;          // S, later the decayed U; then R, later U
+  static constexpr int kV = kU + 2 * kDcRows * kPv;
+  static constexpr int kTotal = kV + kDcRows * kPv;
 };
 
-template <int DK, int DVT, bool FUSE>
-__global__ void __launch_bounds__(256, 1) delta_state_kernel(const DeltaChunkParams p) {
+// 8 * WN warps: warp = (row tile wr, column group wn).  Products with 64 rows and those with the state's rows are dealt so
+// that every warp has part of each.
+template <int DK, int DVT, int WN, bool FUSE>
+__global__ void __launch_bounds__(256 * WN, 1) delta_state_kernel(const DeltaChunkParams p) {
   using L = DeltaStateSmem<DK, DVT>;
-  constexpr int NT = DVT / 8, kPk = L::kPk, kPv = L::kPv;
-  constexpr int N4 = DK == 128 ? NT : NT / 2;      // state columns (in eights) per warp
+  constexpr int kThreads = 256 * WN, kPk = L::kPk, kPv = L::kPv;
+  constexpr int NT = DVT / 8 / WN;                 // octets of columns per warp: K S, Q S, M U
+  constexpr int N2 = NT / 2;                       // ... T R (twice as many warps per row tile)
+  constexpr int N4 = DK == 128 ? NT : NT / 2;      // ... the state
+  static_assert(N2 >= 2 && N2 % 2 == 0, "column octets come in pairs");
   extern __shared__ __align__(16) unsigned char sm[];
-  __shared__ float s_eg[kDcRows], s_ec[kDcRows], s_last;
+  __shared__ float s_eg[kDcRows], s_ec[kDcRows], s_ss[WN][kDcRows], s_last;
   const int ps = blockIdx.z, s = ps + p.n_decode, h = blockIdx.y, c0 = blockIdx.x * DVT, hk = h / (p.heads / p.kv_heads);
   const int len = p.cu[s + 1] - p.cu[s], n_chunks = (len + kDcRows - 1) / kDcRows, chunk0 = p.chunk_off[ps];
   const long long row0 = (long long)p.cu[s] - p.n_decode;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3, wr = warp & 7, wn = warp >> 3;
   const uint32_t base = (uint32_t)__cvta_generic_to_shared(sm);
 
   auto load_qk = [&](int ch, bool key) {           // q or k rows of chunk ch, hi and lo
     constexpr int vecs = DK / 8;
     const int n = min(kDcRows, len - ch * kDcRows);
-    for (int i = threadIdx.x; i < 2 * kDcRows * vecs; i += 256) {
+    for (int i = threadIdx.x; i < 2 * kDcRows * vecs; i += kThreads) {
       const int plane = i / (kDcRows * vecs), r = i / vecs % kDcRows, c = i % vecs;
       const bool on = r < n;
       const __nv_bfloat16* src = p.qk + (((row0 + ch * kDcRows + (on ? r : 0)) * 4 + (key ? 2 : 0) + plane) * p.kv_heads + hk) * DK + c * 8;
@@ -221,23 +227,24 @@ __global__ void __launch_bounds__(256, 1) delta_state_kernel(const DeltaChunkPar
   };
   auto load_tm = [&](int ch, bool m) {
     const __nv_bfloat16* src = p.tm + (((long long)(chunk0 + ch) * p.heads + h) * 4 + (m ? 2 : 0)) * kDcTile;
-    for (int i = threadIdx.x; i < 2 * kDcRows * 8; i += 256)
+    for (int i = threadIdx.x; i < 2 * kDcRows * 8; i += kThreads)
       cp_async16(base + (m ? L::kM : L::kT) + (i >> 3) * kDcPitch + (i & 7) * 16, src + (long long)i * 8, 16u);
   };
   auto load_v = [&](int ch) {
-    constexpr int vecs = DVT / 4;
+    constexpr int vecs = DVT / 8;
     const int n = min(kDcRows, len - ch * kDcRows);
-    for (int i = threadIdx.x; i < kDcRows * vecs; i += 256) {
+    for (int i = threadIdx.x; i < kDcRows * vecs; i += kThreads) {
       const int r = i / vecs, c = i % vecs;
       const bool on = r < n;
-      cp_async16(base + L::kU + r * L::kVPitch + c * 16,
-                 p.v + (row0 + ch * kDcRows + (on ? r : 0)) * p.heads * p.vdim + (long long)h * p.vdim + c0 + c * 4, on ? 16u : 0u);
+      cp_async16(base + L::kV + r * kPv + c * 16,
+                 p.v + (row0 + ch * kDcRows + (on ? r : 0)) * p.heads * p.vdim + (long long)h * p.vdim + c0 + c * 8, on ? 16u : 0u);
     }
   };
   if (n_chunks > 0) { load_qk(0, false); load_qk(0, true); load_tm(0, false); load_tm(0, true); load_v(0); }
   cp_async_commit();
 
-  const int sm_tile = DK == 128 ? warp : warp & 3, sn0 = DK == 128 ? 0 : (warp >> 2) * N4;   // this warp's part of the state
+  const int sm_tile = DK == 128 ? wr : wr & 3;                                        // this warp's part of the state
+  const int sn0 = DK == 128 ? wn * NT : (wn * 2 + (wr >> 2)) * N4;
   float* state = p.state + (((long long)p.slot[s] * p.heads + h) * DK + sm_tile * 16 + g) * p.vdim + c0 + sn0 * 8 + tq * 2;
   float st[N4][4];
   const bool fresh = p.start[s] == 0;
@@ -251,7 +258,7 @@ __global__ void __launch_bounds__(256, 1) delta_state_kernel(const DeltaChunkPar
     st[j][0] = a.x; st[j][1] = a.y; st[j][2] = b.x; st[j][3] = b.y;
   }
   constexpr int kSLo = DK * kPv, kULo = kDcRows * kPv, kQLo = kDcRows * kPk, kTLo = kDcRows * kDcPitch;
-  // 16 x 8 accumulator tiles to a hi / lo pair of bf16 planes
+  // a 16 x 8 accumulator tile to a hi / lo pair of bf16 planes
   auto put = [&](int region, int lo_off, int row, int col8, const float (&v)[4], float f0, float f1) {
     uint32_t hi, lo;
     split2(v[0] * f0, v[1] * f0, hi, lo);
@@ -266,8 +273,24 @@ __global__ void __launch_bounds__(256, 1) delta_state_kernel(const DeltaChunkPar
 #pragma unroll
   for (int j = 0; j < N4; ++j) put(L::kS, kSLo, sm_tile * 16 + g, sn0 + j, st[j], 1.f, 1.f);
 
-  const uint32_t a_off = (lane & 15), a_col = (lane >> 4) * 16;                       // A operand, rows as stored
+  const uint32_t a_off = (lane & 15), a_col = (lane >> 4) * 16;                         // A operand, rows as stored
   const uint32_t t_row = (lane & 7) + ((lane >> 3) & 1) * 8, t_col = (lane >> 4) * 16;  // B operand by transposition: 16 rows x 16 columns
+  // one reduction step of 16: c[0 .. n) += (ah + al) (hi + lo of the B region), without lo * lo
+  auto step16 = [&](float (*c)[4], int n, const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t b, int lo_off) {
+#pragma unroll
+    for (int j = 0; j < n; j += 2) {
+      uint32_t bh[4], bl[4];
+      ldmatrix_x4_trans(b + j * 16, bh[0], bh[1], bh[2], bh[3]);
+      ldmatrix_x4_trans(b + lo_off + j * 16, bl[0], bl[1], bl[2], bl[3]);
+      mma_bf16_acc(c[j], al, bh[0], bh[1]);
+      mma_bf16_acc(c[j + 1], al, bh[2], bh[3]);
+      mma_bf16_acc(c[j], ah, bl[0], bl[1]);
+      mma_bf16_acc(c[j + 1], ah, bl[2], bl[3]);
+      mma_bf16_acc(c[j], ah, bh[0], bh[1]);
+      mma_bf16_acc(c[j + 1], ah, bh[2], bh[3]);
+    }
+  };
+  const int r0 = (wr & 3) * 16 + g;
   for (int ch = 0; ch < n_chunks; ++ch) {
     if (threadIdx.x < kDcRows) {
       const float* gc = p.gcum + ((long long)(chunk0 + ch) * p.heads + h) * kDcRows;
@@ -278,83 +301,66 @@ __global__ void __launch_bounds__(256, 1) delta_state_kernel(const DeltaChunkPar
     }
     cp_async_wait<0>();
     __syncthreads();
-    // K S (warps 0-3) and Q S (warps 4-7), 16 rows each
+    const bool more = ch + 1 < n_chunks;
+    // K S (row tiles 0-3) and Q S (row tiles 4-7)
     float acc[NT][4];
 #pragma unroll
     for (int j = 0; j < NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
     {
-      const uint32_t a_base = base + (warp < 4 ? L::kK : L::kQ) + ((warp & 3) * 16 + a_off) * kPk + a_col;
-      const uint32_t b_base = base + L::kS + t_row * kPv + t_col;
+      const uint32_t a_base = base + (wr < 4 ? L::kK : L::kQ) + ((wr & 3) * 16 + a_off) * kPk + a_col;
+      const uint32_t b_base = base + L::kS + t_row * kPv + wn * NT * 16 + t_col;
 #pragma unroll 2
       for (int k = 0; k < DK / 16; ++k) {
         uint32_t ah[4], al[4];
         ldmatrix_x4(a_base + k * 32, ah[0], ah[1], ah[2], ah[3]);
         ldmatrix_x4(a_base + kQLo + k * 32, al[0], al[1], al[2], al[3]);
-#pragma unroll
-        for (int j = 0; j < NT; j += 2) {
-          uint32_t bh[4], bl[4];
-          ldmatrix_x4_trans(b_base + k * 16 * kPv + j * 16, bh[0], bh[1], bh[2], bh[3]);
-          ldmatrix_x4_trans(b_base + kSLo + k * 16 * kPv + j * 16, bl[0], bl[1], bl[2], bl[3]);
-#pragma unroll
-          for (int n = 0; n < 2; ++n) {
-            mma_bf16_acc(acc[j + n], al, bh[2 * n], bh[2 * n + 1]);
-            mma_bf16_acc(acc[j + n], ah, bl[2 * n], bl[2 * n + 1]);
-            mma_bf16_acc(acc[j + n], ah, bh[2 * n], bh[2 * n + 1]);
-          }
-        }
+        step16(acc, NT, ah, al, b_base + k * 16 * kPv, kSLo);
       }
     }
-    const int r0 = (warp & 3) * 16 + g;
+    __nv_bfloat162 gate[FUSE ? 2 : 1][FUSE ? NT : 1];
     {
       const float e0 = s_eg[r0], e1 = s_eg[r0 + 8];
-      if (warp < 4) {                               // R = V - e^G K S
-        const float* v0 = reinterpret_cast<const float*>(sm + L::kU + r0 * L::kVPitch) + tq * 2;
-        const float* v1 = reinterpret_cast<const float*>(sm + L::kU + (r0 + 8) * L::kVPitch) + tq * 2;
+      if (wr < 4) {                                 // R = V - e^G K S
+        const unsigned char* v0 = sm + L::kV + r0 * kPv + (wn * NT * 8 + tq * 2) * 2;
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
-          const float2 a = *reinterpret_cast<const float2*>(v0 + j * 8), b = *reinterpret_cast<const float2*>(v1 + j * 8);
+          const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(v0 + j * 16));
+          const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(v0 + 8 * kPv + j * 16));
           acc[j][0] = fmaf(-e0, acc[j][0], a.x); acc[j][1] = fmaf(-e0, acc[j][1], a.y);
           acc[j][2] = fmaf(-e1, acc[j][2], b.x); acc[j][3] = fmaf(-e1, acc[j][3], b.y);
+          put(L::kU, kULo, r0, wn * NT + j, acc[j], 1.f, 1.f);
         }
       } else {
 #pragma unroll
         for (int j = 0; j < NT; ++j) { acc[j][0] *= e0; acc[j][1] *= e0; acc[j][2] *= e1; acc[j][3] *= e1; }
+        if constexpr (FUSE) {                       // the output's gates, needed at the end of the chunk
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int t = ch * kDcRows + r0 + 8 * e;
+            const __nv_bfloat16* src = p.gate + (row0 + (t < len ? t : 0)) * p.gate_stride + (long long)h * DVT + wn * NT * 8 + tq * 2;
+#pragma unroll
+            for (int j = 0; j < NT; ++j) gate[e][j] = *reinterpret_cast<const __nv_bfloat162*>(src + j * 8);
+          }
+        }
       }
     }
-    __syncthreads();                                // S, Q and V have been read
-    const bool more = ch + 1 < n_chunks;
-    if (more) load_qk(ch + 1, false);
-    if (warp < 4) {
+    __syncthreads();                                // S, Q and V have been read, R is there
+    if (more) { load_qk(ch + 1, false); load_v(ch + 1); }
+    // U = T R
+    float u[N2][4];
+    const int un0 = (wn * 2 + (wr >> 2)) * N2;
 #pragma unroll
-      for (int j = 0; j < NT; ++j) put(L::kU, kULo, r0, j, acc[j], 1.f, 1.f);
-    }
-    __syncthreads();
-    // U = T R: row tile warp & 3, half of the columns
-    float u[NT / 2][4];
-    const int un0 = (warp >> 2) * (NT / 2);
-#pragma unroll
-    for (int j = 0; j < NT / 2; ++j) u[j][0] = u[j][1] = u[j][2] = u[j][3] = 0.f;
+    for (int j = 0; j < N2; ++j) u[j][0] = u[j][1] = u[j][2] = u[j][3] = 0.f;
     {
-      const uint32_t a_base = base + L::kT + ((warp & 3) * 16 + a_off) * kDcPitch + a_col;
+      const uint32_t a_base = base + L::kT + ((wr & 3) * 16 + a_off) * kDcPitch + a_col;
       const uint32_t b_base = base + L::kU + t_row * kPv + un0 * 16 + t_col;
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
-        if (k > (warp & 3)) break;                  // T is lower triangular
+        if (k > (wr & 3)) break;                    // T is lower triangular
         uint32_t ah[4], al[4];
         ldmatrix_x4(a_base + k * 32, ah[0], ah[1], ah[2], ah[3]);
         ldmatrix_x4(a_base + kTLo + k * 32, al[0], al[1], al[2], al[3]);
-#pragma unroll
-        for (int j = 0; j < NT / 2; j += 2) {
-          uint32_t bh[4], bl[4];
-          ldmatrix_x4_trans(b_base + k * 16 * kPv + j * 16, bh[0], bh[1], bh[2], bh[3]);
-          ldmatrix_x4_trans(b_base + kULo + k * 16 * kPv + j * 16, bl[0], bl[1], bl[2], bl[3]);
-#pragma unroll
-          for (int n = 0; n < 2; ++n) {
-            mma_bf16_acc(u[j + n], al, bh[2 * n], bh[2 * n + 1]);
-            mma_bf16_acc(u[j + n], ah, bl[2 * n], bl[2 * n + 1]);
-            mma_bf16_acc(u[j + n], ah, bh[2 * n], bh[2 * n + 1]);
-          }
-        }
+        step16(u, N2, ah, al, b_base + k * 16 * kPv, kULo);
       }
     }
     __syncthreads();                                // R and T have been read
@@ -362,32 +368,32 @@ __global__ void __launch_bounds__(256, 1) delta_state_kernel(const DeltaChunkPar
     {
       const float d0 = s_ec[r0], d1 = s_ec[r0 + 8];
 #pragma unroll
-      for (int j = 0; j < NT / 2; ++j) {
+      for (int j = 0; j < N2; ++j) {
         put(L::kU, kULo, r0, un0 + j, u[j], 1.f, 1.f);
         put(L::kS, kSLo, r0, un0 + j, u[j], d0, d1);   // decayed to the end of the chunk
       }
     }
     __syncthreads();
-    if (warp >= 4) {                                // O += M U
-      const uint32_t a_base = base + L::kM + ((warp & 3) * 16 + a_off) * kDcPitch + a_col;
-      const uint32_t b_base = base + L::kU + t_row * kPv + t_col;
+    if (wr >= 4) {                                  // O += M U
+      const uint32_t a_base = base + L::kM + ((wr & 3) * 16 + a_off) * kDcPitch + a_col;
+      const uint32_t b_base = base + L::kU + t_row * kPv + wn * NT * 16 + t_col;
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
-        if (k > (warp & 3)) break;
+        if (k > (wr & 3)) break;
         uint32_t ah[4], al[4];
         ldmatrix_x4(a_base + k * 32, ah[0], ah[1], ah[2], ah[3]);
         ldmatrix_x4(a_base + kTLo + k * 32, al[0], al[1], al[2], al[3]);
+        step16(acc, NT, ah, al, b_base + k * 16 * kPv, kULo);
+      }
+      if constexpr (FUSE) {
 #pragma unroll
-        for (int j = 0; j < NT; j += 2) {
-          uint32_t bh[4], bl[4];
-          ldmatrix_x4_trans(b_base + k * 16 * kPv + j * 16, bh[0], bh[1], bh[2], bh[3]);
-          ldmatrix_x4_trans(b_base + kULo + k * 16 * kPv + j * 16, bl[0], bl[1], bl[2], bl[3]);
+        for (int e = 0; e < 2; ++e) {
+          float ss = 0.f;
 #pragma unroll
-          for (int n = 0; n < 2; ++n) {
-            mma_bf16_acc(acc[j + n], al, bh[2 * n], bh[2 * n + 1]);
-            mma_bf16_acc(acc[j + n], ah, bl[2 * n], bl[2 * n + 1]);
-            mma_bf16_acc(acc[j + n], ah, bh[2 * n], bh[2 * n + 1]);
-          }
+          for (int j = 0; j < NT; ++j) ss += acc[j][2 * e] * acc[j][2 * e] + acc[j][2 * e + 1] * acc[j][2 * e + 1];
+          ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+          ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+          if (tq == 0) s_ss[wn][r0 + 8 * e] = ss;
         }
       }
     }
@@ -403,52 +409,37 @@ __global__ void __launch_bounds__(256, 1) delta_state_kernel(const DeltaChunkPar
         uint32_t ah[4], al[4];
         ldmatrix_x4_trans(a_base + k * 16 * kPk, ah[0], ah[1], ah[2], ah[3]);
         ldmatrix_x4_trans(a_base + kQLo + k * 16 * kPk, al[0], al[1], al[2], al[3]);
-#pragma unroll
-        for (int j = 0; j < N4; j += 2) {
-          uint32_t bh[4], bl[4];
-          ldmatrix_x4_trans(b_base + k * 16 * kPv + j * 16, bh[0], bh[1], bh[2], bh[3]);
-          ldmatrix_x4_trans(b_base + kSLo + k * 16 * kPv + j * 16, bl[0], bl[1], bl[2], bl[3]);
-#pragma unroll
-          for (int n = 0; n < 2; ++n) {
-            mma_bf16_acc(st[j + n], al, bh[2 * n], bh[2 * n + 1]);
-            mma_bf16_acc(st[j + n], ah, bl[2 * n], bl[2 * n + 1]);
-            mma_bf16_acc(st[j + n], ah, bh[2 * n], bh[2 * n + 1]);
-          }
-        }
+        step16(st, N4, ah, al, b_base + k * 16 * kPv, kSLo);
       }
     }
     __syncthreads();                                // K, M, U and the decayed U have been read
-    if (more) { load_qk(ch + 1, true); load_tm(ch + 1, true); load_v(ch + 1); }
+    if (more) { load_qk(ch + 1, true); load_tm(ch + 1, true); }
     cp_async_commit();
     if (more) {
 #pragma unroll
       for (int j = 0; j < N4; ++j) put(L::kS, kSLo, sm_tile * 16 + g, sn0 + j, st[j], 1.f, 1.f);
     }
-    if (warp >= 4) {                                // rows r0, r0 + 8 of the chunk
+    if (wr >= 4) {                                  // rows r0, r0 + 8 of the chunk
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int t = ch * kDcRows + r0 + 8 * e;
+        if (t >= len) continue;
         if constexpr (FUSE) {
           float ss = 0.f;
 #pragma unroll
-          for (int j = 0; j < NT; ++j) ss += acc[j][2 * e] * acc[j][2 * e] + acc[j][2 * e + 1] * acc[j][2 * e + 1];
-          ss += __shfl_xor_sync(0xffffffffu, ss, 1);
-          ss += __shfl_xor_sync(0xffffffffu, ss, 2);
-          if (t < len) {
-            const float inv = 1.f / sqrtf(ss / (float)DVT + p.eps);
-            const __nv_bfloat16* gate = p.gate + (row0 + t) * p.gate_stride + (long long)h * DVT + tq * 2;
-            __nv_bfloat16* out = p.out + (row0 + t) * p.out_stride + (long long)h * DVT + tq * 2;
+          for (int w = 0; w < WN; ++w) ss += s_ss[w][r0 + 8 * e];
+          const float inv = 1.f / sqrtf(ss / (float)DVT + p.eps);
+          __nv_bfloat16* out = p.out + (row0 + t) * p.out_stride + (long long)h * DVT + wn * NT * 8 + tq * 2;
 #pragma unroll
-            for (int j = 0; j < NT; ++j) {
-              const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + j * 8));
-              const float2 w = *reinterpret_cast<const float2*>(p.w_norm + j * 8 + tq * 2);
-              *reinterpret_cast<__nv_bfloat162*>(out + j * 8) =
-                  __floats2bfloat162_rn(acc[j][2 * e] * inv * w.x * __fdividef(z.x, 1.f + __expf(-z.x)),
-                                        acc[j][2 * e + 1] * inv * w.y * __fdividef(z.y, 1.f + __expf(-z.y)));
-            }
+          for (int j = 0; j < NT; ++j) {
+            const float2 z = __bfloat1622float2(gate[e][j]);
+            const float2 w = *reinterpret_cast<const float2*>(p.w_norm + (wn * NT + j) * 8 + tq * 2);
+            *reinterpret_cast<__nv_bfloat162*>(out + j * 8) =
+                __floats2bfloat162_rn(acc[j][2 * e] * inv * w.x * __fdividef(z.x, 1.f + __expf(-z.x)),
+                                      acc[j][2 * e + 1] * inv * w.y * __fdividef(z.y, 1.f + __expf(-z.y)));
           }
-        } else if (t < len) {
-          float* o = p.o + ((row0 + t) * p.heads + h) * p.vdim + c0 + tq * 2;
+        } else {
+          float* o = p.o + ((row0 + t) * p.heads + h) * p.vdim + c0 + wn * NT * 8 + tq * 2;
 #pragma unroll
           for (int j = 0; j < NT; ++j) *reinterpret_cast<float2*>(o + j * 8) = make_float2(acc[j][2 * e], acc[j][2 * e + 1]);
         }
@@ -465,8 +456,8 @@ __global__ void __launch_bounds__(256, 1) delta_state_kernel(const DeltaChunkPar
 
 template <int DK>
 int launch_delta_chunk(const DeltaChunkParams& p, cudaStream_t stream) {
-  constexpr size_t smem = (size_t)4 * kDcRows * (DK * 2 + 16) + 2 * kDcRows * 65 * 4;
-  static_assert(4 * kDcRows * (DK * 2 + 16) >= kDcRows * 68 * 4, "the triangular matrix lies over the operands");
+  constexpr size_t operands = (size_t)4 * kDcRows * (DK * 2 + 16), square = (size_t)kDcRows * (68 + 65 + 65) * 4;
+  constexpr size_t smem = operands > square ? operands : square;
   static DeviceSmem configured{};
   MSA_OK_OR_RETURN(ensure_dynamic_smem(delta_chunk_kernel<DK>, smem, configured));
   delta_chunk_kernel<DK><<<dim3((unsigned)p.n_chunks, (unsigned)p.kv_heads), 128, smem, stream>>>(p);
@@ -476,11 +467,12 @@ int launch_delta_chunk(const DeltaChunkParams& p, cudaStream_t stream) {
 template <int DK, int DVT, bool FUSE>
 int launch_delta_state(const DeltaChunkParams& p, cudaStream_t stream) {
   constexpr size_t smem = DeltaStateSmem<DK, DVT>::kTotal;
+  constexpr int WN = DVT >= 64 ? 2 : 1;
   static_assert(smem <= 226 * 1024, "shared memory");
   static DeviceSmem configured{};
-  MSA_OK_OR_RETURN(ensure_dynamic_smem(delta_state_kernel<DK, DVT, FUSE>, smem, configured));
+  MSA_OK_OR_RETURN(ensure_dynamic_smem(delta_state_kernel<DK, DVT, WN, FUSE>, smem, configured));
   const dim3 grid((unsigned)(p.vdim / DVT), (unsigned)p.heads, (unsigned)(p.n_seq - p.n_decode));
-  delta_state_kernel<DK, DVT, FUSE><<<grid, 256, smem, stream>>>(p);
+  delta_state_kernel<DK, DVT, WN, FUSE><<<grid, 256 * WN, smem, stream>>>(p);
   MSA_LAUNCH_OK("delta_state_kernel");
   return MSA_OK;
 }
@@ -496,7 +488,7 @@ extern "C" int64_t msa_lm_delta_chunk_workspace(int32_t n_chunks, int32_t heads)
   return (int64_t)n_chunks * heads * (4 * kDcTile * 2 + kDcRows * 4);
 }
 
-extern "C" int msa_lm_delta_chunk(const msa_lm_delta_args* a, const void* qk, const float* v, const float* gates,
+extern "C" int msa_lm_delta_chunk(const msa_lm_delta_args* a, const void* qk, const void* v, const float* gates,
                                   const int32_t* chunk_off, int32_t n_chunks, int32_t tile, void* workspace, float* o,
                                   void* out, int64_t out_stride, void* stream) {
   MSA_REQUIRE(a && qk && v && gates && chunk_off && workspace && out, "delta_chunk: null pointer");
@@ -508,7 +500,7 @@ extern "C" int msa_lm_delta_chunk(const msa_lm_delta_args* a, const void* qk, co
                   a->proj_stride % 2 == 0 && out_stride % 2 == 0 && (a->vdim == tile || o), "delta_chunk: alignment");
   if (a->n_seq == a->n_decode || n_chunks <= 0) return MSA_OK;
   DeltaChunkParams p{};
-  p.qk = (const __nv_bfloat16*)qk; p.v = v; p.gates = gates;
+  p.qk = (const __nv_bfloat16*)qk; p.v = (const __nv_bfloat16*)v; p.gates = gates;
   p.slot = a->slot; p.start = a->start; p.cu = a->cu; p.chunk_off = chunk_off;
   p.n_decode = a->n_decode; p.n_seq = a->n_seq; p.heads = a->heads; p.kv_heads = a->kv_heads; p.dim = a->dim; p.vdim = a->vdim;
   p.n_chunks = n_chunks;

@@ -71,6 +71,72 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
   }
 }
 
+// The same with four elements per access (sizes and strides multiples of 4, rank <= 512): the latent's row is in
+// registers before the token's angles are computed, and the heads' rotated parts are turned two pairs at a time.
+template <typename T>
+__global__ void __launch_bounds__(128) latent_prep_vec_kernel(const LatentPrepParams p) {
+  __shared__ float s_part[32];
+  extern __shared__ float2 s_turn[];
+  const int width = p.rank + p.rot, tid = threadIdx.x;
+  if ((int)blockIdx.x >= p.n_tok) {
+    const int o = (int)blockIdx.x - p.n_tok;
+    const int ps = owner_of(p.old_off, p.n_seq - p.n_decode, o), s = ps + p.n_decode;
+    const int k = o - p.old_off[ps], start = p.start[s];
+    const int first = start - min(start, p.window - 1);
+    const T* src = reinterpret_cast<const T*>(p.ring) + ((long long)p.slot[s] * p.ring_rows + (first + k) % (int)p.ring_rows) * width;
+    T* dst = reinterpret_cast<T*>(p.ctx) + (long long)(p.ctx_off[ps] + k) * width;
+    for (int i = tid * 4; i < width; i += 512) store4(dst + i, load4(src + i));
+    return;
+  }
+  const int n = blockIdx.x, s = p.tok_seq[n], pos = p.pos[n], half = p.rot / 2, hd = p.dim + p.rot;
+  T* row = reinterpret_cast<T*>(p.proj) + (long long)n * p.proj_stride;
+  const T* lat = row + p.heads * hd;
+  const bool on = tid * 4 < p.rank, turns = tid * 4 < p.rot;
+  const float4 c = on ? load4(lat + tid * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+  const float4 w = on ? load4(p.w_norm + tid * 4) : c;
+  float4 kr = turns ? load4(lat + p.rank + tid * 4) : c;
+  const int per_head = p.rot / 4, quads = p.heads * per_head;
+  constexpr int kAhead = 4;
+  float4 q[kAhead];
+#pragma unroll
+  for (int u = 0; u < kAhead; ++u) {
+    const int i = tid + u * 128;
+    if (i < quads) { const int h = i / per_head; q[u] = load4(row + h * hd + p.dim + (i - h * per_head) * 4); }
+  }
+  T* dst;
+  if (n < p.n_decode) {
+    dst = reinterpret_cast<T*>(p.ring) + ((long long)p.slot[s] * p.ring_rows + pos % (int)p.ring_rows) * width;
+  } else {
+    const int start = p.start[s];
+    dst = reinterpret_cast<T*>(p.ctx) + (long long)(p.ctx_off[s - p.n_decode] + min(start, p.window - 1) + (n - p.cu[s])) * width;
+  }
+  for (int j = tid; j < half; j += 128) {
+    float sn, cs;
+    sincosf((float)pos * p.inv_freq[j], &sn, &cs);
+    s_turn[j] = make_float2(cs, sn);
+  }
+  const float inv = 1.f / sqrtf(block_sum(c.x * c.x + c.y * c.y + c.z * c.z + c.w * c.w, s_part) / (float)p.rank + p.eps);
+  if (on) store4(dst + tid * 4, make_float4(c.x * inv * w.x, c.y * inv * w.y, c.z * inv * w.z, c.w * inv * w.w));
+  auto turn = [&](float4 x, int pair) {
+    const float2 a = s_turn[pair], b = s_turn[pair + 1];
+    return make_float4(x.x * a.x - x.y * a.y, x.y * a.x + x.x * a.y, x.z * b.x - x.w * b.y, x.w * b.x + x.z * b.y);
+  };
+  for (int i = tid * 4; i < p.rot; i += 512) {
+    if (i != tid * 4) kr = load4(lat + p.rank + i);
+    store4(dst + p.rank + i, turn(kr, i / 2));
+  }
+#pragma unroll
+  for (int u = 0; u < kAhead; ++u) {
+    const int i = tid + u * 128;
+    if (i < quads) { const int h = i / per_head, j = i - h * per_head; store4(row + h * hd + p.dim + j * 4, turn(q[u], 2 * j)); }
+  }
+  for (int i = tid + kAhead * 128; i < quads; i += 128) {
+    const int h = i / per_head, j = i - h * per_head;
+    T* at = row + h * hd + p.dim + j * 4;
+    store4(at, turn(load4(at), 2 * j));
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 ring_store_kernel(const T* __restrict__ ctx, int width, const int32_t* slot, const int32_t* start, const int32_t* cu,
@@ -188,6 +254,14 @@ extern "C" int msa_lm_latent_prep(void* proj, int64_t proj_stride, const float* 
   if (n_tok == 0) return MSA_OK;
   LatentPrepParams p{proj, proj_stride, w_norm, eps, inv_freq, heads, dim, rot, rank, pos, tok_seq, slot, start, cu, ctx_off,
                      old_off, n_tok, n_seq, n_decode, window, ring, ring_rows, ctx};
+  const int e4 = 4 * (int)dtype_size(dtype);
+  auto ok4 = [&](const void* q) { return q == nullptr || reinterpret_cast<uintptr_t>(q) % e4 == 0; };
+  if (dim % 4 == 0 && rot % 4 == 0 && rank % 4 == 0 && rank <= 512 && proj_stride % 4 == 0 && ok4(proj) && ok4(ring) && ok4(ctx) &&
+      aligned16(w_norm) && ring_rows < (1ll << 31)) {
+    MSA_LM_DISPATCH(dtype, { latent_prep_vec_kernel<T><<<n_tok + n_old, 128, (size_t)rot * 4, (cudaStream_t)stream>>>(p); });
+    MSA_LAUNCH_OK("latent_prep_vec_kernel");
+    return MSA_OK;
+  }
   MSA_LM_DISPATCH(dtype, { latent_prep_kernel<T><<<n_tok + n_old, 128, (size_t)rot * 4, (cudaStream_t)stream>>>(p); });
   MSA_LAUNCH_OK("latent_prep_kernel");
   return MSA_OK;

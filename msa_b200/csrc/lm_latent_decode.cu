@@ -2,16 +2,16 @@
 // [latent | rotated key part]; the values are the latents themselves.  Flash-decode: the visible rows of a sequence are
 // split over CTAs, partial results are merged by a second kernel.
 //
-// One CTA = up to 32 heads x one split, 256 threads.  The queries stay in shared memory; 64-row tiles of the ring are
+// One CTA = up to 32 heads x one split, 512 threads.  The queries stay in shared memory; 64-row tiles of the ring are
 // double-buffered with cp.async (rows are read once from HBM for all heads, which is what bounds this kernel); scores and
-// output on mma.sync.m16n8k16, softmax in fp32.  Warps split the scores over keys (and the two 16-head tiles) and the
-// output over latent columns.
+// output on mma.sync.m16n8k16, softmax in fp32.  Warps split the scores over octets of keys and the two 16-head tiles (with
+// one head tile: over the two halves of the reduction), and the output over latent columns.
 #include "lm_common.cuh"
 #include "mma_helpers.cuh"
 
 namespace msa {
 
-constexpr int kLdThreads = 256, kLdKeys = 64, kLdPPitch = 144;   // P rows: 64 bf16 + 16 bytes of padding
+constexpr int kLdThreads = 512, kLdKeys = 64, kLdPPitch = 144;   // P rows: 64 bf16 + 16 bytes of padding
 
 struct LatentDecodeParams {
   const __nv_bfloat16* qa; long long qa_row, qa_head;
@@ -29,11 +29,17 @@ __device__ __forceinline__ void mma_bf16_full(float (&c)[4], const uint32_t (&a)
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+__device__ __forceinline__ void ldmatrix_x2_trans(uint32_t addr, uint32_t& r0, uint32_t& r1) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
+}
+
+// MT: 16-head tiles; NT: octets of latent columns per warp (rank / 128).
 template <int MT, int NT>
 __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LatentDecodeParams p) {
   extern __shared__ __align__(16) unsigned char sm[];
   __shared__ float s_max[8][32], s_sum[8][32];
-  constexpr int kParts = 8 / MT;                    // warps that share a head tile's keys
+  __shared__ float4 s_half[MT == 1 ? 256 : 1];      // one head tile: scores of the second half of the reduction
+  constexpr int kParts = 8;                         // octets of keys of a tile
   const int width = p.rank + p.rot, pitch = width * 2 + 16, vecs = width / 8;
   unsigned char* s_q = sm;                          // [MT*16][pitch]
   unsigned char* s_p = s_q + MT * 16 * pitch;       // [MT*16][kLdPPitch]
@@ -71,12 +77,13 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
                      : *reinterpret_cast<const uint4*>(p.qb + b * p.qb_row + h * p.qb_head + (c - p.rank));
     *reinterpret_cast<uint4*>(s_q + r * pitch + c * 2) = v;
   }
-  const int mt = warp % MT, part = warp / MT, g = lane >> 2, tq = lane & 3;
+  const int mt = MT == 2 ? warp & 1 : 0, part = MT == 2 ? warp >> 1 : warp & 7, half = MT == 2 ? 0 : warp >> 3;
+  const int steps = width / 32, ks0 = half == 0 ? 0 : steps / 2 * 32, ks1 = MT == 1 && half == 0 ? steps / 2 * 32 : width;
+  const int g = lane >> 2, tq = lane & 3;
   const uint32_t q_addr = (uint32_t)__cvta_generic_to_shared(s_q) + (mt * 16 + (lane & 15)) * pitch + (lane >> 4) * 16;
   const uint32_t p_addr = (uint32_t)__cvta_generic_to_shared(s_p) + (lane & 15) * kLdPPitch + (lane >> 4) * 16;
-  // scores: MT key octets per warp (MT = 2: keys 16*part .. +15; MT = 1: keys 8*part .. +7, two reduction steps per load)
-  const int brow = MT == 2 ? part * 16 + (lane & 7) + ((lane >> 4) << 3) : part * 8 + (lane & 7);
-  const int bcol = MT == 2 ? ((lane >> 3) & 1) * 16 : (lane >> 3) * 16;
+  // scores: keys 8*part .. +7 of the tile, two reduction steps per load
+  const int brow = part * 8 + (lane & 7), bcol = (lane >> 3) * 16;
   float acc[MT][NT][4];
   float m_run[MT][2], l_run[MT][2];
 #pragma unroll
@@ -90,50 +97,42 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     if (t + 1 < n_tiles) { load_tile(t + 1); cp_async_wait<1>(); } else cp_async_wait<0>();
     __syncthreads();
     const uint32_t kb = (uint32_t)__cvta_generic_to_shared(s_k + (t & 1) * kLdKeys * pitch);
-    float s[MT][4], s2[MT][4];            // two chains per tile, added below
-#pragma unroll
-    for (int j = 0; j < MT; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) s[j][e] = s2[j][e] = 0.f;
+    float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};            // two chains, added below
     const uint32_t b_addr = kb + brow * pitch + bcol;
-#pragma unroll 4
-    for (int k = 0; k < width; k += 32) {
-      uint32_t a[4], a2[4], x[4], y[4];
+#pragma unroll 3
+    for (int k = ks0; k < ks1; k += 32) {
+      uint32_t a[4], a2[4], x[4];
       ldmatrix_x4(q_addr + k * 2, a[0], a[1], a[2], a[3]);
       ldmatrix_x4(q_addr + k * 2 + 32, a2[0], a2[1], a2[2], a2[3]);
       ldmatrix_x4(b_addr + k * 2, x[0], x[1], x[2], x[3]);
-      if constexpr (MT == 2) {
-        ldmatrix_x4(b_addr + k * 2 + 32, y[0], y[1], y[2], y[3]);
-        mma_bf16_full(s[0], a, x[0], x[1]);
-        mma_bf16_full(s[1], a, x[2], x[3]);
-        mma_bf16_full(s2[0], a2, y[0], y[1]);
-        mma_bf16_full(s2[1], a2, y[2], y[3]);
-      } else {
-        mma_bf16_full(s[0], a, x[0], x[1]);
-        mma_bf16_full(s2[0], a2, x[2], x[3]);
-      }
+      mma_bf16_full(s, a, x[0], x[1]);
+      mma_bf16_full(s2, a2, x[2], x[3]);
     }
 #pragma unroll
-    for (int j = 0; j < MT; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) s[j][e] += s2[j][e];
-    // s[j][0..1]: row g, keys (octet j of this warp) 2*tq, 2*tq+1; s[j][2..3]: row g+8
+    for (int e = 0; e < 4; ++e) s[e] += s2[e];
+    if constexpr (MT == 1) {
+      if (half == 1) s_half[part * 32 + lane] = make_float4(s[0], s[1], s[2], s[3]);
+      __syncthreads();
+      if (half == 0) {
+        const float4 o = s_half[part * 32 + lane];
+        s[0] += o.x; s[1] += o.y; s[2] += o.z; s[3] += o.w;
+      }
+    }
+    // s[0..1]: row g, keys 8*part + 2*tq, +1; s[2..3]: row g+8
     const int valid = k1 - k0 - t * kLdKeys;
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-    for (int j = 0; j < MT; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int key = part * 8 * MT + j * 8 + tq * 2 + (e & 1);
-        s[j][e] = key < valid ? s[j][e] * p.scale_log2e : -INFINITY;
-        mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
-      }
+    for (int e = 0; e < 4; ++e) {
+      const int key = part * 8 + tq * 2 + (e & 1);
+      s[e] = key < valid ? s[e] * p.scale_log2e : -INFINITY;
+      mx[e >> 1] = fmaxf(mx[e >> 1], s[e]);
+    }
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
       mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
     }
-    if (tq == 0) { s_max[part][mt * 16 + g] = mx[0]; s_max[part][mt * 16 + g + 8] = mx[1]; }
+    if (half == 0 && tq == 0) { s_max[part][mt * 16 + g] = mx[0]; s_max[part][mt * 16 + g + 8] = mx[1]; }
     __syncthreads();
     // every thread follows the running maximum of all rows it accumulates output for
     float corr[MT][2];
@@ -149,20 +148,18 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
       }
     float sum[2] = {0.f, 0.f};
 #pragma unroll
-    for (int j = 0; j < MT; ++j)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const float m = (MT == 1 || mt == 0) ? m_run[0][e] : m_run[MT - 1][e];
-        const float x0 = exp2f(s[j][2 * e] - m), x1 = exp2f(s[j][2 * e + 1] - m);
-        sum[e] += x0 + x1;
-        *reinterpret_cast<uint32_t*>(s_p + (mt * 16 + g + 8 * e) * kLdPPitch + (part * 8 * MT + j * 8 + tq * 2) * 2) = pack_bf16(x0, x1);
-      }
+    for (int e = 0; e < 2; ++e) {
+      const float m = (MT == 1 || mt == 0) ? m_run[0][e] : m_run[MT - 1][e];
+      const float x0 = exp2f(s[2 * e] - m), x1 = exp2f(s[2 * e + 1] - m);
+      sum[e] = x0 + x1;
+      if (half == 0) *reinterpret_cast<uint32_t*>(s_p + (mt * 16 + g + 8 * e) * kLdPPitch + (part * 8 + tq * 2) * 2) = pack_bf16(x0, x1);
+    }
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       sum[e] += __shfl_xor_sync(0xffffffffu, sum[e], 1);
       sum[e] += __shfl_xor_sync(0xffffffffu, sum[e], 2);
     }
-    if (tq == 0) { s_sum[part][mt * 16 + g] = sum[0]; s_sum[part][mt * 16 + g + 8] = sum[1]; }
+    if (half == 0 && tq == 0) { s_sum[part][mt * 16 + g] = sum[0]; s_sum[part][mt * 16 + g + 8] = sum[1]; }
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < MT; ++i)
@@ -180,6 +177,7 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
         acc[i][j][0] *= corr[i][0]; acc[i][j][1] *= corr[i][0];
         acc[i][j][2] *= corr[i][1]; acc[i][j][3] *= corr[i][1];
       }
+    const uint32_t v_last = kb + ((lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (warp * 8 * NT + (NT - 1) * 8) * 2;
     const uint32_t v_addr = kb + ((lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (warp * 8 * NT + (lane >> 4) * 8) * 2;
 #pragma unroll
     for (int k = 0; k < kLdKeys; k += 16) {
@@ -187,7 +185,7 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
 #pragma unroll
       for (int i = 0; i < MT; ++i) ldmatrix_x4(p_addr + i * 16 * kLdPPitch + k * 2, a[i][0], a[i][1], a[i][2], a[i][3]);
 #pragma unroll
-      for (int j = 0; j < NT; j += 2) {
+      for (int j = 0; j + 1 < NT; j += 2) {
         uint32_t v[4];
         ldmatrix_x4_trans(v_addr + k * pitch + j * 16, v[0], v[1], v[2], v[3]);
 #pragma unroll
@@ -195,6 +193,12 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
           mma_bf16_full(acc[i][j], a[i], v[0], v[1]);
           mma_bf16_full(acc[i][j + 1], a[i], v[2], v[3]);
         }
+      }
+      if constexpr (NT % 2 == 1) {
+        uint32_t v[2];
+        ldmatrix_x2_trans(v_last + k * pitch, v[0], v[1]);
+#pragma unroll
+        for (int i = 0; i < MT; ++i) mma_bf16_full(acc[i][NT - 1], a[i], v[0], v[1]);
       }
     }
     __syncthreads();      // the tile's buffer and P are rewritten next
@@ -282,16 +286,16 @@ extern "C" int msa_lm_latent_decode(const void* qa, int64_t qa_row, int64_t qa_h
   cudaStream_t st = (cudaStream_t)stream;
   if (heads <= 16) {
     switch (rank) {
-      case 128: return launch_latent_decode<1, 2>(p, n, st);
-      case 256: return launch_latent_decode<1, 4>(p, n, st);
-      case 384: return launch_latent_decode<1, 6>(p, n, st);
-      default: return launch_latent_decode<1, 8>(p, n, st);
+      case 128: return launch_latent_decode<1, 1>(p, n, st);
+      case 256: return launch_latent_decode<1, 2>(p, n, st);
+      case 384: return launch_latent_decode<1, 3>(p, n, st);
+      default: return launch_latent_decode<1, 4>(p, n, st);
     }
   }
   switch (rank) {
-    case 128: return launch_latent_decode<2, 2>(p, n, st);
-    case 256: return launch_latent_decode<2, 4>(p, n, st);
-    case 384: return launch_latent_decode<2, 6>(p, n, st);
-    default: return launch_latent_decode<2, 8>(p, n, st);
+    case 128: return launch_latent_decode<2, 1>(p, n, st);
+    case 256: return launch_latent_decode<2, 2>(p, n, st);
+    case 384: return launch_latent_decode<2, 3>(p, n, st);
+    default: return launch_latent_decode<2, 4>(p, n, st);
   }
 }

@@ -136,7 +136,7 @@ class GatedDelta:
         qk, v = s.kv_heads * s.dim, s.heads * s.vdim
         self.w_in = w.stack([(prefix + "q", qk), (prefix + "k", qk), (prefix + "v", v), (prefix + "g", v),
                              (prefix + "b", s.heads), (prefix + "a", s.heads)], width, pad=True)
-        self.conv = torch.cat([w.vector(prefix + n + ".conv", r, s.taps) for n, r in (("q", qk), ("k", qk), ("v", v))]).contiguous()
+        self.conv = torch.cat([w.vector(prefix + n + ".conv", r, s.taps) for n, r in (("q", qk), ("k", qk), ("v", v))]).t().contiguous()
         self.a_log, self.dt_bias = w.vector(prefix + "A_log", s.heads), w.vector(prefix + "dt_bias", s.heads)
         self.norm = w.vector(prefix + "norm", s.vdim)
         self.w_o = w.matrix(prefix + "o", width, v)

@@ -170,7 +170,8 @@ def delta_portions(args, spec, step, out) -> None:
     rows, heads = step.n_tok - step.n_decode, spec.heads
     qk = torch.empty((rows, 4 * spec.kv_heads * spec.dim), dtype=torch.bfloat16, device=dev)
     f = dict(dtype=torch.float32, device=dev)
-    v, gates = torch.empty((rows, heads * spec.vdim), **f), torch.empty((rows, 2 * heads), **f)
+    v = torch.empty((rows, heads * spec.vdim), dtype=torch.bfloat16, device=dev)
+    gates = torch.empty((rows, 2 * heads), **f)
     A.call("msa_lm_delta_prep_split", C.byref(args), A.ptr(qk), A.ptr(v), A.ptr(gates), st)
     A.call("msa_lm_delta_conv_store", C.byref(args), st)
     delta_chunks(args, spec, step, qk, v, gates, out)
@@ -180,7 +181,7 @@ def delta_chunks(args, spec, step, qk, v, gates, out) -> None:
     dev, heads = out.device, spec.heads
     tile = delta_tile(step.n_seq - step.n_decode, heads, spec.vdim)
     work = torch.empty(A.lib().msa_lm_delta_chunk_workspace(step.n_chunks, heads), dtype=torch.uint8, device=dev)
-    o = torch.empty_like(v) if tile != spec.vdim else None
+    o = torch.empty(v.shape, dtype=torch.float32, device=dev) if tile != spec.vdim else None
     A.call("msa_lm_delta_chunk", C.byref(args), A.ptr(qk), A.ptr(v), A.ptr(gates), A.ptr(step.chunk_off), step.n_chunks, tile,
            A.ptr(work), A.ptr(o), A.ptr(out), _rows(out), A.stream_ptr(dev))
 
