@@ -2,16 +2,17 @@
 // [latent | rotated key part]; the values are the latents themselves.  Flash-decode: the visible rows of a sequence are
 // split over CTAs, partial results are merged by a second kernel.
 //
-// One CTA = up to 32 heads x one split, 512 threads.  The queries stay in shared memory; 64-row tiles of the ring are
-// double-buffered with cp.async (rows are read once from HBM for all heads, which is what bounds this kernel); scores and
-// output on mma.sync.m16n8k16, softmax in fp32.  Warps split the scores over octets of keys and the two 16-head tiles (with
-// one head tile: over the two halves of the reduction), and the output over latent columns.
+// One CTA = up to 32 heads x one split, 256 threads; 64-row tiles of the ring are double-buffered with cp.async (rows are
+// read once from HBM for all heads).  Scores and output run on mma.sync.m16n8k16.  For the scores the warps split the
+// reduction: a warp keeps its slice of the queries in registers for the whole launch, multiplies all 64 rows by it, and
+// the slices' partial scores are added up in shared memory, where eight (sixteen) threads per head do the fp32 softmax.
+// For the output the warps split the latent columns.
 #include "lm_common.cuh"
 #include "mma_helpers.cuh"
 
 namespace msa {
 
-constexpr int kLdThreads = 512, kLdKeys = 64, kLdPPitch = 144;   // P rows: 64 bf16 + 16 bytes of padding
+constexpr int kLdThreads = 256, kLdKeys = 64, kLdPPitch = 144;   // P rows: 64 bf16 + 16 bytes of padding
 
 struct LatentDecodeParams {
   const __nv_bfloat16* qa; long long qa_row, qa_head;
@@ -29,23 +30,19 @@ __device__ __forceinline__ void mma_bf16_full(float (&c)[4], const uint32_t (&a)
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-__device__ __forceinline__ void ldmatrix_x2_trans(uint32_t addr, uint32_t& r0, uint32_t& r1) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
-}
-
-// MT: 16-head tiles; NT: octets of latent columns per warp (rank / 128).
-template <int MT, int NT>
+// MT: 16-head tiles; NT: octets of latent columns per warp; KS: reduction steps of 16 per warp.
+template <int MT, int NT, int KS>
 __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LatentDecodeParams p) {
+  constexpr int KQ = 8 / MT, kRows = MT * 16, kPart = 68;            // slices of the reduction; floats per partial row
+  constexpr int TPR = kLdThreads / kRows, KPT = kLdKeys / TPR;       // softmax: threads per row, keys per thread
   extern __shared__ __align__(16) unsigned char sm[];
-  __shared__ float s_max[8][32], s_sum[8][32];
-  __shared__ float4 s_half[MT == 1 ? 256 : 1];      // one head tile: scores of the second half of the reduction
-  constexpr int kParts = 8;                         // octets of keys of a tile
-  const int width = p.rank + p.rot, pitch = width * 2 + 16, vecs = width / 8;
-  unsigned char* s_q = sm;                          // [MT*16][pitch]
-  unsigned char* s_p = s_q + MT * 16 * pitch;       // [MT*16][kLdPPitch]
-  unsigned char* s_k = s_p + MT * 16 * kLdPPitch;   // 2 x [64][pitch]
-  const int b = blockIdx.z, h0 = blockIdx.y * MT * 16, split = blockIdx.x;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  __shared__ float s_corr[kRows], s_m[kRows], s_l[kRows];
+  const int width = p.rank + p.rot, pitch = width * 2 + 16, vecs = width / 8, steps = width / 16;
+  float* s_part = reinterpret_cast<float*>(sm);                      // [KQ][kRows][kPart]
+  unsigned char* s_p = sm + KQ * kRows * kPart * 4;                  // [kRows][kLdPPitch]
+  unsigned char* s_k = s_p + kRows * kLdPPitch;                      // 2 x [64][pitch]
+  const int b = blockIdx.z, h0 = blockIdx.y * kRows, split = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
   const int pos = p.pos[b], lo = max(0, pos - p.window + 1), n_keys = pos - lo + 1;
   int chunk = (n_keys + p.splits - 1) / p.splits;
   chunk = (chunk + kLdKeys - 1) / kLdKeys * kLdKeys;
@@ -58,126 +55,114 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
   auto load_tile = [&](int t) {
     const uint32_t dst = k_base + (t & 1) * kLdKeys * pitch;
 #pragma unroll 4
-    for (int r = threadIdx.x >> 5; r < kLdKeys; r += kLdThreads / 32) {     // a warp per row
+    for (int r = warp; r < kLdKeys; r += kLdThreads / 32) {                 // a warp per row
       const int k = k0 + t * kLdKeys + r;
       const uint32_t bytes = k < k1 ? 16u : 0u;
       int row = lo_row + k;                                                 // both terms are below the ring's size
       row = k < k1 ? (row >= n_ring ? row - n_ring : row) : 0;
       const __nv_bfloat16* src = ring + (long long)row * width;
-      for (int c = threadIdx.x & 31; c < vecs; c += 32) cp_async16(dst + r * pitch + c * 16, src + c * 8, bytes);
+      for (int c = lane; c < vecs; c += 32) cp_async16(dst + r * pitch + c * 16, src + c * 8, bytes);
     }
     cp_async_commit();
   };
   if (n_tiles > 0) load_tile(0);
-  for (int i = threadIdx.x; i < MT * 16 * vecs; i += kLdThreads) {
-    const int r = i / vecs, c = (i - r * vecs) * 8, h = h0 + r;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (h < p.heads)
-      v = c < p.rank ? *reinterpret_cast<const uint4*>(p.qa + b * p.qa_row + h * p.qa_head + c)
-                     : *reinterpret_cast<const uint4*>(p.qb + b * p.qb_row + h * p.qb_head + (c - p.rank));
-    *reinterpret_cast<uint4*>(s_q + r * pitch + c * 2) = v;
-  }
-  const int mt = MT == 2 ? warp & 1 : 0, part = MT == 2 ? warp >> 1 : warp & 7, half = MT == 2 ? 0 : warp >> 3;
-  const int steps = width / 32, ks0 = half == 0 ? 0 : steps / 2 * 32, ks1 = MT == 1 && half == 0 ? steps / 2 * 32 : width;
-  const int g = lane >> 2, tq = lane & 3;
-  const uint32_t q_addr = (uint32_t)__cvta_generic_to_shared(s_q) + (mt * 16 + (lane & 15)) * pitch + (lane >> 4) * 16;
-  const uint32_t p_addr = (uint32_t)__cvta_generic_to_shared(s_p) + (lane & 15) * kLdPPitch + (lane >> 4) * 16;
-  // scores: keys 8*part .. +7 of the tile, two reduction steps per load
-  const int brow = part * 8 + (lane & 7), bcol = (lane >> 3) * 16;
-  float acc[MT][NT][4];
-  float m_run[MT][2], l_run[MT][2];
+  const int mt = warp % MT, kq = warp / MT, ks0 = kq * KS;
+  uint32_t q[KS][4];
 #pragma unroll
-  for (int i = 0; i < MT; ++i) {
-    m_run[i][0] = m_run[i][1] = -INFINITY;
-    l_run[i][0] = l_run[i][1] = 0.f;
+  for (int i = 0; i < KS; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {                                           // (row g, g + 8) x (columns 2 tq, 2 tq + 8)
+      const int h = h0 + mt * 16 + g + 8 * (e & 1), c = (ks0 + i) * 16 + tq * 2 + 8 * (e >> 1);
+      uint32_t v = 0u;
+      if (h < p.heads && ks0 + i < steps)
+        v = c < p.rank ? *reinterpret_cast<const uint32_t*>(p.qa + b * p.qa_row + h * p.qa_head + c)
+                       : *reinterpret_cast<const uint32_t*>(p.qb + b * p.qb_row + h * p.qb_head + (c - p.rank));
+      q[i][e] = v;
+    }
+  const uint32_t p_addr = (uint32_t)__cvta_generic_to_shared(s_p) + (lane & 15) * kLdPPitch + (lane >> 4) * 16;
+  const uint32_t b_off = ((lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16 + ks0 * 32;
+  const int srow = threadIdx.x / TPR, skey = threadIdx.x % TPR * KPT;       // the scores this thread looks after
+  float m_run = -INFINITY, l_run = 0.f;
+  float acc[MT][NT][4];
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
 #pragma unroll
     for (int j = 0; j < NT; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
-  }
   for (int t = 0; t < n_tiles; ++t) {
-    if (t + 1 < n_tiles) { load_tile(t + 1); cp_async_wait<1>(); } else cp_async_wait<0>();
-    __syncthreads();
-    const uint32_t kb = (uint32_t)__cvta_generic_to_shared(s_k + (t & 1) * kLdKeys * pitch);
-    float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};            // two chains, added below
-    const uint32_t b_addr = kb + brow * pitch + bcol;
-#pragma unroll 3
-    for (int k = ks0; k < ks1; k += 32) {
-      uint32_t a[4], a2[4], x[4];
-      ldmatrix_x4(q_addr + k * 2, a[0], a[1], a[2], a[3]);
-      ldmatrix_x4(q_addr + k * 2 + 32, a2[0], a2[1], a2[2], a2[3]);
-      ldmatrix_x4(b_addr + k * 2, x[0], x[1], x[2], x[3]);
-      mma_bf16_full(s, a, x[0], x[1]);
-      mma_bf16_full(s2, a2, x[2], x[3]);
-    }
+    cp_async_wait<0>();
+    __syncthreads();                       // the tile is there; the other buffer, the scores and P are free
+    if (t + 1 < n_tiles) load_tile(t + 1);
+    const uint32_t kb = k_base + (t & 1) * kLdKeys * pitch;
+    float s[8][4];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) s[e] += s2[e];
-    if constexpr (MT == 1) {
-      if (half == 1) s_half[part * 32 + lane] = make_float4(s[0], s[1], s[2], s[3]);
-      __syncthreads();
-      if (half == 0) {
-        const float4 o = s_half[part * 32 + lane];
-        s[0] += o.x; s[1] += o.y; s[2] += o.z; s[3] += o.w;
+    for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
+#pragma unroll
+    for (int i = 0; i < KS; ++i) {
+      if (ks0 + i >= steps) break;
+#pragma unroll
+      for (int j = 0; j < 8; j += 2) {
+        uint32_t x[4];
+        ldmatrix_x4(kb + b_off + j * 8 * pitch + i * 32, x[0], x[1], x[2], x[3]);
+        mma_bf16_full(s[j], q[i], x[0], x[1]);
+        mma_bf16_full(s[j + 1], q[i], x[2], x[3]);
       }
     }
-    // s[0..1]: row g, keys 8*part + 2*tq, +1; s[2..3]: row g+8
-    const int valid = k1 - k0 - t * kLdKeys;
-    float mx[2] = {-INFINITY, -INFINITY};
+    {
+      float* dst = s_part + (kq * kRows + mt * 16 + g) * kPart + tq * 2;
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int key = part * 8 + tq * 2 + (e & 1);
-      s[e] = key < valid ? s[e] * p.scale_log2e : -INFINITY;
-      mx[e >> 1] = fmaxf(mx[e >> 1], s[e]);
+      for (int j = 0; j < 8; ++j) {
+        *reinterpret_cast<float2*>(dst + j * 8) = make_float2(s[j][0], s[j][1]);
+        *reinterpret_cast<float2*>(dst + 8 * kPart + j * 8) = make_float2(s[j][2], s[j][3]);
+      }
     }
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
-      mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
-    }
-    if (half == 0 && tq == 0) { s_max[part][mt * 16 + g] = mx[0]; s_max[part][mt * 16 + g + 8] = mx[1]; }
     __syncthreads();
-    // every thread follows the running maximum of all rows it accumulates output for
+    {
+      float x[KPT];
+#pragma unroll
+      for (int i = 0; i < KPT; ++i) x[i] = 0.f;
+#pragma unroll
+      for (int w = 0; w < KQ; ++w)
+#pragma unroll
+        for (int i = 0; i < KPT; i += 4) {
+          const float4 v = load4(s_part + (w * kRows + srow) * kPart + skey + i);
+          x[i] += v.x; x[i + 1] += v.y; x[i + 2] += v.z; x[i + 3] += v.w;
+        }
+      const int valid = k1 - k0 - t * kLdKeys - skey;
+      float m = m_run;
+#pragma unroll
+      for (int i = 0; i < KPT; ++i) {
+        x[i] = i < valid ? x[i] * p.scale_log2e : -INFINITY;
+        m = fmaxf(m, x[i]);
+      }
+#pragma unroll
+      for (int o = 1; o < TPR; o <<= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+      const float corr = exp2f(m_run - m);
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < KPT; ++i) { x[i] = exp2f(x[i] - m); sum += x[i]; }
+      l_run = l_run * corr + sum;          // this thread's keys alone; added up at the end
+      m_run = m;
+      uint32_t* dst = reinterpret_cast<uint32_t*>(s_p + srow * kLdPPitch + skey * 2);
+#pragma unroll
+      for (int i = 0; i < KPT; i += 4) *reinterpret_cast<uint2*>(dst + i / 2) = make_uint2(pack_bf16(x[i], x[i + 1]), pack_bf16(x[i + 2], x[i + 3]));
+      if (skey == 0) s_corr[srow] = corr;
+    }
+    __syncthreads();
     float corr[MT][2];
+    bool same = true;
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        float m = m_run[i][e];
+      for (int e = 0; e < 2; ++e) { corr[i][e] = s_corr[i * 16 + g + 8 * e]; same = same && corr[i][e] == 1.f; }
+    if (!__all_sync(0xffffffffu, same)) {
 #pragma unroll
-        for (int w = 0; w < kParts; ++w) m = fmaxf(m, s_max[w][i * 16 + g + 8 * e]);
-        corr[i][e] = exp2f(m_run[i][e] - m);
-        m_run[i][e] = m;
-      }
-    float sum[2] = {0.f, 0.f};
+      for (int i = 0; i < MT; ++i)
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const float m = (MT == 1 || mt == 0) ? m_run[0][e] : m_run[MT - 1][e];
-      const float x0 = exp2f(s[2 * e] - m), x1 = exp2f(s[2 * e + 1] - m);
-      sum[e] = x0 + x1;
-      if (half == 0) *reinterpret_cast<uint32_t*>(s_p + (mt * 16 + g + 8 * e) * kLdPPitch + (part * 8 + tq * 2) * 2) = pack_bf16(x0, x1);
+        for (int j = 0; j < NT; ++j) {
+          acc[i][j][0] *= corr[i][0]; acc[i][j][1] *= corr[i][0];
+          acc[i][j][2] *= corr[i][1]; acc[i][j][3] *= corr[i][1];
+        }
     }
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      sum[e] += __shfl_xor_sync(0xffffffffu, sum[e], 1);
-      sum[e] += __shfl_xor_sync(0xffffffffu, sum[e], 2);
-    }
-    if (half == 0 && tq == 0) { s_sum[part][mt * 16 + g] = sum[0]; s_sum[part][mt * 16 + g + 8] = sum[1]; }
-    __syncthreads();
-#pragma unroll
-    for (int i = 0; i < MT; ++i)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        float l = l_run[i][e] * corr[i][e];
-#pragma unroll
-        for (int w = 0; w < kParts; ++w) l += s_sum[w][i * 16 + g + 8 * e];
-        l_run[i][e] = l;
-      }
-#pragma unroll
-    for (int i = 0; i < MT; ++i)
-#pragma unroll
-      for (int j = 0; j < NT; ++j) {
-        acc[i][j][0] *= corr[i][0]; acc[i][j][1] *= corr[i][0];
-        acc[i][j][2] *= corr[i][1]; acc[i][j][3] *= corr[i][1];
-      }
-    const uint32_t v_last = kb + ((lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (warp * 8 * NT + (NT - 1) * 8) * 2;
     const uint32_t v_addr = kb + ((lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (warp * 8 * NT + (lane >> 4) * 8) * 2;
 #pragma unroll
     for (int k = 0; k < kLdKeys; k += 16) {
@@ -185,7 +170,7 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
 #pragma unroll
       for (int i = 0; i < MT; ++i) ldmatrix_x4(p_addr + i * 16 * kLdPPitch + k * 2, a[i][0], a[i][1], a[i][2], a[i][3]);
 #pragma unroll
-      for (int j = 0; j + 1 < NT; j += 2) {
+      for (int j = 0; j < NT; j += 2) {
         uint32_t v[4];
         ldmatrix_x4_trans(v_addr + k * pitch + j * 16, v[0], v[1], v[2], v[3]);
 #pragma unroll
@@ -194,24 +179,21 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
           mma_bf16_full(acc[i][j + 1], a[i], v[2], v[3]);
         }
       }
-      if constexpr (NT % 2 == 1) {
-        uint32_t v[2];
-        ldmatrix_x2_trans(v_last + k * pitch, v[0], v[1]);
-#pragma unroll
-        for (int i = 0; i < MT; ++i) mma_bf16_full(acc[i][NT - 1], a[i], v[0], v[1]);
-      }
     }
-    __syncthreads();      // the tile's buffer and P are rewritten next
   }
+#pragma unroll
+  for (int o = 1; o < TPR; o <<= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, o);
+  if (skey == 0) { s_m[srow] = m_run; s_l[srow] = l_run; }
+  __syncthreads();
 #pragma unroll
   for (int i = 0; i < MT; ++i)
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-      const int h = h0 + i * 16 + g + 8 * e;
+      const int r = i * 16 + g + 8 * e, h = h0 + r;
       if (h >= p.heads) continue;
       const long long row = (long long)b * p.heads + h;
       if (p.splits == 1) {
-        const float inv = 1.f / l_run[i][e];
+        const float inv = 1.f / s_l[r];
 #pragma unroll
         for (int j = 0; j < NT; ++j)
           *reinterpret_cast<uint32_t*>(p.out + row * p.rank + warp * 8 * NT + j * 8 + tq * 2) =
@@ -221,8 +203,8 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
 #pragma unroll
         for (int j = 0; j < NT; ++j) *reinterpret_cast<float2*>(o + j * 8) = make_float2(acc[i][j][2 * e], acc[i][j][2 * e + 1]);
         if (warp == 0 && tq == 0) {
-          p.part_ml[(row * p.splits + split) * 2] = m_run[i][e];
-          p.part_ml[(row * p.splits + split) * 2 + 1] = l_run[i][e];
+          p.part_ml[(row * p.splits + split) * 2] = s_m[r];
+          p.part_ml[(row * p.splits + split) * 2 + 1] = s_l[r];
         }
       }
     }
@@ -248,12 +230,13 @@ latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ 
 
 template <int MT, int NT>
 int launch_latent_decode(const LatentDecodeParams& p, int n, cudaStream_t stream) {
+  constexpr int KQ = 8 / MT, KS = (NT * 4 + 4 + KQ - 1) / KQ;               // up to 64 rotated columns
   const size_t pitch = (size_t)(p.rank + p.rot) * 2 + 16;
-  const size_t smem = (size_t)MT * 16 * (pitch + kLdPPitch) + 2 * kLdKeys * pitch;
+  const size_t smem = (size_t)KQ * MT * 16 * 68 * 4 + (size_t)MT * 16 * kLdPPitch + 2 * kLdKeys * pitch;
   static DeviceSmem configured{};
-  MSA_OK_OR_RETURN(ensure_dynamic_smem(latent_decode_kernel<MT, NT>, smem, configured));
+  MSA_OK_OR_RETURN(ensure_dynamic_smem(latent_decode_kernel<MT, NT, KS>, smem, configured));
   const dim3 grid((unsigned)p.splits, (unsigned)((p.heads + MT * 16 - 1) / (MT * 16)), (unsigned)n);
-  latent_decode_kernel<MT, NT><<<grid, kLdThreads, smem, stream>>>(p);
+  latent_decode_kernel<MT, NT, KS><<<grid, kLdThreads, smem, stream>>>(p);
   MSA_LAUNCH_OK("latent_decode_kernel");
   if (p.splits > 1) {
     latent_merge_kernel<<<(unsigned)(n * p.heads), 128, 0, stream>>>(p.part_o, p.part_ml, p.splits, p.rank, p.out);
@@ -286,16 +269,16 @@ extern "C" int msa_lm_latent_decode(const void* qa, int64_t qa_row, int64_t qa_h
   cudaStream_t st = (cudaStream_t)stream;
   if (heads <= 16) {
     switch (rank) {
-      case 128: return launch_latent_decode<1, 1>(p, n, st);
-      case 256: return launch_latent_decode<1, 2>(p, n, st);
-      case 384: return launch_latent_decode<1, 3>(p, n, st);
-      default: return launch_latent_decode<1, 4>(p, n, st);
+      case 128: return launch_latent_decode<1, 2>(p, n, st);
+      case 256: return launch_latent_decode<1, 4>(p, n, st);
+      case 384: return launch_latent_decode<1, 6>(p, n, st);
+      default: return launch_latent_decode<1, 8>(p, n, st);
     }
   }
   switch (rank) {
-    case 128: return launch_latent_decode<2, 1>(p, n, st);
-    case 256: return launch_latent_decode<2, 2>(p, n, st);
-    case 384: return launch_latent_decode<2, 3>(p, n, st);
-    default: return launch_latent_decode<2, 4>(p, n, st);
+    case 128: return launch_latent_decode<2, 2>(p, n, st);
+    case 256: return launch_latent_decode<2, 4>(p, n, st);
+    case 384: return launch_latent_decode<2, 6>(p, n, st);
+    default: return launch_latent_decode<2, 8>(p, n, st);
   }
 }
