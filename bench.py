@@ -1469,6 +1469,19 @@ def hybrid_kernels(torch, dev, model, z, pk, decode_b):
         rows[name] = {"us": round(ms * 1e3, 1), "bound": "tensor" if t_f > t_b else "hbm", "bound_us": round(max(t_f, t_b) * 1e3, 1),
                       "frac": round(max(t_f, t_b) / ms, 3)}
 
+    def leg_rotating(name, fn, flops, nbytes, reps=24):
+        """Short kernels: back to back over several layers' states or weights, more than L2 in all."""
+        for i in range(3):
+            fn(i)
+        graph = torch.cuda.CUDAGraph()            # the launches of a step come from a graph too
+        with torch.cuda.graph(graph):
+            for i in range(reps):
+                fn(i)
+        ms = _time_ms(torch, graph.replay, 3, 2) / reps
+        t_f, t_b = flops / (pk["tflops_burst"] * 1e9), nbytes / (pk["hbm_gbs"] * 1e6)
+        rows[name] = {"us": round(ms * 1e3, 1), "bound": "tensor" if t_f > t_b else "hbm", "bound_us": round(max(t_f, t_b) * 1e3, 1),
+                      "frac": round(max(t_f, t_b) / ms, 3)}
+
     n_seq, t = 4, 2048
     n = n_seq * t
     cache = model.new_cache(max(n_seq, decode_b) + 1, 4096)
@@ -1537,22 +1550,30 @@ def hybrid_kernels(torch, dev, model, z, pk, decode_b):
     q = pl[:, :heads * (s.dim + s.rot_dim)].view(b, heads, s.dim + s.rot_dim)
     qa = torch.bmm(q[..., :s.dim].transpose(0, 1), lat.w_uk)
     lo = torch.empty((b, heads, s.kv_rank), **bf)
-    leg(f"latent_decode + merge (batch {b})", lambda: K.latent_decode(qa.transpose(0, 1), q[..., s.dim:], cache.ring[1], ds.slot, ds.start, lo, window=window, scale=s.scale),
-        2.0 * b * window * heads * (2 * s.kv_rank + s.rot_dim), b * window * (s.kv_rank + s.rot_dim) * 2)
-    da = K.delta_args(pd, d, dlt, cache.conv[0], cache.state[0], 1e-5, ds)
+    rings, states = list(cache.ring.values()), list(cache.state)
+    leg_rotating(f"latent_decode + merge (batch {b})",
+                 lambda i: K.latent_decode(qa.transpose(0, 1), q[..., s.dim:], rings[i % len(rings)], ds.slot, ds.start, lo, window=window, scale=s.scale, status=model.status),
+                 2.0 * b * window * heads * (2 * s.kv_rank + s.rot_dim), b * window * (s.kv_rank + s.rot_dim) * 2)
+    das = [K.delta_args(pd, d, dlt, cache.conv[r], cache.state[r], 1e-5, ds) for r in states]
     od = torch.empty((b, heads * d.vdim), **bf)
-    leg(f"delta_decode (batch {b})", lambda: A.call("msa_lm_delta_decode", ctypes.byref(da), p(od), od.stride(0), st), 0,
-        b * heads * d.dim * d.vdim * 8 + b * d.channels * 2 * (2 * d.taps))
-    lg = K.matmul(hb, moe.router, torch.float32)
+    leg_rotating(f"delta_decode (batch {b})",
+                 lambda i: A.call("msa_lm_delta_decode", ctypes.byref(das[i % len(das)]), p(od), od.stride(0), A.stream_ptr(dev)), 0,
+                 b * heads * d.dim * d.vdim * 8 + b * d.channels * 2 * (2 * d.taps))
+    lg = torch.randn((b, m.experts), dtype=torch.float32, device=dev)
     idx, mix = K.moe_topk(lg, moe.bias, m.top)
     src, inv, off, tiles = K.moe_sort(idx, m.experts, 128)
     used = int((off[1:] > off[:-1]).sum())
-    leg(f"moe_topk + moe_sort (batch {b})", lambda: K.moe_sort(K.moe_topk(lg, moe.bias, m.top)[0], m.experts, 128), 0, b * m.experts * 4)
-    leg(f"moe_gemm_tc gate/up (batch {b})", lambda: K.moe_gemm_tc(hb, src, moe.w_gate_up, off, tiles, entries=b * m.top, act=True, limit=7.0, status=model.status),
-        2.0 * b * m.top * width * 2 * m.ff, used * 2 * m.ff * width * 2)
-    ab = K.moe_gemm_tc(hb, src, moe.w_gate_up, off, tiles, entries=b * m.top, act=True, limit=7.0, status=model.status)
-    leg(f"moe_gemm_tc down (batch {b})", lambda: K.moe_gemm_tc(ab, None, moe.w_down, off, tiles, entries=b * m.top, act=False, status=model.status),
-        2.0 * b * m.top * width * m.ff, used * m.ff * width * 2)
+    ffs = [l.ff for l in model.layers[1:]]
+    leg_rotating(f"moe_topk + moe_sort (batch {b})", lambda i: K.moe_sort(K.moe_topk(lg, moe.bias, m.top)[0], m.experts, 128), 0, b * m.experts * 4)
+    gate_up = lambda i: K.moe_gemm_tc(hb, src, ffs[i % len(ffs)].w_gate_up, off, tiles, entries=b * m.top, act=True, limit=7.0, status=model.status)
+    leg_rotating(f"moe_gemm_tc gate/up (batch {b})", gate_up, 2.0 * b * m.top * width * 2 * m.ff, used * 2 * m.ff * width * 2)
+    ab = gate_up(0)
+    leg_rotating(f"moe_gemm_tc down (batch {b})",
+                 lambda i: K.moe_gemm_tc(ab, None, ffs[i % len(ffs)].w_down, off, tiles, entries=b * m.top, act=False, status=model.status),
+                 2.0 * b * m.top * width * m.ff, used * m.ff * width * 2)
+    xb, yb = torch.randn((b, width), dtype=torch.float32, device=dev), torch.randn((b, width), **bf)
+    leg_rotating(f"residual_norm (batch {b})",
+                 lambda i: K.residual_norm(xb, yb, model.layers[0].norm1b, model.layers[0].norm2, 1e-5, torch.bfloat16, x_out=xb), 0, b * width * 12)
     model.check_status()
     return rows
 
@@ -1657,7 +1678,9 @@ def run_hybrid(args):
         for b in batches:
             cache = model.new_cache(b, z["window"] + 4 * (steps + warmup) + 64)
             g = GraphedDecode(model, cache, b)
-            g.tables.fill([1] * b, [z["window"] + 3] * b, list(range(b)))
+            for state in (*cache.ring.values(), *cache.state.values(), *cache.conv.values()):     # every sequence its own past
+                state.normal_(std=0.1)
+            g.tables.fill(torch.randint(0, 32768, (b,)).tolist(), [z["window"] + 3] * b, list(range(b)))
             ms = _time_ms(torch, g.replay, steps, warmup)
             r[f"decode_batch_{b}"] = {"ms_per_step": ms, "tokens_per_s": b / ms * 1e3}
             model.check_status()

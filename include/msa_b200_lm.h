@@ -89,12 +89,13 @@ int msa_lm_window_attn_tc(const void* q, int64_t q_row, int32_t n_rows, const vo
 
 /* Decode attention over the rings on tensor cores (bf16; rank a multiple of 128 up to 512, rot 0, 32 or 64): sequence i
  * of n at position pos[i] attends with qa [n, heads, rank] and qb [n, heads, rot] (row / head strides) to its ring's
- * visible rows; out [n, heads, rank].  splits > 1: part_o [n, heads, splits, rank], part_ml [n, heads, splits, 2] fp32. */
+ * visible rows; out [n, heads, rank].  splits > 1: part_o [n, heads, splits, rank], part_ml [n, heads, splits, 2] fp32.  A wait
+ * that runs out sets status[0]. */
 int msa_lm_latent_decode_supported(int32_t rank, int32_t rot);
 int msa_lm_latent_decode(const void* qa, int64_t qa_row, int64_t qa_head, const void* qb, int64_t qb_row, int64_t qb_head,
                          const void* ring, int64_t ring_rows, const int32_t* slot, const int32_t* pos, int32_t n,
                          int32_t heads, int32_t rank, int32_t rot, int32_t window, int32_t splits, float scale, void* out,
-                         float* part_o, float* part_ml, void* stream);
+                         float* part_o, float* part_ml, int32_t* status, void* stream);
 
 /* ---- gated delta rule ---------------------------------------------------------------------------------------------
  * proj row = [kv_heads*dim q | kv_heads*dim k | heads*vdim v | heads*vdim gate | heads beta | heads decay].

@@ -61,7 +61,7 @@ def lib() -> C.CDLL:
             "msa_lm_window_attn_tc": [vp, i64, i32, vp, i64, vp, i64, i32, i32, i32, i32, i32, i32, vp, vp, vp, i32, i32, i32, i32,
                                       i32, f32, vp, i64, vp, vp],
             "msa_lm_latent_decode_supported": [i32, i32],
-            "msa_lm_latent_decode": [vp, i64, i64, vp, i64, i64, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp, vp],
+            "msa_lm_latent_decode": [vp, i64, i64, vp, i64, i64, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp, vp, vp],
             "msa_lm_moe_gemm_tc": [vp, i64, i32, vp, vp, i32, vp, vp, i32, i32, i32, i32, f32, vp, i64, vp, vp],
             "msa_lm_delta_decode": [dp, vp, i64, vp],
             "msa_lm_delta_prep": [dp, vp, vp, vp, vp],

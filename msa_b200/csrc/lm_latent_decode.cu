@@ -2,13 +2,14 @@
 // [latent | rotated key part]; the values are the latents themselves.  Flash-decode: the visible rows of a sequence are
 // split over CTAs, partial results are merged by a second kernel.
 //
-// One CTA = up to 32 heads x one split, 256 threads; 64-row tiles of the ring are double-buffered with cp.async (rows are
-// read once from HBM for all heads).  Scores and output run on mma.sync.m16n8k16.  For the scores the warps split the
+// One CTA = up to 32 heads x one split, 256 threads; 64-row tiles of the ring are double-buffered, one bulk copy
+// per row (rows are read once from HBM for all heads; a warp's worth of instructions per tile).  Scores and output run on mma.sync.m16n8k16.  For the scores the warps split the
 // reduction: a warp keeps its slice of the queries in registers for the whole launch, multiplies all 64 rows by it, and
 // the slices' partial scores are added up in shared memory, where eight (sixteen) threads per head do the fp32 softmax.
 // For the output the warps split the latent columns.
 #include "lm_common.cuh"
 #include "mma_helpers.cuh"
+#include "tc_attn_common.cuh"
 
 namespace msa {
 
@@ -23,6 +24,7 @@ struct LatentDecodeParams {
   float scale_log2e;
   __nv_bfloat16* out;       // [n, heads, rank]
   float *part_o, *part_ml;  // [n, heads, splits, rank], [n, heads, splits, 2]
+  int32_t* status;
 };
 
 __device__ __forceinline__ void mma_bf16_full(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -31,12 +33,19 @@ __device__ __forceinline__ void mma_bf16_full(float (&c)[4], const uint32_t (&a)
 }
 
 // MT: 16-head tiles; NT: octets of latent columns per warp; KS: reduction steps of 16 per warp.
+__device__ __forceinline__ void bulk_row(uint32_t dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               ::"r"(dst), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
+}
+
 template <int MT, int NT, int KS>
 __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LatentDecodeParams p) {
-  constexpr int KQ = 8 / MT, kRows = MT * 16, kPart = 68;            // slices of the reduction; floats per partial row
+  constexpr int KQ = 8 / MT, kRows = MT * 16, kPart = 72;            // slices of the reduction; floats per partial row
   constexpr int TPR = kLdThreads / kRows, KPT = kLdKeys / TPR;       // softmax: threads per row, keys per thread
   extern __shared__ __align__(16) unsigned char sm[];
   __shared__ float s_corr[kRows], s_m[kRows], s_l[kRows];
+  __shared__ uint64_t s_full[2];
+  __shared__ int s_abort;
   const int width = p.rank + p.rot, pitch = width * 2 + 16, vecs = width / 8, steps = width / 16;
   float* s_part = reinterpret_cast<float*>(sm);                      // [KQ][kRows][kPart]
   unsigned char* s_p = sm + KQ * kRows * kPart * 4;                  // [kRows][kLdPPitch]
@@ -52,19 +61,23 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
 
   const int n_ring = (int)p.ring_rows, lo_row = lo % n_ring;
   const uint32_t k_base = (uint32_t)__cvta_generic_to_shared(s_k);
-  auto load_tile = [&](int t) {
-    const uint32_t dst = k_base + (t & 1) * kLdKeys * pitch;
-#pragma unroll 4
-    for (int r = warp; r < kLdKeys; r += kLdThreads / 32) {                 // a warp per row
-      const int k = k0 + t * kLdKeys + r;
-      const uint32_t bytes = k < k1 ? 16u : 0u;
-      int row = lo_row + k;                                                 // both terms are below the ring's size
-      row = k < k1 ? (row >= n_ring ? row - n_ring : row) : 0;
-      const __nv_bfloat16* src = ring + (long long)row * width;
-      for (int c = lane; c < vecs; c += 32) cp_async16(dst + r * pitch + c * 16, src + c * 8, bytes);
+  const uint32_t row_bytes = (uint32_t)width * 2;
+  auto load_tile = [&](int t) {             // eight rows per warp; rows past the split's end repeat its first one
+    if (threadIdx.x == 0) mbar_expect_tx(&s_full[t & 1], kLdKeys * row_bytes);
+    if (lane < kLdKeys / 8) {
+      const int r = warp * (kLdKeys / 8) + lane, k = k0 + t * kLdKeys + r;
+      int row = lo_row + (k < k1 ? k : k0);                                 // both terms are below the ring's size
+      row = row >= n_ring ? row - n_ring : row;
+      bulk_row(k_base + ((t & 1) * kLdKeys + r) * pitch, ring + (long long)row * width, row_bytes, &s_full[t & 1]);
     }
-    cp_async_commit();
   };
+  if (threadIdx.x == 0) {
+    mbar_init(&s_full[0], 1);
+    mbar_init(&s_full[1], 1);
+    s_abort = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  __syncthreads();
   if (n_tiles > 0) load_tile(0);
   const int mt = warp % MT, kq = warp / MT, ks0 = kq * KS;
   uint32_t q[KS][4];
@@ -89,8 +102,13 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
 #pragma unroll
     for (int j = 0; j < NT; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
   for (int t = 0; t < n_tiles; ++t) {
-    cp_async_wait<0>();
-    __syncthreads();                       // the tile is there; the other buffer, the scores and P are free
+    const bool there = mbar_wait(&s_full[t & 1], (t >> 1) & 1, &s_abort, p.status, 21);
+    if (!__syncthreads_and(there)) {       // gave up: the copies in flight land before shared memory is released
+      const unsigned long long w0 = global_ns();
+      while (global_ns() - w0 < 1000000ull) {}
+      return;
+    }
+    // the tile is there; the other buffer, the scores and P are free
     if (t + 1 < n_tiles) load_tile(t + 1);
     const uint32_t kb = k_base + (t & 1) * kLdKeys * pitch;
     float s[8][4];
@@ -127,19 +145,21 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
           const float4 v = load4(s_part + (w * kRows + srow) * kPart + skey + i);
           x[i] += v.x; x[i + 1] += v.y; x[i + 2] += v.z; x[i + 3] += v.w;
         }
-      const int valid = k1 - k0 - t * kLdKeys - skey;
-      float m = m_run;
+      if (t + 1 == n_tiles) {
+        const int valid = k1 - k0 - t * kLdKeys - skey;
 #pragma unroll
-      for (int i = 0; i < KPT; ++i) {
-        x[i] = i < valid ? x[i] * p.scale_log2e : -INFINITY;
-        m = fmaxf(m, x[i]);
+        for (int i = 0; i < KPT; ++i) x[i] = i < valid ? x[i] : -INFINITY;
       }
+      float m = x[0];
+#pragma unroll
+      for (int i = 1; i < KPT; ++i) m = fmaxf(m, x[i]);
+      m = fmaxf(m_run, m * p.scale_log2e);     // the scale is positive
 #pragma unroll
       for (int o = 1; o < TPR; o <<= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-      const float corr = exp2f(m_run - m);
+      const float corr = ex2_approx(m_run - m);
       float sum = 0.f;
 #pragma unroll
-      for (int i = 0; i < KPT; ++i) { x[i] = exp2f(x[i] - m); sum += x[i]; }
+      for (int i = 0; i < KPT; ++i) { x[i] = ex2_approx(fmaf(x[i], p.scale_log2e, -m)); sum += x[i]; }
       l_run = l_run * corr + sum;          // this thread's keys alone; added up at the end
       m_run = m;
       uint32_t* dst = reinterpret_cast<uint32_t*>(s_p + srow * kLdPPitch + skey * 2);
@@ -232,7 +252,7 @@ template <int MT, int NT>
 int launch_latent_decode(const LatentDecodeParams& p, int n, cudaStream_t stream) {
   constexpr int KQ = 8 / MT, KS = (NT * 4 + 4 + KQ - 1) / KQ;               // up to 64 rotated columns
   const size_t pitch = (size_t)(p.rank + p.rot) * 2 + 16;
-  const size_t smem = (size_t)KQ * MT * 16 * 68 * 4 + (size_t)MT * 16 * kLdPPitch + 2 * kLdKeys * pitch;
+  const size_t smem = (size_t)KQ * MT * 16 * 72 * 4 + (size_t)MT * 16 * kLdPPitch + 2 * kLdKeys * pitch;
   static DeviceSmem configured{};
   MSA_OK_OR_RETURN(ensure_dynamic_smem(latent_decode_kernel<MT, NT, KS>, smem, configured));
   const dim3 grid((unsigned)p.splits, (unsigned)((p.heads + MT * 16 - 1) / (MT * 16)), (unsigned)n);
@@ -256,16 +276,16 @@ extern "C" int msa_lm_latent_decode_supported(int32_t rank, int32_t rot) {
 extern "C" int msa_lm_latent_decode(const void* qa, int64_t qa_row, int64_t qa_head, const void* qb, int64_t qb_row,
                                     int64_t qb_head, const void* ring, int64_t ring_rows, const int32_t* slot,
                                     const int32_t* pos, int32_t n, int32_t heads, int32_t rank, int32_t rot, int32_t window,
-                                    int32_t splits, float scale, void* out, float* part_o, float* part_ml, void* stream) {
-  MSA_REQUIRE(qa && ring && slot && pos && out && (rot == 0 || qb), "latent_decode: null pointer");
-  MSA_REQUIRE(msa_lm_latent_decode_supported(rank, rot) && heads > 0 && window > 0 && ring_rows > 0 && ring_rows < (1ll << 30), "latent_decode: bad sizes");
+                                    int32_t splits, float scale, void* out, float* part_o, float* part_ml, int32_t* status, void* stream) {
+  MSA_REQUIRE(qa && ring && slot && pos && out && status && (rot == 0 || qb), "latent_decode: null pointer");
+  MSA_REQUIRE(msa_lm_latent_decode_supported(rank, rot) && heads > 0 && window > 0 && scale > 0.f && ring_rows > 0 && ring_rows < (1ll << 30), "latent_decode: bad sizes");
   MSA_REQUIRE(splits >= 1 && splits <= 64 && (splits == 1 || (part_o && part_ml)), "latent_decode: bad splits");
   MSA_REQUIRE(aligned16(qa) && aligned16(ring) && aligned16(out) && (rot == 0 || aligned16(qb)) && qa_row % 8 == 0 &&
                   qa_head % 8 == 0 && qb_row % 8 == 0 && qb_head % 8 == 0, "latent_decode: rows must be 16-byte aligned");
   if (n <= 0) return MSA_OK;
   LatentDecodeParams p{(const __nv_bfloat16*)qa, qa_row, qa_head, (const __nv_bfloat16*)qb, qb_row, qb_head,
                        (const __nv_bfloat16*)ring, ring_rows, slot, pos, heads, rank, rot, window, splits,
-                       scale * 1.4426950408889634f, (__nv_bfloat16*)out, part_o, part_ml};
+                       scale * 1.4426950408889634f, (__nv_bfloat16*)out, part_o, part_ml, status};
   cudaStream_t st = (cudaStream_t)stream;
   if (heads <= 16) {
     switch (rank) {

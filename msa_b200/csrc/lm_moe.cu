@@ -7,14 +7,16 @@ namespace msa {
 constexpr int kMoeMaxExperts = 1024;
 
 // One warp per row.  The winners are taken one at a time in descending order; the softmax runs over them alone.
+// PER: logits per lane.
+template <int PER>
 __global__ void __launch_bounds__(256)
 moe_topk_kernel(const float* __restrict__ logits, long long stride, const float* __restrict__ bias, int n_rows, int experts,
                 int top, int32_t* __restrict__ idx, float* __restrict__ weight) {
   const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (row >= n_rows) return;
-  float z[kMoeMaxExperts / 32];
-  const int per = (experts + 31) / 32;
-  for (int i = 0; i < per; ++i) {
+  float z[PER];
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
     const int e = i * 32 + lane;
     z[i] = e < experts ? logits[(long long)row * stride + e] + (bias ? bias[e] : 0.f) : -INFINITY;
   }
@@ -23,7 +25,8 @@ moe_topk_kernel(const float* __restrict__ logits, long long stride, const float*
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int arg = experts;
-    for (int i = 0; i < per; ++i)
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
       if (!((taken >> i) & 1u) && i * 32 + lane < experts && (arg == experts || z[i] > best)) { best = z[i]; arg = i * 32 + lane; }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
@@ -56,13 +59,22 @@ moe_sort_kernel(const int32_t* __restrict__ idx, int n, int top, int experts, in
   __syncthreads();
   for (int i = threadIdx.x; i < n; i += blockDim.x) atomicAdd(&s_cnt[idx[i]], 1);
   __syncthreads();
-  if (threadIdx.x == 0) {
+  if (threadIdx.x < 32) {                               // one warp: prefix sums over the experts
     int o = 0, t = 0;
-    for (int e = 0; e < experts; ++e) {
-      s_off[e] = o; s_tile[e] = t;
-      o += s_cnt[e]; t += (s_cnt[e] + tile_rows - 1) / tile_rows;
+    for (int e0 = 0; e0 < experts; e0 += 32) {
+      const int e = e0 + threadIdx.x;
+      const int c = e < experts ? s_cnt[e] : 0, ct = (c + tile_rows - 1) / tile_rows;
+      int so = c, stl = ct;
+#pragma unroll
+      for (int d = 1; d < 32; d <<= 1) {
+        const int x = __shfl_up_sync(0xffffffffu, so, d), y = __shfl_up_sync(0xffffffffu, stl, d);
+        if ((int)threadIdx.x >= d) { so += x; stl += y; }
+      }
+      if (e < experts) { s_off[e] = o + so - c; s_tile[e] = t + stl - ct; }
+      o += __shfl_sync(0xffffffffu, so, 31);
+      t += __shfl_sync(0xffffffffu, stl, 31);
     }
-    s_off[experts] = o; s_tile[experts] = t;
+    if (threadIdx.x == 0) { s_off[experts] = o; s_tile[experts] = t; }
   }
   __syncthreads();
   for (int e = threadIdx.x; e <= experts; e += blockDim.x) off[e] = s_off[e];
@@ -222,7 +234,13 @@ extern "C" int msa_lm_moe_topk(const float* logits, int64_t stride, const float*
   MSA_REQUIRE(logits && idx && weight && n_rows >= 0, "moe_topk: bad arguments");
   MSA_REQUIRE(experts > 0 && experts <= kMoeMaxExperts && top > 0 && top <= experts, "moe_topk: 1 <= top <= experts <= 1024");
   if (n_rows == 0) return MSA_OK;
-  moe_topk_kernel<<<(n_rows + 7) / 8, 256, 0, (cudaStream_t)stream>>>(logits, stride, bias, n_rows, experts, top, idx, weight);
+  const unsigned blocks = (unsigned)((n_rows + 7) / 8);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (experts <= 32) moe_topk_kernel<1><<<blocks, 256, 0, st>>>(logits, stride, bias, n_rows, experts, top, idx, weight);
+  else if (experts <= 64) moe_topk_kernel<2><<<blocks, 256, 0, st>>>(logits, stride, bias, n_rows, experts, top, idx, weight);
+  else if (experts <= 128) moe_topk_kernel<4><<<blocks, 256, 0, st>>>(logits, stride, bias, n_rows, experts, top, idx, weight);
+  else if (experts <= 256) moe_topk_kernel<8><<<blocks, 256, 0, st>>>(logits, stride, bias, n_rows, experts, top, idx, weight);
+  else moe_topk_kernel<32><<<blocks, 256, 0, st>>>(logits, stride, bias, n_rows, experts, top, idx, weight);
   MSA_LAUNCH_OK("moe_topk_kernel");
   return MSA_OK;
 }

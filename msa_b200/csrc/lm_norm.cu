@@ -99,6 +99,54 @@ __global__ void residual_norm_kernel(const ResNormParams p) {
   }
 }
 
+// The same for rows that a block of width / 4 threads covers in one pass (everything in registers, all loads in flight
+// before the first reduction): a decode step has few rows and waits for latency, not for bandwidth.
+template <typename T, typename TY>
+__global__ void __launch_bounds__(1024) residual_norm_once_kernel(const ResNormParams p) {
+  __shared__ float s_part[32];
+  const long long r = blockIdx.x;
+  const long long rb = p.rows ? p.rows[r] : r;
+  const int i = threadIdx.x * 4;
+  const bool on = i < p.width;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 x = on && p.base ? load4(p.base + rb * p.base_stride + i) : zero;
+  const float4 wb = on && p.w_branch ? load4(p.w_branch + i) : zero;
+  const float4 wn = on && p.h_out ? load4(p.w_next + i) : zero;
+  float4 b = zero;
+  if (p.y && on) {
+    const TY* y = reinterpret_cast<const TY*>(p.y);
+    if (p.inv) {
+      for (int k0 = 0; k0 < p.top; k0 += 4) {
+        float4 v[4];
+        float w[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const bool in = k0 + k < p.top;
+          w[k] = in ? p.mix[r * p.top + k0 + k] : 0.f;
+          v[k] = in ? load4(y + (long long)p.inv[r * p.top + k0 + k] * p.y_stride + i) : zero;
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          b.x = fmaf(w[k], v[k].x, b.x); b.y = fmaf(w[k], v[k].y, b.y); b.z = fmaf(w[k], v[k].z, b.z); b.w = fmaf(w[k], v[k].w, b.w);
+        }
+      }
+    } else {
+      b = load4(y + r * p.y_stride + i);
+    }
+  }
+  if (p.y && p.w_branch) {
+    const float sc = 1.f / sqrtf(block_sum(b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w, s_part) / (float)p.width + p.eps);
+    x.x += b.x * sc * wb.x; x.y += b.y * sc * wb.y; x.z += b.z * sc * wb.z; x.w += b.w * sc * wb.w;
+  } else {
+    x.x += b.x; x.y += b.y; x.z += b.z; x.w += b.w;
+  }
+  if (on && p.x_out) store4(p.x_out + r * p.width + i, x);
+  if (on && p.cat_out) store4(reinterpret_cast<T*>(p.cat_out) + r * p.cat_stride + i, x);
+  if (!p.h_out) return;
+  const float inv = 1.f / sqrtf(block_sum(x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w, s_part) / (float)p.width + p.eps);
+  if (on) store4(reinterpret_cast<T*>(p.h_out) + r * p.width + i, make_float4(x.x * inv * wn.x, x.y * inv * wn.y, x.z * inv * wn.z, x.w * inv * wn.w));
+}
+
 template <typename T>
 __global__ void embed_kernel(const T* __restrict__ table, const int32_t* __restrict__ token, int width, int vocab,
                              const float* __restrict__ w_next, float eps, float* x_out, T* h_out, T* cat0, T* cat1,
@@ -170,6 +218,15 @@ extern "C" int msa_lm_residual_norm(const float* base, int64_t base_stride, cons
   const size_t smem = (size_t)width * 4;
   const int threads = row_threads(width);
   cudaStream_t st = (cudaStream_t)stream;
+  if (v4 && width <= 4096 && n_rows <= 512) {
+    const int once = (width / 4 + 31) / 32 * 32;
+    MSA_LM_DISPATCH(dtype, {
+      if (y && y_dtype == MSA_BF16) residual_norm_once_kernel<T, __nv_bfloat16><<<n_rows, once, 0, st>>>(p);
+      else residual_norm_once_kernel<T, float><<<n_rows, once, 0, st>>>(p);
+    });
+    MSA_LAUNCH_OK("residual_norm_once_kernel");
+    return MSA_OK;
+  }
   MSA_LM_DISPATCH(dtype, {
     if (y && y_dtype == MSA_BF16) {
       if (v4) residual_norm_kernel<T, __nv_bfloat16, 4><<<n_rows, threads, smem, st>>>(p);

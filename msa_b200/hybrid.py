@@ -113,8 +113,8 @@ class LatentAttention:
             qa = torch.bmm(q[..., :s.dim].transpose(0, 1), self.w_uk)                     # [heads, n, rank]
             lat = torch.empty((n, s.heads, s.kv_rank), dtype=q.dtype, device=q.device)
             K.latent_decode(qa.transpose(0, 1), q[..., s.dim:] if s.rot_dim else None, ring, step.slot, step.start, lat,
-                            window=view.window, scale=s.scale)
-            out.view(n, s.heads, s.vdim).copy_(torch.bmm(lat.transpose(0, 1), self.w_uv.transpose(1, 2)).transpose(0, 1))
+                            window=view.window, scale=s.scale, status=self.status)
+            torch.bmm(lat.transpose(0, 1), self.w_uv.transpose(1, 2), out=out.view(n, s.heads, s.vdim).transpose(0, 1))
             return
         f32 = dict(out_dtype=torch.float32) if q.dtype != torch.float32 else {}
         qa = torch.bmm(q[..., :s.dim].transpose(0, 1), self.w_uk, **f32)                  # [heads, n, rank]

@@ -115,7 +115,7 @@ def window_attn_tc(proj, kv, ctx, spec, out, step, view, status):
 
 
 def latent_decode_supported(spec, dtype) -> bool:
-    return (dtype == torch.bfloat16 and spec.dim % 8 == 0
+    return (dtype == torch.bfloat16 and spec.dim % 8 == 0 and spec.scale > 0
             and bool(A.lib().msa_lm_latent_decode_supported(spec.kv_rank, spec.rot_dim)))
 
 
@@ -125,7 +125,7 @@ def latent_decode_splits(n: int, heads: int, ring_rows: int, n_sm: int = 148) ->
     return max(1, min(n_sm // max(n * groups, 1), (ring_rows + 127) // 128, 64))
 
 
-def latent_decode(qa, qb, ring, slot, pos, out, *, window, scale):
+def latent_decode(qa, qb, ring, slot, pos, out, *, window, scale, status):
     """``qa`` / ``qb`` / ``out`` ``[n, heads, d]`` views, ``ring`` ``[slots, rows, rank + rot]``."""
     n, heads, rank = qa.shape
     rot = 0 if qb is None else qb.shape[2]
@@ -136,7 +136,7 @@ def latent_decode(qa, qb, ring, slot, pos, out, *, window, scale):
         part_o, part_ml = torch.empty((n, heads, splits, rank), **f), torch.empty((n, heads, splits, 2), **f)
     A.call("msa_lm_latent_decode", A.ptr(qa), qa.stride(0), qa.stride(1), A.ptr(qb), 0 if qb is None else qb.stride(0),
            0 if qb is None else qb.stride(1), A.ptr(ring), ring.shape[1], A.ptr(slot), A.ptr(pos), n, heads, rank, rot, window,
-           splits, float(scale), A.ptr(out), A.ptr(part_o), A.ptr(part_ml), A.stream_ptr(qa.device))
+           splits, float(scale), A.ptr(out), A.ptr(part_o), A.ptr(part_ml), A.ptr(status), A.stream_ptr(qa.device))
 
 
 # ---------------------------------------------------------------------------------------------- gated delta rule
