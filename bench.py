@@ -1591,6 +1591,10 @@ def closest_kernels(torch, dev, pk):
     wt = torch.ones(w, dtype=torch.bfloat16, device=dev)
     ms = _time_ms(torch, lambda: ops.add_rmsnorm(x, y, wt, 1e-6), 20, 3)
     out["add_rmsnorm"] = {"us": round(ms * 1e3, 1), "bound": "hbm", "frac": round(n * w * 8 / (ms * pk["hbm_gbs"] * 1e6), 3)}
+    qkv = torch.randn((n, 48 * 128), dtype=torch.bfloat16, device=dev)
+    cs, nw = torch.randn((n, 1, 128), dtype=torch.bfloat16, device=dev), torch.ones(128, dtype=torch.bfloat16, device=dev)
+    ms = _time_ms(torch, lambda: ops.qk_norm_rope(qkv, 32, 8, nw, nw, 1e-6, cs, cs), 20, 3)
+    out["qk_norm_rope"] = {"us": round(ms * 1e3, 1), "bound": "hbm", "frac": round(n * 128 * 2 * (40 * 2 + 2) / (ms * pk["hbm_gbs"] * 1e6), 3)}
     gu = torch.randn((n, 2 * w), dtype=torch.bfloat16, device=dev)
     ms = _time_ms(torch, lambda: ops.silu_mul(gu, w), 20, 3)
     out["silu_mul"] = {"us": round(ms * 1e3, 1), "bound": "hbm", "frac": round(n * w * 6 / (ms * pk["hbm_gbs"] * 1e6), 3)}

@@ -98,10 +98,14 @@ __global__ void __launch_bounds__(128) latent_prep_vec_kernel(const LatentPrepPa
   const int per_head = p.rot / 4, quads = p.heads * per_head;
   constexpr int kAhead = 4;
   float4 q[kAhead];
+  int at[kAhead], pair[kAhead];
+  const float inv_ph = 1.f / (float)max(per_head, 1);      // (i + 0.5) / per_head rounds down to the head for every i that fits
 #pragma unroll
   for (int u = 0; u < kAhead; ++u) {
-    const int i = tid + u * 128;
-    if (i < quads) { const int h = i / per_head; q[u] = load4(row + h * hd + p.dim + (i - h * per_head) * 4); }
+    const int i = tid + u * 128, h = (int)(((float)i + 0.5f) * inv_ph), j = i - h * per_head;
+    at[u] = h * hd + p.dim + j * 4;
+    pair[u] = 2 * j;
+    if (i < quads) q[u] = load4(row + at[u]);
   }
   T* dst;
   if (n < p.n_decode) {
@@ -128,12 +132,12 @@ __global__ void __launch_bounds__(128) latent_prep_vec_kernel(const LatentPrepPa
 #pragma unroll
   for (int u = 0; u < kAhead; ++u) {
     const int i = tid + u * 128;
-    if (i < quads) { const int h = i / per_head, j = i - h * per_head; store4(row + h * hd + p.dim + j * 4, turn(q[u], 2 * j)); }
+    if (i < quads) store4(row + at[u], turn(q[u], pair[u]));
   }
   for (int i = tid + kAhead * 128; i < quads; i += 128) {
     const int h = i / per_head, j = i - h * per_head;
-    T* at = row + h * hd + p.dim + j * 4;
-    store4(at, turn(load4(at), 2 * j));
+    T* x = row + h * hd + p.dim + j * 4;
+    store4(x, turn(load4(x), 2 * j));
   }
 }
 

@@ -79,6 +79,7 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
   }
   __syncthreads();
   if (n_tiles > 0) load_tile(0);
+  grid_launch_dependents();
   const int mt = warp % MT, kq = warp / MT, ks0 = kq * KS;
   uint32_t q[KS][4];
 #pragma unroll
@@ -230,22 +231,38 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     }
 }
 
+// Launched early (programmatic dependent launch): waits for the partial results before it reads them.
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits, int rank, __nv_bfloat16* __restrict__ out) {
   const long long row = blockIdx.x;
+  const int c = threadIdx.x * 4;
+  grid_dependency_wait();
   float m = -INFINITY, l = 0.f;
-  for (int s = 0; s < splits; ++s) m = fmaxf(m, part_ml[(row * splits + s) * 2]);
-  for (int s = 0; s < splits; ++s) l += part_ml[(row * splits + s) * 2 + 1] * exp2f(part_ml[(row * splits + s) * 2] - m);
-  const float inv = 1.f / l;
-  for (int c = threadIdx.x * 4; c < rank; c += 512) {
-    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int s = 0; s < splits; ++s) {
-      const float w = exp2f(part_ml[(row * splits + s) * 2] - m) * inv;   // an empty split has weight 0 and finite sums
-      const float4 v = load4(part_o + (row * splits + s) * rank + c);
-      a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+  float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int s0 = 0; s0 < splits; s0 += 8) {               // eight partial results in flight; an empty one has weight 0
+    float4 v[8];
+    float2 ml[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const bool on = s0 + i < splits;
+      ml[i] = on ? *reinterpret_cast<const float2*>(part_ml + (row * splits + s0 + i) * 2) : make_float2(-INFINITY, 0.f);
+      v[i] = on && c < rank ? load4(part_o + (row * splits + s0 + i) * rank + c) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    store4(out + row * rank + c, a);
+    float mx = m;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) mx = fmaxf(mx, ml[i].x);
+    const float f = m == -INFINITY ? 0.f : exp2f(m - mx);
+    l *= f; a.x *= f; a.y *= f; a.z *= f; a.w *= f;
+    m = mx;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float w = ml[i].x == -INFINITY ? 0.f : exp2f(ml[i].x - m);
+      l = fmaf(w, ml[i].y, l);
+      a.x = fmaf(w, v[i].x, a.x); a.y = fmaf(w, v[i].y, a.y); a.z = fmaf(w, v[i].z, a.z); a.w = fmaf(w, v[i].w, a.w);
+    }
   }
+  const float inv = 1.f / l;
+  if (c < rank) store4(out + row * rank + c, make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv));
 }
 
 template <int MT, int NT>
@@ -259,8 +276,7 @@ int launch_latent_decode(const LatentDecodeParams& p, int n, cudaStream_t stream
   latent_decode_kernel<MT, NT, KS><<<grid, kLdThreads, smem, stream>>>(p);
   MSA_LAUNCH_OK("latent_decode_kernel");
   if (p.splits > 1) {
-    latent_merge_kernel<<<(unsigned)(n * p.heads), 128, 0, stream>>>(p.part_o, p.part_ml, p.splits, p.rank, p.out);
-    MSA_LAUNCH_OK("latent_merge_kernel");
+    MSA_CUDA_OK(launch_kernel_pdl(latent_merge_kernel, dim3((unsigned)(n * p.heads)), dim3(128), 0, stream, true, p.part_o, p.part_ml, p.splits, p.rank, p.out));
   }
   return MSA_OK;
 }
