@@ -90,7 +90,7 @@ class SequenceStateCache(SparseCache):
 
     One slot holds a sequence's state in every layer run; ``acquire`` / ``release`` hand slots out and take them back.
     Nothing is cleared: the kernels take a sequence at position 0 as empty and never read a ring row that the sequence
-    has not written.  ``specs`` lists the runs in order (``model.state_specs()``); a ring has
+    has not written.  One more slot than asked for exists, ``scratch``: rows that only fill up a step work there.  ``specs`` lists the runs in order (``model.state_specs()``); a ring has
     ``min(window, max_len)`` rows.  The protocol of ``SparseCache`` (``meta``, ``record_kwargs``) stays usable, so the
     interleave loop drives a model on this cache unchanged."""
 
@@ -99,16 +99,17 @@ class SequenceStateCache(SparseCache):
         if n_slots < 1 or max_len < 1:
             raise ValueError("SequenceStateCache needs at least one slot and one position")
         self.specs, self.n_slots, self.max_len, self.device, self.dtype = list(specs), n_slots, max_len, torch.device(device), dtype
+        self.scratch, rows_all = n_slots, n_slots + 1
         self.ring: Dict[int, torch.Tensor] = {}
         self.state: Dict[int, torch.Tensor] = {}
         self.conv: Dict[int, torch.Tensor] = {}
         for i, s in enumerate(self.specs):
             if isinstance(s, RingSpec):
                 rows = max_len if s.window is None else min(s.window, max_len)
-                self.ring[i] = torch.zeros((n_slots, rows, s.width), dtype=dtype, device=device)
+                self.ring[i] = torch.zeros((rows_all, rows, s.width), dtype=dtype, device=device)
             else:
-                self.state[i] = torch.zeros((n_slots, s.heads, s.dim, s.vdim), dtype=torch.float32, device=device)
-                self.conv[i] = torch.zeros((n_slots, 2, s.taps - 1, s.channels), dtype=dtype, device=device)
+                self.state[i] = torch.zeros((rows_all, s.heads, s.dim, s.vdim), dtype=torch.float32, device=device)
+                self.conv[i] = torch.zeros((rows_all, 2, s.taps - 1, s.channels), dtype=dtype, device=device)
         self._free: List[int] = list(range(n_slots - 1, -1, -1))
         self._slot: Dict[Hashable, int] = {}
         self._length: Dict[Hashable, int] = {}

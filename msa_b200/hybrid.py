@@ -332,37 +332,32 @@ class HybridForCausalLM:
 
 
 class GraphedDecode:
-    """Decode steps of a fixed number of sequences as one CUDA graph.  ``run`` feeds tokens from the host,
-    ``replay`` continues on the device with what the last step chose (greedy)."""
+    """Decode steps of up to ``n`` sequences as one CUDA graph.  ``run`` feeds tokens from the host (missing rows work in
+    the cache's scratch slot), ``replay`` continues all ``n`` on the device with what the last step chose (greedy)."""
 
-    def __init__(self, model: HybridForCausalLM, cache: SequenceStateCache, n: int):
+    def __init__(self, model: HybridForCausalLM, cache: SequenceStateCache, n: int, pool=None):
         self.model, self.cache, self.n = model, cache, n
         self.tables = DecodeStep(n, cache, model.config.windows)
-        self.logits = self.next = None
         self.graph = torch.cuda.CUDAGraph()
-        # the warm-up and capture passes run on slots 0 .. n-1 at position 0 and leave garbage there: callers capture
-        # before they acquire slots, or pass slots that are free
         side = torch.cuda.Stream(model.device)
         side.wait_stream(torch.cuda.current_stream(model.device))
 
         def body():
             logits = model.step(self.tables, cache)
             return logits, logits.argmax(dim=-1).to(torch.int32)
-        free = list(cache._free)
-        if len(free) < n:
-            raise RuntimeError(f"capturing a decode step of {n} sequences needs {n} free slots")
-        self.tables.fill([0] * n, [0] * n, free[:n])
+        self.tables.fill([0] * n, [0] * n, [cache.scratch] * n)
         with torch.cuda.stream(side):
             for _ in range(2):
                 body()
         torch.cuda.current_stream(model.device).wait_stream(side)
-        with torch.cuda.graph(self.graph):
+        with torch.cuda.graph(self.graph, pool=pool):
             self.logits, self.next = body()
 
     def run(self, tokens, positions, slots) -> torch.Tensor:
-        self.tables.fill(tokens, positions, slots)
+        k = self.n - len(tokens)
+        self.tables.fill(list(tokens) + [0] * k, list(positions) + [0] * k, list(slots) + [self.cache.scratch] * k)
         self.graph.replay()
-        return self.logits
+        return self.logits[:len(tokens)]
 
     def replay(self) -> torch.Tensor:
         self.tables.token.copy_(self.next)

@@ -2,7 +2,8 @@
 
 A request waits for a slot, its prompt is run in portions of at most ``portion`` tokens beside the decode tokens of the
 other requests, then it decodes one token per step until its length or an end token; its slot goes to the next request.
-Every step is one packed ``model.step``; steps that only decode replay a CUDA graph of their batch size (``graphs``).
+Every step is one packed ``model.step``; steps that only decode replay a CUDA graph (``graphs``), one for each of a few batch
+sizes that smaller batches are filled up to.
 """
 from __future__ import annotations
 
@@ -42,6 +43,7 @@ class Scheduler:
         self._rng: Dict[int, torch.Generator] = {}
         self._graphs: Optional[dict] = {} if graphs and model.device.type == "cuda" else None
         self._seen: Dict[int, int] = {}
+        self._pool = None
 
     # ------------------------------------------------------------------ requests
     def check(self, request: SequenceRequest) -> None:
@@ -99,19 +101,22 @@ class Scheduler:
         return entries
 
     def _decode_logits(self, entries) -> Optional[torch.Tensor]:
-        """Logits of a decode-only step from a graph of its batch size, captured once the size has come up three times."""
+        """Logits of a decode-only step from the graph of the next batch size, captured once that has come up three times."""
         if self._graphs is None or any(len(r.tokens) != r.fed for r, _, _ in entries):
             return None
         n = len(entries)
-        if n not in self._graphs:
-            self._seen[n] = self._seen.get(n, 0) + 1
-            if self._seen[n] < 3 or self.cache.free_slots < n:
+        size = min(n if n <= 4 else (n + 7) // 8 * 8, self.max_batch)
+        if size not in self._graphs:
+            self._seen[size] = self._seen.get(size, 0) + 1
+            if self._seen[size] < 3:
                 return None
             from .hybrid import GraphedDecode
-            self._graphs[n] = GraphedDecode(self.model, self.cache, n)
+            if self._pool is None:
+                self._pool = torch.cuda.graph_pool_handle()       # the graphs never run at once: one pool for all
+            self._graphs[size] = GraphedDecode(self.model, self.cache, size, self._pool)
         c = self.cache
-        logits = self._graphs[n].run([t[0] for _, t, _ in entries], [c.length(r.id) for r, _, _ in entries],
-                                     [c.slot(r.id) for r, _, _ in entries])
+        logits = self._graphs[size].run([t[0] for _, t, _ in entries], [c.length(r.id) for r, _, _ in entries],
+                                        [c.slot(r.id) for r, _, _ in entries])
         for r, _, _ in entries:
             c.advance(r.id, 1)
         return logits

@@ -358,8 +358,8 @@ def test_graphed_decode_matches_plain_steps():
     prompts = [U.tokens_of(cfg, n, 50 + n) for n in (5, 130, 64)]
     runs = []
     for graphed in (False, True):
-        cache = m.new_cache(6, 200)
-        g = GraphedDecode(m, cache, 3) if graphed else None
+        cache = m.new_cache(3, 200)
+        g = GraphedDecode(m, cache, 4) if graphed else None          # one row to fill up
         for i in range(3):
             cache.acquire(i)
         tok = m.run([(i, p, [len(p) - 1]) for i, p in enumerate(prompts)], cache).argmax(-1).tolist()
@@ -390,12 +390,12 @@ def oracle_greedy(name, prompt, n):
 def test_scheduler_generates_what_the_oracle_would(name):
     from msa_b200.scheduler import Scheduler, SequenceRequest
     m, cfg = model(name, torch.float32), U.CONFIGS[name]
-    s = Scheduler(m, max_batch=4, max_len=80, portion=11, step_tokens=16)
-    reqs = [SequenceRequest(U.tokens_of(cfg, n, 60 + n), 7) for n in (23, 1, 40, 9, 2, 17)]
+    s = Scheduler(m, max_batch=6, max_len=80, portion=11, step_tokens=16)
+    reqs = [SequenceRequest(U.tokens_of(cfg, n, 60 + n), 7) for n in (23, 1, 40, 9, 2, 17, 30, 5, 11)]
     for r in reqs:
         s.submit(r)
     s.run()
-    assert s.cache.free_slots == 4
+    assert s.cache.free_slots == 6 and s._graphs          # decode-only steps came from graphs
     for r in reqs:
         assert r.output == oracle_greedy(name, r.tokens, 7)
 

@@ -66,8 +66,8 @@ def cpu_cache(n_slots=3, max_len=50):
 
 def test_slots_are_handed_out_and_taken_back():
     c = cpu_cache()
-    assert c.ring[0].shape == (3, 8, 6) and c.ring[2].shape == (3, 50, 6)
-    assert c.state[1].shape == (3, 2, 3, 4) and c.conv[1].shape == (3, 2, 2, 20)
+    assert c.ring[0].shape == (4, 8, 6) and c.ring[2].shape == (4, 50, 6) and c.scratch == 3      # one slot to spare
+    assert c.state[1].shape == (4, 2, 3, 4) and c.conv[1].shape == (4, 2, 2, 20)
     slots = {s: c.acquire(s) for s in "abc"}
     assert sorted(slots.values()) == [0, 1, 2] and c.free_slots == 0
     with pytest.raises(RuntimeError):
