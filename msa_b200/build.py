@@ -20,7 +20,7 @@ LIB_LM = os.path.join(HERE, "libmsa_b200_lm.so")
 SOURCES = ["cabi.cu", "pool.cu", "bookkeeping.cu", "route_simt.cu", "route_tc.cu", "route_modes.cu", "route_dec.cu", "topk.cu", "gather.cu", "decode_attn.cu", "prefill_attn.cu", "attn_generic.cu", "doc_attn_tc.cu", "decode_dense.cu"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC"]
-LM_SOURCES = ["cabi.cu", "lm_norm.cu", "lm_latent.cu", "lm_attn_tc.cu", "lm_latent_decode.cu", "lm_delta.cu", "lm_delta_chunk.cu", "lm_moe.cu", "lm_moe_tc.cu"]
+LM_SOURCES = ["cabi.cu", "lm_norm.cu", "lm_latent.cu", "lm_attn_tc.cu", "lm_latent_decode.cu", "lm_delta.cu", "lm_delta_chunk.cu", "lm_group.cu", "lm_linear.cu", "lm_linear_chunk.cu", "lm_moe.cu", "lm_moe_tc.cu"]
 # name -> (library, sources, extra flags, headers outside csrc).  The decoder designs keep the full accuracy of 32-bit
 # divisions, exponentials and angles.
 LIBRARIES = {

@@ -69,20 +69,25 @@ class SparseCacheOnCPU(SparseCache):
 
 @dataclass(frozen=True)
 class RingSpec:
-    """A windowed layer's state: the last rows of ``width`` elements (``window`` None: every row)."""
+    """A windowed layer's state: the last rows of ``width`` elements (``window`` None: every row) and, where a short
+    convolution feeds them, its last ``taps - 1`` inputs over ``channels`` channels."""
     width: int
     window: Optional[int]
+    channels: int = 0
+    taps: int = 1
 
 
 @dataclass(frozen=True)
 class RecurrentSpec:
     """A recurrent layer's state: a ``[heads, dim, vdim]`` fp32 matrix per head and the last ``taps - 1`` inputs of its
-    convolution over ``channels`` channels (double-buffered by the parity of the sequence's position)."""
+    convolution over ``channels`` channels (double-buffered by the parity of the sequence's position); ``shift``: width of
+    the layer's input if the previous token's is kept."""
     heads: int
     dim: int
     vdim: int
-    channels: int
-    taps: int
+    channels: int = 0
+    taps: int = 1
+    shift: int = 0
 
 
 class SequenceStateCache(SparseCache):
@@ -91,7 +96,7 @@ class SequenceStateCache(SparseCache):
     One slot holds a sequence's state in every layer run; ``acquire`` / ``release`` hand slots out and take them back.
     Nothing is cleared: the kernels take a sequence at position 0 as empty and never read a ring row that the sequence
     has not written.  One more slot than asked for exists, ``scratch``: rows that only fill up a step work there.  ``specs`` lists the runs in order (``model.state_specs()``); a ring has
-    ``min(window, max_len)`` rows.  The protocol of ``SparseCache`` (``meta``, ``record_kwargs``) stays usable, so the
+    ``min(window, max_len)`` rows.  ``last_token`` keeps every sequence's previous token (for embeddings that read it).  The protocol of ``SparseCache`` (``meta``, ``record_kwargs``) stays usable, so the
     interleave loop drives a model on this cache unchanged."""
 
     def __init__(self, specs: Sequence, n_slots: int, max_len: int, device, dtype: torch.dtype):
@@ -103,12 +108,17 @@ class SequenceStateCache(SparseCache):
         self.ring: Dict[int, torch.Tensor] = {}
         self.state: Dict[int, torch.Tensor] = {}
         self.conv: Dict[int, torch.Tensor] = {}
+        self.shift: Dict[int, torch.Tensor] = {}
+        self.last_token = torch.zeros(rows_all, dtype=torch.int32, device=device)
         for i, s in enumerate(self.specs):
             if isinstance(s, RingSpec):
                 rows = max_len if s.window is None else min(s.window, max_len)
                 self.ring[i] = torch.zeros((rows_all, rows, s.width), dtype=dtype, device=device)
             else:
                 self.state[i] = torch.zeros((rows_all, s.heads, s.dim, s.vdim), dtype=torch.float32, device=device)
+                if s.shift:
+                    self.shift[i] = torch.zeros((rows_all, s.shift), dtype=dtype, device=device)
+            if s.channels:
                 self.conv[i] = torch.zeros((rows_all, 2, s.taps - 1, s.channels), dtype=dtype, device=device)
         self._free: List[int] = list(range(n_slots - 1, -1, -1))
         self._slot: Dict[Hashable, int] = {}
@@ -143,7 +153,7 @@ class SequenceStateCache(SparseCache):
         self._length[seq] += n
 
     def state_bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for d in (self.ring, self.state, self.conv) for t in d.values())
+        return sum(t.numel() * t.element_size() for d in (self.ring, self.state, self.conv, self.shift) for t in d.values())
 
 
 @dataclass

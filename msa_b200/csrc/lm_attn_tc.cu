@@ -28,7 +28,10 @@ struct WindowAttnTcParams {
   const int32_t *start, *cu, *ctx_off;   // ctx_off counts from seq0
   int seq0, heads, window;
   int q_row0;                            // packed row of the first query row of the map
-  int q_head, k_head, v_head, v_col, r_col;   // column strides of a head, first value column, rotated column of the context
+  int q_head, k_head, v_head;            // column strides of a head
+  int group;                             // query heads per key / value head
+  int sink;                              // one more entry per softmax, with score 0 and no value
+  const __nv_bfloat16* gate; long long gate_row;   // null, or one logit per row and head
   float scale_log2e;
   long long n_sh, n_items;               // sequences * heads; times the row blocks of the longest portion
   __nv_bfloat16* out; long long out_row;
@@ -137,14 +140,14 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
           if (!(ok = mbar_wait(&s_k_empty[st], ph ^ 1u, abort_flag, p.status, 1))) break;
           mbar_expect_tx(&s_k_full[st], QB * kWaKBlk);
 #pragma unroll
-          for (int c = 0; c < DB; ++c) tma_load_2d(ks + c * kWaKBlk, &tmap_k, it.h * p.k_head + 64 * c, y, &s_k_full[st]);
+          for (int c = 0; c < DB; ++c) tma_load_2d(ks + c * kWaKBlk, &tmap_k, it.h / p.group * p.k_head + 64 * c, y, &s_k_full[st]);
 #pragma unroll
-          for (int c = 0; c < RB; ++c) tma_load_2d(ks + (DB + c) * kWaKBlk, &tmap_r, p.r_col + 64 * c, y, &s_k_full[st]);
+          for (int c = 0; c < RB; ++c) tma_load_2d(ks + (DB + c) * kWaKBlk, &tmap_r, 64 * c, y, &s_k_full[st]);
           if (!(ok = mbar_wait(&s_v_empty[st], ph ^ 1u, abort_flag, p.status, 1))) break;
           mbar_expect_tx(&s_v_full[st], VB * kWaKBlk);
 #pragma unroll
           for (int c = 0; c < VB; ++c)
-            tma_load_2d(ks + (QB + c) * kWaKBlk, &tmap_v, p.v_col + it.h * p.v_head + 64 * c, y, &s_v_full[st]);
+            tma_load_2d(ks + (QB + c) * kWaKBlk, &tmap_v, it.h / p.group * p.v_head + 64 * c, y, &s_v_full[st]);
         }
         ++n_it;
       }
@@ -240,7 +243,7 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
     for (long long w = blockIdx.x; w < p.n_items && ok; w += gridDim.x) {
       const WaItem it = wa_item(p, w);
       if (!it.valid || it.a[q] == it.b[q]) continue;
-      float m_ref = -1e30f, l_run = 0.f;
+      float m_ref = p.sink ? 0.f : -1e30f, l_run = p.sink ? 1.f : 0.f;
       const int row0 = it.r0 + q * kWaRows + wq * 32;          // first row of this warp
       for (int t = it.a[q]; t < it.b[q]; ++t, ++n_c) {
         const uint32_t sb = n_c & 1u;
@@ -285,12 +288,12 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
         mx = fmaxf(mx, mx2);
         const bool move = (mx - m_ref) * p.scale_log2e > kWaRescale;
         if (__any_sync(0xffffffffu, move)) {
+          const float f = move ? exp2f((m_ref - mx) * p.scale_log2e) : 1.f;
           if (t > it.a[q]) {   // wait for the PV in flight, then rescale this warp's rows of O in place
             ok = mbar_wait(&s_o_full[q][(n_c - 1u) & 1u], ((n_c - 1u) >> 1) & 1u, abort_flag, p.status, 6);
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
             tc_fence_after();
-            const float f = move ? exp2f((m_ref - mx) * p.scale_log2e) : 1.f;
 #pragma unroll
             for (int c = 0; c < VB * 4; ++c) {
               uint32_t v[16];
@@ -300,8 +303,8 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
               for (int i = 0; i < 16; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * f);
               tmem_st16(lane_base + col_o + 16 * c, v);
             }
-            l_run *= f;
           }
+          l_run *= f;
           if (move) m_ref = mx;
         }
         const float neg_m = -m_ref * p.scale_log2e;
@@ -346,7 +349,9 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      const float inv = 1.f / l_run;
+      float inv = 1.f / l_run;
+      if (p.gate && row0 + lane < it.len)
+        inv *= sigmoid_f(__bfloat162float(p.gate[(it.q_row + q * kWaRows + wq * 32 + lane) * p.gate_row + it.h]));
       unsigned char* stg = out_stage + warp * kWaStage;
       __nv_bfloat16* dst0 = p.out + (long long)(it.q_row + q * kWaRows + wq * 32) * p.out_row + (long long)it.h * VB * 64;
 #pragma unroll
@@ -405,31 +410,36 @@ extern "C" int msa_lm_window_attn_tc_supported(int32_t dim, int32_t rot, int32_t
   return (dim == 64 || dim == 128) && (rot == 0 || rot == 64) && (vdim == 64 || vdim == 128);
 }
 
-extern "C" int msa_lm_window_attn_tc(const void* q, int64_t q_row, int32_t n_rows, const void* kv, int64_t kv_row,
-                                     const void* ctx, int64_t ctx_row, int32_t n_ctx, int32_t heads, int32_t dim, int32_t rot,
-                                     int32_t vdim, int32_t rank, const int32_t* start, const int32_t* cu,
-                                     const int32_t* ctx_off, int32_t seq0, int32_t seq1, int32_t row0, int32_t max_len,
-                                     int32_t window, float scale, void* out, int64_t out_row, int32_t* status, void* stream) {
-  MSA_REQUIRE(q && kv && ctx && start && cu && ctx_off && out && status, "window_attn_tc: null pointer");
+extern "C" int msa_lm_window_attn_tc(const msa_lm_attn_args* args, int32_t n_rows, int32_t n_ctx, int32_t row0, int32_t* status, void* stream) {
+  MSA_REQUIRE(args, "window_attn_tc: null arguments");
+  const msa_lm_attn_args a = *args;
+  const int dim = a.da, rot = a.db, vdim = a.dv;
+  MSA_REQUIRE(a.qa && a.ka && a.v && a.start && a.cu && a.ctx_off && a.out && status && a.ring_rows == 0, "window_attn_tc: null pointer");
+  MSA_REQUIRE(a.dtype == MSA_BF16 && a.qa_dtype == MSA_BF16 && a.out_dtype == MSA_BF16, "window_attn_tc: bf16 only");
   MSA_REQUIRE(msa_lm_window_attn_tc_supported(dim, rot, vdim), "window_attn_tc: unsupported head sizes (%d, %d, %d)", dim, rot, vdim);
-  MSA_REQUIRE(heads > 0 && window > 0 && rank > 0 && rank % 8 == 0 && scale > 0.f, "window_attn_tc: bad sizes");
-  MSA_REQUIRE(aligned16(q) && aligned16(kv) && aligned16(ctx) && aligned16(out) && q_row % 8 == 0 && kv_row % 8 == 0 &&
-                  ctx_row % 8 == 0 && out_row % 8 == 0, "window_attn_tc: rows must be 16-byte aligned");
-  if (seq1 <= seq0 || max_len <= 0 || n_rows <= 0) return MSA_OK;
+  MSA_REQUIRE(a.heads > 0 && a.window > 0 && a.scale > 0.f && a.group > 0 && a.heads % a.group == 0, "window_attn_tc: bad sizes");
+  MSA_REQUIRE(rot == 0 || (a.kb && a.kb_head == 0 && a.qb == (const __nv_bfloat16*)a.qa + dim && a.qb_head == a.qa_head),
+              "window_attn_tc: the rotated parts must follow the plain query part and be shared by the keys");
+  MSA_REQUIRE(aligned16(a.qa) && aligned16(a.ka) && aligned16(a.v) && aligned16(a.out) && (rot == 0 || aligned16(a.kb)) &&
+                  a.qa_row % 8 == 0 && a.ka_row % 8 == 0 && a.v_row % 8 == 0 && a.out_row % 8 == 0 && a.kb_row % 8 == 0 &&
+                  a.qa_head % 8 == 0 && a.ka_head % 8 == 0 && a.v_head % 8 == 0 && a.out_head == vdim, "window_attn_tc: rows must be 16-byte aligned");
+  if (a.seq1 <= a.seq0 || a.max_len <= 0 || n_rows <= 0) return MSA_OK;
+  const int kv_heads = a.heads / a.group;
   CUtensorMap mq, mk, mr, mv;
-  MSA_OK_OR_RETURN(make_map(&mq, q, n_rows, (uint64_t)heads * (dim + rot), q_row, 64, kWaRows));
-  MSA_OK_OR_RETURN(make_map(&mk, kv, n_ctx, (uint64_t)heads * (dim + vdim), kv_row, 64, kWaKeys));
-  mv = mk;
-  if (rot) MSA_OK_OR_RETURN(make_map(&mr, ctx, n_ctx, (uint64_t)rank + rot, ctx_row, 64, kWaKeys));
+  MSA_OK_OR_RETURN(make_map(&mq, a.qa, n_rows, (uint64_t)(a.heads - 1) * a.qa_head + dim + rot, a.qa_row, 64, kWaRows));
+  MSA_OK_OR_RETURN(make_map(&mk, a.ka, n_ctx, (uint64_t)(kv_heads - 1) * a.ka_head + dim, a.ka_row, 64, kWaKeys));
+  MSA_OK_OR_RETURN(make_map(&mv, a.v, n_ctx, (uint64_t)(kv_heads - 1) * a.v_head + vdim, a.v_row, 64, kWaKeys));
+  if (rot) MSA_OK_OR_RETURN(make_map(&mr, a.kb, n_ctx, (uint64_t)rot, a.kb_row, 64, kWaKeys));
   else mr = mk;
   WindowAttnTcParams p{};
-  p.start = start; p.cu = cu; p.ctx_off = ctx_off;
-  p.seq0 = seq0; p.heads = heads; p.window = window; p.q_row0 = row0;
-  p.q_head = dim + rot; p.k_head = dim; p.v_head = vdim; p.v_col = heads * dim; p.r_col = rank;
-  p.scale_log2e = scale * 1.4426950408889634f;
-  p.n_sh = (long long)(seq1 - seq0) * heads;
-  p.n_items = p.n_sh * ((max_len + kWaRows * kWaTiles - 1) / (kWaRows * kWaTiles));
-  p.out = (__nv_bfloat16*)out; p.out_row = out_row; p.status = status;
+  p.start = a.start; p.cu = a.cu; p.ctx_off = a.ctx_off;
+  p.seq0 = a.seq0; p.heads = a.heads; p.window = a.window; p.q_row0 = row0;
+  p.q_head = (int)a.qa_head; p.k_head = (int)a.ka_head; p.v_head = (int)a.v_head;
+  p.group = a.group; p.sink = a.sink; p.gate = (const __nv_bfloat16*)a.gate; p.gate_row = a.gate_row;
+  p.scale_log2e = a.scale * 1.4426950408889634f;
+  p.n_sh = (long long)(a.seq1 - a.seq0) * a.heads;
+  p.n_items = p.n_sh * ((a.max_len + kWaRows * kWaTiles - 1) / (kWaRows * kWaTiles));
+  p.out = (__nv_bfloat16*)a.out; p.out_row = a.out_row; p.status = status;
   cudaStream_t st = (cudaStream_t)stream;
   const int key = (dim / 64) * 100 + (rot / 64) * 10 + vdim / 64;
   switch (key) {

@@ -66,6 +66,10 @@ __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
+// silu in front of a rounding to T.
+template <typename T> __device__ __forceinline__ float silu_act(float z) { return silu_f(z); }
+template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+
 // Index of the sequence that owns position `i` of a prefix-sum table off[0 .. n].
 __device__ __forceinline__ int owner_of(const int32_t* off, int n, int i) {
   int lo = 0, hi = n - 1;

@@ -9,6 +9,7 @@
 #include <type_traits>
 
 #include "lm_common.cuh"
+#include "lm_conv.cuh"
 
 namespace msa {
 
@@ -72,21 +73,8 @@ delta_prep_kernel(const msa_lm_delta_args a, float* __restrict__ qk, float* __re
 // head of q or k, or 128 channels of v), so every input is loaded once.
 constexpr int kPrepRows = 8;
 
-template <typename T> __device__ __forceinline__ float silu_act(float z) { return silu_f(z); }
-template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
-
 // SPLIT: q and k leave as pairs of bf16 numbers whose sum they are, [rows, 2 (q, k), 2 (hi, lo), kv_heads, dim], and v in
 // bf16.
-template <typename T> struct Raw4;
-template <> struct Raw4<float> { using type = float4; };
-template <> struct Raw4<__nv_bfloat16> { using type = uint2; };
-__device__ __forceinline__ float4 widen(float4 v) { return v; }
-__device__ __forceinline__ float4 widen(uint2 r) {
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
-  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
-  return make_float4(a.x, a.y, b.x, b.y);
-}
-
 template <typename T, int TAPS, bool SPLIT>
 __global__ void __launch_bounds__(256)
 delta_prep_vec_kernel(const msa_lm_delta_args a, void* __restrict__ qk_out, void* __restrict__ v_out, float* __restrict__ gates) {

@@ -156,8 +156,8 @@ ring_store_kernel(const T* __restrict__ ctx, int width, const int32_t* slot, con
   }
 }
 
-// General attention: 8 rows per block, a row = (token, head).  With shared keys and values a block's rows run over the
-// heads of a token first; otherwise a block stays in one head.  A tile of up to 32 keys and values is staged in shared
+// General attention: 8 rows per block, a row = (token, head).  A block's rows run over the heads that share a key / value
+// head first.  A tile of up to 32 keys and values is staged in shared
 // memory as fp32; lane = key for the scores, lane = value column for the output.
 constexpr int kGaRows = 8, kGaThreads = 128;
 
@@ -188,7 +188,8 @@ __global__ void __launch_bounds__(kGaThreads) window_attn_kernel(const msa_lm_at
   const int p_lo = start + t_lo, p_hi = start + t_hi;
   const int j0 = max(0, p_lo - a.window + 1);
   const int first = start - min(start, a.window - 1);
-  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  const float m0 = a.sink ? 0.f : -INFINITY, l0 = a.sink ? 1.f : 0.f;     // the sink: one entry with score 0 and no value
+  float m[2] = {m0, m0}, l[2] = {l0, l0};
   for (int jt = j0; jt <= p_hi; jt += tile) {
     const int nk = min(tile, p_hi - jt + 1);
     __syncthreads();
@@ -196,9 +197,9 @@ __global__ void __launch_bounds__(kGaThreads) window_attn_kernel(const msa_lm_at
       const int k = i / (dq + a.dv), c = i % (dq + a.dv), j = jt + k;
       const long long row = a.ring_rows > 0 ? (long long)a.slot[s] * a.ring_rows + j % a.ring_rows
                                             : (long long)a.ctx_off[s - a.seq0] + (j - first);
-      if (c < a.da) s_k[k * kstr + c] = load_any(a.ka, a.dtype, row * a.ka_row + h0 * a.ka_head + c);
-      else if (c < dq) s_k[k * kstr + c] = load_any(a.kb, a.dtype, row * a.kb_row + h0 * a.kb_head + (c - a.da));
-      else s_v[k * a.dv + (c - dq)] = load_any(a.v, a.dtype, row * a.v_row + h0 * a.v_head + (c - dq));
+      if (c < a.da) s_k[k * kstr + c] = load_any(a.ka, a.dtype, row * a.ka_row + blockIdx.y * a.ka_head + c);
+      else if (c < dq) s_k[k * kstr + c] = load_any(a.kb, a.dtype, row * a.kb_row + blockIdx.y * a.kb_head + (c - a.da));
+      else s_v[k * a.dv + (c - dq)] = load_any(a.v, a.dtype, row * a.v_row + blockIdx.y * a.v_head + (c - dq));
     }
     __syncthreads();
 #pragma unroll
@@ -235,8 +236,9 @@ __global__ void __launch_bounds__(kGaThreads) window_attn_kernel(const msa_lm_at
     const long long rr = r0 + r;
     const long long tok = a.cu[s] - a.cu[a.seq0] + rr / hg;
     const int h = h0 + (int)(rr % hg);
+    const float inv = (a.gate ? sigmoid_f(load_any(a.gate, a.dtype, tok * a.gate_row + h)) : 1.f) / l[q];
     for (int c = lane; c < a.dv; c += 32)
-      store_any(a.out, a.out_dtype, tok * a.out_row + h * a.out_head + c, s_o[r * a.dv + c] / l[q]);
+      store_any(a.out, a.out_dtype, tok * a.out_row + h * a.out_head + c, s_o[r * a.dv + c] * inv);
   }
 }
 
@@ -295,8 +297,8 @@ extern "C" int msa_lm_window_attn(const msa_lm_attn_args* args, void* stream) {
   MSA_REQUIRE(a.ring_rows > 0 ? a.slot != nullptr : a.ctx_off != nullptr, "window_attn: no key addressing");
   MSA_REQUIRE(a.heads > 0 && a.da > 0 && a.db >= 0 && a.dv > 0 && a.window > 0, "window_attn: bad sizes");
   if (a.seq1 <= a.seq0 || a.max_len <= 0) return MSA_OK;
-  const bool shared = a.ka_head == 0 && a.v_head == 0 && (a.db == 0 || a.kb_head == 0);
-  const int hg = shared ? a.heads : 1;
+  MSA_REQUIRE(a.group > 0 && a.heads % a.group == 0, "window_attn: heads must be a multiple of group");
+  const int hg = a.group;
   const int dq = a.da + a.db;
   int tile = 32;
   auto bytes = [&](int t) { return (size_t)4 * ((size_t)kGaRows * (dq + a.dv) + (size_t)t * (dq + 1 + a.dv)); };

@@ -8,6 +8,7 @@
 // the slices' partial scores are added up in shared memory, where eight (sixteen) threads per head do the fp32 softmax.
 // For the output the warps split the latent columns.
 #include "lm_common.cuh"
+#include "lm_merge.cuh"
 #include "mma_helpers.cuh"
 #include "tc_attn_common.cuh"
 
@@ -231,40 +232,6 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     }
 }
 
-// Launched early (programmatic dependent launch): waits for the partial results before it reads them.
-__global__ void __launch_bounds__(128)
-latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits, int rank, __nv_bfloat16* __restrict__ out) {
-  const long long row = blockIdx.x;
-  const int c = threadIdx.x * 4;
-  grid_dependency_wait();
-  float m = -INFINITY, l = 0.f;
-  float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-  for (int s0 = 0; s0 < splits; s0 += 8) {               // eight partial results in flight; an empty one has weight 0
-    float4 v[8];
-    float2 ml[8];
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const bool on = s0 + i < splits;
-      ml[i] = on ? *reinterpret_cast<const float2*>(part_ml + (row * splits + s0 + i) * 2) : make_float2(-INFINITY, 0.f);
-      v[i] = on && c < rank ? load4(part_o + (row * splits + s0 + i) * rank + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
-    float mx = m;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) mx = fmaxf(mx, ml[i].x);
-    const float f = m == -INFINITY ? 0.f : exp2f(m - mx);
-    l *= f; a.x *= f; a.y *= f; a.z *= f; a.w *= f;
-    m = mx;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const float w = ml[i].x == -INFINITY ? 0.f : exp2f(ml[i].x - m);
-      l = fmaf(w, ml[i].y, l);
-      a.x = fmaf(w, v[i].x, a.x); a.y = fmaf(w, v[i].y, a.y); a.z = fmaf(w, v[i].z, a.z); a.w = fmaf(w, v[i].w, a.w);
-    }
-  }
-  const float inv = 1.f / l;
-  if (c < rank) store4(out + row * rank + c, make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv));
-}
-
 template <int MT, int NT>
 int launch_latent_decode(const LatentDecodeParams& p, int n, cudaStream_t stream) {
   constexpr int KQ = 8 / MT, KS = (NT * 4 + 4 + KQ - 1) / KQ;               // up to 64 rotated columns
@@ -276,7 +243,8 @@ int launch_latent_decode(const LatentDecodeParams& p, int n, cudaStream_t stream
   latent_decode_kernel<MT, NT, KS><<<grid, kLdThreads, smem, stream>>>(p);
   MSA_LAUNCH_OK("latent_decode_kernel");
   if (p.splits > 1) {
-    MSA_CUDA_OK(launch_kernel_pdl(latent_merge_kernel, dim3((unsigned)(n * p.heads)), dim3(128), 0, stream, true, p.part_o, p.part_ml, p.splits, p.rank, p.out));
+    const MergeParams m{p.part_o, p.part_ml, p.heads, p.splits, p.rank, 0, nullptr, 0, p.out, (long long)p.heads * p.rank};
+    return launch_merge(m, n, stream);
   }
   return MSA_OK;
 }

@@ -23,25 +23,35 @@ def matmul(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
     return torch.mm(x, w.t(), out_dtype=out_dtype)
 
 
-def embed(table, token, w_next, eps, cat: Optional[torch.Tensor] = None, cat_both: bool = False, status=None):
-    """``(x fp32, h)``: the embedding rows and, with ``w_next``, their norm.  ``cat`` [n, 2*width]: its right half (with
-    ``cat_both`` its left half too) receives the rows."""
+def embed(table, token, w_next, eps, cat: Optional[torch.Tensor] = None, cat_both: bool = False, status=None, *, w_next2=None,
+          x_copy: Optional[torch.Tensor] = None, pair=None, step=None, last_token=None):
+    """``(x fp32, h)``: the embedding rows and, with ``w_next``, their norm (``w_next2``: a second one, ``(x, h, h2)``).
+    ``cat`` [n, 2*width]: its right half (with ``cat_both`` its left half too) receives the rows; ``x_copy`` fp32 too.
+    ``pair`` = (table, buckets, mul_prev, mul_cur): hashed rows of (previous token, token) join, from the tables of ``step``
+    and ``last_token`` [slots]."""
     A.need_cuda(table, token)
     n, width = token.shape[0], table.shape[1]
     x = torch.empty((n, width), dtype=torch.float32, device=table.device)
     h = torch.empty((n, width), dtype=table.dtype, device=table.device) if w_next is not None else None
-    cat0 = A.ptr(cat) if cat is not None and cat_both else 0
-    cat1 = A.ptr(cat) + width * cat.element_size() if cat is not None else 0
-    A.call("msa_lm_embed", A.ptr(table), A.ptr(token), n, width, table.shape[0], A.ptr(w_next), float(eps), A.ptr(x),
-           A.ptr(h), cat0, cat1, _rows(cat) if cat is not None else 0, A.ptr(status), A.dtype_code(table.dtype),
-           A.stream_ptr(table.device))
-    return x, h
+    h2 = torch.empty_like(h) if w_next2 is not None else None
+    args = A.EmbedArgs(table=A.ptr(table), token=A.ptr(token), w_next=A.ptr(w_next), w_next2=A.ptr(w_next2), x_out=A.ptr(x), x_copy=A.ptr(x_copy),
+                       h_out=A.ptr(h), h_out2=A.ptr(h2), cat0=A.ptr(cat) if cat is not None and cat_both else 0,
+                       cat1=A.ptr(cat) + width * cat.element_size() if cat is not None else 0,
+                       cat_stride=_rows(cat) if cat is not None else 0, status=A.ptr(status), n_rows=n, width=width, vocab=table.shape[0],
+                       eps=float(eps), dtype=A.dtype_code(table.dtype))
+    if pair is not None:
+        args.pair_table, args.buckets, args.mul_prev, args.mul_cur = A.ptr(pair[0]), pair[1], pair[2], pair[3]
+        args.last_token, args.tok_seq, args.slot = A.ptr(last_token), A.ptr(step.tok_seq), A.ptr(step.slot)
+        args.start, args.cu = A.ptr(step.start), A.ptr(step.cu)
+    A.call("msa_lm_embed", C.byref(args), A.stream_ptr(table.device))
+    return (x, h) if w_next2 is None else (x, h, h2)
 
 
 def residual_norm(base, y, w_branch, w_next, eps, dtype, *, x_out=None, want_h=True, cat=None, inv=None, mix=None,
-                  rows=None, broadcast=False):
-    """One launch of ``msa_lm_residual_norm``; returns ``h`` (or None).  ``base`` fp32 rows (``broadcast``: one vector),
-    ``y`` the branch or the expert outputs when ``inv`` / ``mix`` [n, top] are given."""
+                  rows=None, broadcast=False, add=None, w_next2=None):
+    """One launch of ``msa_lm_residual_norm``; returns ``h`` (or None; with ``w_next2`` a pair).  ``base`` fp32 rows
+    (``broadcast``: one vector), ``y`` the branch or the expert outputs when ``inv`` / ``mix`` [n, top] are given, ``add``
+    further fp32 rows."""
     A.need_cuda(base, y)
     width = (base if base is not None else y).shape[-1]
     if rows is not None:
@@ -52,18 +62,48 @@ def residual_norm(base, y, w_branch, w_next, eps, dtype, *, x_out=None, want_h=T
         n = y.shape[0] if y is not None else base.shape[0]
     dev = (base if base is not None else y).device
     h = torch.empty((n, width), dtype=dtype, device=dev) if want_h and w_next is not None else None
+    h2 = torch.empty_like(h) if h is not None and w_next2 is not None else None
     A.call("msa_lm_residual_norm", A.ptr(base), 0 if broadcast or base is None else _rows(base), A.ptr(y),
            A.dtype_code(y.dtype) if y is not None else 0, _rows(y) if y is not None else 0, A.ptr(inv), A.ptr(mix),
            inv.shape[1] if inv is not None else 0, A.ptr(w_branch), A.ptr(w_next) if h is not None else 0, float(eps),
-           A.ptr(rows), n, width, A.ptr(x_out), A.ptr(h), A.ptr(cat), _rows(cat) if cat is not None else 0,
-           A.dtype_code(dtype), A.stream_ptr(dev))
-    return h
+           A.ptr(rows), n, width, A.ptr(x_out), A.ptr(h), A.ptr(cat), _rows(cat) if cat is not None else 0, A.ptr(add),
+           A.ptr(w_next2) if h2 is not None else 0, A.ptr(h2), A.dtype_code(dtype), A.stream_ptr(dev))
+    return h if w_next2 is None else (h, h2)
 
 
-def silu_mul(gu: torch.Tensor, ff: int) -> torch.Tensor:
+def silu_mul(gu: torch.Tensor, ff: int, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     A.need_cuda(gu)
-    out = torch.empty((gu.shape[0], ff), dtype=gu.dtype, device=gu.device)
-    A.call("msa_lm_silu_mul", A.ptr(gu), _rows(gu), gu.shape[0], ff, A.ptr(out), A.dtype_code(gu.dtype), A.stream_ptr(gu.device))
+    if out is None:
+        out = torch.empty((gu.shape[0], ff), dtype=gu.dtype, device=gu.device)
+    A.call("msa_lm_silu_mul", A.ptr(gu), _rows(gu), gu.shape[0], ff, A.ptr(out), _rows(out), A.dtype_code(gu.dtype), A.stream_ptr(gu.device))
+    return out
+
+
+def softcap(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    """In place on fp32 logits."""
+    if logits.numel():
+        A.call("msa_lm_softcap", A.ptr(logits), logits.numel(), float(cap), A.stream_ptr(logits.device))
+    return logits
+
+
+def token_shift(h, mu, step, shift):
+    """``[mixes, n, width]``: every row of ``h`` mixed with its sequence's previous one (``shift`` keeps the last rows)."""
+    A.need_cuda(h, mu)
+    out = torch.empty((mu.shape[0],) + h.shape, dtype=h.dtype, device=h.device)
+    A.call("msa_lm_token_shift", A.ptr(h), A.ptr(mu), mu.shape[0], h.shape[0], h.shape[1], A.ptr(step.tok_seq), A.ptr(step.slot),
+           A.ptr(step.start), A.ptr(step.cu), A.ptr(shift), A.ptr(out), A.dtype_code(h.dtype), A.stream_ptr(h.device))
+    return out
+
+
+def tanh_split(x: torch.Tensor, dtype: torch.dtype, parts: int) -> torch.Tensor:
+    out = torch.empty((x.shape[0], parts * x.shape[1]), dtype=dtype, device=x.device)
+    A.call("msa_lm_tanh_split", A.ptr(x), x.shape[0], x.shape[1], parts, A.ptr(out), A.dtype_code(dtype), A.stream_ptr(x.device))
+    return out
+
+
+def part_norm(x, w, parts, eps, out):
+    A.call("msa_lm_part_norm", A.ptr(x), _rows(x), A.ptr(w), x.shape[0], x.shape[1], parts, float(eps), A.ptr(out), _rows(out),
+           A.dtype_code(out.dtype), A.stream_ptr(x.device))
     return out
 
 
@@ -83,35 +123,38 @@ def ring_store(ctx, step, view, ring):
            A.dtype_code(ctx.dtype), A.stream_ptr(ctx.device))
 
 
-def window_attn(qa, qb, ka, kb, v, out, *, scale, window, start, cu, seq0, seq1, max_len, slot=None, ctx_off=None, ring_rows=0):
-    """General windowed attention.  ``qa`` / ``qb`` / ``out`` are ``[tokens, heads, d]`` views of the query rows,
-    ``ka`` / ``kb`` / ``v`` ``[rows, heads or 1, d]`` views of the key rows (1: shared by the heads)."""
+def attn_args(qa, qb, ka, kb, v, out, *, scale, window, start, cu, seq0, seq1, max_len, slot=None, ctx_off=None, ring_rows=0,
+              sink=False, gate=None) -> A.AttnArgs:
+    """``qa`` / ``qb`` / ``out`` are ``[tokens, heads, d]`` views of the query rows, ``ka`` / ``kb`` / ``v`` ``[rows, kv heads, d]``
+    views of the key rows; ``gate`` ``[tokens, heads]`` logits."""
     head = lambda t: 0 if t is None or t.shape[1] == 1 else t.stride(1)
     row = lambda t: 0 if t is None else t.stride(0)
     for t in (qa, qb, ka, kb, v, out):
         if t is not None and t.stride(2) != 1:
-            raise A.MsaError("window_attn: contiguous last axis expected")
-    args = A.AttnArgs(
+            raise A.MsaError("window attention: contiguous last axis expected")
+    return A.AttnArgs(
         qa=A.ptr(qa), qa_row=row(qa), qa_head=qa.stride(1), qb=A.ptr(qb), qb_row=row(qb), qb_head=qb.stride(1) if qb is not None else 0,
         ka=A.ptr(ka), ka_row=row(ka), ka_head=head(ka), kb=A.ptr(kb), kb_row=row(kb), kb_head=head(kb),
         v=A.ptr(v), v_row=row(v), v_head=head(v), out=A.ptr(out), out_row=row(out), out_head=out.stride(1),
-        slot=A.ptr(slot), start=A.ptr(start), cu=A.ptr(cu), ctx_off=A.ptr(ctx_off), ring_rows=ring_rows, seq0=seq0, seq1=seq1,
+        gate=A.ptr(gate), gate_row=row(gate), slot=A.ptr(slot), start=A.ptr(start), cu=A.ptr(cu), ctx_off=A.ptr(ctx_off),
+        ring_rows=ring_rows, group=qa.shape[1] // max(ka.shape[1], v.shape[1]), sink=1 if sink else 0, seq0=seq0, seq1=seq1,
         max_len=max_len, heads=qa.shape[1], da=qa.shape[2], db=qb.shape[2] if qb is not None else 0, dv=v.shape[2], window=window,
         qa_dtype=A.dtype_code(qa.dtype), out_dtype=A.dtype_code(out.dtype), dtype=A.dtype_code(ka.dtype), scale=float(scale))
-    A.call("msa_lm_window_attn", C.byref(args), A.stream_ptr(qa.device))
 
 
-def window_attn_tc_supported(spec, dtype) -> bool:
-    return (dtype == torch.bfloat16 and spec.kv_rank % 8 == 0 and spec.scale > 0
-            and bool(A.lib().msa_lm_window_attn_tc_supported(spec.dim, spec.rot_dim, spec.vdim)))
+def window_attn(qa, qb, ka, kb, v, out, **kw):
+    """General windowed attention (any sizes, both dtypes)."""
+    A.call("msa_lm_window_attn", C.byref(attn_args(qa, qb, ka, kb, v, out, **kw)), A.stream_ptr(qa.device))
 
 
-def window_attn_tc(proj, kv, ctx, spec, out, step, view, status):
-    """The portions of a step on the tensor cores: ``proj`` / ``out`` from the first portion row on."""
-    A.call("msa_lm_window_attn_tc", A.ptr(proj), _rows(proj), proj.shape[0], A.ptr(kv), _rows(kv), A.ptr(ctx), _rows(ctx),
-           ctx.shape[0], spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank, A.ptr(step.start), A.ptr(step.cu),
-           A.ptr(view.ctx_off), step.n_decode, step.n_seq, step.n_decode, step.max_len, view.window, float(spec.scale),
-           A.ptr(out), _rows(out), A.ptr(status), A.stream_ptr(proj.device))
+def window_attn_tc_supported(dim, rot, vdim, dtype, scale) -> bool:
+    return dtype == torch.bfloat16 and scale > 0 and bool(A.lib().msa_lm_window_attn_tc_supported(dim, rot, vdim))
+
+
+def window_attn_tc(qa, qb, ka, kb, v, out, *, row0, status, **kw):
+    """The portions of a step on the tensor cores: ``qa`` / ``out`` from the first portion row (packed row ``row0``) on."""
+    args = attn_args(qa, qb, ka, kb, v, out, **kw)
+    A.call("msa_lm_window_attn_tc", C.byref(args), qa.shape[0], ka.shape[0], row0, A.ptr(status), A.stream_ptr(qa.device))
 
 
 def latent_decode_supported(spec, dtype) -> bool:
@@ -137,6 +180,97 @@ def latent_decode(qa, qb, ring, slot, pos, out, *, window, scale, status):
     A.call("msa_lm_latent_decode", A.ptr(qa), qa.stride(0), qa.stride(1), A.ptr(qb), 0 if qb is None else qb.stride(0),
            0 if qb is None else qb.stride(1), A.ptr(ring), ring.shape[1], A.ptr(slot), A.ptr(pos), n, heads, rank, rot, window,
            splits, float(scale), A.ptr(out), A.ptr(part_o), A.ptr(part_ml), A.ptr(status), A.stream_ptr(qa.device))
+
+
+# ---------------------------------------------------------------------------------------------- grouped attention
+def group_prep(proj, spec, w, step, view, ring, conv_state, q, ctx):
+    """Convolve, rotate and place the rows of a step: queries in ``q`` [n, heads, pitch], keys and values in ring and context."""
+    args = A.GroupArgs(proj=A.ptr(proj), proj_stride=_rows(proj), conv_w=A.ptr(w.conv), inv_freq=A.ptr(w.inv_freq), conv_state=A.ptr(conv_state),
+                       q_out=A.ptr(q), ring=A.ptr(ring), ctx=A.ptr(ctx), pos=A.ptr(step.pos), tok_seq=A.ptr(step.tok_seq), slot=A.ptr(step.slot),
+                       start=A.ptr(step.start), cu=A.ptr(step.cu), ctx_off=A.ptr(view.ctx_off), old_off=A.ptr(view.old_off),
+                       ring_rows=ring.shape[1], heads=spec.heads, kv_heads=spec.kv_heads, dim=spec.dim, vdim=spec.vdim, rot=spec.rot_dims,
+                       taps=spec.taps, q_pitch=w.dim, k_pitch=w.dim, v_pitch=w.vdim, n_tok=step.n_tok, n_seq=step.n_seq,
+                       n_decode=step.n_decode, n_old=view.n_old, window=view.window, dtype=A.dtype_code(proj.dtype))
+    A.call("msa_lm_group_prep", C.byref(args), A.stream_ptr(proj.device))
+
+
+def conv_store(proj, channels, taps, step, conv_state):
+    """The portions' last convolution inputs; ``proj`` from the first convolved column on."""
+    if taps > 1 and step.n_seq > step.n_decode:
+        A.call("msa_lm_conv_store", A.ptr(proj), _rows(proj), channels, taps, A.ptr(conv_state), A.ptr(step.slot), A.ptr(step.start),
+               A.ptr(step.cu), step.n_seq, step.n_decode, A.dtype_code(proj.dtype), A.stream_ptr(proj.device))
+
+
+def group_decode_supported(dim, vdim, dtype) -> bool:
+    return dtype == torch.bfloat16 and bool(A.lib().msa_lm_group_decode_supported(dim, vdim))
+
+
+def group_decode_splits(n: int, heads: int, kv_heads: int, ring_rows: int, n_sm: int = 148) -> int:
+    """CTAs per sequence and head group: two per SM, at least 64 rows each."""
+    group = heads // kv_heads
+    tiles = kv_heads * ((group + 15) // 16 if group > 8 else 1)
+    return max(1, min(2 * n_sm // max(n * tiles, 1), (ring_rows + 63) // 64, 64))
+
+
+def group_decode(q, ring, kv_heads, step, out, *, window, scale, sink, gate):
+    """``q`` [n, heads, dim], ``out`` [n, heads, vdim] views, ``ring`` [slots, rows, kv_heads * (dim + vdim)]."""
+    n, heads, dim = q.shape
+    vdim = out.shape[2]
+    splits = group_decode_splits(n, heads, kv_heads, ring.shape[1])
+    part_o = part_ml = None
+    if splits > 1:
+        f = dict(dtype=torch.float32, device=q.device)
+        part_o, part_ml = torch.empty((n, heads, splits, vdim), **f), torch.empty((n, heads, splits, 2), **f)
+    A.call("msa_lm_group_decode", A.ptr(q), q.stride(0), A.ptr(ring), ring.shape[1], A.ptr(step.slot), A.ptr(step.start), n, heads, kv_heads, dim,
+           vdim, window, splits, float(scale), 1 if sink else 0, A.ptr(gate), gate.stride(0) if gate is not None else 0, A.ptr(out),
+           out.stride(0), A.ptr(part_o), A.ptr(part_ml), A.stream_ptr(q.device))
+
+
+# ---------------------------------------------------------------------------------------------- decaying outer products
+def wkv_mix(rkvg, decay, spec, w, state, eps, step, out):
+    """``rkvg`` [4, n, heads*dim], ``decay`` fp32 [n, heads*dim] (overwritten); advances the states, fills ``out``."""
+    args = A.WkvArgs(r=A.ptr(rkvg[0]), k=A.ptr(rkvg[1]), v=A.ptr(rkvg[2]), g=A.ptr(rkvg[3]), row_stride=rkvg.stride(1), decay=A.ptr(decay),
+                     w0=A.ptr(w.w0), u=A.ptr(w.u), norm=A.ptr(w.norm), state=A.ptr(state), tok_seq=A.ptr(step.tok_seq), slot=A.ptr(step.slot),
+                     start=A.ptr(step.start), cu=A.ptr(step.cu), n_tok=step.n_tok, n_seq=step.n_seq, n_decode=step.n_decode,
+                     heads=spec.heads, dim=spec.dim, eps=float(eps), dtype=A.dtype_code(rkvg.dtype))
+    dev, st = rkvg.device, A.stream_ptr(rkvg.device)
+    if step.n_decode:
+        A.call("msa_lm_wkv_decode", C.byref(args), A.ptr(out), _rows(out), st)
+    rows = step.n_tok - step.n_decode
+    if not rows:
+        return out
+    tail, f = out[step.n_decode:], dict(dtype=torch.float32, device=dev)
+    if rkvg.dtype == torch.bfloat16 and A.lib().msa_lm_wkv_chunk_supported(spec.dim):
+        work = torch.empty((step.n_chunks, spec.heads, spec.dim, spec.dim), **f)
+        A.call("msa_lm_wkv_chunk", C.byref(args), A.ptr(step.chunk_off), step.n_chunks, A.ptr(work), A.ptr(tail), _rows(tail), st)
+    else:
+        o = torch.empty((rows, spec.heads * spec.dim), **f)
+        A.call("msa_lm_wkv_scan", C.byref(args), A.ptr(o), A.ptr(tail), _rows(tail), st)
+    return out
+
+
+def ssd_mix(proj, spec, w, conv_state, state, eps, step, out):
+    """From the projections to the input of the output product; advances the states, fills ``out``."""
+    dev, st, f = proj.device, A.stream_ptr(proj.device), dict(dtype=torch.float32, device=proj.device)
+    y = torch.empty((step.n_tok, spec.inner), **f)
+    args = A.SsdArgs(proj=A.ptr(proj), proj_stride=_rows(proj), conv_w=A.ptr(w.conv), conv_b=A.ptr(w.conv_b), dt_bias=A.ptr(w.dt_bias),
+                     a_log=A.ptr(w.a_log), d_skip=A.ptr(w.d_skip), conv_state=A.ptr(conv_state), state=A.ptr(state), tok_seq=A.ptr(step.tok_seq),
+                     slot=A.ptr(step.slot), start=A.ptr(step.start), cu=A.ptr(step.cu), y=A.ptr(y), n_tok=step.n_tok, n_seq=step.n_seq,
+                     n_decode=step.n_decode, heads=spec.heads, vdim=spec.vdim, n_state=spec.state, groups=spec.groups, taps=spec.taps,
+                     dtype=A.dtype_code(proj.dtype))
+    if step.n_decode:
+        A.call("msa_lm_ssd_decode", C.byref(args), st)
+    rows = step.n_tok - step.n_decode
+    if rows:
+        xbc, dt = torch.empty((rows, spec.channels), dtype=proj.dtype, device=dev), torch.empty((rows, spec.heads), **f)
+        A.call("msa_lm_ssd_prep", C.byref(args), A.ptr(xbc), A.ptr(dt), st)
+        conv_store(proj[:, spec.inner:], spec.channels, spec.taps, step, conv_state)
+        if proj.dtype == torch.bfloat16 and A.lib().msa_lm_ssd_chunk_supported(spec.state, spec.vdim):
+            gcum, work = torch.empty((rows, spec.heads), **f), torch.empty((step.n_chunks, spec.heads, spec.state, spec.vdim), **f)
+            A.call("msa_lm_ssd_chunk", C.byref(args), A.ptr(xbc), A.ptr(dt), A.ptr(step.chunk_off), step.n_chunks, A.ptr(gcum), A.ptr(work), st)
+        else:
+            A.call("msa_lm_ssd_scan", C.byref(args), A.ptr(xbc), A.ptr(dt), st)
+    return part_norm(y, w.norm, spec.norm_groups, eps, out)
 
 
 # ---------------------------------------------------------------------------------------------- gated delta rule

@@ -11,6 +11,8 @@ from typing import Any, Callable, Dict
 
 import torch
 
+from .hybrid_config import DESIGNS as HYBRID_DESIGNS
+
 
 @dataclass(frozen=True)
 class Design:
@@ -62,4 +64,5 @@ def _load_hybrid(path, device, dtype):
 
 
 register(Design("MSAForCausalLM", "memory", _load_msa, (torch.bfloat16, torch.float32)))
-register(Design("Mutuvik", "states", _load_hybrid, (torch.bfloat16, torch.float32)))
+for _name in HYBRID_DESIGNS:
+    register(Design(_name, "states", _load_hybrid, (torch.bfloat16, torch.float32)))
