@@ -249,10 +249,10 @@ int msa_lm_ssd_decode(const msa_lm_ssd_args* a, void* stream);
 int msa_lm_ssd_prep(const msa_lm_ssd_args* a, void* xbc, float* dt, void* stream);
 /* ... the recurrence token by token (n_state up to 256). */
 int msa_lm_ssd_scan(const msa_lm_ssd_args* a, const void* xbc, const float* dt, void* stream);
-/* ... or in chunks of 64 tokens on tensor cores (bf16; n_state and vdim multiples of 8 up to 128): gcum [rows, heads] and
- * work [n_chunks, heads, n_state, vdim] fp32. */
+/* ... or in chunks of 64 tokens on tensor cores (bf16; n_state and vdim multiples of 8 up to 128): gcum [rows, heads]
+ * fp64 and work [n_chunks, heads, n_state, vdim] fp32 are scratch. */
 int msa_lm_ssd_chunk_supported(int32_t n_state, int32_t vdim);
-int msa_lm_ssd_chunk(const msa_lm_ssd_args* a, const void* xbc, const float* dt, const int32_t* chunk_off, int32_t n_chunks, float* gcum,
+int msa_lm_ssd_chunk(const msa_lm_ssd_args* a, const void* xbc, const float* dt, const int32_t* chunk_off, int32_t n_chunks, double* gcum,
                      float* work, void* stream);
 
 /* out = x / rms(x) * w, every row in `parts` equal parts with a root mean square each. */

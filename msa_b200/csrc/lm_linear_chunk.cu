@@ -2,7 +2,9 @@
 //   1. per chunk, what its tokens add to the state:      dS = sum_i (e^(G_C - G_i) k_i) v_i^T
 //   2. along the chunks, elementwise:                    S_(c+1) = e^(G_C) S_c + dS_c
 //   3. per chunk, the read-out from S_c and from the chunk's own tokens.
-// G is the running sum of the log decays inside the chunk (in units of log 2), per key channel (wkv) or per head (ssd).
+// G is the running sum of the log decays inside the chunk (in units of log 2), per key channel (wkv) or per head (ssd).  A
+// difference of two running sums loses what a steep token between the chunk's start and both has cost: wkv's sums restart
+// every 16 rows (and no token counts for more than 2^-160, which is zero already), ssd's are 64-bit numbers.
 //
 // 32-bit operands enter the products as the sum of two bf16 numbers (16 to 17 significant bits), accumulated in fp32; what
 // is bf16 by nature (projections, convolved activations) enters as it is.  Decays, sums and the states are plain fp32.
@@ -16,7 +18,7 @@
 namespace msa {
 
 constexpr int kLcRows = 64;
-constexpr float kLcSteep = 100.f;
+constexpr float kLcSteep = 100.f, kLcGone = -160.f;
 
 __device__ __forceinline__ void lc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -68,9 +70,10 @@ __device__ __forceinline__ void lc_load_split(unsigned char* dst, int pitch, int
 }
 
 // ---- step 2 for both ----------------------------------------------------------------------------------------------------
-// g: running log2 decays [rows.., stride]; the chunk's total stands in its last row.  A thread carries four elements.
-template <bool CHANNEL>
-__global__ void __launch_bounds__(128) linear_carry_kernel(float* __restrict__ work, const float* __restrict__ g, long long g_stride, int g_row0,
+// g: running log2 decays [rows.., stride]; the chunk's total stands in its last row (CHANNEL: the sum of its blocks' last
+// rows).  A thread carries four elements.
+template <bool CHANNEL, typename G>
+__global__ void __launch_bounds__(128) linear_carry_kernel(float* __restrict__ work, const G* __restrict__ g, long long g_stride, int g_row0,
                                                            float* __restrict__ state, const int32_t* slot, const int32_t* start,
                                                            const int32_t* cu, const int32_t* chunk_off, int n_decode, int heads, int dk, int dv) {
   const int e = (blockIdx.x * 128 + threadIdx.x) * 4, h = blockIdx.y, ps = blockIdx.z, s = ps + n_decode;
@@ -79,7 +82,7 @@ __global__ void __launch_bounds__(128) linear_carry_kernel(float* __restrict__ w
   const long long step = (long long)heads * dk * dv;
   float* w = work + ((long long)chunk_off[ps] * heads + h) * dk * dv + e;
   float* st = state + ((long long)slot[s] * heads + h) * dk * dv + e;
-  const float* gp = g + ((long long)cu[s] - g_row0) * g_stride + (CHANNEL ? h * dk + d : h);
+  const G* gp = g + ((long long)cu[s] - g_row0) * g_stride + (CHANNEL ? h * dk + d : h);
   float4 S = start[s] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(st);
   constexpr int kAhead = 8;
   for (int c0 = 0; c0 < n; c0 += kAhead) {
@@ -89,7 +92,15 @@ __global__ void __launch_bounds__(128) linear_carry_kernel(float* __restrict__ w
     for (int i = 0; i < kAhead; ++i) {
       if (c0 + i >= n) break;
       x[i] = load4(w + (c0 + i) * step);
-      f[i] = gp[(long long)(min((c0 + i + 1) * kLcRows, len) - 1) * g_stride];
+      const int last = min((c0 + i + 1) * kLcRows, len) - 1;
+      f[i] = (float)gp[(long long)last * g_stride];
+      if constexpr (CHANNEL) {
+#pragma unroll
+        for (int b = 0; b < kLcRows / 16 - 1; ++b) {
+          const int r = (c0 + i) * kLcRows + 16 * b + 15;
+          if (r < last) f[i] += gp[(long long)r * g_stride];
+        }
+      }
     }
 #pragma unroll
     for (int i = 0; i < kAhead; ++i) {
@@ -110,13 +121,13 @@ struct WkvChunkParams {
   __nv_bfloat16* out; long long out_stride;
 };
 
-// Step 1; the decays become running sums in place.
+// Step 1; the decays become running sums, one for every 16 rows, in place.
 template <int D>
 __global__ void __launch_bounds__(2 * D) wkv_add_kernel(const WkvChunkParams p) {
   constexpr int kP = D * 2 + 16, kThreads = 2 * D;
   extern __shared__ __align__(16) unsigned char sm[];
   unsigned char *s_k = sm, *s_v = sm + 2 * kLcRows * kP;      // decayed keys (hi, lo), values
-  float* s_tot = reinterpret_cast<float*>(s_v + kLcRows * kP);   // [2][D]
+  float* s_tot = reinterpret_cast<float*>(s_v + kLcRows * kP);   // [D]: the chunk's second half
   const msa_lm_wkv_args& a = p.a;
   const int h = blockIdx.y, dim = a.dim;
   const LcChunk ch = lc_chunk(p.chunk_off, a.cu, a.n_decode, a.n_seq, blockIdx.x);
@@ -129,26 +140,32 @@ __global__ void __launch_bounds__(2 * D) wkv_add_kernel(const WkvChunkParams p) 
     float* dec = a.decay + ch.n0 * a.heads * dim + h * dim + d;
     const __nv_bfloat16* key = reinterpret_cast<const __nv_bfloat16*>(a.k) + row + d;
     const float w0 = on ? a.w0[h * dim + d] : 0.f;
-    float g[32], sum = 0.f;
+    float g[32];
 #pragma unroll
     for (int i = 0; i < 32; ++i) g[i] = on && r0 + i < ch.len ? dec[(long long)(r0 + i) * a.heads * dim] : -INFINITY;
     __nv_bfloat16 k[32];
 #pragma unroll
     for (int i = 0; i < 32; ++i) k[i] = on && r0 + i < ch.len ? key[(long long)(r0 + i) * a.row_stride] : __float2bfloat16_rn(0.f);
+    float sum = 0.f;
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
-      sum -= 1.4426950408889634f * expf(g[i] + w0);
-      g[i] = sum;
+      g[i] = fmaxf(kLcGone, -1.4426950408889634f * expf(g[i] + w0));
+      sum = i % 16 ? sum + g[i] : g[i];
+      if (on && r0 + i < ch.len) dec[(long long)(r0 + i) * a.heads * dim] = sum;
     }
-    s_tot[part * D + d] = sum;
-    __syncthreads();
-    const float before = part ? s_tot[d] : 0.f, total = s_tot[d] + s_tot[D + d];
+    if (part) {
+      sum = 0.f;
 #pragma unroll
-    for (int i = 0; i < 32; ++i) {
+      for (int i = 0; i < 32; ++i) sum += g[i];
+      s_tot[d] = sum;
+    }
+    __syncthreads();
+    float rest = part ? 0.f : s_tot[d];                  // what a key decays by until the chunk's end
+#pragma unroll
+    for (int i = 31; i >= 0; --i) {
       const int r = r0 + i;
-      g[i] += before;
-      if (on && r < ch.len) dec[(long long)r * a.heads * dim] = g[i];
-      const float x = __bfloat162float(k[i]) * exp2f(total - g[i]);
+      const float x = __bfloat162float(k[i]) * exp2f(rest);
+      rest += g[i];
       const __nv_bfloat16 hi = __float2bfloat16_rn(x);
       *reinterpret_cast<__nv_bfloat16*>(s_k + r * kP + d * 2) = hi;
       *reinterpret_cast<__nv_bfloat16*>(s_k + (kLcRows + r) * kP + d * 2) = __float2bfloat16_rn(x - __bfloat162float(hi));
@@ -218,12 +235,11 @@ __global__ void __launch_bounds__(128) wkv_read_kernel(const WkvChunkParams p) {
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3, r0 = warp * 16 + g;
   if (warp * 16 >= ch.len) return;
-  const float* ref = s_g + (warp * 16 - 1) * kG;      // running sums in front of this warp's rows (warp 0: zero)
   bool steep;
   {
     float span = 0.f;
     const float* end = s_g + (warp * 16 + 15) * kG;
-    for (int d = lane; d < dim; d += 32) span = fmaxf(span, (warp ? ref[d] : 0.f) - end[d]);
+    for (int d = lane; d < dim; d += 32) span = fmaxf(span, -end[d]);
     steep = warp_max_f(span) > kLcSteep;
   }
   float o[D / 8][4], s[8][4];
@@ -238,21 +254,28 @@ __global__ void __launch_bounds__(128) wkv_read_kernel(const WkvChunkParams p) {
   for (int kk = 0; kk < D / 16; ++kk) {
     if (kk * 16 >= dim) break;
     uint32_t fh[4], fl[4], th[4], tl[4];               // rows from the chunk's start, from the block's start
-    float2 base[2];
+    float2 sum[2][4], after[2][4];                     // per block of 16 keys: its decay, that of the blocks up to this warp's
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
       const int c = kk * 16 + tq * 2 + 8 * x;
-      base[x] = warp ? *reinterpret_cast<const float2*>(ref + c) : make_float2(0.f, 0.f);
+      float2 run = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int b = 3; b >= 0; --b) {
+        sum[x][b] = b < warp ? *reinterpret_cast<const float2*>(s_g + (16 * b + 15) * kG + c) : make_float2(0.f, 0.f);
+        after[x][b] = run;
+        run.x += sum[x][b].x;
+        run.y += sum[x][b].y;
+      }
       const float2 u = c < dim ? *reinterpret_cast<const float2*>(a.u + h * dim + c) : make_float2(0.f, 0.f);
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int t = r0 + 8 * e;
         const float2 r = lc_pair(s_r + t * kP + c * 2), k = lc_pair(s_k + t * kP + c * 2);
-        const float2 gt = t ? *reinterpret_cast<const float2*>(s_g + (t - 1) * kG + c) : make_float2(0.f, 0.f);
+        const float2 gt = t & 15 ? *reinterpret_cast<const float2*>(s_g + (t - 1) * kG + c) : make_float2(0.f, 0.f);
         own[e] = fmaf(r.x * u.x, k.x, own[e]);
         own[e] = fmaf(r.y * u.y, k.y, own[e]);
-        lc_split2(r.x * exp2f(gt.x), r.y * exp2f(gt.y), fh[2 * x + e], fl[2 * x + e]);
-        lc_split2(r.x * exp2f(gt.x - base[x].x), r.y * exp2f(gt.y - base[x].y), th[2 * x + e], tl[2 * x + e]);
+        lc_split2(r.x * exp2f(gt.x + run.x), r.y * exp2f(gt.y + run.y), fh[2 * x + e], fl[2 * x + e]);
+        lc_split2(r.x * exp2f(gt.x), r.y * exp2f(gt.y), th[2 * x + e], tl[2 * x + e]);
       }
     }
 #pragma unroll
@@ -276,7 +299,8 @@ __global__ void __launch_bounds__(128) wkv_read_kernel(const WkvChunkParams p) {
         for (int x = 0; x < 2; ++x) {
           const int c = kk * 16 + tq * 2 + 8 * x;
           const float2 k = lc_pair(s_k + key * kP + c * 2), gi = *reinterpret_cast<const float2*>(s_g + key * kG + c);
-          lc_split2(k.x * exp2f(base[x].x - gi.x), k.y * exp2f(base[x].y - gi.y), bh[x], bl[x]);
+          const float2 m = sum[x][n / 2], f = after[x][n / 2];
+          lc_split2(k.x * exp2f((m.x - gi.x) + f.x), k.y * exp2f((m.y - gi.y) + f.y), bh[x], bl[x]);
         }
         lc_mma(s[n], tl, bh[0], bh[1]);
         lc_mma(s[n], th, bl[0], bl[1]);
@@ -362,7 +386,7 @@ int launch_wkv_chunk(const WkvChunkParams& p, int n_chunks, cudaStream_t st) {
   wkv_add_kernel<D><<<grid, 2 * D, add, st>>>(p);
   MSA_LAUNCH_OK("wkv_add_kernel");
   const dim3 carry((unsigned)((a.dim * a.dim / 4 + 127) / 128), (unsigned)a.heads, (unsigned)(a.n_seq - a.n_decode));
-  linear_carry_kernel<true><<<carry, 128, 0, st>>>(p.work, a.decay, (long long)a.heads * a.dim, 0, a.state, a.slot, a.start, a.cu, p.chunk_off,
+  linear_carry_kernel<true, float><<<carry, 128, 0, st>>>(p.work, a.decay, (long long)a.heads * a.dim, 0, a.state, a.slot, a.start, a.cu, p.chunk_off,
                                                    a.n_decode, a.heads, a.dim, a.dim);
   MSA_LAUNCH_OK("linear_carry_kernel");
   wkv_read_kernel<D><<<grid, 128, read, st>>>(p);
@@ -376,7 +400,8 @@ struct SsdChunkParams {
   const __nv_bfloat16* xbc;      // [rows, inner | groups*n_state | groups*n_state]
   const float* dt;               // [rows, heads]
   const int32_t* chunk_off;
-  float *gcum, *work;            // [rows, heads], [chunks, heads, n_state, vdim]
+  double* gcum;                  // [rows, heads]
+  float* work;                   // [chunks, heads, n_state, vdim]
 };
 
 // Step 1; leaves the running sums of the log2 decays in gcum.
@@ -395,19 +420,19 @@ __global__ void __launch_bounds__(2 * N) ssd_add_kernel(const SsdChunkParams p) 
   cp_async_commit();
   if (threadIdx.x < 32) {
     const int lane = threadIdx.x, r = 2 * lane;
-    const float rate = -1.4426950408889634f * expf(a.a_log[h]);
+    const double rate = -1.4426950408889634 * expf(a.a_log[h]);
     const float d0 = r < ch.len ? p.dt[(row0 + r) * a.heads + h] : 0.f, d1 = r + 1 < ch.len ? p.dt[(row0 + r + 1) * a.heads + h] : 0.f;
-    float sum = rate * d0 + rate * d1;
+    double sum = rate * d0 + rate * d1;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const float x = __shfl_up_sync(0xffffffffu, sum, o);
+      const double x = __shfl_up_sync(0xffffffffu, sum, o);
       if (lane >= o) sum += x;
     }
-    const float total = __shfl_sync(0xffffffffu, sum, 31), g0 = sum - rate * d1;
+    const double total = __shfl_sync(0xffffffffu, sum, 31), g0 = sum - rate * d1;
     if (r < ch.len) p.gcum[(row0 + r) * a.heads + h] = g0;
     if (r + 1 < ch.len) p.gcum[(row0 + r + 1) * a.heads + h] = sum;
-    s_w[r] = d0 * exp2f(total - g0);
-    s_w[r + 1] = d1 * exp2f(total - sum);
+    s_w[r] = d0 * exp2f((float)(total - g0));
+    s_w[r + 1] = d1 * exp2f((float)(total - sum));
   }
   __syncthreads();
   for (int i = threadIdx.x; i < kLcRows * (V / 4); i += kThreads) {
@@ -461,7 +486,8 @@ __global__ void __launch_bounds__(128) ssd_read_kernel(const SsdChunkParams p) {
   constexpr int kPn = N * 2 + 16, kPv = V * 2 + 16;
   extern __shared__ __align__(16) unsigned char sm[];
   unsigned char *s_c = sm, *s_b = s_c + kLcRows * kPn, *s_x = s_b + kLcRows * kPn, *s_s = s_x + kLcRows * kPv;
-  __shared__ float s_g[kLcRows], s_dt[kLcRows];
+  __shared__ double s_g[kLcRows];
+  __shared__ float s_dt[kLcRows];
   const msa_lm_ssd_args& a = p.a;
   const int h = blockIdx.y, inner = a.heads * a.vdim, bc = a.groups * a.n_state, chan = inner + 2 * bc, gr = h / (a.heads / a.groups);
   const LcChunk ch = lc_chunk(p.chunk_off, a.cu, a.n_decode, a.n_seq, blockIdx.x);
@@ -515,9 +541,9 @@ __global__ void __launch_bounds__(128) ssd_read_kernel(const SsdChunkParams p) {
       }
     }
   }
-  const float g0 = s_g[r0], g1 = s_g[r0 + 8];
+  const double g0 = s_g[r0], g1 = s_g[r0 + 8];
   {
-    const float f0 = exp2f(g0), f1 = exp2f(g1);
+    const float f0 = exp2f((float)g0), f1 = exp2f((float)g1);
 #pragma unroll
     for (int j = 0; j < V / 8; ++j) { o[j][0] *= f0; o[j][1] *= f0; o[j][2] *= f1; o[j][3] *= f1; }
   }
@@ -529,13 +555,14 @@ __global__ void __launch_bounds__(128) ssd_read_kernel(const SsdChunkParams p) {
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
       const int i = (2 * m + x) * 8 + tq * 2;
-      const float2 gi = *reinterpret_cast<const float2*>(s_g + i), di = *reinterpret_cast<const float2*>(s_dt + i);
+      const double gx = s_g[i], gy = s_g[i + 1];
+      const float2 di = *reinterpret_cast<const float2*>(s_dt + i);
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int t = r0 + 8 * e;
-        const float gt = e ? g1 : g0;
-        const float p0 = i <= t ? s[2 * m + x][2 * e] * exp2f(gt - gi.x) * di.x : 0.f;
-        const float p1 = i + 1 <= t ? s[2 * m + x][2 * e + 1] * exp2f(gt - gi.y) * di.y : 0.f;
+        const double gt = e ? g1 : g0;
+        const float p0 = i <= t ? s[2 * m + x][2 * e] * exp2f((float)(gt - gx)) * di.x : 0.f;
+        const float p1 = i + 1 <= t ? s[2 * m + x][2 * e + 1] * exp2f((float)(gt - gy)) * di.y : 0.f;
         lc_split2(p0, p1, ah[2 * x + e], al[2 * x + e]);
       }
     }
@@ -580,7 +607,7 @@ int launch_ssd_chunk(const SsdChunkParams& p, int n_chunks, cudaStream_t st) {
   ssd_add_kernel<N, V><<<grid, 2 * N, add, st>>>(p);
   MSA_LAUNCH_OK("ssd_add_kernel");
   const dim3 carry((unsigned)((a.n_state * a.vdim / 4 + 127) / 128), (unsigned)a.heads, (unsigned)(a.n_seq - a.n_decode));
-  linear_carry_kernel<false><<<carry, 128, 0, st>>>(p.work, p.gcum, a.heads, a.n_decode, a.state, a.slot, a.start, a.cu, p.chunk_off, a.n_decode,
+  linear_carry_kernel<false, double><<<carry, 128, 0, st>>>(p.work, p.gcum, a.heads, a.n_decode, a.state, a.slot, a.start, a.cu, p.chunk_off, a.n_decode,
                                                     a.heads, a.n_state, a.vdim);
   MSA_LAUNCH_OK("linear_carry_kernel");
   ssd_read_kernel<N, V><<<grid, 128, read, st>>>(p);
@@ -620,7 +647,7 @@ extern "C" int msa_lm_ssd_chunk_supported(int32_t n_state, int32_t vdim) {
 }
 
 extern "C" int msa_lm_ssd_chunk(const msa_lm_ssd_args* a, const void* xbc, const float* dt, const int32_t* chunk_off, int32_t n_chunks,
-                                float* gcum, float* work, void* stream) {
+                                double* gcum, float* work, void* stream) {
   MSA_OK_OR_RETURN(ssd_check(a, "ssd_chunk"));
   MSA_REQUIRE(a->dtype == MSA_BF16 && msa_lm_ssd_chunk_supported(a->n_state, a->vdim) && xbc && dt && chunk_off && gcum && work,
               "ssd_chunk: unsupported sizes or null pointer");

@@ -266,7 +266,8 @@ def ssd_mix(proj, spec, w, conv_state, state, eps, step, out):
         A.call("msa_lm_ssd_prep", C.byref(args), A.ptr(xbc), A.ptr(dt), st)
         conv_store(proj[:, spec.inner:], spec.channels, spec.taps, step, conv_state)
         if proj.dtype == torch.bfloat16 and A.lib().msa_lm_ssd_chunk_supported(spec.state, spec.vdim):
-            gcum, work = torch.empty((rows, spec.heads), **f), torch.empty((step.n_chunks, spec.heads, spec.state, spec.vdim), **f)
+            gcum = torch.empty((rows, spec.heads), dtype=torch.float64, device=dev)
+            work = torch.empty((step.n_chunks, spec.heads, spec.state, spec.vdim), **f)
             A.call("msa_lm_ssd_chunk", C.byref(args), A.ptr(xbc), A.ptr(dt), A.ptr(step.chunk_off), step.n_chunks, A.ptr(gcum), A.ptr(work), st)
         else:
             A.call("msa_lm_ssd_scan", C.byref(args), A.ptr(xbc), A.ptr(dt), st)

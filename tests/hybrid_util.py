@@ -16,6 +16,19 @@ def delta(heads, kv_heads, dim, vdim, conv):
     return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}
 
 
+def attention(heads, kv_heads, dim, vdim, window, rot, conv, base=500.0, scale=None):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv, "scale": scale or dim ** -0.5,
+            "rot": {"base": base, "dims": rot}, "mask": {"size": window}}
+
+
+def wkv(heads, dim):
+    return {"heads": heads, "dim": dim}
+
+
+def mamba2(heads, vdim, state, groups, norm_groups, conv):
+    return {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "norm_groups": norm_groups, "conv": conv}
+
+
 def dense(ff):
     return {"kind": "dense", "ff": ff}
 
@@ -30,6 +43,12 @@ def layer(kind, mixer, mlp):
 
 def config(width, vocab, layers, loop=None, eps=1e-5):
     return {"architecture": "Mutuvik", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": layers, "loop": loop}
+
+
+def parallel(width, vocab, layers, loop=None, eps=1e-5, bigram=None, cap=None):
+    pair = None if bigram is None else {"buckets": bigram[0], "mul_prev": bigram[1], "mul_cur": bigram[2]}
+    return {"architecture": "Nazerax", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": layers, "loop": loop,
+            "embedding": {"bigram": pair}, "logit_softcap": cap}
 
 
 # uneven sizes everywhere, two windows, a layer without a feed-forward, a loop in the middle with a tail behind it
@@ -56,7 +75,34 @@ WIDE = config(256, 320, [
     layer("latent_attention", latent(8, 64, 32, 64, 128, 160, base=10000.0), dense(128)),
 ])
 
-CONFIGS = {"mixed": MIXED, "odd": ODD, "wide": WIDE}
+# the parallel frame: uneven sizes, two windows, a convolution of one tap, a layer without a feed-forward, a loop with a tail
+PAR_MIXED = parallel(72, 203, [
+    layer("wkv", wkv(3, 24), dense(112)),
+    layer("attention", attention(6, 2, 20, 28, 17, 12, 3), dense(60)),
+    layer("mamba2", mamba2(6, 12, 20, 3, 2, 4), None),
+    layer("attention", attention(4, 4, 16, 8, 33, 16, 1, base=77.0), dense(88)),
+    layer("wkv", wkv(2, 40), dense(52)),
+], loop={"start": 1, "stop": 4, "times": 3}, eps=3e-4, bigram=(61, 31, 5), cap=9.0)
+
+# nothing is a multiple of 4; the loop starts with the first layer; no bigram, no cap; window 1 and a wide one, no rotation
+PAR_ODD = parallel(51, 97, [
+    layer("wkv", wkv(3, 7), dense(33)),
+    layer("mamba2", mamba2(3, 5, 7, 1, 5, 3), dense(9)),
+    layer("attention", attention(3, 1, 9, 5, 1, 4, 2), dense(21)),
+    layer("attention", attention(3, 3, 5, 7, 400, 0, 6), None),
+], loop={"start": 0, "stop": 2, "times": 2})
+
+# sizes that the tensor-core kernels take; a single pass of the loop
+PAR_WIDE = parallel(256, 320, [
+    layer("wkv", wkv(4, 64), dense(320)),
+    layer("attention", attention(8, 2, 64, 128, 100, 32, 4, base=10000.0), dense(256)),
+    layer("mamba2", mamba2(6, 64, 128, 2, 3, 4), dense(192)),
+    layer("wkv", wkv(2, 128), dense(128)),
+    layer("attention", attention(20, 2, 128, 64, 160, 64, 4, base=10000.0), dense(256)),
+    layer("mamba2", mamba2(4, 32, 48, 1, 4, 2), dense(64)),
+], loop={"start": 2, "stop": 4, "times": 1}, bigram=(127, 11, 3), cap=20.0)
+
+CONFIGS = {"mixed": MIXED, "odd": ODD, "wide": WIDE, "par-mixed": PAR_MIXED, "par-odd": PAR_ODD, "par-wide": PAR_WIDE}
 
 
 def make_weights(cfg, seed=0, sharp=2.0):
@@ -66,13 +112,19 @@ def make_weights(cfg, seed=0, sharp=2.0):
     mat = lambda n, r, c, s=1.0: w.__setitem__(n, torch.randn(r, c, generator=g) * (s / c ** 0.5))
     vec = lambda n, k, mean, std: w.__setitem__(n, mean + std * torch.randn(k, generator=g))
     w["embed"] = torch.randn(cfg["vocab"], width, generator=g)
-    if cfg["loop"]:
+    par = cfg["architecture"] == "Nazerax"
+    mid = 0.0 if par else 1.0                      # what the frame's norm weights are stored around
+    if par:
+        mat("head", cfg["vocab"], width, 3.0)
+        if cfg["embedding"]["bigram"]:
+            w["bigram"] = torch.randn(cfg["embedding"]["bigram"]["buckets"] + 1, width, generator=g)
+    elif cfg["loop"]:
         mat("loop.in", width, 2 * width)
         w["loop.step"] = 0.5 * torch.randn(cfg["loop"]["times"], width, generator=g)
     for i, entry in enumerate(cfg["layers"]):
         p, m = f"l{i}.", entry["mixer"]
-        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if entry["mlp"] else ()):
-            vec(p + n, width, 1.0, 0.2)
+        for n in ("norm1", "norm2") if par else ("norm1", "norm1b") + (("norm2", "norm2b") if entry["mlp"] else ()):
+            vec(p + n, width, mid, 0.2)
         x = p + "mix."
         if entry["type"] == "delta":
             qk, v = m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
@@ -86,6 +138,34 @@ def make_weights(cfg, seed=0, sharp=2.0):
             vec(x + "dt_bias", m["heads"], 0.0, 1.0)
             vec(x + "norm", m["vdim"], 1.0, 0.2)
             mat(x + "o", width, v)
+        elif entry["type"] == "wkv":
+            inner, rank = m["heads"] * m["dim"], 4 + m["dim"] // 8
+            for n in "rkvgw":
+                w[x + "mu." + n] = torch.rand(width, generator=g)
+            for n in "rkvg":
+                mat(x + n, inner, width)
+            mat(x + "w1", rank, width, 2.0)
+            mat(x + "w2", inner, rank, 1.5)
+            w[x + "w0"] = torch.rand(inner, generator=g) * 6 - 5
+            w[x + "u"] = 0.5 * torch.randn(m["heads"], m["dim"], generator=g)
+            vec(x + "norm", inner, 1.0, 0.2)
+            mat(x + "o", width, inner)
+        elif entry["type"] == "mamba2":
+            inner, chan = m["heads"] * m["vdim"], m["heads"] * m["vdim"] + 2 * m["groups"] * m["state"]
+            mat(x + "in", inner + chan + m["heads"], width)
+            w[x + "conv"] = torch.randn(chan, m["conv"], generator=g) * 0.6
+            vec(x + "conv.b", chan, 0.0, 0.3)
+            vec(x + "dt_bias", m["heads"], -1.0, 1.0)
+            w[x + "A_log"] = torch.rand(m["heads"], generator=g) * 3 - 2.5
+            vec(x + "D", m["heads"], 1.0, 0.5)
+            vec(x + "norm", inner, 1.0, 0.2)
+            mat(x + "o", width, inner)
+        elif entry["type"] == "attention":
+            for n, r in (("q", m["heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["kv_heads"] * m["vdim"])):
+                mat(x + n, r, width, sharp if n == "q" else 1.0)
+                w[x + n + ".conv"] = torch.randn(r, m["conv"], generator=g) * 0.6
+            mat(x + "g", m["heads"], width)
+            mat(x + "o", width, m["heads"] * m["vdim"])
         else:
             mat(x + "q", m["heads"] * (m["dim"] + m["rot_dim"]), width, sharp)
             mat(x + "dkv", m["kv_rank"] + m["rot_dim"], width)
@@ -104,7 +184,7 @@ def make_weights(cfg, seed=0, sharp=2.0):
             for e in range(f["router"]["experts"]):
                 for n, r, c in (("gate", e_ff, width), ("up", e_ff, width), ("down", width, e_ff)):
                     mat(f"{p}mlp.e{e}.{n}", r, c, 1.5)
-    vec("final.norm", width, 1.0, 0.2)
+    vec("final.norm", width, mid, 0.2)
     return {k: v.to(torch.bfloat16) for k, v in w.items()}
 
 

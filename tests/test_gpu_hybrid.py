@@ -52,6 +52,7 @@ def close(got, want, dtype):
 
 DTYPES = pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], ids=["f32", "bf16"])
 NAMES = pytest.mark.parametrize("name", list(U.CONFIGS))
+BOTH = pytest.mark.parametrize("name", ["mixed", "par-mixed"])
 
 
 # ------------------------------------------------------------------------------------------ mechanisms alone
@@ -64,7 +65,7 @@ class OneMixer:
         w = H.Weights({"m." + k: v for k, v in weights.items()}, "cuda:0", dtype)
         self.mixer = H.MIXERS[kind](s, w, "m.", width, eps)
         w.check_all_used()
-        self.dtype, self.windows = dtype, (getattr(s, "window", None),) if kind == "latent_attention" else ()
+        self.dtype, self.windows = dtype, (s.window,) if hasattr(s, "window") else ()
 
     def cache(self, n_slots, max_len):
         from msa_b200.cache import SequenceStateCache
@@ -77,7 +78,7 @@ class OneMixer:
         step = PackedStep([(s, [0] * h.shape[0], range(h.shape[0])) for s, h in entries], cache, self.windows)
         packed = torch.empty((step.n_tok, entries[0][1].shape[1]), dtype=self.dtype, device="cuda:0")
         packed[step.want_rows.long()] = torch.cat([h for _, h in entries]).to("cuda:0", self.dtype)
-        y = K.matmul(self.mixer.mix(K.matmul(packed, self.mixer.w_in), step, cache, 0), self.mixer.w_o)
+        y = K.matmul(self.mixer.forward(packed, step, cache, 0), self.mixer.w_o)
         step.commit(cache)
         return list(y[step.want_rows.long()].float().cpu().split([h.shape[0] for _, h in entries]))
 
@@ -85,8 +86,7 @@ class OneMixer:
 def mixer_case(kind, spec, width, seed, sharp=2.0):
     cfg = U.config(width, 8, [U.layer(kind, spec, None)])
     w = {k[len("l0.mix."):]: v for k, v in U.make_weights(cfg, seed, sharp).items() if k.startswith("l0.mix.")}
-    return w, lambda h, s=spec: {"latent_attention": O.latent_attention, "delta": O.delta_mixer}[kind](
-        h.double(), {k: v.double() for k, v in w.items()}, s, EPS)
+    return w, lambda h, s=spec: O.MIXERS[kind](h.double(), {k: v.double() for k, v in w.items()}, s, EPS)
 
 
 def bf16_rows(n, width, seed):
@@ -108,6 +108,29 @@ MIXER_CASES = {
     "delta-64": ("delta", U.delta(6, 2, 64, 96, 4), 96),
     "delta-192": ("delta", U.delta(2, 1, 192, 64, 2), 64),
     "delta-32": ("delta", U.delta(2, 2, 32, 64, 4), 64),
+    "group": ("attention", U.attention(6, 2, 20, 28, 17, 12, 3), 72),
+    "group-odd": ("attention", U.attention(3, 1, 7, 5, 6, 2, 2), 33),
+    "group-window1": ("attention", U.attention(4, 2, 8, 8, 1, 8, 4), 32),
+    "group-taps6": ("attention", U.attention(4, 2, 16, 8, 40, 6, 6), 40),
+    "group-plain": ("attention", U.attention(5, 5, 24, 16, 70, 0, 1), 40),
+    "group-64": ("attention", U.attention(8, 2, 64, 64, 150, 32, 4), 128),
+    "group-128": ("attention", U.attention(24, 2, 128, 128, 300, 128, 4), 128),
+    "group-unequal": ("attention", U.attention(6, 3, 96, 40, 64, 30, 3), 96),
+    "group-192": ("attention", U.attention(2, 1, 192, 160, 90, 64, 2), 64),
+    "wkv": ("wkv", U.wkv(3, 24), 72),
+    "wkv-odd": ("wkv", U.wkv(3, 7), 33),
+    "wkv-16": ("wkv", U.wkv(1, 16), 32),
+    "wkv-64": ("wkv", U.wkv(4, 64), 128),
+    "wkv-72": ("wkv", U.wkv(2, 72), 64),
+    "wkv-128": ("wkv", U.wkv(2, 128), 96),
+    "wkv-160": ("wkv", U.wkv(2, 160), 64),
+    "mamba2": ("mamba2", U.mamba2(6, 12, 20, 3, 2, 4), 72),
+    "mamba2-odd": ("mamba2", U.mamba2(3, 5, 7, 1, 5, 3), 33),
+    "mamba2-taps1": ("mamba2", U.mamba2(2, 16, 16, 2, 1, 1), 32),
+    "mamba2-taps6": ("mamba2", U.mamba2(4, 16, 24, 2, 4, 6), 40),
+    "mamba2-128": ("mamba2", U.mamba2(8, 64, 128, 1, 4, 4), 128),
+    "mamba2-wide": ("mamba2", U.mamba2(4, 128, 64, 4, 8, 4), 96),
+    "mamba2-192": ("mamba2", U.mamba2(2, 24, 192, 1, 1, 2), 64),
 }
 
 
@@ -117,7 +140,7 @@ def mixer_close(got, want, dtype):
     if dtype == torch.float32:
         assert float(e.max()) < 5e-5, (float(e.max()), int(e.argmax()))
     else:
-        assert float(e.max()) < 0.1 and float(e.median()) < 0.015, (float(e.max()), int(e.argmax()), float(e.median()))
+        assert float(e.max()) < 0.1 and (len(e) < 10 or float(e.median()) < 0.015), (float(e.max()), int(e.argmax()), float(e.median()))
 
 
 @DTYPES
@@ -330,9 +353,10 @@ def test_unequal_requests_side_by_side_with_slots_used_again(name, dtype):
     close(torch.cat([torch.cat(got[i]) for i in toks]), torch.cat([U.oracle_logits(name, 0, toks[i], dtype) for i in toks]), dtype)
 
 
-def test_batch_mates_do_not_change_a_sequence():
+@BOTH
+def test_batch_mates_do_not_change_a_sequence(name):
     """The same portion alone and beside others differs by rounding at most (fp32)."""
-    m, cfg = model("mixed", torch.float32), U.CONFIGS["mixed"]
+    m, cfg = model(name, torch.float32), U.CONFIGS[name]
     a, b = U.tokens_of(cfg, 50, 31), U.tokens_of(cfg, 77, 32)
     cache = m.new_cache(2, 100)
     cache.acquire("a")
@@ -343,18 +367,20 @@ def test_batch_mates_do_not_change_a_sequence():
     assert float(U.row_errors(both, alone).max()) < 2e-5
 
 
-def test_long_decoding():
-    m, cfg = model("mixed", torch.float32), U.CONFIGS["mixed"]
+@BOTH
+def test_long_decoding(name):
+    m, cfg = model(name, torch.float32), U.CONFIGS[name]
     toks = U.tokens_of(cfg, 420, 41)
     cache = m.new_cache(2, 420)
     cache.acquire("other"), cache.acquire("a")
     got = feed(m, cache, "a", toks, (9, 1))
-    close(got, U.oracle_logits("mixed", 0, toks), torch.float32)
+    close(got, U.oracle_logits(name, 0, toks), torch.float32)
 
 
-def test_graphed_decode_matches_plain_steps():
+@pytest.mark.parametrize("name", ["wide", "par-wide", "par-mixed"])
+def test_graphed_decode_matches_plain_steps(name):
     from msa_b200.hybrid import GraphedDecode
-    m, cfg = model("wide", torch.bfloat16), U.CONFIGS["wide"]
+    m, cfg = model(name, torch.bfloat16), U.CONFIGS[name]
     prompts = [U.tokens_of(cfg, n, 50 + n) for n in (5, 130, 64)]
     runs = []
     for graphed in (False, True):
@@ -400,9 +426,10 @@ def test_scheduler_generates_what_the_oracle_would(name):
         assert r.output == oracle_greedy(name, r.tokens, 7)
 
 
-def test_forward_takes_left_padded_batches():
+@BOTH
+def test_forward_takes_left_padded_batches(name):
     """The interleave loop's call: padded rows, masked steps, states advanced for unmasked tokens only."""
-    m, cfg = model("mixed", torch.float32), U.CONFIGS["mixed"]
+    m, cfg = model(name, torch.float32), U.CONFIGS[name]
     a, b = U.tokens_of(cfg, 9, 71), U.tokens_of(cfg, 5, 72)
     cache = m.new_cache(2, 32)
     ids = torch.tensor([a[:8], [0] * 4 + b[:4]])
@@ -411,21 +438,22 @@ def test_forward_takes_left_padded_batches():
     assert first.shape == (2, 1, cfg["vocab"])
     second = m(input_ids=torch.tensor([[a[8]], [0]]), attention_mask=torch.tensor([[1], [0]]), past_key_values=cache).logits
     third = m(input_ids=torch.tensor([[0], [b[4]]]), attention_mask=torch.tensor([[0], [1]]), past_key_values=cache).logits
-    wa, wb = U.oracle_logits("mixed", 0, a), U.oracle_logits("mixed", 0, b)
+    wa, wb = U.oracle_logits(name, 0, a), U.oracle_logits(name, 0, b)
     for got, want in ((first[0, 0], wa[7]), (first[1, 0], wb[3]), (second[0, 0], wa[8]), (third[1, 0], wb[4])):
         assert float(U.row_errors(got[None], want[None])) < 2e-4
     assert float(second[1].abs().max()) == 0 and cache.length(0) == 9 and cache.length(1) == 5
 
 
+@BOTH
 @pytest.mark.timeout(300)
-def test_engine_and_command_line_generate(tmp_path, capfd):
+def test_engine_and_command_line_generate(name, tmp_path, capfd):
     from msa_b200.__main__ import main
     from msa_b200.engine import GenerateConfig, MSAEngine
     from msa_b200.memory import ModelConfig
-    cfg = U.CONFIGS["mixed"]
+    cfg = U.CONFIGS[name]
     U.save(cfg, U.make_weights(cfg, 0), str(tmp_path))
     prompts = [U.tokens_of(cfg, n, 80 + n) for n in (12, 3, 30)]
-    want = [" ".join(map(str, oracle_greedy("mixed", p, 5))) for p in prompts]
+    want = [" ".join(map(str, oracle_greedy(name, p, 5))) for p in prompts]
     gen = GenerateConfig(devices=[0], max_generate_tokens=5, max_context=64, state_slots=2)
     with MSAEngine(gen, ModelConfig(model_path=str(tmp_path), dtype="float32")) as e:
         texts, _, tag = e.generate([prompts[0], " ".join(map(str, prompts[1])), prompts[2]], userdata="t")

@@ -48,9 +48,38 @@ def test_configuration_reads_every_choice():
         HybridConfig.parse(bad)
 
 
+def test_configuration_of_the_parallel_frame():
+    c = HybridConfig.parse(U.PAR_MIXED)
+    assert c.structure.block == "parallel" and c.structure.norm_offset == 1.0 and not c.structure.tied
+    assert (c.bigram.buckets, c.bigram.mul_prev, c.bigram.mul_cur, c.logit_softcap) == (61, 31, 5, 9.0)
+    assert c.windows == (17, 33) and c.runs() == [(0, None)] + [(i, t) for t in range(3) for i in (1, 2, 3)] + [(4, None)]
+    att, ssd = c.layers[1].mixer, c.layers[2].mixer
+    assert (att.heads, att.kv_heads, att.dim, att.vdim, att.rot_dims, att.rot_base, att.taps, att.window) == (6, 2, 20, 28, 12, 500.0, 3, 17)
+    assert att.sink and att.gate and att.channels == 8 * 20 + 2 * 28
+    assert (ssd.inner, ssd.channels, ssd.norm_groups, ssd.taps) == (72, 72 + 2 * 60, 2, 4) and c.layers[2].mlp is None
+    odd = HybridConfig.parse(U.PAR_ODD)
+    assert odd.bigram is None and odd.logit_softcap is None and odd.layers[3].mixer.rot_dims == 0
+    bad = json.loads(json.dumps(U.PAR_MIXED))
+    bad["layers"][1]["mixer"]["kv_heads"] = 4
+    with pytest.raises(ValueError, match="multiple"):
+        HybridConfig.parse(bad)
+    bad = json.loads(json.dumps(U.PAR_MIXED))
+    bad["layers"][2]["mixer"]["norm_groups"] = 5
+    with pytest.raises(ValueError, match="divide"):
+        HybridConfig.parse(bad)
+    bad = json.loads(json.dumps(U.PAR_MIXED))
+    bad["layers"][0]["mlp"] = U.moe(4, 2, 8, 1.0)
+    with pytest.raises(ValueError, match="dense"):
+        HybridConfig.parse(bad)
+    with pytest.raises(ValueError, match="architecture"):
+        HybridConfig.parse({**U.PAR_MIXED, "architecture": "Unheard"})
+
+
 def test_registry_tells_designs_apart(tmp_path):
     from msa_b200.registry import design_of
-    (tmp_path / "a").mkdir(), (tmp_path / "b").mkdir(), (tmp_path / "c").mkdir()
+    (tmp_path / "a").mkdir(), (tmp_path / "b").mkdir(), (tmp_path / "c").mkdir(), (tmp_path / "d").mkdir()
+    (tmp_path / "d" / "config.json").write_text(json.dumps(U.PAR_ODD))
+    assert design_of(str(tmp_path / "d")).name == "Nazerax" and design_of(str(tmp_path / "d")).serves == "states"
     (tmp_path / "a" / "config.json").write_text(json.dumps(U.ODD))
     (tmp_path / "b" / "config.json").write_text(json.dumps({"architectures": ["MSAForCausalLM"], "msa_config": {}}))
     (tmp_path / "c" / "config.json").write_text(json.dumps({"architectures": ["Something"]}))
@@ -77,6 +106,13 @@ def test_slots_are_handed_out_and_taken_back():
     assert "b" not in c and c.acquire("d") == slots["b"] and c.length("d") == 0
     with pytest.raises(KeyError):
         c.acquire("d")
+
+
+def test_state_of_every_kind_of_layer():
+    c = SequenceStateCache([RingSpec(6, 8, channels=10, taps=4), RecurrentSpec(2, 3, 3, shift=12), RecurrentSpec(2, 5, 4, 18, 1)], 2, 50, "cpu",
+                           torch.float32)
+    assert c.conv[0].shape == (3, 2, 3, 10) and c.shift[1].shape == (3, 12) and 1 not in c.conv and c.conv[2].shape == (3, 2, 0, 18)
+    assert c.state[1].shape == (3, 2, 3, 3) and c.last_token.shape == (3,) and c.last_token.dtype == torch.int32
 
 
 def test_step_tables_put_single_tokens_first_and_find_the_wanted_rows():
@@ -225,3 +261,32 @@ def test_oracle_state_carries_over_and_window_counts_the_token_itself():
     p = O.rotate_interleaved(torch.tensor([[1.0, 0.0, 0.0, 2.0]]).double(), torch.tensor([3]), 100.0)[0]
     c = torch.cos(torch.tensor([3.0, 0.3]).double()), torch.sin(torch.tensor([3.0, 0.3]).double())
     assert torch.allclose(p, torch.stack([c[0][0], c[1][0], -2 * c[1][1], 2 * c[0][1]]))
+
+
+def test_oracle_of_the_parallel_mechanisms_by_hand():
+    g = torch.Generator().manual_seed(1)
+    r = lambda *s: torch.randn(*s, generator=g, dtype=torch.float64)
+    # a bonus-less read-out sees earlier tokens only; a decay of zero forgets everything but the last one
+    q, k, v, w = r(5, 1, 3), r(5, 1, 3), r(5, 1, 3), torch.rand(5, 1, 3, generator=g).double()
+    out, _ = O.wkv_recurrence(q, k, v, w, torch.zeros(1, 3).double())
+    assert float(out[0].abs().max()) == 0
+    want = (q[2, 0] * (w[1, 0] * k[0, 0])).sum() * v[0, 0] + (q[2, 0] * k[1, 0]).sum() * v[1, 0]
+    assert torch.allclose(out[2, 0], want)
+    out, s = O.wkv_recurrence(q, k, v, torch.zeros_like(w), torch.ones(1, 3).double())
+    assert torch.allclose(out[3, 0], (q[3, 0] * k[2, 0]).sum() * v[2, 0] + (q[3, 0] * k[3, 0]).sum() * v[3, 0])
+    assert torch.allclose(s[0], torch.outer(k[4, 0], v[4, 0]))
+    # the current token is read with its full step
+    out, _ = O.ssd_recurrence(q, k, v, torch.log(w[..., 0]), torch.full((5, 1), 2.0).double())
+    assert torch.allclose(out[1, 0], 2 * (q[1, 0] * k[1, 0]).sum() * v[1, 0] + 2 * w[1, 0, 0] * (q[1, 0] * k[0, 0]).sum() * v[0, 0])
+    p = O.softmax_plus_one(torch.tensor([[0.0, float("-inf"), 0.0], [50.0, 0.0, 0.0]]).double())
+    assert torch.allclose(p[0], torch.tensor([1 / 3, 0.0, 1 / 3]).double()) and float(p[1, 0]) > 1 - 1e-9
+    x = torch.arange(1.0, 5.0).double()[:, None]
+    assert O.causal_conv(x, torch.tensor([[10.0, 1.0]]).double(), torch.tensor([0.5]).double())[:, 0].tolist() == [1.5, 12.5, 23.5, 34.5]
+    assert O.shifted(x)[:, 0].tolist() == [0.0, 1.0, 2.0, 3.0]
+    y = O.group_norm(torch.tensor([[3.0, 4.0, 0.0, 2.0]]).double(), 2, 0.0)
+    assert torch.allclose(y, torch.tensor([[3.0, 4.0, 0.0, 2.0]]).double() / torch.tensor([12.5, 12.5, 2.0, 2.0]).double().sqrt())
+    cfg = {"embedding": {"bigram": {"buckets": 5, "mul_prev": 3, "mul_cur": 2}}}
+    w = {"embed": torch.zeros(9, 1), "bigram": torch.arange(6.0)[:, None]}
+    assert O.embedding(cfg, w, [4, 7, 4], torch.float64)[:, 0].tolist() == [5.0, (12 + 14) % 5, (21 + 8) % 5]
+    rot = O.rotate_leading(torch.tensor([[1.0, 0.0, 7.0]]).double(), torch.tensor([2]), 100.0, 2)[0]
+    assert torch.allclose(rot, torch.tensor([torch.cos(torch.tensor(2.0)), torch.sin(torch.tensor(2.0)), 7.0]).double())
