@@ -66,6 +66,8 @@ def parse():
                     choices=["routing", "pooling", "decode", "fetch", "route-decode", "prefill", "stage1", "generate", "hybrid"],
                     help="routing = the headline (default); the others time one secondary kernel each")
     ap.add_argument("--hybrid-sizes", default="2k,4k", help="hybrid workload: model sizes to run")
+    ap.add_argument("--hybrid-design", default="Mutuvik", choices=["Mutuvik", "Nazerax"],
+                    help="hybrid workload: Mutuvik beside the memory decoder, or Nazerax beside Mutuvik with dense feed-forwards")
     return ap.parse_args()
 
 
@@ -1412,44 +1414,59 @@ HYBRID_SIZES = {   # width, heads, kv heads of the delta layers, window, dense f
 }
 
 
-def hybrid_config(z, vocab=32768):
+def hybrid_config(z, vocab=32768, dense=False):
     delta = {"type": "delta", "mixer": {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128, "conv": 4}}
     latent = {"type": "latent_attention", "mixer": {
         "heads": z["heads"], "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
         "rot": {"base": 10000.0, "dims": 64}, "mask": {"size": z["window"]}}}
-    moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["eff"], "limit": 7.0}}
+    moe = {"kind": "dense", "ff": z["ff"]} if dense else {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["eff"], "limit": 7.0}}
     return {"architecture": "Mutuvik", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-5},
             "layers": [{**delta, "mlp": {"kind": "dense", "ff": z["ff"]}}, {**latent, "mlp": moe}, {**delta, "mlp": moe}, {**latent, "mlp": moe}],
             "loop": {"start": 1, "stop": 4, "times": 2}}
 
 
-def hybrid_model(torch, dev, z):
+def nazerax_config(z, vocab=32768):
+    """The same width, layer runs, window and dense feed-forward: wkv heads of 64, attention of ``heads`` x 128 over 8 (4)
+    key / value heads, a state-space layer of twice the width."""
+    width = z["width"]
+    wkv = {"type": "wkv", "mixer": {"heads": width // 64, "dim": 64}}
+    att = {"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["heads"] // 4, "dim": 128, "vdim": 128, "conv": 4, "scale": 128 ** -0.5,
+                                          "rot": {"base": 10000.0, "dims": 64}, "mask": {"size": z["window"]}}}
+    ssd = {"type": "mamba2", "mixer": {"heads": width // 32, "vdim": 64, "state": 128, "groups": 8, "norm_groups": 8, "conv": 4}}
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    return {"architecture": "Nazerax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}},
+            "layers": [{**wkv, "mlp": mlp}, {**att, "mlp": mlp}, {**ssd, "mlp": mlp}, {**att, "mlp": mlp}],
+            "loop": {"start": 1, "stop": 4, "times": 2}}
+
+
+def hybrid_model(torch, dev, cfg):
     from msa_b200.hybrid import HybridForCausalLM, Weights
     from msa_b200.hybrid_config import HybridConfig
     gen = torch.Generator(device=dev)
     gen.manual_seed(3)
 
     class Drawn(Weights):
+        def shape(self, name):                        # sizes that only a checkpoint's tensors tell
+            return (64, cfg["width"])
+
         def raw(self, name, *shape):
             t = torch.randn(shape, generator=gen, device=dev, dtype=torch.float32)
-            if len(shape) == 2 and not name.endswith(".conv") and name not in ("embed", "loop.step"):
+            if len(shape) == 2 and not name.endswith(".conv") and name not in ("embed", "loop.step", "bigram"):
                 t *= shape[1] ** -0.5
             elif "norm" in name:
-                t = 1 + 0.1 * t
+                t = 0.1 * t + (0.0 if cfg["architecture"] == "Nazerax" and ".mix." not in name else 1.0)
             elif name.endswith("A_log"):
                 t -= 1.0
+            elif name.endswith(".w0"):
+                t -= 2.0
             return t.to(torch.bfloat16)
-    return HybridForCausalLM(HybridConfig.parse(hybrid_config(z)), Drawn({}, dev, torch.bfloat16), dev)
+    return HybridForCausalLM(HybridConfig.parse(cfg), Drawn({}, dev, torch.bfloat16), dev)
 
 
-def hybrid_kernels(torch, dev, model, z, pk, decode_b):
-    """Every kernel of the design alone: time, algorithmic flops and bytes, and the fraction of the bound that applies
-    (the larger of flops over the burst bf16 rate and bytes over the copy bandwidth)."""
-    import ctypes
-
-    from msa_b200 import _cabi_lm as A, lm_ops as K
-    from msa_b200.cache import DecodeStep, PackedStep
-    rows, heads, width, window = {}, z["heads"], z["width"], z["window"]
+def kernel_legs(torch, dev, pk):
+    """``(rows, leg, leg_rotating)``: timers of one kernel that fill ``rows`` with time, algorithmic bound and fraction."""
+    rows = {}
     flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
 
     def leg(name, fn, flops, nbytes, reps=10):
@@ -1482,45 +1499,112 @@ def hybrid_kernels(torch, dev, model, z, pk, decode_b):
         rows[name] = {"us": round(ms * 1e3, 1), "bound": "tensor" if t_f > t_b else "hbm", "bound_us": round(max(t_f, t_b) * 1e3, 1),
                       "frac": round(max(t_f, t_b) / ms, 3)}
 
-    n_seq, t = 4, 2048
+    return rows, leg, leg_rotating
+
+
+def nazerax_kernels(torch, dev, model, z, pk, decode_b):
+    """Every kernel of Nazerax alone, as ``hybrid_kernels``."""
+    import ctypes
+
+    from msa_b200 import _cabi_lm as A, lm_ops as K
+    from msa_b200.cache import DecodeStep, PackedStep
+    from msa_b200.hybrid import portion_attention
+    rows, leg, leg_rotating = kernel_legs(torch, dev, pk)
+    width, window = z["width"], z["window"]
+    n_seq, t, b = 4, 2048, decode_b
     n = n_seq * t
-    cache = model.new_cache(max(n_seq, decode_b) + 1, 4096)
+    cache = model.new_cache(max(n_seq, b) + 1, 4096)
     for i in range(n_seq):
         cache.acquire(i)
     step = PackedStep([(i, [1] * t, []) for i in range(n_seq)], cache, model.config.windows)
-    lat, dlt, moe = model.layers[1].mixer, model.layers[0].mixer, model.layers[1].ff
-    view = step.views[window]
-    bf = dict(dtype=torch.bfloat16, device=dev)
-    h = torch.randn((n, width), **bf)
-    x = torch.randn((n, width), dtype=torch.float32, device=dev)
-    y = torch.randn((n, width), **bf)
-    leg("residual_norm", lambda: K.residual_norm(x, y, model.layers[0].norm1b, model.layers[0].norm2, 1e-5, torch.bfloat16, x_out=x),
-        0, n * width * 12)
-    s = lat.spec
-    proj = K.matmul(h, lat.w_in)
-    ctx = torch.empty((n, s.kv_rank + s.rot_dim), **bf)
-    leg("latent_prep", lambda: K.latent_prep(proj, s, lat.norm, lat.inv_freq, 1e-5, step, view, cache.ring[1], ctx), 0,
-        n * 2 * (2 * heads * s.rot_dim + 2 * (s.kv_rank + s.rot_dim)))
-    kv = K.matmul(ctx[:, :s.kv_rank], lat.w_kv)
-    out = torch.empty((n, heads * s.vdim), **bf)
+    wkv, att, ssd = (model.layers[i].mixer for i in range(3))
+    l0, ff = model.layers[0], model.layers[0].ff
+    bf, f32 = dict(dtype=torch.bfloat16, device=dev), dict(dtype=torch.float32, device=dev)
+    h, y, x = torch.randn((n, width), **bf), torch.randn((n, width), **bf), torch.randn((n, width), **f32)
+    p, st = A.ptr, A.stream_ptr(dev)
+    tok = torch.randint(0, model.config.vocab, (n,), dtype=torch.int32, device=dev)
+    leg("embed + bigram + two norms", lambda: K.embed(model.embed, tok, l0.norm1, 1e-5, w_next2=l0.norm2, x_copy=x, pair=model.pair, step=step,
+                                                      last_token=cache.last_token), 0, n * width * (4 + 8 + 4))
+    leg("residual_norm (two norms)", lambda: K.residual_norm(x, y, None, l0.norm1, 1e-5, torch.bfloat16, x_out=x, w_next2=l0.norm2), 0, n * width * 14)
+    leg("token_shift", lambda: K.token_shift(h, wkv.mu, step, cache.shift[0]), 0, n * width * 12)
+    mixes = K.token_shift(h, wkv.mu, step, cache.shift[0])
+    s = wkv.spec
+    leg("cuBLAS r, k, v, gate (reference)", lambda: torch.bmm(mixes[:4], wkv.w_in.transpose(1, 2)), 8.0 * n * width * s.inner,
+        8 * n * width + 8 * n * s.inner + wkv.w_in.numel() * 2)
+    rkvg = torch.bmm(mixes[:4], wkv.w_in.transpose(1, 2))
+    lowin = K.matmul(mixes[4], wkv.w1, torch.float32)
+    leg("tanh_split", lambda: K.tanh_split(lowin, torch.bfloat16, wkv.parts), 0, lowin.numel() * 8)
+    raw = K.matmul(K.tanh_split(lowin, torch.bfloat16, wkv.parts), wkv.w2, torch.float32)
+    out = torch.empty((n, s.inner), **bf)
+    macs = n * s.heads * (2 * s.dim * s.dim + 64 * s.dim)
+    leg("wkv chunks (add, carry, read)", lambda: K.wkv_mix(rkvg, raw, s, wkv, cache.state[0], 1e-5, step, out), 2.0 * macs,
+        n * s.inner * (8 + 4 + 2) + n_seq * s.heads * s.dim * s.dim * 8)
+    g = att.spec
+    view, width_row = step.views[window], g.kv_heads * (g.dim + g.vdim)
+    proj = K.matmul(h, att.w_in)
+    q, ctx = torch.empty((n, g.heads, g.dim), **bf), torch.empty((n, width_row), **bf)
+    leg("group_prep", lambda: K.group_prep(proj, g, att, step, view, cache.ring[1], cache.conv[1], q, ctx), 0, n * g.channels * 4)
+    oa = torch.empty((n, g.heads, g.vdim), **bf)
+    gate = proj[:, g.channels:g.channels + g.heads]
+    k, v = ctx[:, :g.kv_heads * g.dim].unflatten(1, (g.kv_heads, g.dim)), ctx[:, g.kv_heads * g.dim:].unflatten(1, (g.kv_heads, g.vdim))
     pairs = n_seq * sum(min(i + 1, window) for i in range(t))
-    leg("window_attn_tc (prompt)", lambda: K.window_attn_tc(proj, kv, ctx, s, out, step, view, model.status),
-        2.0 * pairs * heads * (s.dim + s.rot_dim + s.vdim), n * heads * 2 * (s.dim + s.rot_dim + s.dim + 2 * s.vdim))
-    leg("ring_store", lambda: K.ring_store(ctx, step, view, cache.ring[1]), 0, n_seq * min(t, window) * (s.kv_rank + s.rot_dim) * 4)
-    d = dlt.spec
-    projd = K.matmul(h, dlt.w_in)
-    args = K.delta_args(projd, d, dlt, cache.conv[0], cache.state[0], 1e-5, step)
-    f32 = dict(dtype=torch.float32, device=dev)
-    v, gates = torch.empty((n, heads * d.vdim), **bf), torch.empty((n, 2 * heads), **f32)
-    qk, outd, st = torch.empty((n, 4 * d.kv_heads * d.dim), **bf), torch.empty((n, heads * d.vdim), **bf), A.stream_ptr(dev)
-    p = A.ptr
-    leg("delta_prep", lambda: A.call("msa_lm_delta_prep_split", ctypes.byref(args), p(qk), p(v), p(gates), st), 0,
-        n * (d.channels * 2 + 2 * d.kv_heads * d.dim * 4 + heads * d.vdim * 2))
-    # flops of the chunked form, once each: S products, the triangular ones at half
-    c = 64
-    macs = n * heads * (3 * d.dim * d.vdim + c * d.vdim) + n * d.kv_heads * c * d.dim + n * heads * c * c / 6
-    leg("delta_chunk + delta_state", lambda: K.delta_chunks(args, d, step, qk, v, gates, outd), 2.0 * macs,
-        n * (d.kv_heads * d.dim * 8 + heads * d.vdim * (2 + 2 + 2)) + n_seq * heads * d.dim * d.vdim * 4)
+    leg("window_attn_tc (prompt)", lambda: portion_attention((q, None, k, None, v, oa), True, model.status, step, view, g.scale, sink=True, gate=gate),
+        2.0 * pairs * g.heads * (g.dim + g.vdim), n * 2 * (g.heads * (g.dim + g.vdim) + width_row))
+    leg("ring_store", lambda: K.ring_store(ctx, step, view, cache.ring[1]), 0, n_seq * min(t, window) * width_row * 4)
+    d = ssd.spec
+    projd = K.matmul(h, ssd.w_in)
+    yd, od = torch.empty((n, d.inner), **f32), torch.empty((n, d.inner), **bf)
+    xbc, dt = torch.empty((n, d.channels), **bf), torch.empty((n, d.heads), **f32)
+
+    def ssd_args(pr, stp, run, yy):
+        return A.SsdArgs(proj=p(pr), proj_stride=pr.stride(0), conv_w=p(ssd.conv), conv_b=p(ssd.conv_b), dt_bias=p(ssd.dt_bias), a_log=p(ssd.a_log),
+                         d_skip=p(ssd.d_skip), conv_state=p(cache.conv[run]), state=p(cache.state[run]), tok_seq=p(stp.tok_seq), slot=p(stp.slot),
+                         start=p(stp.start), cu=p(stp.cu), y=p(yy), n_tok=stp.n_tok, n_seq=stp.n_seq, n_decode=stp.n_decode, heads=d.heads,
+                         vdim=d.vdim, n_state=d.state, groups=d.groups, taps=d.taps, dtype=A.dtype_code(torch.bfloat16))
+    sa = ssd_args(projd, step, 2, yd)
+    leg("ssd_prep", lambda: A.call("msa_lm_ssd_prep", ctypes.byref(sa), p(xbc), p(dt), st), 0, n * d.channels * 4)
+    gcum, work = torch.empty((n, d.heads), dtype=torch.float64, device=dev), torch.empty((step.n_chunks, d.heads, d.state, d.vdim), **f32)
+    macs = n * d.heads * (2 * d.state * d.vdim + 32 * d.vdim) + n * d.groups * 32 * d.state
+    leg("ssd chunks (add, carry, read)", lambda: A.call("msa_lm_ssd_chunk", ctypes.byref(sa), p(xbc), p(dt), p(step.chunk_off), step.n_chunks, p(gcum), p(work), st),
+        2.0 * macs, n * (d.channels * 2 + d.inner * 6 + d.heads * 4) + n_seq * d.heads * d.state * d.vdim * 8)
+    leg("part_norm", lambda: K.part_norm(yd, ssd.norm, d.norm_groups, 1e-5, od), 0, n * d.inner * 6)
+    del work, gcum
+    gu, act = K.matmul(h, ff.w_gate_up), torch.empty((n, ff.ff), **bf)
+    leg("silu_mul", lambda: K.silu_mul(gu, ff.ff, act), 0, n * ff.ff * 6)
+    leg("cuBLAS in-projection (reference)", lambda: K.matmul(h, ssd.w_in), 2.0 * n * width * ssd.w_in.shape[0], (n * width + ssd.w_in.numel() + n * ssd.w_in.shape[0]) * 2)
+    for i in range(n_seq):
+        cache.release(i)
+    del proj, projd, yd, od, xbc, gu, act, mixes, rkvg, raw
+    ds = DecodeStep(b, cache, model.config.windows)
+    ds.fill([1] * b, [window + 5] * b, list(range(b)))
+    hb, xb, yb = torch.randn((b, width), **bf), torch.randn((b, width), **f32), torch.randn((b, width), **bf)
+    mb = K.token_shift(hb, wkv.mu, ds, cache.shift[0])
+    leg_rotating(f"token_shift (batch {b})", lambda i: K.token_shift(hb, wkv.mu, ds, cache.shift[0]), 0, b * width * 14)
+    rb, rawb, ob = torch.bmm(mb[:4], wkv.w_in.transpose(1, 2)), torch.randn((b, s.inner), **f32), torch.empty((b, s.inner), **bf)
+    more = [torch.randn((b + 2, s.heads, s.dim, s.dim), **f32) for _ in range(8)]            # several layers' states
+    leg_rotating(f"wkv_decode (batch {b})", lambda i: K.wkv_mix(rb, rawb, s, wkv, more[i % 8], 1e-5, ds, ob), 0, b * s.heads * s.dim * s.dim * 8 + b * s.inner * 14)
+    pb, qb = K.matmul(hb, att.w_in), torch.empty((b, g.heads, g.dim), **bf)
+    leg_rotating(f"group_prep (batch {b})", lambda i: K.group_prep(pb, g, att, ds, ds.views[window], cache.ring[1], cache.conv[1], qb, None), 0,
+                 b * g.channels * 2 * (2 * g.taps))
+    rings, oab, gb = list(cache.ring.values()), torch.empty((b, g.heads, g.vdim), **bf), pb[:, g.channels:g.channels + g.heads]
+    leg_rotating(f"group_decode + merge (batch {b})",
+                 lambda i: K.group_decode(qb, rings[i % len(rings)], g.kv_heads, ds, oab, window=window, scale=g.scale, sink=True, gate=gb),
+                 2.0 * b * window * g.heads * (g.dim + g.vdim), b * window * width_row * 2)
+    pd, yb2, ob2 = K.matmul(hb, ssd.w_in), torch.empty((b, d.inner), **f32), torch.empty((b, d.inner), **bf)
+    runs = [r for r, sp in enumerate(cache.specs) if r in cache.state and getattr(sp, "channels", 0)]
+    das = [ssd_args(pd, ds, r, yb2) for r in runs]
+    leg_rotating(f"ssd_decode (batch {b})", lambda i: A.call("msa_lm_ssd_decode", ctypes.byref(das[i % len(das)]), A.stream_ptr(dev)), 0,
+                 b * d.heads * d.state * d.vdim * 8 + b * d.channels * 2 * (2 * d.taps))
+    leg_rotating(f"part_norm (batch {b})", lambda i: K.part_norm(yb2, ssd.norm, d.norm_groups, 1e-5, ob2), 0, b * d.inner * 6)
+    leg_rotating(f"residual_norm (two norms, batch {b})",
+                 lambda i: K.residual_norm(xb, yb, None, l0.norm1, 1e-5, torch.bfloat16, x_out=xb, w_next2=l0.norm2), 0, b * width * 14)
+    lg = torch.randn((b, model.config.vocab), **f32)
+    leg_rotating(f"softcap (batch {b})", lambda i: K.softcap(lg, 30.0), 0, lg.numel() * 8)
+    model.check_status()
+    return rows
+
+
+def hybrid_expert_kernels(torch, K, leg, model, moe, h, x, n, width):
     m = moe.spec
     logits = K.matmul(h, moe.router, torch.float32)
     leg("moe_topk", lambda: K.moe_topk(logits, moe.bias, m.top), 0, n * m.experts * 4)
@@ -1538,6 +1622,67 @@ def hybrid_kernels(torch, dev, model, z, pk, decode_b):
         2.0 * ent * width * m.ff, moe.w_down.numel() * 2 + ent * (m.ff + width) * 2)
     leg("residual_norm over experts", lambda: K.residual_norm(x, ye, model.layers[1].norm2b, model.layers[2].norm1, 1e-5, torch.bfloat16, x_out=x, inv=inv, mix=mix),
         0, n * width * 10 + ent * width * 2)
+
+
+def hybrid_kernels(torch, dev, model, z, pk, decode_b):
+    """Every kernel of the design alone: time, algorithmic flops and bytes, and the fraction of the bound that applies
+    (the larger of flops over the burst bf16 rate and bytes over the copy bandwidth)."""
+    import ctypes
+
+    from msa_b200 import _cabi_lm as A, lm_ops as K
+    from msa_b200.cache import DecodeStep, PackedStep
+    from msa_b200.hybrid import portion_attention
+    rows, leg, leg_rotating = kernel_legs(torch, dev, pk)
+    heads, width, window = z["heads"], z["width"], z["window"]
+    n_seq, t = 4, 2048
+    n = n_seq * t
+    cache = model.new_cache(max(n_seq, decode_b) + 1, 4096)
+    for i in range(n_seq):
+        cache.acquire(i)
+    step = PackedStep([(i, [1] * t, []) for i in range(n_seq)], cache, model.config.windows)
+    lat, dlt, moe = model.layers[1].mixer, model.layers[0].mixer, model.layers[1].ff
+    experts = hasattr(moe, "router")
+    view = step.views[window]
+    bf = dict(dtype=torch.bfloat16, device=dev)
+    h = torch.randn((n, width), **bf)
+    x = torch.randn((n, width), dtype=torch.float32, device=dev)
+    y = torch.randn((n, width), **bf)
+    leg("residual_norm", lambda: K.residual_norm(x, y, model.layers[0].norm1b, model.layers[0].norm2, 1e-5, torch.bfloat16, x_out=x),
+        0, n * width * 12)
+    s = lat.spec
+    proj = K.matmul(h, lat.w_in)
+    ctx = torch.empty((n, s.kv_rank + s.rot_dim), **bf)
+    leg("latent_prep", lambda: K.latent_prep(proj, s, lat.norm, lat.inv_freq, 1e-5, step, view, cache.ring[1], ctx), 0,
+        n * 2 * (2 * heads * s.rot_dim + 2 * (s.kv_rank + s.rot_dim)))
+    kv = K.matmul(ctx[:, :s.kv_rank], lat.w_kv)
+    out = torch.empty((n, heads * s.vdim), **bf)
+    pairs = n_seq * sum(min(i + 1, window) for i in range(t))
+    qp, kr = proj[:, :heads * (s.dim + s.rot_dim)].unflatten(1, (heads, s.dim + s.rot_dim)), ctx[:, s.kv_rank:].unsqueeze(1)
+    kx, vx = (kv[:, c:c + heads * w].unflatten(1, (heads, w)) for c, w in ((0, s.dim), (heads * s.dim, s.vdim)))
+    leg("window_attn_tc (prompt)",
+        lambda: portion_attention((qp[..., :s.dim], qp[..., s.dim:], kx, kr, vx, out.unflatten(1, (heads, s.vdim))), True, model.status, step, view, s.scale),
+        2.0 * pairs * heads * (s.dim + s.rot_dim + s.vdim), n * heads * 2 * (s.dim + s.rot_dim + s.dim + 2 * s.vdim))
+    leg("ring_store", lambda: K.ring_store(ctx, step, view, cache.ring[1]), 0, n_seq * min(t, window) * (s.kv_rank + s.rot_dim) * 4)
+    d = dlt.spec
+    projd = K.matmul(h, dlt.w_in)
+    args = K.delta_args(projd, d, dlt, cache.conv[0], cache.state[0], 1e-5, step)
+    f32 = dict(dtype=torch.float32, device=dev)
+    v, gates = torch.empty((n, heads * d.vdim), **bf), torch.empty((n, 2 * heads), **f32)
+    qk, outd, st = torch.empty((n, 4 * d.kv_heads * d.dim), **bf), torch.empty((n, heads * d.vdim), **bf), A.stream_ptr(dev)
+    p = A.ptr
+    leg("delta_prep", lambda: A.call("msa_lm_delta_prep_split", ctypes.byref(args), p(qk), p(v), p(gates), st), 0,
+        n * (d.channels * 2 + 2 * d.kv_heads * d.dim * 4 + heads * d.vdim * 2))
+    # flops of the chunked form, once each: S products, the triangular ones at half
+    c = 64
+    macs = n * heads * (3 * d.dim * d.vdim + c * d.vdim) + n * d.kv_heads * c * d.dim + n * heads * c * c / 6
+    leg("delta_chunk + delta_state", lambda: K.delta_chunks(args, d, step, qk, v, gates, outd), 2.0 * macs,
+        n * (d.kv_heads * d.dim * 8 + heads * d.vdim * (2 + 2 + 2)) + n_seq * heads * d.dim * d.vdim * 4)
+    if not experts:
+        gu, act = K.matmul(h, moe.w_gate_up), torch.empty((n, moe.ff), **bf)
+        leg("silu_mul", lambda: K.silu_mul(gu, moe.ff, act), 0, n * moe.ff * 6)
+        del gu, act
+    else:
+        hybrid_expert_kernels(torch, K, leg, model, moe, h, x, n, width)
     leg("cuBLAS in-projection (reference)", lambda: K.matmul(h, dlt.w_in), 2.0 * n * width * dlt.w_in.shape[0], (n * width + dlt.w_in.numel() + n * dlt.w_in.shape[0]) * 2)
     # decode: every sequence past its window
     for i in range(n_seq):
@@ -1559,18 +1704,20 @@ def hybrid_kernels(torch, dev, model, z, pk, decode_b):
     leg_rotating(f"delta_decode (batch {b})",
                  lambda i: A.call("msa_lm_delta_decode", ctypes.byref(das[i % len(das)]), p(od), od.stride(0), A.stream_ptr(dev)), 0,
                  b * heads * d.dim * d.vdim * 8 + b * d.channels * 2 * (2 * d.taps))
-    lg = torch.randn((b, m.experts), dtype=torch.float32, device=dev)
-    idx, mix = K.moe_topk(lg, moe.bias, m.top)
-    src, inv, off, tiles = K.moe_sort(idx, m.experts, 128)
-    used = int((off[1:] > off[:-1]).sum())
-    ffs = [l.ff for l in model.layers[1:]]
-    leg_rotating(f"moe_topk + moe_sort (batch {b})", lambda i: K.moe_sort(K.moe_topk(lg, moe.bias, m.top)[0], m.experts, 128), 0, b * m.experts * 4)
-    gate_up = lambda i: K.moe_gemm_tc(hb, src, ffs[i % len(ffs)].w_gate_up, off, tiles, entries=b * m.top, act=True, limit=7.0, status=model.status)
-    leg_rotating(f"moe_gemm_tc gate/up (batch {b})", gate_up, 2.0 * b * m.top * width * 2 * m.ff, used * 2 * m.ff * width * 2)
-    ab = gate_up(0)
-    leg_rotating(f"moe_gemm_tc down (batch {b})",
-                 lambda i: K.moe_gemm_tc(ab, None, ffs[i % len(ffs)].w_down, off, tiles, entries=b * m.top, act=False, status=model.status),
-                 2.0 * b * m.top * width * m.ff, used * m.ff * width * 2)
+    if experts:
+        m = moe.spec
+        lg = torch.randn((b, m.experts), dtype=torch.float32, device=dev)
+        idx, mix = K.moe_topk(lg, moe.bias, m.top)
+        src, inv, off, tiles = K.moe_sort(idx, m.experts, 128)
+        used = int((off[1:] > off[:-1]).sum())
+        ffs = [l.ff for l in model.layers[1:]]
+        leg_rotating(f"moe_topk + moe_sort (batch {b})", lambda i: K.moe_sort(K.moe_topk(lg, moe.bias, m.top)[0], m.experts, 128), 0, b * m.experts * 4)
+        gate_up = lambda i: K.moe_gemm_tc(hb, src, ffs[i % len(ffs)].w_gate_up, off, tiles, entries=b * m.top, act=True, limit=7.0, status=model.status)
+        leg_rotating(f"moe_gemm_tc gate/up (batch {b})", gate_up, 2.0 * b * m.top * width * 2 * m.ff, used * 2 * m.ff * width * 2)
+        ab = gate_up(0)
+        leg_rotating(f"moe_gemm_tc down (batch {b})",
+                     lambda i: K.moe_gemm_tc(ab, None, ffs[i % len(ffs)].w_down, off, tiles, entries=b * m.top, act=False, status=model.status),
+                     2.0 * b * m.top * width * m.ff, used * m.ff * width * 2)
     xb, yb = torch.randn((b, width), dtype=torch.float32, device=dev), torch.randn((b, width), **bf)
     leg_rotating(f"residual_norm (batch {b})",
                  lambda i: K.residual_norm(xb, yb, model.layers[0].norm1b, model.layers[0].norm2, 1e-5, torch.bfloat16, x_out=xb), 0, b * width * 12)
@@ -1648,60 +1795,75 @@ def closest_model(torch, dev, z, runs, decode_batches, steps, warmup):
     return out
 
 
-def run_hybrid(args):
-    """Prompt and decode throughput of the layered decoder at a few sizes, its kernels one by one, and the memory
-    decoder at equal size.  Prompts: 4 x 2,048 tokens in one step, logits of each last token; decode: one token for every
-    sequence from a full window, CUDA graph, tokens fed back on the device."""
-    import torch
+def hybrid_throughput(torch, dev, model, z, steps, warmup, batches):
+    """Prompts: 4 x 2,048 tokens in one step, logits of each last token; decode: one token for every sequence from a full
+    window, CUDA graph, tokens fed back on the device.  Also the kernel launches of the prompt steps."""
     from msa_b200 import _cabi_lm as A
     from msa_b200.cache import PackedStep
     from msa_b200.hybrid import GraphedDecode
+    r = {"layer_runs": len(model.config.runs())}
+    n_seq, t = 4, 2048
+    cache = model.new_cache(n_seq, t)
+    for i in range(n_seq):
+        cache.acquire(i)
+    ids = torch.randint(0, 32768, (n_seq, t)).tolist()
+    step = PackedStep([(i, ids[i], [t - 1]) for i in range(n_seq)], cache, model.config.windows)
+    l0 = A.launches
+    model.step(step, cache)
+    launches = (A.launches - l0) * (max(3, steps // 2) + 3)
+    ms = _time_ms(torch, lambda: model.step(step, cache), max(3, steps // 2), 3)
+    r["prompt_4x2048"] = {"ms": ms, "tokens_per_s": n_seq * t / ms * 1e3}
+    del cache, step
+    for b in batches:
+        cache = model.new_cache(b, z["window"] + 4 * (steps + warmup) + 64)
+        g = GraphedDecode(model, cache, b)
+        for state in (*cache.ring.values(), *cache.state.values(), *cache.conv.values()):     # every sequence its own past
+            state.normal_(std=0.1)
+        g.tables.fill(torch.randint(0, 32768, (b,)).tolist(), [z["window"] + 3] * b, list(range(b)))
+        ms = _time_ms(torch, g.replay, steps, warmup)
+        r[f"decode_batch_{b}"] = {"ms_per_step": ms, "tokens_per_s": b / ms * 1e3}
+        model.check_status()
+        del g, cache
+        torch.cuda.empty_cache()
+    return r, launches
+
+
+def run_hybrid(args):
+    """Prompt and decode throughput of a layered decoder at a few sizes, its kernels one by one, and the closest other model
+    at equal size: the memory decoder beside Mutuvik, Mutuvik with dense feed-forwards beside Nazerax."""
+    import torch
     torch.cuda.set_device(0)
     dev, pk = torch.device("cuda", 0), peaks()
     steps, warmup = max(args.steps, 20), max(args.warmup, 3)
     sampler = ClockSampler(0)
     sampler.start()
     sizes, launches, batches = {}, 0, (1, 32, 128)
+    ours = args.hybrid_design == "Nazerax"
     for name in args.hybrid_sizes.split(","):
         z = HYBRID_SIZES[name]
-        model = hybrid_model(torch, dev, z)
-        runs = len(model.config.runs())
-        r = {"layer_runs": runs}
-        n_seq, t = 4, 2048
-        cache = model.new_cache(n_seq, t)
-        for i in range(n_seq):
-            cache.acquire(i)
-        ids = torch.randint(0, 32768, (n_seq, t)).tolist()
-        step = PackedStep([(i, ids[i], [t - 1]) for i in range(n_seq)], cache, model.config.windows)
-        l0 = A.launches
-        model.step(step, cache)
-        launches += (A.launches - l0) * (max(3, steps // 2) + 3)
-        ms = _time_ms(torch, lambda: model.step(step, cache), max(3, steps // 2), 3)
-        r["prompt_4x2048"] = {"ms": ms, "tokens_per_s": n_seq * t / ms * 1e3}
-        del cache, step
-        for b in batches:
-            cache = model.new_cache(b, z["window"] + 4 * (steps + warmup) + 64)
-            g = GraphedDecode(model, cache, b)
-            for state in (*cache.ring.values(), *cache.state.values(), *cache.conv.values()):     # every sequence its own past
-                state.normal_(std=0.1)
-            g.tables.fill(torch.randint(0, 32768, (b,)).tolist(), [z["window"] + 3] * b, list(range(b)))
-            ms = _time_ms(torch, g.replay, steps, warmup)
-            r[f"decode_batch_{b}"] = {"ms_per_step": ms, "tokens_per_s": b / ms * 1e3}
-            model.check_status()
-            del g, cache
-            torch.cuda.empty_cache()
-        r["kernels"] = hybrid_kernels(torch, dev, model, z, pk, 32)
+        model = hybrid_model(torch, dev, nazerax_config(z) if ours else hybrid_config(z))
+        r, n = hybrid_throughput(torch, dev, model, z, steps, warmup, batches)
+        launches += n
+        r["kernels"] = (nazerax_kernels if ours else hybrid_kernels)(torch, dev, model, z, pk, 32)
         del model
         torch.cuda.empty_cache()
-        r["memory_decoder"] = closest_model(torch, dev, z, runs, batches, steps, warmup)
+        if ours:
+            model = hybrid_model(torch, dev, hybrid_config(z, dense=True))
+            r["Mutuvik, dense"], _ = hybrid_throughput(torch, dev, model, z, steps, warmup, batches)
+            r["Mutuvik, dense"]["kernels"] = hybrid_kernels(torch, dev, model, z, pk, 32)
+            del model
+            torch.cuda.empty_cache()
+        else:
+            r["memory_decoder"] = closest_model(torch, dev, z, r["layer_runs"], batches, steps, warmup)
         sizes[name] = r
-    closest = closest_kernels(torch, dev, pk)
     first = sizes[args.hybrid_sizes.split(",")[-1]]
     print(json.dumps({"metric": "layered decoder prompt tokens/s", "value": first["prompt_4x2048"]["tokens_per_s"], "unit": "tokens/s",
                       "n_gpus": 1, "steps": steps, "warmup": warmup, "ms_per_step": first["prompt_4x2048"]["ms"], "higher_is_better": True,
                       "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic, random weights",
-                      "config": {"workload": "hybrid", "sizes": {k: HYBRID_SIZES[k] for k in sizes}, "l2": "kernel legs flush L2"},
-                      "gpu_launches": launches, "clocks": sampler.stop(), "peaks": pk, "results": sizes, "memory_decoder_kernels": closest}))
+                      "config": {"workload": "hybrid", "design": args.hybrid_design, "sizes": {k: HYBRID_SIZES[k] for k in sizes},
+                                 "l2": "kernel legs flush L2"},
+                      "gpu_launches": launches, "clocks": sampler.stop(), "peaks": pk, "results": sizes,
+                      **({} if ours else {"memory_decoder_kernels": closest_kernels(torch, dev, pk)})}))
 
 
 def run_generate(args):
