@@ -81,7 +81,7 @@ inline int pass_groups(int dv, int v) { return dv / v >= kLinThreads ? 1 : kLinT
 
 // One block per (head, sequence).
 template <typename T, int V>
-__global__ void __launch_bounds__(kLinThreads) wkv_decode_kernel(const msa_lm_wkv_args a, T* __restrict__ out, long long out_stride) {
+__global__ void __launch_bounds__(kLinThreads, 4) wkv_decode_kernel(const msa_lm_wkv_args a, T* __restrict__ out, long long out_stride) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float s_part[32];
   const int h = blockIdx.x, b = blockIdx.y, dim = a.dim, pad = (dim + 3) / 4 * 4;
@@ -120,7 +120,7 @@ struct SsdLayout {
 };
 
 template <typename T, int V>
-__global__ void __launch_bounds__(kLinThreads) ssd_decode_kernel(const msa_lm_ssd_args a) {
+__global__ void __launch_bounds__(kLinThreads, 4) ssd_decode_kernel(const msa_lm_ssd_args a) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float s_part[32];
   const SsdLayout L(a);

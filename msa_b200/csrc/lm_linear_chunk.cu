@@ -57,15 +57,25 @@ __device__ __forceinline__ void lc_load_rows(uint32_t dst, int pitch, const __nv
 template <int ROWS, int TILE, int THREADS>
 __device__ __forceinline__ void lc_load_split(unsigned char* dst, int pitch, int lo_off, const float* src, int rows, int cols) {
   constexpr int kVecs = TILE / 4;
-#pragma unroll 4
-  for (int i = threadIdx.x; i < ROWS * kVecs; i += THREADS) {
-    const int r = i / kVecs, c = i % kVecs * 4;
-    const float4 x = r < rows && c < cols ? load4(src + (long long)r * cols + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-    uint2 hi, lo;
-    lc_split2(x.x, x.y, hi.x, lo.x);
-    lc_split2(x.z, x.w, hi.y, lo.y);
-    *reinterpret_cast<uint2*>(dst + r * pitch + c * 2) = hi;
-    *reinterpret_cast<uint2*>(dst + lo_off + r * pitch + c * 2) = lo;
+  constexpr int kAll = ROWS * kVecs / THREADS, kStep = kAll <= 8 ? kAll : (kAll % 8 == 0 ? 8 : 6);
+  static_assert(ROWS * kVecs % THREADS == 0 && kAll % kStep == 0, "whole turns");
+#pragma unroll 1
+  for (int u = 0; u < kAll; u += kStep) {
+    float4 x[kStep];
+#pragma unroll
+    for (int k = 0; k < kStep; ++k) {
+      const int i = threadIdx.x + (u + k) * THREADS, r = i / kVecs, c = i % kVecs * 4;
+      x[k] = r < rows && c < cols ? load4(src + (long long)r * cols + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int k = 0; k < kStep; ++k) {
+      const int i = threadIdx.x + (u + k) * THREADS, r = i / kVecs, c = i % kVecs * 4;
+      uint2 hi, lo;
+      lc_split2(x[k].x, x[k].y, hi.x, lo.x);
+      lc_split2(x[k].z, x[k].w, hi.y, lo.y);
+      *reinterpret_cast<uint2*>(dst + r * pitch + c * 2) = hi;
+      *reinterpret_cast<uint2*>(dst + lo_off + r * pitch + c * 2) = lo;
+    }
   }
 }
 
@@ -480,10 +490,10 @@ __global__ void __launch_bounds__(2 * N) ssd_add_kernel(const SsdChunkParams p) 
   }
 }
 
-// Step 3 with the skip and the gate.  Four warps, 16 rows each.
+// Step 3 with the skip and the gate.  Eight warps: 16 rows and half of the value columns each.
 template <int N, int V>
-__global__ void __launch_bounds__(128) ssd_read_kernel(const SsdChunkParams p) {
-  constexpr int kPn = N * 2 + 16, kPv = V * 2 + 16;
+__global__ void __launch_bounds__(256, 2) ssd_read_kernel(const SsdChunkParams p) {
+  constexpr int kPn = N * 2 + 16, kPv = V * 2 + 16, VH = V / 2;
   extern __shared__ __align__(16) unsigned char sm[];
   unsigned char *s_c = sm, *s_b = s_c + kLcRows * kPn, *s_x = s_b + kLcRows * kPn, *s_s = s_x + kLcRows * kPv;
   __shared__ double s_g[kLcRows];
@@ -494,11 +504,11 @@ __global__ void __launch_bounds__(128) ssd_read_kernel(const SsdChunkParams p) {
   const long long row0 = ch.n0 - a.n_decode;
   const __nv_bfloat16* src = p.xbc + row0 * chan;
   auto sp = [](const void* q) { return (uint32_t)__cvta_generic_to_shared(q); };
-  lc_load_rows<N, 128>(sp(s_b), kPn, src + inner + gr * a.n_state, chan, a.n_state, ch.len);
-  lc_load_rows<N, 128>(sp(s_c), kPn, src + inner + bc + gr * a.n_state, chan, a.n_state, ch.len);
-  lc_load_rows<V, 128>(sp(s_x), kPv, src + h * a.vdim, chan, a.vdim, ch.len);
+  lc_load_rows<N, 256>(sp(s_b), kPn, src + inner + gr * a.n_state, chan, a.n_state, ch.len);
+  lc_load_rows<N, 256>(sp(s_c), kPn, src + inner + bc + gr * a.n_state, chan, a.n_state, ch.len);
+  lc_load_rows<V, 256>(sp(s_x), kPv, src + h * a.vdim, chan, a.vdim, ch.len);
   cp_async_commit();
-  lc_load_split<N, V, 128>(s_s, kPv, N * kPv, p.work + ((long long)blockIdx.x * a.heads + h) * a.n_state * a.vdim, a.n_state, a.vdim);
+  lc_load_split<N, V, 256>(s_s, kPv, N * kPv, p.work + ((long long)blockIdx.x * a.heads + h) * a.n_state * a.vdim, a.n_state, a.vdim);
   if (threadIdx.x < kLcRows) {
     const int r = min((int)threadIdx.x, ch.len - 1);
     s_g[threadIdx.x] = p.gcum[(row0 + r) * a.heads + h];
@@ -506,22 +516,23 @@ __global__ void __launch_bounds__(128) ssd_read_kernel(const SsdChunkParams p) {
   }
   cp_async_wait<0>();
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3, r0 = warp * 16 + g;
-  if (warp * 16 >= ch.len) return;
-  float o[V / 8][4], s[8][4];
+  const int warp = threadIdx.x >> 5 & 3, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3, r0 = warp * 16 + g;
+  const int c0 = (threadIdx.x >> 7) * VH;              // this warp's first column
+  if (warp * 16 >= ch.len || c0 >= a.vdim) return;
+  float o[VH / 8][4], s[8][4];
 #pragma unroll
-  for (int j = 0; j < V / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  for (int j = 0; j < VH / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
 #pragma unroll
   for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
   const uint32_t a_base = sp(s_c) + (warp * 16 + (lane & 15)) * kPn + (lane >> 4) * 16;
   const uint32_t k_base = sp(s_b) + ((lane & 7) + ((lane >> 4) << 3)) * kPn + ((lane >> 3) & 1) * 16;
-  const uint32_t s_base = sp(s_s) + ((lane & 7) + ((lane >> 3) & 1) * 8) * kPv + (lane >> 4) * 16;
+  const uint32_t s_base = sp(s_s) + c0 * 2 + ((lane & 7) + ((lane >> 3) & 1) * 8) * kPv + (lane >> 4) * 16;
 #pragma unroll 2
   for (int kk = 0; kk < N / 16; ++kk) {
     uint32_t c[4];
     ldmatrix_x4(a_base + kk * 32, c[0], c[1], c[2], c[3]);
 #pragma unroll
-    for (int j = 0; j < V / 8; j += 2) {
+    for (int j = 0; j < VH / 8; j += 2) {
       uint32_t bh[4], bl[4];
       ldmatrix_x4_trans(s_base + kk * 16 * kPv + j * 16, bh[0], bh[1], bh[2], bh[3]);
       ldmatrix_x4_trans(s_base + (N + kk * 16) * kPv + j * 16, bl[0], bl[1], bl[2], bl[3]);
@@ -545,9 +556,9 @@ __global__ void __launch_bounds__(128) ssd_read_kernel(const SsdChunkParams p) {
   {
     const float f0 = exp2f((float)g0), f1 = exp2f((float)g1);
 #pragma unroll
-    for (int j = 0; j < V / 8; ++j) { o[j][0] *= f0; o[j][1] *= f0; o[j][2] *= f1; o[j][3] *= f1; }
+    for (int j = 0; j < VH / 8; ++j) { o[j][0] *= f0; o[j][1] *= f0; o[j][2] *= f1; o[j][3] *= f1; }
   }
-  const uint32_t x_base = sp(s_x) + ((lane & 7) + ((lane >> 3) & 1) * 8) * kPv + (lane >> 4) * 16;
+  const uint32_t x_base = sp(s_x) + c0 * 2 + ((lane & 7) + ((lane >> 3) & 1) * 8) * kPv + (lane >> 4) * 16;
 #pragma unroll
   for (int m = 0; m < 4; ++m) {
     if (m > warp) break;
@@ -567,7 +578,7 @@ __global__ void __launch_bounds__(128) ssd_read_kernel(const SsdChunkParams p) {
       }
     }
 #pragma unroll
-    for (int j = 0; j < V / 8; j += 2) {
+    for (int j = 0; j < VH / 8; j += 2) {
       uint32_t b[4];
       ldmatrix_x4_trans(x_base + m * 16 * kPv + j * 16, b[0], b[1], b[2], b[3]);
 #pragma unroll
@@ -585,9 +596,9 @@ __global__ void __launch_bounds__(128) ssd_read_kernel(const SsdChunkParams p) {
     const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(a.proj) + (ch.n0 + t) * a.proj_stride + h * a.vdim;
     float* dst = a.y + (ch.n0 + t) * inner + h * a.vdim;
 #pragma unroll
-    for (int j = 0; j < V / 8; ++j) {
-      if (j * 8 >= a.vdim) break;
-      const int c = j * 8 + tq * 2;
+    for (int j = 0; j < VH / 8; ++j) {
+      if (c0 + j * 8 >= a.vdim) break;
+      const int c = c0 + j * 8 + tq * 2;
       const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + c)), x = lc_pair(s_x + t * kPv + c * 2);
       *reinterpret_cast<float2*>(dst + c) = make_float2(fmaf(skip, x.x, o[j][2 * e]) * silu_act<__nv_bfloat16>(z.x),
                                                         fmaf(skip, x.y, o[j][2 * e + 1]) * silu_act<__nv_bfloat16>(z.y));
@@ -610,7 +621,7 @@ int launch_ssd_chunk(const SsdChunkParams& p, int n_chunks, cudaStream_t st) {
   linear_carry_kernel<false, double><<<carry, 128, 0, st>>>(p.work, p.gcum, a.heads, a.n_decode, a.state, a.slot, a.start, a.cu, p.chunk_off, a.n_decode,
                                                     a.heads, a.n_state, a.vdim);
   MSA_LAUNCH_OK("linear_carry_kernel");
-  ssd_read_kernel<N, V><<<grid, 128, read, st>>>(p);
+  ssd_read_kernel<N, V><<<grid, 256, read, st>>>(p);
   MSA_LAUNCH_OK("ssd_read_kernel");
   return MSA_OK;
 }
