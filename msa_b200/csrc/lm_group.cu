@@ -10,7 +10,7 @@
 
 namespace msa {
 
-constexpr int kGpRows = 8;      // packed rows per block
+constexpr int kGpRows = 8;      // packed rows per block, at most (a step of few rows: one)
 
 struct GroupLayout {
   int nq, nk, nv, chan, width;  // columns of q, k and v, all of them; elements of a ring row
@@ -93,16 +93,16 @@ __global__ void __launch_bounds__(256) group_prep_kernel(const msa_lm_group_args
   }
 }
 
-// Four channels per thread, eight packed rows per block: every input is loaded once.
+// Four channels per thread, up to eight packed rows per block: every input is loaded once.
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256) group_prep_vec_kernel(const msa_lm_group_args a, int row_blocks) {
+__global__ void __launch_bounds__(256) group_prep_vec_kernel(const msa_lm_group_args a, int row_blocks, int rows) {
   extern __shared__ float2 s_turn[];            // [rows][rot / 2]
   const GroupLayout L(a);
   if ((int)blockIdx.x >= row_blocks) {
     if (blockIdx.y == 0) copy_old_row<T, 4>(a, L, (int)blockIdx.x - row_blocks);
     return;
   }
-  const int row0 = blockIdx.x * kGpRows, n_here = min(kGpRows, a.n_tok - row0), half = a.rot / 2;
+  const int row0 = blockIdx.x * rows, n_here = min(rows, a.n_tok - row0), half = a.rot / 2;
   const int c = (blockIdx.y * 256 + threadIdx.x) * 4;
   const bool on = c < L.chan;
   const ConvSource<T> src{reinterpret_cast<const T*>(a.proj), a.proj_stride, reinterpret_cast<T*>(a.conv_state), L.chan, TAPS};
@@ -381,14 +381,14 @@ extern "C" int msa_lm_group_prep(const msa_lm_group_args* args, void* stream) {
   if (a.taps <= 4 && a.dim % 4 == 0 && a.vdim % 4 == 0 && a.proj_stride % 4 == 0 && a.q_pitch % 4 == 0 && a.k_pitch % 4 == 0 &&
       a.v_pitch % 4 == 0 && kGpRows * turn <= 48 * 1024 && ok4(a.proj) && ok4(a.conv_state) && ok4(a.q_out) && ok4(a.ring) && ok4(a.ctx) &&
       aligned16(a.conv_w)) {
-    const int row_blocks = (a.n_tok + kGpRows - 1) / kGpRows;
+    const int rows = a.n_tok <= 256 ? 1 : kGpRows, row_blocks = (a.n_tok + rows - 1) / rows;
     const dim3 grid((unsigned)(row_blocks + a.n_old), (unsigned)((L.chan + 1023) / 1024));
     MSA_LM_DISPATCH(a.dtype, {
       switch (a.taps) {
-        case 1: group_prep_vec_kernel<T, 1><<<grid, 256, kGpRows * turn, st>>>(a, row_blocks); break;
-        case 2: group_prep_vec_kernel<T, 2><<<grid, 256, kGpRows * turn, st>>>(a, row_blocks); break;
-        case 3: group_prep_vec_kernel<T, 3><<<grid, 256, kGpRows * turn, st>>>(a, row_blocks); break;
-        default: group_prep_vec_kernel<T, 4><<<grid, 256, kGpRows * turn, st>>>(a, row_blocks);
+        case 1: group_prep_vec_kernel<T, 1><<<grid, 256, rows * turn, st>>>(a, row_blocks, rows); break;
+        case 2: group_prep_vec_kernel<T, 2><<<grid, 256, rows * turn, st>>>(a, row_blocks, rows); break;
+        case 3: group_prep_vec_kernel<T, 3><<<grid, 256, rows * turn, st>>>(a, row_blocks, rows); break;
+        default: group_prep_vec_kernel<T, 4><<<grid, 256, rows * turn, st>>>(a, row_blocks, rows);
       }
     });
     MSA_LAUNCH_OK("group_prep_vec_kernel");

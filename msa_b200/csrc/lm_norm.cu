@@ -269,7 +269,7 @@ __global__ void token_shift_kernel(const T* __restrict__ h, const float* __restr
   const bool from_state = t == 0, none = from_state && start[s] == 0;
   const T* before = from_state ? state : h + (r - 1) * width;
   const T* last = h + (long long)(cu[s + 1] - 1) * width;
-  for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+  for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * V; i < width; i += gridDim.y * blockDim.x * V) {
     if constexpr (V == 4) {
       const float4 x = load4(h + r * width + i);
       float4 d = none ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(before + i);
@@ -407,9 +407,10 @@ extern "C" int msa_lm_token_shift(const void* h, const float* mu, int32_t n_mix,
   const int e = (int)dtype_size(dtype);
   const bool v4 = width % 4 == 0 && vec4_ok(h, e) && vec4_ok(mu, 4) && vec4_ok(shift, e) && vec4_ok(out, e);
   const int per = v4 ? width / 4 : width, threads = per >= 256 ? 256 : (per + 31) / 32 * 32;
+  const dim3 grid((unsigned)n_tok, n_tok <= 256 ? (unsigned)((per + threads - 1) / threads) : 1u);   // few rows: spread the columns
   MSA_LM_DISPATCH(dtype, {
-    if (v4) token_shift_kernel<T, 4><<<n_tok, threads, 0, (cudaStream_t)stream>>>((const T*)h, mu, n_mix, n_tok, width, tok_seq, slot, start, cu, (T*)shift, (T*)out);
-    else token_shift_kernel<T, 1><<<n_tok, threads, 0, (cudaStream_t)stream>>>((const T*)h, mu, n_mix, n_tok, width, tok_seq, slot, start, cu, (T*)shift, (T*)out);
+    if (v4) token_shift_kernel<T, 4><<<grid, threads, 0, (cudaStream_t)stream>>>((const T*)h, mu, n_mix, n_tok, width, tok_seq, slot, start, cu, (T*)shift, (T*)out);
+    else token_shift_kernel<T, 1><<<grid, threads, 0, (cudaStream_t)stream>>>((const T*)h, mu, n_mix, n_tok, width, tok_seq, slot, start, cu, (T*)shift, (T*)out);
   });
   MSA_LAUNCH_OK("token_shift_kernel");
   return MSA_OK;
