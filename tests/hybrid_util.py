@@ -99,7 +99,7 @@ PAR_WIDE = parallel(256, 320, [
     layer("mamba2", mamba2(6, 64, 128, 2, 3, 4), dense(192)),
     layer("wkv", wkv(2, 128), dense(128)),
     layer("attention", attention(20, 2, 128, 64, 160, 64, 4, base=10000.0), dense(256)),
-    layer("mamba2", mamba2(4, 32, 48, 1, 4, 2), dense(64)),
+    layer("mamba2", mamba2(4, 32, 40, 1, 4, 2), dense(64)),
 ], loop={"start": 2, "stop": 4, "times": 1}, bigram=(127, 11, 3), cap=20.0)
 
 CONFIGS = {"mixed": MIXED, "odd": ODD, "wide": WIDE, "par-mixed": PAR_MIXED, "par-odd": PAR_ODD, "par-wide": PAR_WIDE}
